@@ -1,0 +1,101 @@
+// Windowed causal attention over the paged cache for any head sizes, block size and activation type (bf16 or fp32): one
+// warp per (query row, head).  This is the fp32 path of the models and takes the head shapes that the tensor-core kernels
+// (fmha_sm100.cu for prompt portions, gqa_decode.cu for single tokens) do not.
+//
+//   lane = key     32 scores at a time, each lane reads its key row
+//   lane = column  P V, value rows read coalesced
+// Scores, softmax and the accumulation over the values are fp32.
+#include "../include/omni_vec.cuh"
+
+namespace omni {
+
+constexpr int AA_WARPS = 4;
+constexpr int AA_MAXV = 16;      // value columns per lane: d_v <= 512
+
+template <typename T>
+__global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
+    const T* __restrict__ q, int q_ld, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
+    const int64_t* __restrict__ positions, const int* __restrict__ q_to_seq, const int64_t* __restrict__ slots,
+    const int* __restrict__ block_table, int bt_ld, int rows, int Hq, int Hkv, int dk, int dv, int block_size, int window,
+    float scale, T* __restrict__ out, int out_ld) {
+  extern __shared__ float aa_q[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * AA_WARPS + warp;
+  if (item >= (long long)rows * Hq) return;      // no block-level synchronisation below
+  const int t = (int)(item / Hq), h = (int)(item % Hq), hk = h / (Hq / Hkv);
+  float* sq = aa_q + warp * dk;
+  T* orow = out + (size_t)t * out_ld + h * dv;
+  if (slots[t] < 0) {                            // padding row
+    for (int d = lane; d < dv; d += 32) orow[d] = from_f32<T>(0.f);
+    return;
+  }
+  for (int d = lane; d < dk; d += 32) sq[d] = to_f32(q[(size_t)t * q_ld + h * dk + d]);
+  __syncwarp();
+  const int pos = (int)positions[t];
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int* bt = block_table + (size_t)q_to_seq[t] * bt_ld;
+  float m = -INFINITY, l = 0.f, acc[AA_MAXV];
+#pragma unroll
+  for (int i = 0; i < AA_MAXV; ++i) acc[i] = 0.f;
+  for (int k0 = lo; k0 <= pos; k0 += 32) {
+    const int key = k0 + lane;
+    float s = -INFINITY;
+    size_t head = 0;
+    if (key <= pos) {
+      head = ((size_t)bt[key / block_size] * block_size + key % block_size) * Hkv + hk;
+      const T* kr = k_cache + head * dk;
+      float dot = 0.f;
+      for (int d = 0; d < dk; ++d) dot = fmaf(sq[d], to_f32(kr[d]), dot);
+      s = dot * scale;
+    }
+    float mx = s;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float m_new = fmaxf(m, mx);            // finite: at least one key of the group is visible
+    const float f = expf(m - m_new);
+    const float p = expf(s - m_new);
+    l = l * f + warp_sum32(p);
+    m = m_new;
+#pragma unroll
+    for (int i = 0; i < AA_MAXV; ++i) acc[i] *= f;
+    const int n = min(32, pos - k0 + 1);
+    for (int j = 0; j < n; ++j) {
+      const float pj = __shfl_sync(0xffffffffu, p, j);
+      const T* vr = v_cache + (size_t)__shfl_sync(0xffffffffu, (unsigned long long)head, j) * dv;
+#pragma unroll
+      for (int i = 0; i < AA_MAXV; ++i)
+        if (i * 32 + lane < dv) acc[i] = fmaf(pj, to_f32(vr[i * 32 + lane]), acc[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < AA_MAXV; ++i)
+    if (i * 32 + lane < dv) orow[i * 32 + lane] = from_f32<T>(acc[i] / l);
+}
+
+template <typename T>
+static int launch_attn_any(const void* q, int q_ld, const void* k, const void* v, const int64_t* positions,
+                           const int* q_to_seq, const int64_t* slots, const int* bt, int bt_ld, int rows, int Hq, int Hkv,
+                           int dk, int dv, int block_size, int window, float scale, void* out, int out_ld, cudaStream_t st) {
+  const long long items = (long long)rows * Hq;
+  attn_any_kernel<T><<<(unsigned)((items + AA_WARPS - 1) / AA_WARPS), AA_WARPS * 32, AA_WARPS * dk * sizeof(float), st>>>(
+      (const T*)q, q_ld, (const T*)k, (const T*)v, positions, q_to_seq, slots, bt, bt_ld, rows, Hq, Hkv, dk, dv, block_size,
+      window, scale, (T*)out, out_ld);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace omni
+
+using namespace omni;
+
+extern "C" int omni_attn_any(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int64_t* positions,
+                             const int* q_to_seq, const int64_t* slots, const int* block_table, int bt_ld, int rows, int Hq,
+                             int Hkv, int dk, int dv, int block_size, int window, float scale, void* out, int out_ld, int f32,
+                             cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (Hkv < 1 || Hq % Hkv != 0 || dk < 1 || dk > 2048 || dv < 1 || dv > 32 * AA_MAXV || block_size < 1 || window < 0) return -1;
+  if (f32)
+    return launch_attn_any<float>(q, q_ld, k_cache, v_cache, positions, q_to_seq, slots, block_table, bt_ld, rows, Hq, Hkv, dk,
+                                  dv, block_size, window, scale, out, out_ld, st);
+  return launch_attn_any<__nv_bfloat16>(q, q_ld, k_cache, v_cache, positions, q_to_seq, slots, block_table, bt_ld, rows, Hq,
+                                        Hkv, dk, dv, block_size, window, scale, out, out_ld, st);
+}

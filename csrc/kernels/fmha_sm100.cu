@@ -7,6 +7,10 @@
 // The key dimension may come from two tensors: `k` (per kv head) and `k2` (shared by all heads).  That is how
 // MLA prefill runs without materialising [k_nope | k_pe]: k/v are column slices of the kv_b_proj output,
 // k2 is the roped k_pe slice of the latent rows.  GQA (Qwen) uses k only, with q heads mapped to kv heads.
+// omni_fmha_paged: the same kernel reading K and V tiles from the paged cache through the block table (any head sizes
+// up to 192 / 128 that are multiples of 8: the tensor maps are [rows, heads, head size], so a partial 64-wide chunk is
+// zero-filled), with an optional sliding window - key tiles outside every query's window are never loaded - and with the
+// softmax weights carried as a pair of bf16 values (p = hi + lo, two MMAs), i.e. to 16 bits of mantissa.
 // Causal mask is aligned to the end of the key range (query i of a request with Lq queries and Lk keys sees
 // keys <= Lk - Lq + i), which also covers chunked prefill and prefix-cache hits.
 //
@@ -28,7 +32,13 @@ struct FmhaParams {
   int nk1, nk2;      // number of 64-wide key chunks taken from k and from k2
   float scale_log2;
   int causal;
-  __nv_bfloat16* out;  // [Tq, Hq * 128]
+  __nv_bfloat16* out;  // [Tq, Hq * dv], row pitch out_ld
+  int dv, out_ld;
+  // paged variant: keys of request b live in blocks of the cache, kv_len[b] of them (cu_k is not used)
+  const int* kv_len;
+  const int* block_table;
+  int bt_ld, block_size;
+  int window;          // a query sees the last `window` keys up to its own; 0 = all
   OmniStatus* status;
 };
 
@@ -41,7 +51,7 @@ constexpr int FM_K_STAGE = FM_MAXC * FM_KCHUNK; // 24 KB
 constexpr int FM_V_STAGE = 2 * FM_KCHUNK;       // 16 KB
 constexpr int FM_SMEM = FM_MAXC * FM_QCHUNK + FM_STAGES * (FM_K_STAGE + FM_V_STAGE) + 1024 + 1024;
 constexpr int FM_THREADS = 192;
-constexpr int FT_O = 0, FT_S = 128, FT_P = 256, FT_COLS = 512;
+constexpr int FT_O = 0, FT_S = 128, FT_P = 256, FT_PLO = 320, FT_COLS = 512;
 
 __device__ __forceinline__ void fm_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc,
                                            uint32_t accumulate) {
@@ -52,14 +62,15 @@ __device__ __forceinline__ void fm_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uin
       : "memory");
 }
 
+template <bool PAGED>
 __global__ void __launch_bounds__(FM_THREADS, 1)
 fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                    const __grid_constant__ CUtensorMap tmap_k2, const __grid_constant__ CUtensorMap tmap_v,
                    const FmhaParams p) {
   const int b = blockIdx.y, h = blockIdx.z;
   const int q_begin = p.cu_q[b], q_end = p.cu_q[b + 1];
-  const int k_begin = p.cu_k[b], k_end = p.cu_k[b + 1];
-  const int Lq = q_end - q_begin, Lk = k_end - k_begin;
+  const int k_begin = PAGED ? 0 : p.cu_k[b];
+  const int Lq = q_end - q_begin, Lk = PAGED ? p.kv_len[b] : p.cu_k[b + 1] - k_begin;
   const int q0 = blockIdx.x * FM_BQ;
   if (q0 >= Lq) return;  // uniform for the whole CTA, before any barrier / TMEM use
   const int ctx = Lk - Lq;
@@ -67,7 +78,10 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const int nc = p.nk1 + p.nk2;
   // keys this tile can see
   int k_hi = p.causal ? min(Lk, ctx + q0 + FM_BQ) : Lk;
-  const int n = (k_hi + FM_BK - 1) / FM_BK;
+  int t_first = 0;                                     // first key tile inside the window of the tile's first query
+  if (PAGED && p.window > 0) t_first = max(0, ctx + q0 - p.window + 1) / FM_BK;
+  const int n = (k_hi + FM_BK - 1) / FM_BK - t_first;
+  const int nv = PAGED ? (p.dv + 63) / 64 : 2;         // 64-wide chunks of the value size
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -112,29 +126,39 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   if (warp == 0) {
     if (lane == 0) {
       mbar_expect_tx(q_full, nc * FM_QCHUNK);
-      for (int c = 0; c < nc; ++c)
-        tma_load_2d(sq + c * FM_QCHUNK, &tmap_q, q_full, h * p.q_head_stride + c * 64, q_begin + q0);
+      for (int c = 0; c < nc; ++c) {
+        if (PAGED) tma_load_3d(sq + c * FM_QCHUNK, &tmap_q, q_full, c * 64, h, q_begin + q0);
+        else tma_load_2d(sq + c * FM_QCHUNK, &tmap_q, q_full, h * p.q_head_stride + c * 64, q_begin + q0);
+      }
       for (int i = 0; i < n; ++i) {
         const int st = i % FM_STAGES;
         const uint32_t ph = (i / FM_STAGES) & 1;
-        const int row = k_begin + i * FM_BK;
+        int row = k_begin + i * FM_BK;
+        if (PAGED) {
+          const int key0 = (t_first + i) * FM_BK;
+          row = p.block_table[(size_t)b * p.bt_ld + key0 / p.block_size] * p.block_size + key0 % p.block_size;
+        }
         if (!mbar_wait(&k_empty[st], ph ^ 1, abort_flag, p.status, 11, i)) break;
         mbar_expect_tx(&k_full[st], nc * FM_KCHUNK);
-        for (int c = 0; c < p.nk1; ++c)
-          tma_load_2d(sk + st * FM_K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], hk * p.k_head_stride + c * 64, row);
+        for (int c = 0; c < p.nk1; ++c) {
+          if (PAGED) tma_load_3d(sk + st * FM_K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], c * 64, hk, row);
+          else tma_load_2d(sk + st * FM_K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], hk * p.k_head_stride + c * 64, row);
+        }
         for (int c = 0; c < p.nk2; ++c)
           tma_load_2d(sk + st * FM_K_STAGE + (p.nk1 + c) * FM_KCHUNK, &tmap_k2, &k_full[st], p.k2_col0 + c * 64, row);
         if (!mbar_wait(&v_empty[st], ph ^ 1, abort_flag, p.status, 12, i)) break;
-        mbar_expect_tx(&v_full[st], 2 * FM_KCHUNK);
-        for (int c = 0; c < 2; ++c)
-          tma_load_2d(sv + st * FM_V_STAGE + c * FM_KCHUNK, &tmap_v, &v_full[st],
-                      hk * p.v_head_stride + p.v_col0 + c * 64, row);
+        mbar_expect_tx(&v_full[st], nv * FM_KCHUNK);
+        for (int c = 0; c < nv; ++c) {
+          if (PAGED) tma_load_3d(sv + st * FM_V_STAGE + c * FM_KCHUNK, &tmap_v, &v_full[st], c * 64, hk, row);
+          else tma_load_2d(sv + st * FM_V_STAGE + c * FM_KCHUNK, &tmap_v, &v_full[st],
+                           hk * p.v_head_stride + p.v_col0 + c * 64, row);
+        }
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr uint32_t idesc_qk = umma_idesc(128, FM_BK, 1, 1, 0, 0);
-      constexpr uint32_t idesc_pv = umma_idesc(128, FM_DV, 1, 1, 0, 1);
+      const uint32_t idesc_pv = umma_idesc(128, nv * 64, 1, 1, 0, 1);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 13, 0);
       auto issue_qk = [&](int j) -> bool {
         const int st = j % FM_STAGES;
@@ -168,6 +192,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
           const uint64_t bd = umma_desc_mnmajor_sw128(vbase + k * 2048, FM_KCHUNK, 1024);
           fm_umma_ts(tmem_base + FT_O, tmem_base + FT_P + (i & 1) * (FM_BK / 2) + k * 8, bd, idesc_pv,
                      (i > 0 || k > 0) ? 1u : 0u);
+          if (PAGED) fm_umma_ts(tmem_base + FT_O, tmem_base + FT_PLO + (i & 1) * (FM_BK / 2) + k * 8, bd, idesc_pv, 1u);
         }
         umma_commit(&v_empty[st]);
         umma_commit(o_done);
@@ -185,9 +210,11 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     for (int i = 0; i < n; ++i) {
       if (!mbar_wait(&s_full[i & 1], (i >> 1) & 1, abort_flag, p.status, 17, i)) { ok = false; break; }
       tc_fence_after();
-      const int kbase = i * FM_BK;
+      const int kbase = (t_first + i) * FM_BK;
       int lim = Lk - kbase;                        // keys beyond the request end are masked
       if (p.causal) lim = min(lim, q_pos - kbase + 1);
+      int low = 0;                                 // and those before the window
+      if (PAGED && p.window > 0) low = q_pos - p.window + 1 - kbase;
       float s[FM_BK];
       float mx = -INFINITY;
 #pragma unroll
@@ -197,23 +224,22 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         tmem_ld_wait();
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
-          s[c0 + j] = (c0 + j < lim) ? __uint_as_float(sv32[j]) * p.scale_log2 : -INFINITY;
+          s[c0 + j] = (c0 + j < lim && (!PAGED || c0 + j >= low)) ? __uint_as_float(sv32[j]) * p.scale_log2 : -INFINITY;
           mx = fmaxf(mx, s[c0 + j]);
         }
       }
-      // rows past the end of the request (and, never in practice, fully masked rows) stay finite
-      const float m_cand = fmaxf(m, mx);
-      const float m_new = (m_cand == -INFINITY) ? 0.f : m_cand;
-      const bool grow = (m_new - m) > 8.0f;
-      if (i == 0) {
-        m = m_new;
-      } else if (__any_sync(0xffffffffu, grow)) {
+      // A row that has seen no key yet (its window starts in a later tile, or it lies past the end of the request)
+      // has nothing accumulated: it takes the maximum over as it is.
+      const float m_new = fmaxf(m, mx);
+      const bool grow = m != -INFINITY && (m_new - m) > 8.0f;
+      if (m == -INFINITY) m = m_new;
+      if (i > 0 && __any_sync(0xffffffffu, grow)) {
         if (!mbar_wait(o_done, (i - 1) & 1, abort_flag, p.status, 18, i)) { ok = false; break; }
         tc_fence_after();
         const float f = grow ? exp2f(m - m_new) : 1.0f;
         if (grow) { l *= f; m = m_new; }
 #pragma unroll 1
-        for (int c = 0; c < FM_DV; c += 32) {
+        for (int c = 0; c < nv * 64; c += 32) {
           uint32_t ov[32];
           tmem_ld_x32(lane_addr + FT_O + c, ov);
           tmem_ld_wait();
@@ -223,17 +249,24 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         }
         tmem_st_wait();
       }
-      uint32_t pk[32];
+      uint32_t pk[32], pl[32];
       float rs = 0.f;
+      const float m_ref = m == -INFINITY ? 0.f : m;
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
-        const float p0 = exp2f(s[2 * j] - m), p1 = exp2f(s[2 * j + 1] - m);
+        const float p0 = exp2f(s[2 * j] - m_ref), p1 = exp2f(s[2 * j + 1] - m_ref);
         rs += p0 + p1;
         __nv_bfloat162 h2 = __floats2bfloat162_rn(p0, p1);
         pk[j] = *reinterpret_cast<uint32_t*>(&h2);
+        if (PAGED) {      // what the rounding to bf16 left over
+          const float2 hf = __bfloat1622float2(h2);
+          h2 = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
+          pl[j] = *reinterpret_cast<uint32_t*>(&h2);
+        }
       }
       l += rs;
       tmem_st_x32(lane_addr + FT_P + (i & 1) * (FM_BK / 2), pk);
+      if (PAGED) tmem_st_x32(lane_addr + FT_PLO + (i & 1) * (FM_BK / 2), pl);
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
@@ -244,15 +277,16 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       tc_fence_after();
       const bool row_ok = (q0 + row) < Lq;
       const float inv_l = l > 0.f ? 1.0f / l : 0.f;
-      __nv_bfloat16* orow = p.out + ((size_t)(q_begin + q0 + row) * p.Hq + h) * FM_DV;
+      __nv_bfloat16* orow = p.out + (size_t)(q_begin + q0 + row) * p.out_ld + h * p.dv;
 #pragma unroll 1
-      for (int c = 0; c < FM_DV; c += 32) {
+      for (int c = 0; c < p.dv; c += 32) {
         uint32_t ov[32];
         tmem_ld_x32(lane_addr + FT_O + c, ov);
         tmem_ld_wait();
         if (row_ok) {
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
+            if (PAGED && c + j >= p.dv) break;
             __nv_bfloat16 o8[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) o8[e] = __float2bfloat16(__uint_as_float(ov[j + e]) * inv_l);
@@ -304,9 +338,41 @@ extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q
   p.k_head_stride = k_head_stride; p.v_head_stride = v_head_stride; p.v_col0 = v_col0; p.k2_col0 = k2_col0;
   p.nk1 = d_k1 / 64; p.nk2 = d_k2 / 64; p.scale_log2 = scale * 1.4426950408889634f; p.causal = causal;
   p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
+  p.dv = FM_DV; p.out_ld = Hq * FM_DV;
+  p.kv_len = nullptr; p.block_table = nullptr; p.bt_ld = 0; p.block_size = 0; p.window = 0;
   static bool configured[64] = {false};
-  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel, FM_SMEM, configured)) return e;
+  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel<false>, FM_SMEM, configured)) return e;
   dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
-  fmha_varlen_kernel<<<grid, FM_THREADS, FM_SMEM, stream>>>(tq, tk, tk2, tv, p);
+  fmha_varlen_kernel<false><<<grid, FM_THREADS, FM_SMEM, stream>>>(tq, tk, tk2, tv, p);
+  return (int)cudaGetLastError();
+}
+
+// Ragged queries against the paged cache.  q: rows of pitch q_ld holding Hq heads of d_k; k_cache / v_cache
+// [slots, Hkv, d_k / d_v]; kv_len[b] keys of request b, of which its cu_q segment is the end; out rows of pitch out_ld.
+extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const void* k_cache, const void* v_cache,
+                               long long slots, const int* cu_q, const int* kv_len, const int* block_table, int bt_ld, int B,
+                               int max_q, int Hq, int Hkv, int d_k, int d_v, int block_size, int window, float scale,
+                               void* out, int out_ld, void* status, cudaStream_t stream) {
+  if (B <= 0 || max_q <= 0) return 0;
+  if (d_k < 8 || d_v < 8 || d_k % 8 != 0 || d_v % 8 != 0 || d_k > 64 * FM_MAXC || d_v > FM_DV) return -1;
+  if (Hkv < 1 || Hq % Hkv != 0 || B > 65535 || Hq > 65535 || window < 0) return -2;
+  if (block_size < FM_BK || block_size % FM_BK != 0 || q_ld % 8 != 0 || out_ld % 8 != 0) return -3;
+  if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % 16 != 0) return -4;
+  CUtensorMap tq, tk, tv;
+  if (make_tmap_3d(&tq, q, 2, d_k, Hq, (uint64_t)q_rows, (uint64_t)d_k * 2, (uint64_t)q_ld * 2, 64, 1, FM_BQ, true)) return -10;
+  if (make_tmap_3d(&tk, k_cache, 2, d_k, Hkv, (uint64_t)slots, (uint64_t)d_k * 2, (uint64_t)Hkv * d_k * 2, 64, 1, FM_BK, true))
+    return -11;
+  if (make_tmap_3d(&tv, v_cache, 2, d_v, Hkv, (uint64_t)slots, (uint64_t)d_v * 2, (uint64_t)Hkv * d_v * 2, 64, 1, FM_BK, true))
+    return -13;
+  FmhaParams p;
+  memset(&p, 0, sizeof(p));
+  p.cu_q = cu_q; p.Hq = Hq; p.Hkv = Hkv; p.nk1 = (d_k + 63) / 64; p.nk2 = 0;
+  p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
+  p.dv = d_v; p.out_ld = out_ld; p.kv_len = kv_len; p.block_table = block_table; p.bt_ld = bt_ld;
+  p.block_size = block_size; p.window = window;
+  static bool configured[64] = {false};
+  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel<true>, FM_SMEM, configured)) return e;
+  dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
+  fmha_varlen_kernel<true><<<grid, FM_THREADS, FM_SMEM, stream>>>(tq, tk, tk, tv, p);
   return (int)cudaGetLastError();
 }

@@ -25,6 +25,7 @@
 //   NACC  1 = one accumulator; 2 = two weight tiles (gate rows, up rows) share the X tile
 //   EPI   0 = store (optional per-row multiplier, bf16 or fp32 output)
 //         1 = SwiGLU: silu(gate) * up -> bf16
+//         3 = gelu(gate) * up -> bf16, gelu in its tanh form (bf16 operands only)
 //         2 = SwiGLU then e4m3 quantisation with one scale per (row, 128 output features);
 //             the 128 accumulator lanes of a tile are exactly one quantisation block.
 //
@@ -444,7 +445,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
           }
         }
       } else {
-        // SwiGLU on (gate, up) held by the same lane
+        // gated activation of (gate, up) held by the same lane
 #pragma unroll
         for (int c0 = 0; c0 < CW; c0 += 16) {
           float act[16];
@@ -454,12 +455,15 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
             tmem_ld_x16(lane_addr + bufc * ACC_COLS + BN + c_lo + c0, vu);
             tmem_ld_wait();
 #pragma unroll
-            for (int j = 0; j < 16; ++j) act[j] = silu_f(__uint_as_float(vg[j])) * __uint_as_float(vu[j]);
+            for (int j = 0; j < 16; ++j) {
+              const float g = __uint_as_float(vg[j]);
+              act[j] = (EPI == 3 ? gelu_tanh_f(g) : silu_f(g)) * __uint_as_float(vu[j]);
+            }
           } else {
 #pragma unroll
             for (int j = 0; j < 16; ++j) act[j] = silu_f(accv(0, c0 + j)) * accv(NACC - 1, c0 + j);
           }
-          if (EPI == 1) {
+          if (EPI == 1 || EPI == 3) {
             if (c_lo + c0 < rows && n_ok) {
 #pragma unroll
               for (int j = 0; j < 16; ++j)
@@ -552,7 +556,7 @@ static int launch_gemm(const CUtensorMap& tw, const CUtensorMap& tx, const GemmP
 using namespace omni;
 
 
-// kind: 0 bf16, 1 fp8 block-scaled.  epi: 0 store, 1 swiglu->bf16, 2 swiglu->fp8+scales.
+// kind: 0 bf16, 1 fp8 block-scaled.  epi: 0 store, 1 swiglu->bf16, 2 swiglu->fp8+scales, 3 geglu->bf16.
 // bn: token tile (16, 32, 64, 128, 256); 0 picks from `t_hint` (expected rows per group).
 // x_rows: number of addressable rows of X (and of `out`); rows beyond it read as zero.
 // Returns 0 on success, a negative value for bad arguments, a positive CUDA error otherwise.
@@ -618,6 +622,7 @@ extern "C" int omni_gemm(int kind, int epi, const void* w, const void* x, void* 
   if (kind == KIND_ && bn == BN_ && epi == EPI_) return launch_gemm<KIND_, BN_, NACC_, EPI_>(tw, tx, p, grid, stream);
   OMNI_GEMM_CASE(0, 32, 1, 0) OMNI_GEMM_CASE(0, 64, 1, 0) OMNI_GEMM_CASE(0, 128, 1, 0) OMNI_GEMM_CASE(0, 256, 1, 0)
   OMNI_GEMM_CASE(0, 32, 2, 1) OMNI_GEMM_CASE(0, 64, 2, 1) OMNI_GEMM_CASE(0, 128, 2, 1)
+  OMNI_GEMM_CASE(0, 32, 2, 3) OMNI_GEMM_CASE(0, 64, 2, 3) OMNI_GEMM_CASE(0, 128, 2, 3)
   OMNI_GEMM_CASE(1, 32, 1, 0) OMNI_GEMM_CASE(1, 64, 1, 0) OMNI_GEMM_CASE(1, 128, 1, 0)
   OMNI_GEMM_CASE(1, 32, 2, 1) OMNI_GEMM_CASE(1, 64, 2, 1)
   OMNI_GEMM_CASE(1, 32, 2, 2) OMNI_GEMM_CASE(1, 64, 2, 2)

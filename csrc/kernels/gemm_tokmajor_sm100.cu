@@ -25,7 +25,7 @@
 // The 256 weight rows of a tile are two blocks of 128 (each with its own weight scale).  EPI 0 = store: the
 // blocks are consecutive output features (bf16 or fp32 output, optional per-row multiplier).  EPI 1 / 2 =
 // SwiGLU: W holds n_out gate rows, then n_out up rows, per group; block 0 is 128 gate rows, block 1 the
-// matching up rows, and the tile produces 128 output features: EPI 1 -> bf16, EPI 2 -> e4m3 with one scale
+// matching up rows, and the tile produces 128 output features: EPI 1 -> bf16 (EPI 3: the same with gelu), EPI 2 -> e4m3 with one scale
 // per token and 128 output features (exactly one tile).
 //
 // KIND 0 = bf16 operands: the whole K range accumulates in TMEM and the epilogue runs once per tile.
@@ -484,16 +484,16 @@ gemm_tokmajor_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_co
           }
         }
       } else {
-        // SwiGLU on (gate, up) held by the same thread; overwrite the gate accumulator with the activation
+        // gated activation of (gate, up) held by the same thread; overwrite the gate accumulator with the activation
         const int n0 = nt * TM_BN + c_lo;
         float amax = 0.f;
 #pragma unroll
         for (int j = 0; j < TM_CW / 2; ++j) {
-          acc[0][j].x = silu_f(acc[0][j].x) * acc[NB - 1][j].x;
-          acc[0][j].y = silu_f(acc[0][j].y) * acc[NB - 1][j].y;
+          acc[0][j].x = (EPI == 3 ? gelu_tanh_f(acc[0][j].x) : silu_f(acc[0][j].x)) * acc[NB - 1][j].x;
+          acc[0][j].y = (EPI == 3 ? gelu_tanh_f(acc[0][j].y) : silu_f(acc[0][j].y)) * acc[NB - 1][j].y;
           amax = fmaxf(amax, fmaxf(fabsf(acc[0][j].x), fabsf(acc[0][j].y)));
         }
-        if (EPI == 1) {
+        if (EPI == 1 || EPI == 3) {
           if (row_ok) {
             __nv_bfloat16* o = (__nv_bfloat16*)p.out + row * p.out_ld + n0;
             const bool wide = ((uintptr_t)o & 31) == 0;
@@ -633,7 +633,7 @@ extern "C" int omni_gemm_tm2(int kind, int epi, const void* w, const void* x, vo
   if (kind == 1 && ((x_scale_ld % 4) != 0 || ((uintptr_t)x_scale % 16) != 0)) return -7;
   if (epi == 2 && (out_scale == nullptr || kind != 1)) return -5;
   if ((n_out % 8) != 0 || (out_ld % 8) != 0 || (out_group_col % 8) != 0) return -8;
-  if (epi < 0 || epi > 2) return -9;
+  if (epi < 0 || epi > 3 || (epi == 3 && kind != 0)) return -9;
   TmGemmParams p;
   memset(&p, 0, sizeof(p));
   p.G = G; p.n_out = n_out; p.K = K; p.T = T; p.seg_start = seg_start; p.seg_len = seg_len;
@@ -672,6 +672,7 @@ extern "C" int omni_gemm_tm2(int kind, int epi, const void* w, const void* x, vo
   if (kind == 0) {
     if (epi == 0) return launch_tm<0, 0>(tx, tw, p, grid, stream);
     if (epi == 1) return launch_tm<0, 1>(tx, tw, p, grid, stream);
+    if (epi == 3) return launch_tm<0, 3>(tx, tw, p, grid, stream);
     return -9;
   }
   if (epi == 0) return launch_tm<1, 0>(tx, tw, p, grid, stream);

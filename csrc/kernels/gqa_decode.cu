@@ -20,6 +20,11 @@
 // log-sum-exps that a small second kernel combines.  This is a bandwidth-bound op on a few query rows, so the
 // warp-level MMA is enough: the tensor pipe is idle most of the time either way.
 //
+// omni_gqa_paged_decode_window runs the general form of the same kernel: key and value sizes of their own (multiples of
+// 8 up to 256; staged rows are DP = 64, 128 or 256 wide and the columns past the real size stay zero), any number of query
+// heads per KV head (16 per CTA), a sliding window (tiles before it are not read), and softmax weights carried as a pair
+// of bf16 values (two MMAs per value tile), i.e. to 16 bits of mantissa.
+//
 // Reference counterpart: the paged decode attention of the GQA backend
 // (omni/models/common/layers/attention/backend/attention.py:507-702).
 #include <cuda_bf16.h>
@@ -29,18 +34,26 @@
 
 namespace omni {
 
-constexpr int GQ_D = 128;
+constexpr int GQ_D = 128;                              // head size of the special form
 constexpr int GQ_TILE = 32;                            // keys per warp tile
-constexpr int GQ_ROW_BYTES = GQ_D * 2;                 // 256
-constexpr int GQ_STAGE_BYTES = 2 * GQ_TILE * GQ_ROW_BYTES;   // K and V of one tile: 16 KB
 constexpr int GQ_WARPS = 4;
-constexpr int GQ_Q_BYTES = 16 * GQ_ROW_BYTES;          // 16 query rows (zero padded)
-constexpr int GQ_SMEM = GQ_WARPS * GQ_STAGE_BYTES + GQ_Q_BYTES;
-static_assert(GQ_WARPS * GQ_STAGE_BYTES >= GQ_WARPS * 16 * GQ_D * 4 + 2 * GQ_WARPS * 16 * 4,
-              "the staging area is reused for the merge of the four warps");
+template <int DP>
+struct GqSmem {
+  static constexpr int ROW_BYTES = DP * 2;
+  static constexpr int STAGE_BYTES = 2 * GQ_TILE * ROW_BYTES;   // K and V of one tile: 16 KB for DP = 128
+  static constexpr int Q_BYTES = 16 * ROW_BYTES;                // 16 query rows (zero padded)
+  static constexpr int TOTAL = GQ_WARPS * STAGE_BYTES + Q_BYTES;
+  static_assert(GQ_WARPS * STAGE_BYTES >= GQ_WARPS * 16 * DP * 4 + 2 * GQ_WARPS * 16 * 4,
+                "the staging area is reused for the merge of the four warps");
+};
+
+struct GqShape {           // used by the general form only
+  int q_ld, out_ld, dk, dv, window;
+};
 
 __device__ __forceinline__ uint32_t gq_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ uint32_t gq_swz(int row, int chunk) { return (uint32_t)(row * GQ_ROW_BYTES + ((chunk ^ (row & 7)) << 4)); }
+template <int DP>
+__device__ __forceinline__ uint32_t gq_swz(int row, int chunk) { return (uint32_t)(row * DP * 2 + ((chunk ^ (row & 7)) << 4)); }
 
 __device__ __forceinline__ void gq_cp_async16(uint32_t dst, const void* src, bool valid) {
   const int n = valid ? 16 : 0;     // 0 source bytes: the 16 destination bytes are zero-filled
@@ -68,45 +81,67 @@ __device__ __forceinline__ uint32_t gq_pack(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
 }
+__device__ __forceinline__ uint32_t gq_rest(uint32_t packed, float lo, float hi) {
+  const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&packed));
+  return gq_pack(lo - f.x, hi - f.y);
+}
 
-__global__ void __launch_bounds__(GQ_WARPS * 32, 3)
+template <int DP, bool GEN>
+__global__ void __launch_bounds__(GQ_WARPS * 32, DP > 128 ? 1 : 3)
 gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                   const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_table, int bt_ld,
                   const int* __restrict__ seq_lens, int block_size, int Hq, int Hkv, float scale_log2, int splits,
-                  float* __restrict__ o_part, float* __restrict__ lse_part, __nv_bfloat16* __restrict__ out) {
+                  float* __restrict__ o_part, float* __restrict__ lse_part, __nv_bfloat16* __restrict__ out,
+                  const GqShape sh) {
   extern __shared__ __align__(1024) uint8_t gq_smem[];
-  const int hk = blockIdx.x, split = blockIdx.y, b = blockIdx.z;
-  const int G = Hq / Hkv;
+  using SM = GqSmem<DP>;
+  const int split = blockIdx.y, b = blockIdx.z;
+  const int Gall = Hq / Hkv;
+  const int nsub = GEN ? (Gall + 15) >> 4 : 1;                // CTAs per KV head
+  const int hk = GEN ? blockIdx.x / nsub : blockIdx.x;
+  const int g0 = GEN ? (blockIdx.x - hk * nsub) * 16 : 0;     // first query head of this CTA within the group
+  const int G = GEN ? min(16, Gall - g0) : Gall;
+  const int dk = GEN ? sh.dk : DP, dv = GEN ? sh.dv : DP;
+  const int q_ld = GEN ? sh.q_ld : Hq * DP, out_ld = GEN ? sh.out_ld : Hq * DP;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int L = seq_lens[b];
-  const int tiles = (L + GQ_TILE - 1) / GQ_TILE;
+  const int low = (GEN && sh.window > 0) ? max(0, L - sh.window) : 0;     // first visible key
+  const int tile0 = low / GQ_TILE;
+  const int tiles = (L + GQ_TILE - 1) / GQ_TILE - tile0;
   const int tps = (tiles + splits - 1) / splits;
-  const int t_begin = split * tps, t_end = min(tiles, t_begin + tps);
+  const int t_begin = tile0 + split * tps, t_end = min(tile0 + tiles, t_begin + tps);
 
-  uint8_t* stage = gq_smem + warp * GQ_STAGE_BYTES;           // [K tile 8 KB][V tile 8 KB]
-  uint8_t* sq = gq_smem + GQ_WARPS * GQ_STAGE_BYTES;          // 16 x 128 bf16, swizzled like the tiles
-  const uint32_t stage_k = gq_smem_u32(stage), stage_v = stage_k + GQ_TILE * GQ_ROW_BYTES, sq_addr = gq_smem_u32(sq);
+  uint8_t* stage = gq_smem + warp * SM::STAGE_BYTES;          // [K tile][V tile]
+  uint8_t* sq = gq_smem + GQ_WARPS * SM::STAGE_BYTES;         // 16 x DP bf16, swizzled like the tiles
+  const uint32_t stage_k = gq_smem_u32(stage), stage_v = stage_k + GQ_TILE * SM::ROW_BYTES, sq_addr = gq_smem_u32(sq);
 
   // query rows of this group (rows >= G are zero)
-  for (int i = threadIdx.x; i < 16 * 16; i += blockDim.x) {
-    const int row = i >> 4, chunk = i & 15;
+  constexpr int CH = DP / 8;                                  // 16-byte chunks of a staged row
+  for (int i = threadIdx.x; i < 16 * CH; i += blockDim.x) {
+    const int row = i / CH, chunk = i % CH;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (row < G) v = *reinterpret_cast<const uint4*>(q + ((size_t)b * Hq + hk * G + row) * GQ_D + chunk * 8);
-    *reinterpret_cast<uint4*>(sq + gq_swz(row, chunk)) = v;
+    if (row < G && chunk * 8 < dk)
+      v = *reinterpret_cast<const uint4*>(q + (size_t)b * q_ld + (hk * Gall + g0 + row) * dk + chunk * 8);
+    *reinterpret_cast<uint4*>(sq + gq_swz<DP>(row, chunk)) = v;
+  }
+  if (GEN && (dk < DP || dv < DP)) {                          // the columns past the head size are never staged
+    for (int i = threadIdx.x; i < GQ_WARPS * SM::STAGE_BYTES / 16; i += blockDim.x)
+      reinterpret_cast<uint4*>(gq_smem)[i] = make_uint4(0u, 0u, 0u, 0u);
   }
   __syncthreads();
-  // A fragments of Q for the eight 16-wide steps over the head dimension
-  uint32_t qa[8][4];
+  // A fragments of Q for the 16-wide steps over the head dimension
+  constexpr int KS = DP / 16, JT = DP / 8;                    // 16-wide steps over the head size, 8-wide output tiles
+  uint32_t qa[KS][4];
   {
     const int row = ((lane >> 3) & 1) * 8 + (lane & 7), chalf = lane >> 4;
 #pragma unroll
-    for (int ks = 0; ks < 8; ++ks) gq_ldmatrix_x4(sq_addr + gq_swz(row, ks * 2 + chalf), qa[ks]);
+    for (int ks = 0; ks < KS; ++ks) gq_ldmatrix_x4(sq_addr + gq_swz<DP>(row, ks * 2 + chalf), qa[ks]);
   }
 
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  float o[16][4];
+  float o[JT][4];
 #pragma unroll
-  for (int j = 0; j < 16; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
+  for (int j = 0; j < JT; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
 
   for (int t = t_begin + warp; t < t_end; t += GQ_WARPS) {
     // ---- stage the tile: lane `r` knows where key row r of the tile lives
@@ -115,13 +150,13 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
     long long my_slot = 0;
     if (my_valid) my_slot = (long long)block_table[(size_t)b * bt_ld + my_key / block_size] * block_size + my_key % block_size;
 #pragma unroll 4
-    for (int it = 0; it < 16; ++it) {
-      const int row = it * 2 + (lane >> 4), chunk = lane & 15;
+    for (int it = 0; it < GQ_TILE * CH / 32; ++it) {
+      const int row = (it * 32 + lane) / CH, chunk = (it * 32 + lane) % CH;
       const long long slot = __shfl_sync(0xffffffffu, my_slot, row);
       const bool valid = __shfl_sync(0xffffffffu, (int)my_valid, row) != 0;
-      const size_t off = ((size_t)slot * Hkv + hk) * GQ_D + chunk * 8;
-      gq_cp_async16(stage_k + gq_swz(row, chunk), k_cache + off, valid);
-      gq_cp_async16(stage_v + gq_swz(row, chunk), v_cache + off, valid);
+      const size_t head = (size_t)slot * Hkv + hk;
+      if (!GEN || chunk * 8 < dk) gq_cp_async16(stage_k + gq_swz<DP>(row, chunk), k_cache + head * dk + chunk * 8, valid);
+      if (!GEN || chunk * 8 < dv) gq_cp_async16(stage_v + gq_swz<DP>(row, chunk), v_cache + head * dv + chunk * 8, valid);
     }
     gq_cp_async_wait_all();
     __syncwarp();
@@ -134,9 +169,9 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
     for (int j = 0; j < 4; ++j) {
       const int krow = j * 8 + (lane & 7);
 #pragma unroll
-      for (int kp = 0; kp < 4; ++kp) {          // two 16-wide steps per ldmatrix.x4
+      for (int kp = 0; kp < KS / 2; ++kp) {     // two 16-wide steps per ldmatrix.x4
         uint32_t kb[4];
-        gq_ldmatrix_x4(stage_k + gq_swz(krow, kp * 4 + (lane >> 3)), kb);
+        gq_ldmatrix_x4(stage_k + gq_swz<DP>(krow, kp * 4 + (lane >> 3)), kb);
         gq_mma(s[j], qa[2 * kp], kb[0], kb[1]);
         gq_mma(s[j], qa[2 * kp + 1], kb[2], kb[3]);
       }
@@ -149,7 +184,7 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + j * 8 + (e & 1);
-        const float v = key < L ? s[j][e] * scale_log2 : -INFINITY;
+        const float v = (key < L && (!GEN || key >= low)) ? s[j][e] * scale_log2 : -INFINITY;
         s[j][e] = v;
         mt[e >> 1] = fmaxf(mt[e >> 1], v);
       }
@@ -180,8 +215,8 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
       l[r] = l[r] * f[r] + rs[r];
     }
 #pragma unroll
-    for (int j = 0; j < 16; ++j) { o[j][0] *= f[0]; o[j][1] *= f[0]; o[j][2] *= f[1]; o[j][3] *= f[1]; }
-    // ---- O += P V : two 16-key steps, sixteen 8-wide output tiles
+    for (int j = 0; j < JT; ++j) { o[j][0] *= f[0]; o[j][1] *= f[0]; o[j][2] *= f[1]; o[j][3] *= f[1]; }
+    // ---- O += P V : two 16-key steps, 8-wide output tiles
 #pragma unroll
     for (int ks = 0; ks < 2; ++ks) {
       uint32_t pa[4];
@@ -189,13 +224,24 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
       pa[1] = gq_pack(s[2 * ks][2], s[2 * ks][3]);
       pa[2] = gq_pack(s[2 * ks + 1][0], s[2 * ks + 1][1]);
       pa[3] = gq_pack(s[2 * ks + 1][2], s[2 * ks + 1][3]);
+      uint32_t pl[4];                           // general form: what the rounding of the weights left over
+      if (GEN) {
+        pl[0] = gq_rest(pa[0], s[2 * ks][0], s[2 * ks][1]);
+        pl[1] = gq_rest(pa[1], s[2 * ks][2], s[2 * ks][3]);
+        pl[2] = gq_rest(pa[2], s[2 * ks + 1][0], s[2 * ks + 1][1]);
+        pl[3] = gq_rest(pa[3], s[2 * ks + 1][2], s[2 * ks + 1][3]);
+      }
       const int vrow = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
 #pragma unroll
-      for (int jp = 0; jp < 8; ++jp) {          // two output tiles per ldmatrix.x4.trans
+      for (int jp = 0; jp < JT / 2; ++jp) {     // two output tiles per ldmatrix.x4.trans
         uint32_t vb[4];
-        gq_ldmatrix_x4_trans(stage_v + gq_swz(vrow, jp * 2 + (lane >> 4)), vb);
+        gq_ldmatrix_x4_trans(stage_v + gq_swz<DP>(vrow, jp * 2 + (lane >> 4)), vb);
         gq_mma(o[2 * jp], pa, vb[0], vb[1]);
         gq_mma(o[2 * jp + 1], pa, vb[2], vb[3]);
+        if (GEN) {
+          gq_mma(o[2 * jp], pl, vb[0], vb[1]);
+          gq_mma(o[2 * jp + 1], pl, vb[2], vb[3]);
+        }
       }
     }
     __syncwarp();      // every lane is done with the staged tile before the next copies land
@@ -203,15 +249,15 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 
   // ---- merge the four warps (staging memory is free now)
   __syncthreads();
-  float* s_o = reinterpret_cast<float*>(gq_smem);                     // [4][16][128]
-  float* s_m = s_o + GQ_WARPS * 16 * GQ_D;                            // [4][16]
+  float* s_o = reinterpret_cast<float*>(gq_smem);                     // [4][16][DP]
+  float* s_m = s_o + GQ_WARPS * 16 * DP;                              // [4][16]
   float* s_l = s_m + GQ_WARPS * 16;
   {
     const int g = lane >> 2, c = (lane & 3) * 2;
 #pragma unroll
-    for (int j = 0; j < 16; ++j) {
-      float* r0 = s_o + ((size_t)warp * 16 + g) * GQ_D + j * 8 + c;
-      float* r1 = s_o + ((size_t)warp * 16 + g + 8) * GQ_D + j * 8 + c;
+    for (int j = 0; j < JT; ++j) {
+      float* r0 = s_o + ((size_t)warp * 16 + g) * DP + j * 8 + c;
+      float* r1 = s_o + ((size_t)warp * 16 + g + 8) * DP + j * 8 + c;
       r0[0] = o[j][0]; r0[1] = o[j][1]; r1[0] = o[j][2]; r1[1] = o[j][3];
     }
     if ((lane & 3) == 0) {
@@ -220,8 +266,9 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
     }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < G * GQ_D; idx += blockDim.x) {
-    const int g = idx / GQ_D, d = idx - g * GQ_D;
+  for (int idx = threadIdx.x; idx < G * DP; idx += blockDim.x) {
+    const int g = idx / DP, d = idx - g * DP;
+    if (GEN && d >= dv) continue;
     float mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < GQ_WARPS; ++w) mm = fmaxf(mm, s_m[w * 16 + g]);
@@ -232,24 +279,25 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
         const float mw = s_m[w * 16 + g];
         const float fw = mw == -INFINITY ? 0.f : exp2f(mw - mm);
         ll += s_l[w * 16 + g] * fw;
-        acc += s_o[((size_t)w * 16 + g) * GQ_D + d] * fw;
+        acc += s_o[((size_t)w * 16 + g) * DP + d] * fw;
       }
     }
-    const int hq = hk * G + g;
+    const int hq = hk * Gall + g0 + g;
     if (splits == 1) {
-      out[((size_t)b * Hq + hq) * GQ_D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
     } else {
-      o_part[(((size_t)b * splits + split) * Hq + hq) * GQ_D + d] = ll > 0.f ? acc / ll : 0.f;
+      o_part[(((size_t)b * splits + split) * Hq + hq) * dv + d] = ll > 0.f ? acc / ll : 0.f;
       if (d == 0) lse_part[((size_t)b * splits + split) * Hq + hq] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
     }
   }
 }
 
 __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part, int splits,
-                                   int Hq, __nv_bfloat16* out) {
+                                   int Hq, int dv, int out_ld, __nv_bfloat16* out) {
   const int bh = blockIdx.x;
   const int b = bh / Hq, h = bh - b * Hq;
   const int d = threadIdx.x;
+  if (d >= dv) return;
   float mx = -INFINITY;
   for (int s = 0; s < splits; ++s) mx = fmaxf(mx, lse_part[((size_t)b * splits + s) * Hq + h]);
   float den = 0.f, acc = 0.f;
@@ -258,14 +306,40 @@ __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float
     if (v == -INFINITY) continue;
     const float w = exp2f(v - mx);
     den += w;
-    acc += w * o_part[(((size_t)b * splits + s) * Hq + h) * GQ_D + d];
+    acc += w * o_part[(((size_t)b * splits + s) * Hq + h) * dv + d];
   }
-  out[(size_t)bh * GQ_D + d] = __float2bfloat16(den > 0.f ? acc / den : 0.f);
+  out[(size_t)b * out_ld + h * dv + d] = __float2bfloat16(den > 0.f ? acc / den : 0.f);
 }
 
 }  // namespace omni
 
 using namespace omni;
+
+template <int DP, bool GEN>
+static int launch_gqa(dim3 grid, const void* q, const void* k_cache, const void* v_cache, const int* block_table, int bt_ld,
+                      const int* seq_lens, int B, int block_size, int Hq, int Hkv, float scale, int splits, float* o_part,
+                      float* lse_part, void* out, const GqShape& sh, int dv, int out_ld, cudaStream_t stream) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaError_t e = cudaGetDevice(&dev);
+  if (e != cudaSuccess) return (int)e;
+  if (dev < 0 || dev >= 64 || !configured[dev]) {
+    e = cudaFuncSetAttribute(gqa_decode_kernel<DP, GEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, GqSmem<DP>::TOTAL);
+    if (e != cudaSuccess) return (int)e;
+    if (dev >= 0 && dev < 64) configured[dev] = true;
+  }
+  gqa_decode_kernel<DP, GEN><<<grid, GQ_WARPS * 32, GqSmem<DP>::TOTAL, stream>>>(
+      (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_table, bt_ld, seq_lens,
+      block_size, Hq, Hkv, scale * 1.4426950408889634f, splits, o_part, lse_part, (__nv_bfloat16*)out, sh);
+  e = cudaGetLastError();
+  if (e != cudaSuccess) return (int)e;
+  if (splits > 1) {
+    gqa_combine_kernel<<<B * Hq, (dv + 31) / 32 * 32, 0, stream>>>(o_part, lse_part, splits, Hq, dv, out_ld,
+                                                                   (__nv_bfloat16*)out);
+    e = cudaGetLastError();
+  }
+  return (int)e;
+}
 
 extern "C" int omni_gqa_paged_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                                      int bt_ld, const int* seq_lens, int B, int Hq, int Hkv, int D, int block_size,
@@ -274,25 +348,29 @@ extern "C" int omni_gqa_paged_decode(const void* q, const void* k_cache, const v
   if (B <= 0) return 0;
   if (D != GQ_D || Hq % Hkv != 0 || Hq / Hkv > 16 || splits < 1) return -1;
   if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaError_t e = cudaGetDevice(&dev);
-  if (e != cudaSuccess) return (int)e;
-  if (dev < 0 || dev >= 64 || !configured[dev]) {
-    e = cudaFuncSetAttribute(gqa_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, GQ_SMEM);
-    if (e != cudaSuccess) return (int)e;
-    if (dev >= 0 && dev < 64) configured[dev] = true;
-  }
-  dim3 grid(Hkv, splits, B);
-  gqa_decode_kernel<<<grid, GQ_WARPS * 32, GQ_SMEM, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache,
-                                                             (const __nv_bfloat16*)v_cache, block_table, bt_ld, seq_lens,
-                                                             block_size, Hq, Hkv, scale * 1.4426950408889634f, splits, o_part,
-                                                             lse_part, (__nv_bfloat16*)out);
-  e = cudaGetLastError();
-  if (e != cudaSuccess) return (int)e;
-  if (splits > 1) {
-    gqa_combine_kernel<<<B * Hq, GQ_D, 0, stream>>>(o_part, lse_part, splits, Hq, (__nv_bfloat16*)out);
-    e = cudaGetLastError();
-  }
-  return (int)e;
+  GqShape sh = {};
+  return launch_gqa<GQ_D, false>(dim3(Hkv, splits, B), q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq,
+                                 Hkv, scale, splits, o_part, lse_part, out, sh, GQ_D, Hq * GQ_D, stream);
+}
+
+// General form: q rows of pitch q_ld, key size dk, value size dv, out rows of pitch out_ld, window 0 = all keys.
+extern "C" int omni_gqa_paged_decode_window(const void* q, int q_ld, const void* k_cache, const void* v_cache,
+                                            const int* block_table, int bt_ld, const int* seq_lens, int B, int Hq, int Hkv,
+                                            int dk, int dv, int block_size, int window, float scale, int splits,
+                                            float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (Hkv < 1 || Hq % Hkv != 0 || splits < 1 || splits > 65535 || B > 65535 || window < 0) return -1;
+  if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;
+  if (dk < 8 || dv < 8 || dk % 8 != 0 || dv % 8 != 0 || dk > 256 || dv > 256) return -3;
+  if (q_ld % 8 != 0 || ((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16 != 0) return -4;
+  const GqShape sh = {q_ld, out_ld, dk, dv, window};
+  const dim3 grid(Hkv * ((Hq / Hkv + 15) / 16), splits, B);
+  const int d = dk > dv ? dk : dv;
+#define GQA_CASE(DP)                                                                                                     \
+  if (d <= DP)                                                                                                           \
+    return launch_gqa<DP, true>(grid, q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq, Hkv, scale,  \
+                                splits, o_part, lse_part, out, sh, dv, out_ld, stream);
+  GQA_CASE(64) GQA_CASE(128) GQA_CASE(256)
+#undef GQA_CASE
+  return -5;
 }

@@ -36,7 +36,8 @@ class DecodeGraphs:
             q_seq_lens=torch.zeros(n, dtype=torch.int32, device=dev),
             q_to_seq=(torch.arange(n, dtype=torch.int32, device=dev) // tpr).int(),
             max_seq_len=r.cfg.max_model_len,
-            num_valid=torch.zeros(1, dtype=torch.int32, device=dev))
+            num_valid=torch.zeros(1, dtype=torch.int32, device=dev),
+            state_slots=torch.full((padded,), -1, dtype=torch.int32, device=dev) if r.has_state else None)
         ids = torch.zeros(n, dtype=torch.int64, device=dev)
         return ids, md
 
@@ -72,6 +73,8 @@ class DecodeGraphs:
         s_md.block_table.copy_(md.block_table)
         s_md.seq_lens.copy_(md.seq_lens)
         s_md.q_seq_lens.copy_(md.q_seq_lens)
+        if md.state_slots is not None:
+            s_md.state_slots.copy_(md.state_slots)
         if md.num_valid is not None:
             s_md.num_valid.copy_(md.num_valid)
         else:

@@ -71,6 +71,7 @@ class ModelRunner:
         self._bt_width = (cfg.max_model_len + cfg.block_size - 1) // cfg.block_size + 1
         self.step_times: list = []
         self.omni = None
+        self.has_state = model_cfg.has_recurrent_state     # one slot of recurrent state per live request
         self._agreements_done = 0      # per-step host agreements completed (the first ones belong to start-up)
 
     # ------------------------------------------------------------------ model / cache set-up
@@ -78,6 +79,13 @@ class ModelRunner:
         cfg = self.model_cfg
         t0 = time.time()
         self.setup_tensor_parallel()
+        if cfg.layers is not None:
+            if get_parallel_state().world_size > 1 and (self.cfg.attn_tp or self.cfg.vocab_parallel or get_parallel_state().pp_size > 1):
+                raise ValueError("layer-list models run whole on every rank (data parallel)")
+            if self.kv_connector is not None and self.has_state:
+                raise ValueError("KV hand-over between instances does not carry recurrent state")
+            # positions are unbounded by design: the rotation tables cover what this engine may reach
+            cfg.max_position_embeddings = max(cfg.max_position_embeddings, self.cfg.max_model_len + 64)
         self.model = build_model(cfg, device=self.device, planner=self.planner,
                                  seed=seed if weights is None else None)
         from ...models.deepseek_mtp import DeepseekV3MTP
@@ -237,6 +245,8 @@ class ModelRunner:
 
     def kv_bytes_per_block(self) -> int:
         cfg = self.model_cfg
+        if cfg.layers is not None:
+            return max(1, self.cfg.block_size * self.model.kv_bytes_per_token())
         layers = self.model.num_kv_layers + len(self.drafters)
         esz = 4 if cfg.dtype == "float32" else 2
         return layers * self.cfg.block_size * cfg.kv_bytes_per_token(esz)
@@ -248,6 +258,8 @@ class ModelRunner:
             return 256
         free, total = torch.cuda.mem_get_info(self.device)
         budget = free - int(total * (1.0 - self.cfg.gpu_memory_utilization))
+        if self.has_state:
+            budget -= self.model.state_bytes(self.cfg.max_num_seqs)
         return max(16, int(budget // self.kv_bytes_per_block()))
 
     def initialize_kv_cache(self, num_blocks: int) -> None:
@@ -270,6 +282,14 @@ class ModelRunner:
             return (zeros(num_blocks, bs, cfg.local_kv_heads, cfg.head_dim),
                     zeros(num_blocks, bs, cfg.local_kv_heads, cfg.head_dim))
 
+        if cfg.layers is not None:      # page pools and state slots, one entry per layer
+            self.kv_caches = self.model.allocate_caches(
+                num_blocks, bs, self.cfg.max_num_seqs, lambda *shape, dtype: torch.zeros(*shape, dtype=dtype, device=self.device))
+            self.drafter_kv = []
+            if self.kv_connector is not None:
+                self.kv_connector.register_kv_caches([c for c, s in zip(self.kv_caches, cfg.layers)
+                                                      if s.attention is not None and s.attention.owns_kv])
+            return
         self.kv_caches = [one() for _ in range(self.model.num_kv_layers)]
         self.drafter_kv = [[one()] for _ in self.drafters]
         if self.kv_connector is not None:
@@ -278,6 +298,8 @@ class ModelRunner:
     def enable_omni_attn(self, state, num_window_blocks: int) -> None:
         """Compressed layers get a cache of per-request windows; decode runs eagerly from here on."""
         cfg, bs = self.model_cfg, self.cfg.block_size
+        if cfg.layers is not None:
+            raise ValueError("Omni-Attention compresses the caches of the uniform attention stacks only")
         self.omni = state
         dt = self.model.model.dtype
         ipc = (self.kv_connector is not None and getattr(self.kv_connector, "transport", "inproc") != "inproc"
@@ -356,7 +378,8 @@ class ModelRunner:
     def _prepare_prefill(self, so: SchedulerOutput):
         ids, pos, slots, cu_q, cu_k, qlens, ctx, sample_idx, seq_lens = [], [], [], [0], [0], [], [], [], []
         gather, need_gather = [], False
-        bt_rows = []
+        bt_rows, q_to_seq, state_slots = [], [], []
+        layer_list = self.model_cfg.layers is not None      # attention reads the pages: nothing is gathered
         for s in so.scheduled:
             r = s.request
             st, n = r.num_computed_tokens, s.num_scheduled_tokens
@@ -369,8 +392,12 @@ class ModelRunner:
             qlens.append(n)
             ctx.append(st)
             seq_lens.append(st + n)
-            need_gather |= st > 0
-            gather += self._slots(r.block_ids, 0, st + n)
+            if layer_list:
+                q_to_seq += [len(qlens) - 1] * n
+                state_slots.append(r.state_slot)
+            else:
+                need_gather |= st > 0
+                gather += self._slots(r.block_ids, 0, st + n)
             sample_idx.append(cu_q[-1] - 1)
             bt_rows.append(r.block_ids + [0] * (self._bt_width - len(r.block_ids)))
         md = AttnMetadata(
@@ -379,6 +406,8 @@ class ModelRunner:
             cu_q=self._to_dev(cu_q, torch.int32), cu_k=self._to_dev(cu_k, torch.int32), query_lens=qlens,
             context_lens=ctx, max_q=max(qlens), max_k=max(seq_lens),
             kv_gather_slots=self._to_dev(gather, torch.int64) if need_gather else None,
+            q_to_seq=self._to_dev(q_to_seq, torch.int32) if layer_list else None,
+            state_slots=self._to_dev(state_slots, torch.int32) if layer_list else None,
             sample_indices=self._to_dev(sample_idx, torch.int64))
         if self.omni is not None:
             oslots = []
@@ -398,8 +427,9 @@ class ModelRunner:
         B = len(so.scheduled)
         n = padded * tpr
         # int64 section: ids | positions | slots ; int32 section: q_seq_lens | seq_lens | q_to_seq | num_valid | block table
+        # | state slots (models with recurrent state)
         n64 = 3 * n
-        n32 = n + padded + n + 2 + padded * W
+        n32 = n + padded + n + 2 + padded * W + (padded if self.has_state else 0)
         total_bytes = n64 * 8 + n32 * 4
         key = (padded, tpr)
         stage = getattr(self, "_stage", None)
@@ -417,7 +447,10 @@ class ModelRunner:
         seq_lens = a32[o:o + padded]; o += padded
         q_to_seq = a32[o:o + n]; o += n
         num_valid = a32[o:o + 2]; o += 2
-        bt = a32[o:o + padded * W].reshape(padded, W)
+        bt = a32[o:o + padded * W].reshape(padded, W); o += padded * W
+        if self.has_state:
+            a32[o:o + padded] = -1
+            a32[o:o + B] = [s.request.state_slot for s in so.scheduled]
         ids[:] = 0
         bt[:] = 0
         st = np.zeros(padded, dtype=np.int64)
@@ -451,11 +484,11 @@ class ModelRunner:
         d_seq = d32[o:o + padded]; o += padded
         d_q2s = d32[o:o + n]; o += n
         d_nv = d32[o:o + 1]; o += 2
-        d_bt = d32[o:o + padded * W].view(padded, W)
+        d_bt = d32[o:o + padded * W].view(padded, W); o += padded * W
         md = AttnMetadata(
             is_prefill=False, positions=d64[n:2 * n], slot_mapping=d64[2 * n:3 * n], block_table=d_bt, seq_lens=d_seq,
             tokens_per_req=tpr, q_seq_lens=d_q, q_to_seq=d_q2s, max_seq_len=max_seq,
-            num_valid=d_nv if padded != B else None)
+            num_valid=d_nv if padded != B else None, state_slots=d32[o:o + padded] if self.has_state else None)
         if self.omni is not None:
             nb = self.omni.spec.blocks_per_request
             wt = [list(s.request.omni_block_ids) for s in so.scheduled] + [[0] * nb] * (padded - B)
@@ -536,6 +569,13 @@ class ModelRunner:
         ids, md = self._prepare_prefill(so)
         rounds = self._agree_finish(handle, 1)
         hidden = self.model(ids, md, self.kv_caches)
+        if any(s.want_logits is not None for s in so.scheduled):
+            first = [0]
+            for s in so.scheduled:
+                first.append(first[-1] + s.num_scheduled_tokens)
+            rows = [a + k for a, s in zip(first, so.scheduled) for k in s.want_logits or ()]
+            logits = self.model.compute_logits(hidden[self._to_dev(rows, torch.int64)]) if rows else None
+            return ModelRunnerOutput([r.request_id for r in reqs], [[[] for _ in reqs]], None, logits=logits)
         pp = self._pipeline()
         if pp is None or pp.is_last:
             last_h = hidden[md.sample_indices]
@@ -601,6 +641,10 @@ class ModelRunner:
         spec_final = None
         for step in range(so.num_step):
             hidden, logits = self._forward_decode(ids, md, padded)
+            if any(s.want_logits is not None for s in so.scheduled):
+                rows = [i for i, s in enumerate(so.scheduled) if s.want_logits]
+                return ModelRunnerOutput([r.request_id for r in reqs], [[[] for _ in reqs]], None,
+                                         logits=logits[self._to_dev(rows, torch.int64)] if rows else None)
             pp = self._pipeline()
             toks = self._sample(logits, reqs, tpr) if logits is not None else None
             if pp is not None:
@@ -680,6 +724,7 @@ class ModelRunner:
                           self._to_dev([blocks], torch.int32), self._to_dev([n], torch.int32),
                           cu_q=self._to_dev([0, n], torch.int32), cu_k=self._to_dev([0, n], torch.int32),
                           query_lens=[n], context_lens=[0], max_q=n, max_k=n,
+                          q_to_seq=torch.zeros(n, dtype=torch.int32, device=self.device), state_slots=self._to_dev([0], torch.int32),
                           sample_indices=self._to_dev([n - 1], torch.int64))
         h = self.model(ids, md, self.kv_caches)
         self.model.compute_logits(h[md.sample_indices])

@@ -52,12 +52,39 @@ def _run(cmd, log: Path | None = None) -> None:
         raise RuntimeError("build command failed: " + " ".join(str(c) for c in cmd))
 
 
-def build_kernels(verbose: bool = False) -> Path:
-    """Compile every ``csrc/kernels/*.cu`` for sm_100a and link ``libomni_kernels.so``."""
+# Kernel sources (stems) that one architecture needs when it is served alone
+ARCH_KERNELS = {
+    "Forovik": ("attn_any", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "mamba2", "post_norm_ops",
+                "sampler_misc"),
+}
+
+
+def _kernel_inputs(stems=None):
+    headers = sorted((CSRC / "include").glob("*"))
+    return headers, [s for s in sorted((CSRC / "kernels").glob("*.cu")) if stems is None or s.stem in stems]
+
+
+def ensure_kernels(architecture: str) -> Path:
+    """Path of a library that holds the architecture's kernels: the full one if it is up to date, else one with only what
+    the architecture needs, compiled now if it has not been before."""
+    import fcntl
+    headers, every = _kernel_inputs()
+    if not _newer([*every, *headers], KERNEL_LIB):
+        return KERNEL_LIB
+    stems = ARCH_KERNELS.get(architecture)
+    if stems is None:
+        return build_kernels()
+    LIB_DIR.mkdir(exist_ok=True)
+    with open(LIB_DIR / ".build.lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_kernels(stems=stems, lib=LIB_DIR / f"libomni_kernels_{architecture.lower()}.so")
+
+
+def build_kernels(verbose: bool = False, stems=None, lib: Path = KERNEL_LIB) -> Path:
+    """Compile every ``csrc/kernels/*.cu`` (or those named by ``stems``) for sm_100a and link them into ``lib``."""
     LIB_DIR.mkdir(exist_ok=True)
     OBJ_DIR.mkdir(exist_ok=True)
-    headers = sorted((CSRC / "include").glob("*"))
-    sources = sorted((CSRC / "kernels").glob("*.cu"))
+    headers, sources = _kernel_inputs(stems)
     nvcc = _nvcc()
     jobs = []
     objs = []
@@ -70,11 +97,13 @@ def build_kernels(verbose: bool = False) -> Path:
     if jobs:
         with cf.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             list(ex.map(lambda j: _run(*j), jobs))
-    if jobs or _newer(objs, KERNEL_LIB):
-        _run([nvcc, "-shared", "-o", KERNEL_LIB, *objs])
+    if jobs or _newer(objs, lib):
+        part = lib.with_suffix(".part")
+        _run([nvcc, "-shared", "-o", part, *objs])
+        os.replace(part, lib)
     if verbose:
-        print(f"built {KERNEL_LIB} from {len(sources)} sources ({len(jobs)} recompiled)")
-    return KERNEL_LIB
+        print(f"built {lib} from {len(sources)} sources ({len(jobs)} recompiled)")
+    return lib
 
 
 def build_placement(verbose: bool = False) -> Path | None:

@@ -536,6 +536,8 @@ def main(argv=None) -> int:
     ap.add_argument("--model-overrides", default=None, help="JSON of model-config fields to override (e.g. fewer layers)")
     ap.add_argument("--gpu-memory-utilization", type=float, default=0.9)
     ap.add_argument("--enable-chunked-prefill", action="store_true")
+    ap.add_argument("--mixed-batches", action="store_true",
+                    help="with chunked prefill: decoding requests take part in the steps that run portions of prompts")
     ap.add_argument("--scheduling-policy", default="fcfs", choices=["fcfs", "priority"])
     ap.add_argument("--reasoning-parser", default=None, help="split chat answers into reasoning and content (pangu)")
     ap.add_argument("--tool-call-parser", default=None, help="turn tool-call blocks of chat answers into tool_calls (pangu)")
@@ -545,7 +547,8 @@ def main(argv=None) -> int:
                        max_num_batched_tokens=a.max_num_batched_tokens, block_size=a.block_size, num_kv_blocks=a.num_kv_blocks,
                        num_speculative_tokens=a.num_speculative_tokens, tp_size=a.tensor_parallel_size,
                        enforce_eager=a.enforce_eager, gpu_memory_utilization=a.gpu_memory_utilization,
-                       enable_chunked_prefill=a.enable_chunked_prefill, scheduling_policy=a.scheduling_policy,
+                       enable_chunked_prefill=a.enable_chunked_prefill or a.mixed_batches, mixed_batches=a.mixed_batches,
+                       scheduling_policy=a.scheduling_policy,
                        model_overrides=json.loads(a.model_overrides) if a.model_overrides else {},
                        kv_transfer_config=json.loads(a.kv_transfer_config) if a.kv_transfer_config else None)
     if a.additional_config:

@@ -46,6 +46,7 @@ class EngineConfig:
     async_schedule: bool = False
     enable_prefix_caching: bool = False
     enable_chunked_prefill: bool = os.environ.get("FORCE_ENABLE_CHUNK_PREFILL", "0") == "1"
+    mixed_batches: bool = False      # with chunked prefill: running requests decode in the steps that also run prompts
     decode_gear_list: list = field(default_factory=list)
     enforce_eager: bool = False
     ep_backend: str = "fused"
@@ -99,6 +100,9 @@ class EngineCore:
             planner = OmniPlanner.from_config(pc, self.model_cfg)
             self.worker.planner = self.worker.runner.planner = planner
         self.planner = planner
+        if weights is None and os.path.isdir(cfg.model) and any(f.endswith(".safetensors") for f in os.listdir(cfg.model)):
+            from ..quantization.loader import iter_safetensors
+            weights = iter_safetensors(cfg.model)
         self.worker.load_model(weights, seed=cfg.seed)
         if self.state is not None and not rc.num_kv_blocks and self.state.get("num_kv_blocks"):
             rc.num_kv_blocks = int(self.state.get("num_kv_blocks"))      # skips the profile run; ranks still agree on the minimum
@@ -113,14 +117,16 @@ class EngineCore:
             if planner is not None and ema is not None:
                 # handed to the balancer when the dynamic machinery is built
                 planner.pending_ema = (self.state.get_array("placement_positions"), ema)
-        self.kv = KVCacheManager(n_blocks, cfg.block_size, cfg.enable_prefix_caching)
+        self.kv = KVCacheManager(n_blocks, cfg.block_size, cfg.enable_prefix_caching,
+                                 num_state_slots=cfg.max_num_seqs if self.model_cfg.has_recurrent_state else None)
         if cfg.enable_omni_attn:
             from ..accelerators.cache import apply_omni_attn_patch
             apply_omni_attn_patch(self, cfg.omni_attn_config or {})
         sc = SchedulerConfig(max_num_seqs=cfg.max_num_seqs, max_num_batched_tokens=cfg.max_num_batched_tokens,
                              max_model_len=cfg.max_model_len, num_speculative_tokens=cfg.num_speculative_tokens,
                              num_step=cfg.num_step, async_schedule=cfg.async_schedule,
-                             enable_chunked_prefill=cfg.enable_chunked_prefill, policy=cfg.scheduling_policy)
+                             enable_chunked_prefill=cfg.enable_chunked_prefill, policy=cfg.scheduling_policy,
+                             mixed_batches=cfg.mixed_batches)
         self.scheduler = Scheduler(sc, self.kv, connector=sched_conn)
         self._ids = itertools.count()
         from ..parallel import get_parallel_state

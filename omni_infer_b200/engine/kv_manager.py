@@ -1,4 +1,5 @@
-"""Paged KV-cache block manager: free list, reference counts, optional hash-based prefix caching.
+"""Paged KV-cache block manager: free list, reference counts, optional hash-based prefix caching, and one state slot per
+live request for models with recurrent layers.
 
 Block size defaults to 128 tokens as in the reference deployment (omni/adaptors/vllm/platform.py:226).
 Block 0 is reserved as the padding target of CUDA-graph padded rows."""
@@ -13,12 +14,17 @@ from .request import Request
 
 class KVCacheManager:
     def __init__(self, num_blocks: int, block_size: int = 128, enable_prefix_caching: bool = False,
-                 reserve_null_block: bool = True):
+                 reserve_null_block: bool = True, num_state_slots: Optional[int] = None):
         self.num_blocks, self.block_size = num_blocks, block_size
         self.enable_prefix_caching = enable_prefix_caching
         first = 1 if reserve_null_block else 0
         self.free_blocks: deque = deque(range(first, num_blocks))
         self.ref: list = [0] * num_blocks
+        # None: the model keeps no state beside its cache.  A slot is taken with a request's first blocks and given back
+        # with them; it is not cleared, a request that starts at position 0 reads nothing of it.
+        self.free_state_slots: Optional[deque] = deque(range(num_state_slots)) if num_state_slots is not None else None
+        if enable_prefix_caching and num_state_slots is not None:
+            raise ValueError("cached prefixes carry no recurrent state: prefix caching is not combined with such models")
         self.hash_to_block: dict = {}
         self.block_hash: dict = {}
         self.evictable: OrderedDict = OrderedDict()    # cached, unreferenced blocks in LRU order
@@ -83,6 +89,8 @@ class KVCacheManager:
                        lookahead: int = 0) -> Optional[list]:
         """Make sure ``req`` owns blocks for ``num_computed_tokens + num_new_tokens + lookahead`` tokens.
         Returns the newly added block ids, or None when memory is short (nothing is changed then)."""
+        if self.free_state_slots is not None and req.state_slot < 0 and not self.free_state_slots:
+            return None
         took_prefix = bool(computed_blocks) and not req.block_ids
         if took_prefix:
             for b in computed_blocks:
@@ -91,6 +99,7 @@ class KVCacheManager:
             req.block_ids = list(computed_blocks)
         need = self.blocks_needed(req.num_computed_tokens + num_new_tokens + lookahead) - len(req.block_ids)
         if need <= 0:
+            self._take_state_slot(req)
             return []
         if need > self.num_free_blocks:
             if took_prefix:
@@ -102,7 +111,12 @@ class KVCacheManager:
             self.ref[b] = 1
             new.append(b)
         req.block_ids.extend(new)
+        self._take_state_slot(req)
         return new
+
+    def _take_state_slot(self, req: Request) -> None:
+        if self.free_state_slots is not None and req.state_slot < 0:
+            req.state_slot = self.free_state_slots.popleft()
 
     def free(self, req: Request) -> None:
         for b in reversed(req.block_ids):
@@ -115,6 +129,9 @@ class KVCacheManager:
                 else:
                     self.free_blocks.append(b)
         req.block_ids = []
+        if req.state_slot >= 0:
+            self.free_state_slots.append(req.state_slot)
+            req.state_slot = -1
 
     def get_block_ids(self, req: Optional[Request]) -> list:
         """Unknown requests answer with an empty group instead of raising (the KV connector may ask about a

@@ -65,6 +65,7 @@ class Request:
     num_computed_tokens: int = 0
     num_cached_tokens: int = 0                           # prefix-cache hits at admission
     block_ids: list = field(default_factory=list)
+    state_slot: int = -1                                 # slot of the recurrent state (models that have one)
     first_token_time: Optional[float] = None
     finish_time: Optional[float] = None
     num_preemptions: int = 0
@@ -105,6 +106,8 @@ class ScheduledRequest:
     num_scheduled_tokens: int      # tokens run through the model this step (prompt chunk, or 1 + drafts)
     is_prefill: bool
     spec_token_ids: list = field(default_factory=list)
+    # rows (offsets into the scheduled tokens) whose logits are returned; None = sample from the last row
+    want_logits: Optional[list] = None
 
 
 @dataclass
@@ -131,6 +134,7 @@ class ModelRunnerOutput:
     finished_sending: set = field(default_factory=set)
     finished_recving: set = field(default_factory=set)
     failed_recving: set = field(default_factory=set)     # remote KV never arrived: prefill locally instead
+    logits: Any = None                                   # [rows, vocab] of the rows asked for, in the order of the batch
     step_time_s: float = 0.0
 
 

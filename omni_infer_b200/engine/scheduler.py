@@ -40,6 +40,13 @@ class SchedulerConfig:
     async_schedule: bool = False
     enable_chunked_prefill: bool = os.environ.get("FORCE_ENABLE_CHUNK_PREFILL", "0") == "1"
     policy: str = "fcfs"                    # fcfs | priority
+    # With chunked prefill: a step that runs portions of prompts also carries one token of every decoding request, as a
+    # portion of one (no drafts, one model step).  Off: a step is all prompts or all decode.
+    mixed_batches: bool = False
+
+    def __post_init__(self):
+        if self.mixed_batches and (not self.enable_chunked_prefill or self.num_speculative_tokens):
+            raise ValueError("mixed batches need chunked prefill and run without speculative tokens")
 
 
 class Scheduler:
@@ -158,6 +165,16 @@ class Scheduler:
                     self.waiting.remove(req)
                     self.running.append(req)
 
+        # -- mixed batches: decoding requests ride along with the portions of prompts that follow
+        if cfg.mixed_batches and (self.waiting or any(r.num_tokens - r.num_computed_tokens > 1 for r in self.running)):
+            for req in self.running:
+                if budget <= 0:
+                    break
+                if req.num_tokens - req.num_computed_tokens == 1 and self.kv.allocate_slots(req, 1) is not None:
+                    scheduled.append(ScheduledRequest(req, 1, True))
+                    budget -= 1
+        riders = {id(s) for s in scheduled}
+
         # -- 0. partially prefilled running requests (chunked prefill) go on first: they are older than anything
         # waiting, and admitting newcomers ahead of them can take the blocks they need to ever finish.  When the
         # pool is exhausted the last running request is preempted, as in the decode phase.
@@ -249,6 +266,9 @@ class Scheduler:
         for r in reversed(skipped):
             self.waiting.appendleft(r)
 
+        # nothing but riders: a plain decode step (which may also preempt, where riding along may not)
+        if all(id(s) in riders for s in scheduled):
+            scheduled = []
         if scheduled:
             for s in scheduled:
                 if s.request not in self.running:

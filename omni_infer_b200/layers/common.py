@@ -35,10 +35,11 @@ class AttnMetadata:
     # decode
     tokens_per_req: int = 1                 # 1 + speculative tokens
     q_seq_lens: Optional[torch.Tensor] = None   # [B * tokens_per_req] int32 visible kv tokens per q row
-    q_to_seq: Optional[torch.Tensor] = None     # [B * tokens_per_req] int32
+    q_to_seq: Optional[torch.Tensor] = None     # [B * tokens_per_req] int32 (prefill: [T], the request of every row)
     max_seq_len: int = 0
     num_valid: Optional[torch.Tensor] = None    # device int32 scalar: rows beyond are padding
     sample_indices: Optional[torch.Tensor] = None  # rows of hidden states that produce logits
+    state_slots: Optional[torch.Tensor] = None     # [B] int32 recurrent-state slot per request, -1 = padding row
     # Omni-Attention (compressed layers): per-layer-group overrides
     omni: Optional[dict] = None
 
@@ -88,6 +89,52 @@ class RMSNorm(nn.Module):
     def forward(self, x, residual=None, quant=False):
         """Returns y, or (y, y_q, scale) with ``quant``; ``residual`` is updated in place to x + residual."""
         return ops.rmsnorm(x, self.weight, self.eps, residual=residual, quant=quant)
+
+
+class PaddedLinear(Linear):
+    """Linear whose stored weight has both sizes rounded up to a multiple of 8 (TMA row pitch, 16-byte output vectors).  The
+    padding is zero and activations carry zeros in their padding columns, so the product is that of the real sizes."""
+
+    def __init__(self, in_features: int, out_features: int, *, dtype=torch.bfloat16, device=None):
+        super().__init__((in_features + 7) // 8 * 8, (out_features + 7) // 8 * 8, dtype=dtype, device=device)
+        self.real_in, self.real_out = in_features, out_features
+        self.zero_padding()
+
+    def zero_padding(self):
+        self.weight.data[self.real_out:] = 0
+        self.weight.data[:, self.real_in:] = 0
+
+
+class GeGLUMLP(nn.Module):
+    """gate_up (merged, gate rows first, each block padded to a multiple of 8) -> gelu (tanh form) of the gate times up,
+    in the GEMM epilogue where the width allows -> down."""
+
+    def __init__(self, hidden: int, inter: int, *, dtype=torch.bfloat16, device=None):
+        super().__init__()
+        self.inter, self.block = inter, (inter + 7) // 8 * 8
+        self.gate_up_proj = PaddedLinear(hidden, 2 * self.block, dtype=dtype, device=device)
+        self.down_proj = PaddedLinear(inter, hidden, dtype=dtype, device=device)
+
+    def zero_padding(self):
+        w = self.gate_up_proj.weight.data
+        w[self.inter:self.block] = 0
+        w[self.block + self.inter:] = 0
+
+    def forward(self, x):
+        return ops.gemm(ops.gemm(x, self.gate_up_proj.weight, epi="geglu"), self.down_proj.weight)
+
+
+class PostNorm(nn.Module):
+    """Norm on a sublayer's output: residual (fp32, in place) += rmsnorm(y) * weight, in one kernel with the activation copy
+    that the next sublayer reads.  The weight is kept in fp32."""
+
+    def __init__(self, hidden: int, eps: float, device=None):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(hidden, dtype=torch.float32, device=device), requires_grad=False)
+        self.eps = eps
+
+    def forward(self, y, residual):
+        return ops.layer_list.post_norm_add(y, self.weight, residual, self.eps)
 
 
 class SwiGLUMLP(nn.Module):

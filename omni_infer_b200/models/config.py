@@ -1,16 +1,98 @@
 """Architecture description shared by all model families (DeepSeek-V2/V3 MLA+MoE, MTP drafters,
-Qwen2 dense GQA, Qwen3-MoE GQA) plus the named configurations used by the benchmarks."""
+Qwen2 dense GQA, Qwen3-MoE GQA, layer-list models) plus the named configurations used by the benchmarks."""
 from __future__ import annotations
 
 import json
+import re
 from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any, Optional
 
 
 @dataclass
+class AttentionSpec:
+    """Softmax attention of one layer of a layer-list model."""
+    heads: int
+    kv_heads: int
+    dim: int                                 # query / key size per head
+    vdim: int                                # value size per head
+    scale: float
+    window: int = 0                          # a query sees itself and the window - 1 tokens before it; 0 = all
+    rot_dims: int = 0                        # leading dimensions of each head that are rotated; 0 = none
+    rot_base: float = 10000.0
+    rot_factor: float = 1.0                  # linear scaling: every frequency is divided by it
+    kv_from: Optional[int] = None            # attends to the cached keys and values of this earlier layer
+
+    @property
+    def owns_kv(self) -> bool:
+        return self.kv_from is None
+
+    def cache_elems_per_token(self) -> int:
+        return self.kv_heads * (self.dim + self.vdim) if self.owns_kv else 0
+
+
+@dataclass
+class Mamba2Spec:
+    """Mamba-2 recurrence of one layer of a layer-list model."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int = 1
+    conv: int = 4                            # taps of the short convolution
+    norm_groups: int = 1
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass
+class LayerSpec:
+    """One entry of a layer-list model: a mixer and an optional gated dense feed-forward."""
+    attention: Optional[AttentionSpec] = None
+    mamba2: Optional[Mamba2Spec] = None
+    ff: int = 0                              # width of the feed-forward, 0 = the layer has none
+
+    @classmethod
+    def from_dict(cls, i: int, d: dict) -> "LayerSpec":
+        """Entry ``i`` of the ``layers`` list of a config.json.  The type may carry a running number (several mixers of
+        one kind with sizes of their own)."""
+        kind, m = re.sub(r"_\d+$", "", d["type"]), d["mixer"]
+        s = cls()
+        if kind == "attention":
+            rot = m.get("rot") or {}
+            s.attention = AttentionSpec(
+                heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]),
+                window=int((m.get("mask") or {}).get("size") or 0), rot_dims=int(rot.get("dims", 0)),
+                rot_base=float(rot.get("base", 10000.0)),
+                rot_factor=float((rot.get("scaling") or {}).get("factor", 1.0)), kv_from=m.get("kv_from"))
+            if s.attention.heads % s.attention.kv_heads or s.attention.rot_dims % 2 or s.attention.rot_dims > s.attention.dim:
+                raise ValueError(f"layer {i}: heads must divide over the key/value heads, rotated dimensions be even and "
+                                 "fit the head")
+        elif kind == "mamba2":
+            s.mamba2 = Mamba2Spec(heads=m["heads"], vdim=m["vdim"], state=m["state"], groups=m["groups"], conv=m["conv"],
+                                  norm_groups=m["norm_groups"])
+            if s.mamba2.heads % s.mamba2.groups or s.mamba2.inner % s.mamba2.norm_groups:
+                raise ValueError(f"layer {i}: heads must divide over the groups, the inner width over the norm groups")
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {d['type']!r}")
+        mlp = d.get("mlp")
+        if mlp:
+            if mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            s.ff = int(mlp["ff"])
+        return s
+
+
+@dataclass
 class ModelConfig:
     architecture: str = "DeepseekV3ForCausalLM"
+    # layer-list models: one LayerSpec per layer; None = the uniform stacks described by the fields below
+    layers: Optional[list] = None
     # tensor-parallel attention: heads sharded over attn_tp_size ranks, hidden states sharded by token rows between
     # layers (set by the model runner; 1 = every rank runs whole attention layers on its own requests)
     attn_tp_size: int = 1
@@ -95,7 +177,15 @@ class ModelConfig:
             scale = scale * m * m
         return scale
 
+    @property
+    def has_recurrent_state(self) -> bool:
+        """Does a request hold state besides its cached tokens (one slot per live request)?"""
+        return any(s.mamba2 is not None for s in self.layers or ())
+
     def kv_bytes_per_token(self, elem_bytes: int = 2) -> int:
+        if self.layers is not None:     # mean over the layers that hold a cache
+            per = [s.attention.cache_elems_per_token() for s in self.layers if s.attention is not None and s.attention.owns_kv]
+            return sum(per) * elem_bytes // max(1, len(per))
         if self.use_mla:
             return (self.kv_lora_rank + self.qk_rope_head_dim) * elem_bytes
         return 2 * self.local_kv_heads * self.head_dim * elem_bytes
@@ -111,6 +201,8 @@ class ModelConfig:
     @classmethod
     def from_hf_dict(cls, d: dict[str, Any]) -> "ModelConfig":
         arch = (d.get("architectures") or [d.get("architecture", "DeepseekV3ForCausalLM")])[0]
+        if isinstance(d.get("layers"), list):
+            return cls.from_layer_list(arch, d)
         c = cls(architecture=arch)
         for k in ("vocab_size", "hidden_size", "num_hidden_layers", "num_attention_heads", "intermediate_size",
                   "moe_intermediate_size", "n_routed_experts", "n_shared_experts", "num_experts_per_tok",
@@ -138,6 +230,23 @@ class ModelConfig:
         elif qc.get("quant_method") in ("ascend_compressed_tensors", "compressed-tensors", "compressed_tensors"):
             c.quantization = "w8a8_int8"
         return c
+
+    @classmethod
+    def from_layer_list(cls, arch: str, d: dict[str, Any]) -> "ModelConfig":
+        """config.json whose ``layers`` list describes every layer (mixer and feed-forward sizes of its own)."""
+        layers = [LayerSpec.from_dict(i, e) for i, e in enumerate(d["layers"])]
+        for i, s in enumerate(layers):
+            a = s.attention
+            if a is None or a.owns_kv:
+                continue
+            src = layers[a.kv_from].attention if 0 <= a.kv_from < i else None
+            if src is None or not src.owns_kv:
+                raise ValueError(f"layer {i} takes its keys from layer {a.kv_from}, which holds none")
+            if (src.kv_heads, src.dim, src.vdim) != (a.kv_heads, a.dim, a.vdim):
+                raise ValueError(f"layers {i} and {a.kv_from} share keys but differ in their head sizes")
+        return cls(architecture=arch, layers=layers, vocab_size=d["vocab"], hidden_size=d["width"],
+                   num_hidden_layers=len(layers), rms_norm_eps=float(d["norm"]["eps"]), use_mla=False,
+                   tie_word_embeddings=True, n_routed_experts=0, name=arch)
 
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
@@ -239,7 +348,37 @@ def tiny_qwen3_moe(**kw) -> ModelConfig:
     return c
 
 
+def forovik(width=2048, layers=12, vocab=32768, heads=16, kv_heads=4, dim=128, window=1024, ff=5632, m_heads=64, m_vdim=64,
+            state=128, groups=1, conv=4, norm_groups=1, **kw) -> ModelConfig:
+    """Layer-list model in the shape of a small hybrid: groups of one windowed-attention layer (with feed-forward) and two
+    Mamba-2 layers; every second attention layer reads the keys and values of the one before it."""
+    specs, last_kv = [], None
+    for i in range(layers):
+        if i % 3 == 0:
+            share = last_kv if (i // 3) % 2 == 1 else None
+            specs.append(LayerSpec(AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window, dim // 2, 1e6, 4.0, share),
+                                   None, ff))
+            last_kv = i if share is None else last_kv
+        else:
+            specs.append(LayerSpec(None, Mamba2Spec(m_heads, m_vdim, state, groups, conv, norm_groups)))
+    c = ModelConfig(architecture="Forovik", name="forovik", layers=specs, vocab_size=vocab, hidden_size=width,
+                    num_hidden_layers=layers, use_mla=False, tie_word_embeddings=True, rms_norm_eps=1e-5)
+    for k, v in kw.items():
+        setattr(c, k, v)
+    return c
+
+
+def tiny_forovik(**kw) -> ModelConfig:
+    """CPU-sized layer-list model."""
+    kw.setdefault("dtype", "float32")
+    kw.setdefault("name", "tiny-forovik")
+    return forovik(width=64, layers=6, vocab=512, heads=4, kv_heads=2, dim=16, window=40, ff=96, m_heads=4, m_vdim=16,
+                   state=32, groups=2, conv=4, norm_groups=2, **kw)
+
+
 PRESETS = {
+    "forovik": forovik,
+    "tiny-forovik": tiny_forovik,
     "tiny-deepseek-v3": tiny_deepseek_v3,
     "tiny-qwen3-moe": tiny_qwen3_moe,
     "small-deepseek": small_deepseek_gpu,

@@ -16,6 +16,7 @@ def _lazy():
         return
     from .deepseek import DeepseekV2ForCausalLM, DeepseekV3ForCausalLM
     from .deepseek_mtp import DeepSeekMTPModel, DeepSeekMTPModelDuo, DeepSeekMTPModelTres
+    from .layer_list import LayerListForCausalLM
     from .qwen import Qwen2ForCausalLM, Qwen3MoeForCausalLM
 
     table = {
@@ -26,6 +27,7 @@ def _lazy():
         "DeepSeekMTPModelTres": DeepSeekMTPModelTres,
         "Qwen2ForCausalLM": Qwen2ForCausalLM,
         "Qwen3MoeForCausalLM": Qwen3MoeForCausalLM,
+        "Forovik": LayerListForCausalLM,
     }
     if any(os.environ.get(k) == "1" for k in ("RANDOM_MODE", "CAPTURE_MODE", "REPLAY_MODE")):
         from .mock import mock_model_class_factory

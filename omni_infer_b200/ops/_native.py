@@ -31,6 +31,15 @@ def available() -> bool:
     return _LIB_PATH.exists()
 
 
+def use_library(path) -> None:
+    """Load the kernels from ``path`` instead of the full library (a library with one architecture's kernels only, see
+    ``omni_infer_b200.build.ensure_kernels``).  Before the first kernel call."""
+    global _LIB_PATH
+    if _lib is not None and Path(path) != _LIB_PATH:
+        raise RuntimeError("the kernel library has been loaded already")
+    _LIB_PATH = Path(path)
+
+
 # kernels launched by one call of each entry point (entry points not listed launch one)
 _KERNELS_PER_CALL = {"omni_moe_align": 2}
 

@@ -13,7 +13,7 @@ from . import _native as nat
 
 FP8 = torch.float8_e4m3fn
 FP8_MAX = 448.0
-_EPI = {"store": 0, "swiglu": 1, "swiglu_quant": 2}
+_EPI = {"store": 0, "swiglu": 1, "swiglu_quant": 2, "geglu": 3}
 
 
 def quant_fp8_block_ref(x: torch.Tensor, block: int = 128, ld: int | None = None):
@@ -83,7 +83,9 @@ def gemm_ref(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, 
             continue
         acc = xf[s:s + l] @ wf[g].t()
         if epi != "store":
-            acc = torch.nn.functional.silu(acc[:, :n_out]) * acc[:, n_out:]
+            gate = acc[:, :n_out]
+            act = torch.nn.functional.gelu(gate, approximate="tanh") if epi == "geglu" else torch.nn.functional.silu(gate)
+            acc = act * acc[:, n_out:]
         y[s:s + l] = acc
     if row_scale is not None:
         y = y * row_scale.float().unsqueeze(-1)
@@ -123,7 +125,9 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
     x: [T, K] bf16 or e4m3 (then ``x_scale`` is [K/128, ld] fp32, K-block major).
     w: [N, K] or [G, N, K]; e4m3 weights carry ``w_scale`` [G, N/128, K/128].
     seg_start/seg_len: int32 [G] row segments per group (grouped GEMM).
-    epi: "store" | "swiglu" (w holds gate rows then up rows) | "swiglu_quant" (returns (q, scale_t)).
+    epi: "store" | "swiglu" (w holds gate rows then up rows) | "geglu" (the same with the tanh form of gelu) |
+    "swiglu_quant" (returns (q, scale_t)).
+    fp32 operands run a plain fp32 kernel (dense, "store" and "geglu" only).
     """
     if out_dtype is None:
         out_dtype = torch.bfloat16 if (x.dtype == FP8 or x.is_cuda) else x.dtype
@@ -131,6 +135,8 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
         return gemm_ref(x, w, w_scale=w_scale, x_scale=x_scale, seg_start=seg_start, seg_len=seg_len,
                         epi=epi, row_scale=row_scale, out_dtype=out_dtype)
     L = nat.lib()
+    if x.dtype == torch.float32:
+        return _gemm_f32(x, w, epi, seg_len, row_scale, out)
     if w.dim() == 2:
         w = w.unsqueeze(0)
     G, n_w, K = w.shape
@@ -142,6 +148,9 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
         assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     e = _EPI[epi]
     n_out = n_w if e == 0 else n_w // 2
+    if e == 3 and n_out % 128 != 0:
+        from .layer_list import gelu_mul
+        return gelu_mul(gemm(x, w, seg_start=seg_start, seg_len=seg_len, row_scale=row_scale, bn=bn, t_hint=t_hint), n_out, n_out)
     if e == 1 and n_out % 128 != 0:
         # the fused SwiGLU epilogue pairs 128-row gate and up blocks; odd widths (e.g. 10944) take the plain GEMM
         # and a separate activation kernel
@@ -182,6 +191,20 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
     if e == 2:
         return out, out_scale
     return out
+
+
+def _gemm_f32(x, w, epi, seg_len, row_scale, out):
+    assert w.dtype == torch.float32 and w.dim() == 2 and seg_len is None and row_scale is None and epi in ("store", "geglu")
+    assert x.shape[1] == w.shape[1] and x.stride(1) == 1 and w.stride(1) == 1
+    T, n = x.shape[0], w.shape[0]
+    y = out if out is not None and epi == "store" else torch.empty(T, n, dtype=torch.float32, device=x.device)
+    rc = nat.lib().omni_gemm_f32(nat.ptr(x), nat.ptr(w), nat.ptr(y), nat.c_int(T), nat.c_int(n), nat.c_int(x.shape[1]),
+                                 nat.c_int(x.stride(0)), nat.c_int(w.stride(0)), nat.c_int(y.stride(0)), nat.stream())
+    nat.check_rc(rc, "omni_gemm_f32")
+    if epi == "geglu":
+        from .layer_list import gelu_mul
+        return gelu_mul(y, n // 2, n // 2)
+    return y
 
 
 def bmm_heads_ref(x, w):

@@ -1,0 +1,298 @@
+"""Ops of the layer-list models: the fp32 residual stream with norms on the sublayers' outputs, windowed attention over the
+paged cache with a q/k norm over the whole projection, and the Mamba-2 layer between its projections.
+
+CUDA tensors run ``csrc/kernels/post_norm_ops.cu``, ``attn_any.cu``, ``fmha_sm100.cu``, ``gqa_decode.cu`` and
+``mamba2.cu``; CPU tensors run the fp32 references here.  Activations are bf16 or fp32.  Rows may be wider than their
+content (a multiple of 8 columns, so that they can be TMA operands); the columns past it are zero.
+
+Ragged batches: the rows of request r are ``cu_q[r]:cu_q[r + 1]``, its rows' positions ascend by one, ``q_to_seq[row] = r``.
+``cu_q=None``: one row per request (decode)."""
+from __future__ import annotations
+
+import torch
+import torch.nn.functional as F
+
+from . import _native as nat
+
+
+def pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def _f32(t) -> int:
+    assert t.dtype in (torch.float32, torch.bfloat16)
+    return int(t.dtype == torch.float32)
+
+
+def _segments(cu_q, rows: int):
+    """(request, first row, end row) of every request with rows."""
+    if cu_q is None:
+        return [(i, i, i + 1) for i in range(rows)]
+    c = cu_q.tolist()
+    return [(i, c[i], c[i + 1]) for i in range(len(c) - 1) if c[i + 1] > c[i]]
+
+
+# ----------------------------------------------------------------------------- residual stream
+def embed_residual(ids, table):
+    """Embedding rows -> (fp32 residual, activations).  fp32 activations are the residual itself."""
+    if not table.is_cuda:
+        x = table[ids].float()
+        return x, (x if table.dtype == torch.float32 else x.to(table.dtype))
+    T, ld = ids.shape[0], table.shape[1]
+    x = torch.empty(T, ld, dtype=torch.float32, device=table.device)
+    xa = None if table.dtype == torch.float32 else torch.empty(T, ld, dtype=table.dtype, device=table.device)
+    rc = nat.lib().omni_embed_residual(nat.ptr(ids), nat.ptr(table), nat.c_int(table.shape[0]), nat.c_int(T), nat.c_int(ld),
+                                       nat.ptr(x), nat.ptr(xa), nat.c_int(_f32(table)), nat.stream())
+    nat.check_rc(rc, "omni_embed_residual")
+    return x, (x if xa is None else xa)
+
+
+def rms_ref(x, w, eps):
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w
+
+
+def post_norm_add(y, w, x, eps):
+    """x (fp32, in place) += rmsnorm(y) * w; returns the activations for the next sublayer (x itself in fp32 runs)."""
+    H = w.shape[0]
+    f32 = y.dtype == torch.float32
+    if not y.is_cuda:
+        x[:, :H] += rms_ref(y[:, :H].float(), w, eps)
+        return x if f32 else x.to(y.dtype)
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and y.stride(1) == 1 and x.is_contiguous()
+    xa = None if f32 else torch.empty(x.shape, dtype=y.dtype, device=y.device)
+    rc = nat.lib().omni_post_norm_add(nat.ptr(y), nat.c_int(y.stride(0)), nat.ptr(w), nat.ptr(x), nat.ptr(xa),
+                                      nat.c_int(y.shape[0]), nat.c_int(H), nat.c_int(x.shape[1]), nat.c_float(eps),
+                                      nat.c_int(_f32(y)), nat.stream())
+    nat.check_rc(rc, "omni_post_norm_add")
+    return x if f32 else xa
+
+
+def rmsnorm_residual(x, w, eps, dtype):
+    """Norm of the fp32 residual, as activations of ``dtype``."""
+    H = w.shape[0]
+    if not x.is_cuda:
+        out = torch.zeros(x.shape, dtype=dtype)
+        out[:, :H] = rms_ref(x[:, :H], w, eps).to(dtype)
+        return out
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+    rc = nat.lib().omni_rmsnorm_residual(nat.ptr(x), nat.ptr(w), nat.ptr(out), nat.c_int(x.shape[0]), nat.c_int(H),
+                                         nat.c_int(x.shape[1]), nat.c_float(eps), nat.c_int(_f32(out)), nat.stream())
+    nat.check_rc(rc, "omni_rmsnorm_residual")
+    return out
+
+
+# ----------------------------------------------------------------------------- q/k norm, rotation, cache write
+def _rotate_half_ref(x, cos_sin, positions, rot):
+    """x [T, heads, D] fp32; rotates the first ``rot`` entries of every head."""
+    if rot == 0:
+        return x
+    cs = cos_sin[positions]
+    c, s = cs[:, None, : rot // 2], cs[:, None, rot // 2:]
+    u, v = x[..., : rot // 2], x[..., rot // 2: rot]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., rot:]], -1)
+
+
+def qk_norm_rope_cache(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, positions, slots, k_cache, v_cache):
+    """``qkv`` rows are q heads | k heads | v heads (``hkv=0``: q only).  RMSNorm over the whole q and the whole k
+    projection, rotate-half RoPE on the first ``rot`` dimensions of every head; q in place, k and v into the caches
+    [blocks, block, hkv, d] at ``slots`` (-1: not stored)."""
+    T, nq, nk = qkv.shape[0], hq * dk, hkv * dk
+    if not qkv.is_cuda:
+        q = rms_ref(qkv[:, :nq].float(), q_w, eps).view(T, hq, dk)
+        qkv[:, :nq] = _rotate_half_ref(q, cos_sin, positions, rot).reshape(T, nq).to(qkv.dtype)
+        if hkv:
+            k = rms_ref(qkv[:, nq:nq + nk].float(), k_w, eps).view(T, hkv, dk)
+            k = _rotate_half_ref(k, cos_sin, positions, rot)
+            ok = slots >= 0
+            k_cache.view(-1, hkv, dk)[slots[ok]] = k[ok].to(k_cache.dtype)
+            v_cache.view(-1, hkv, dv)[slots[ok]] = qkv[:, nq + nk:nq + nk + hkv * dv].view(T, hkv, dv)[ok]
+        return
+    assert qkv.stride(1) == 1 and (not hkv or k_cache.dtype == qkv.dtype)
+    rc = nat.lib().omni_qk_norm_rope_cache(
+        nat.ptr(qkv), nat.c_int(qkv.stride(0)), nat.c_int(hq), nat.c_int(hkv), nat.c_int(dk), nat.c_int(dv), nat.ptr(q_w),
+        nat.ptr(k_w), nat.c_float(eps), nat.ptr(cos_sin), nat.c_int(rot), nat.ptr(positions), nat.ptr(slots),
+        nat.ptr(k_cache if hkv else None), nat.ptr(v_cache if hkv else None), nat.c_int(T), nat.c_int(_f32(qkv)), nat.stream())
+    nat.check_rc(rc, "omni_qk_norm_rope_cache")
+
+
+# ----------------------------------------------------------------------------- windowed attention over the paged cache
+def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, out):
+    hq, dk = q.shape[1], q.shape[2]
+    bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    kf, vf = k_cache.view(-1, hkv, dk), v_cache.view(-1, hkv, dv)
+    rep = hq // hkv
+    out.zero_()
+    for t in range(q.shape[0]):
+        if int(slots[t]) < 0:
+            continue
+        p = int(positions[t])
+        pos = torch.arange(max(0, p - window + 1) if window else 0, p + 1)
+        rows = block_table[int(q_to_seq[t]), pos // bs].long() * bs + pos % bs
+        k = kf[rows].float().repeat_interleave(rep, 1)
+        v = vf[rows].float().repeat_interleave(rep, 1)
+        s = torch.einsum("hd,lhd->hl", q[t].float(), k) * scale
+        o = torch.einsum("hl,lhd->hd", torch.softmax(s, -1), v)
+        out[t, :hq * dv] = o.reshape(-1).to(out.dtype)
+    return out
+
+
+def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_table, seq_lens, scale, window=0, cu_q=None,
+                    max_q=1, max_seq_len=0, any_shape=False):
+    """q [T, hq, dk] (rows of any pitch) against the cached keys of the rows' requests, each row seeing the ``window``
+    positions up to its own (0: all of them).  Returns [T, pad8(hq * dv)].
+
+    bf16 portions of prompts run on tcgen05 (``omni_fmha_paged``), bf16 single tokens on the split-KV decode kernel; fp32
+    and head shapes those two do not take - or ``any_shape`` - go to ``omni_attn_any``."""
+    T, hq, dk = q.shape
+    bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    ld = pad8(hq * dv)
+    alloc = torch.empty if ld == hq * dv else torch.zeros
+    out = alloc(T, ld, dtype=q.dtype, device=q.device)
+    if not q.is_cuda:
+        return paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, out)
+    assert q.stride(2) == 1 and q.stride(1) == dk and k_cache.dtype == q.dtype and block_table.stride(1) == 1
+    f32 = _f32(q)
+    lib = nat.lib()
+    tc = not any_shape and not f32 and dk % 8 == 0 and dv % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+    if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0:
+        rc = lib.omni_fmha_paged(
+            nat.ptr(q), nat.c_int64(T), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache),
+            nat.c_int64(k_cache.shape[0] * bs), nat.ptr(cu_q), nat.ptr(seq_lens), nat.ptr(block_table),
+            nat.c_int(block_table.stride(0)), nat.c_int(cu_q.shape[0] - 1), nat.c_int(max_q), nat.c_int(hq), nat.c_int(hkv),
+            nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(out), nat.c_int(ld),
+            nat.ptr(nat.status_buffer(q.device)), nat.stream())
+        nat.check_rc(rc, "omni_fmha_paged")
+        return out
+    if tc and cu_q is None and dk <= 256 and dv <= 256:
+        ctas = T * hkv * ((hq // hkv + 15) // 16)
+        span = min(max_seq_len, window) if window else max_seq_len
+        tiles = (span + 31) // 32 + 1
+        splits = max(1, min((444 + ctas - 1) // ctas, tiles // 8, 32)) if ctas < 444 else 1
+        o_part = lse = None
+        if splits > 1:
+            o_part = torch.empty(T * splits * hq * dv, dtype=torch.float32, device=q.device)
+            lse = torch.empty(T * splits * hq, dtype=torch.float32, device=q.device)
+        rc = lib.omni_gqa_paged_decode_window(
+            nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.ptr(block_table),
+            nat.c_int(block_table.stride(0)), nat.ptr(seq_lens), nat.c_int(T), nat.c_int(hq), nat.c_int(hkv), nat.c_int(dk),
+            nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.c_int(splits), nat.ptr(o_part),
+            nat.ptr(lse), nat.ptr(out), nat.c_int(ld), nat.stream())
+        nat.check_rc(rc, "omni_gqa_paged_decode_window")
+        return out
+    rc = lib.omni_attn_any(
+        nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.ptr(positions), nat.ptr(q_to_seq),
+        nat.ptr(slots), nat.ptr(block_table), nat.c_int(block_table.stride(0)), nat.c_int(T), nat.c_int(hq), nat.c_int(hkv),
+        nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(out), nat.c_int(ld),
+        nat.c_int(f32), nat.stream())
+    nat.check_rc(rc, "omni_attn_any")
+    return out
+
+
+# ----------------------------------------------------------------------------- gated feed-forward
+def gelu_mul(x, inter, up_off):
+    """gelu(x[:, :inter]) * x[:, up_off:up_off + inter] -> [T, pad8(inter)]."""
+    T, ld = x.shape[0], pad8(inter)
+    if not x.is_cuda:
+        g, u = x[:, :inter].float(), x[:, up_off:up_off + inter].float()
+        return F.pad(F.gelu(g, approximate="tanh") * u, (0, ld - inter)).to(x.dtype)
+    out = torch.empty(T, ld, dtype=x.dtype, device=x.device)
+    rc = nat.lib().omni_gelu_mul(nat.ptr(x), nat.c_int(x.stride(0)), nat.c_int(up_off), nat.ptr(out), nat.c_int(ld),
+                                 nat.c_int(T), nat.c_int(inter), nat.c_int(_f32(x)), nat.stream())
+    nat.check_rc(rc, "omni_gelu_mul")
+    return out
+
+
+# ----------------------------------------------------------------------------- Mamba-2
+def conv_silu_ref(u, w, bias, state, positions, state_slots, cu_q, out):
+    taps, C = w.shape
+    for r, a, b in _segments(cu_q, u.shape[0]):
+        slot = int(state_slots[r])
+        if slot < 0:
+            out[a:b, :C] = 0
+            continue
+        old = state[slot].float() if taps > 1 else u.new_zeros(0, C).float()
+        pos0 = int(positions[a])
+        if pos0 < taps - 1:                       # entries before the start of the sequence
+            old = old.clone()
+            old[: taps - 1 - pos0] = 0
+        full = torch.cat([old, u[a:b, :C].float()])
+        y = sum(full[k:k + b - a] * w[k] for k in range(taps)) + bias
+        out[a:b, :C] = F.silu(y).to(out.dtype)
+        if taps > 1:
+            state[slot] = full[b - a:].to(state.dtype)
+    return out
+
+
+def conv_silu(u, w, bias, state, *, positions, state_slots, q_to_seq=None, cu_q=None):
+    """Causal convolution per channel (``w`` [taps, C], last tap = current token), bias, silu.  u [T, C] (rows of any
+    pitch); ``state`` [slots, taps - 1, C] holds the last inputs of every request and is moved on.  -> [T, pad8(C)]."""
+    T, (taps, C) = u.shape[0], w.shape
+    out = torch.empty(T, pad8(C), dtype=u.dtype, device=u.device)
+    if not u.is_cuda:
+        return conv_silu_ref(u, w, bias, state, positions, state_slots, cu_q, out)
+    assert u.stride(1) == 1 and state.dtype == u.dtype and w.is_contiguous()
+    B = T if cu_q is None else cu_q.shape[0] - 1
+    rc = nat.lib().omni_conv_silu(
+        nat.ptr(u), nat.c_int(u.stride(0)), nat.c_int(C), nat.c_int(taps), nat.ptr(w), nat.ptr(bias), nat.ptr(state),
+        nat.ptr(positions), nat.ptr(q_to_seq), nat.ptr(cu_q), nat.ptr(state_slots), nat.c_int(B), nat.c_int(T), nat.ptr(out),
+        nat.c_int(out.shape[1]), nat.c_int(_f32(u)), nat.stream())
+    nat.check_rc(rc, "omni_conv_silu")
+    return out
+
+
+def ssm_scan_ref(xbc, dt, A_log, dt_bias, D, state, positions, state_slots, cu_q, H, P, N, G, out):
+    inner = H * P
+    of = torch.arange(H) // (H // G)
+    A = -torch.exp(A_log)
+    for r, a, b in _segments(cu_q, xbc.shape[0]):
+        slot = int(state_slots[r])
+        if slot < 0:
+            out[a:b] = 0
+            continue
+        S = state[slot] if int(positions[a]) > 0 else torch.zeros_like(state[slot])      # [H, P, N]
+        for t in range(a, b):
+            x = xbc[t, :inner].float().view(H, P)
+            B = xbc[t, inner:inner + G * N].float().view(G, N)[of]
+            C = xbc[t, inner + G * N:inner + 2 * G * N].float().view(G, N)[of]
+            d = F.softplus(dt[t].float() + dt_bias, threshold=1e9)
+            S = torch.exp(A * d)[:, None, None] * S + (d[:, None] * x)[:, :, None] * B[:, None, :]
+            y = torch.einsum("hpn,hn->hp", S, C) + D[:, None] * x
+            out[t, :inner] = y.reshape(-1).to(out.dtype)
+        state[slot] = S
+    return out
+
+
+def ssm_scan(xbc, dt, A_log, dt_bias, D, state, *, H, P, N, G, positions, state_slots, cu_q=None, by_rows=False):
+    """S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x with dt = softplus(dt + dt_bias), per head; ``xbc`` rows are
+    x | B | C, ``dt`` [T, H] (rows of any pitch), ``state`` [slots, H, P, N] fp32.  Requests that start at position 0 start
+    from zeros.  ``by_rows``: token by token even where the chunked tensor-core form applies.  -> y [T, pad8(H P)]."""
+    T = xbc.shape[0]
+    out = torch.empty(T, pad8(H * P), dtype=xbc.dtype, device=xbc.device)
+    if not xbc.is_cuda:
+        return ssm_scan_ref(xbc, dt, A_log, dt_bias, D, state, positions, state_slots, cu_q, H, P, N, G, out)
+    assert xbc.stride(1) == 1 and dt.dtype == xbc.dtype and dt.stride(1) == 1 and state.dtype == torch.float32
+    B = T if cu_q is None else cu_q.shape[0] - 1
+    rc = nat.lib().omni_ssm_scan(
+        nat.ptr(xbc), nat.c_int(xbc.stride(0)), nat.ptr(dt), nat.c_int(dt.stride(0)), nat.ptr(A_log), nat.ptr(dt_bias),
+        nat.ptr(D), nat.ptr(state), nat.ptr(cu_q), nat.ptr(positions), nat.ptr(state_slots), nat.c_int(B), nat.ptr(out),
+        nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N), nat.c_int(G), nat.c_int(_f32(xbc)),
+        nat.c_int(int(by_rows)), nat.stream())
+    nat.check_rc(rc, "omni_ssm_scan")
+    return out
+
+
+def gated_group_norm(y, z, w, parts, eps):
+    """RMSNorm of y * silu(z) in ``parts`` equal parts, times w.  y, z: rows of at least len(w) columns."""
+    T, inner = y.shape[0], w.shape[0]
+    ld = pad8(inner)
+    if not y.is_cuda:
+        g = y[:, :inner].float() * F.silu(z[:, :inner].float())
+        g = g.view(T, parts, -1)
+        g = g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)
+        return F.pad(g.reshape(T, inner) * w, (0, ld - inner)).to(y.dtype)
+    out = torch.empty(T, ld, dtype=y.dtype, device=y.device)
+    rc = nat.lib().omni_gated_group_norm(
+        nat.ptr(y), nat.c_int(y.stride(0)), nat.ptr(z), nat.c_int(z.stride(0)), nat.ptr(w), nat.ptr(out), nat.c_int(ld),
+        nat.c_int(T), nat.c_int(inner), nat.c_int(parts), nat.c_float(eps), nat.c_int(_f32(y)), nat.stream())
+    nat.check_rc(rc, "omni_gated_group_norm")
+    return out

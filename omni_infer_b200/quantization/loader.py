@@ -3,6 +3,7 @@
 Accepted weight formats (per tensor):
   * bf16 / fp16 / fp32
   * HF DeepSeek-V3 e4m3 + ``weight_scale_inv`` fp32 per 128x128 block (loaded as is)
+  * models with ``checkpoint_targets`` (layer-list models): their own names, every tensor required, none left over
   * compressed-tensors int8 w8a8: ``weight`` int8 [out,in] + ``weight_scale`` [out,1] (+ ``weight_offset``)
     as produced for the reference (omni/quantization/compressed_tensors/schemes/compressed_tensors_w8a8_int8.py:33-69,
     omni/quantization/compressed_tensors/compressed_tensors_moe.py:34-92); dequantised at load and re-quantised
@@ -40,6 +41,8 @@ class WeightLoader:
         self.model, self.cfg, self.planner, self.mtp_layer = model, cfg, planner, mtp_layer
         self.params = dict(model.named_parameters())
         self.loaded: set = set()
+        # models that name their own checkpoint tensors: {tensor: (parameter, first row, rows, columns)}
+        self.targets = model.checkpoint_targets() if hasattr(model, "checkpoint_targets") else None
         self._pending: dict = {}     # base name -> {"weight":..., "scale":..., "offset":...}
 
     # -- write one logical weight (float or fp8+scale) into (a row slice of) a parameter
@@ -79,8 +82,23 @@ class WeightLoader:
             return self.planner.local_slots_of(moe.moe_index, expert)
         return moe.local_slots_of(expert)
 
+    def _store_target(self, name: str, w):
+        """One tensor of a model with ``checkpoint_targets``; columns None: a vector, negative: stored transposed."""
+        if name not in self.targets:
+            raise KeyError(f"checkpoint tensor {name!r} belongs to no parameter of this model")
+        p, r0, rows, cols = self.targets[name]
+        want = (rows,) if cols is None else ((-cols, rows) if cols < 0 else (rows, cols))
+        if tuple(w.shape) != want:
+            raise ValueError(f"checkpoint tensor {name!r} has shape {tuple(w.shape)}, the configuration asks for {want}")
+        w = w.t() if cols is not None and cols < 0 else w
+        tgt = p.data[r0:r0 + rows] if cols is None else p.data[r0:r0 + rows, :abs(cols)]
+        tgt.copy_(w.to(p.dtype))
+        self.loaded.add(name)
+
     def _route(self, name: str, w, scale, offset):
         cfg = self.cfg
+        if self.targets is not None:
+            return self._store_target(name, w)
         m = re.match(r"model\.layers\.(\d+)\.(.*)", name)
         if self.mtp_layer is not None:
             # drafter: only layer `mtp_layer`; its sub-names map onto enorm / hnorm / eh_proj / shared_head / decoder
@@ -231,6 +249,8 @@ class WeightLoader:
             if "weight" in ent:
                 self._route(base, ent["weight"], ent.get("scale"), ent.get("offset"))
         self._pending.clear()
+        if self.targets is not None and len(self.loaded) < len(self.targets):
+            raise KeyError(f"checkpoint lacks {sorted(set(self.targets) - self.loaded)[:4]}")
         self.model.process_weights_after_loading()
         return self.loaded
 
