@@ -48,7 +48,7 @@ FINISH_REASON = {RequestStatus.FINISHED_STOPPED: "stop", RequestStatus.FINISHED_
                  RequestStatus.FINISHED_ABORTED: "abort", RequestStatus.FINISHED_IGNORED: "ignored"}
 
 
-@dataclass
+@dataclass(eq=False)       # a request is itself: the scheduler looks it up in its lists at every step
 class Request:
     request_id: str
     prompt_token_ids: list
