@@ -9,7 +9,7 @@ import torch
 
 import layer_list_cases as cases
 import layer_list_oracle as oracle
-from layer_list_cases import CONFIGS, error, expected, tokens
+from layer_list_cases import CONFIGS, error, expected, row_errors, tokens
 from omni_infer_b200.engine.engine_core import LLM, EngineConfig, EngineCore
 from omni_infer_b200.engine.kv_manager import KVCacheManager
 from omni_infer_b200.engine.request import Request, SamplingParams
@@ -18,7 +18,10 @@ from omni_infer_b200.models.config import ModelConfig, get_config
 
 RUNS = [pytest.param("cpu", "float32", id="cpu-float32"), pytest.param("cuda", "float32", id="cuda-float32", marks=pytest.mark.gpu),
         pytest.param("cuda", "bfloat16", id="cuda-bfloat16", marks=pytest.mark.gpu)]
-TOL = {"float32": 2e-5, "bfloat16": 0.06}
+# largest row error, typical row error.  Rounding to bf16 alone (the CPU references) gives 0.06 and 0.015 here.
+TOL = {"float32": 2e-5, "bfloat16": 0.15}
+TYPICAL = {"float32": 1e-5, "bfloat16": 0.03}
+ONE_LAYER = {"float32": 1e-5, "bfloat16": 0.03}
 
 
 @pytest.fixture(autouse=True)
@@ -70,8 +73,8 @@ def portions(n, sizes):
 
 
 def check(name, got, toks, dtype, seed=0):
-    e = error(got, expected(name, seed, toks))
-    assert e < TOL[dtype], e
+    e = row_errors(got, expected(name, seed, toks))
+    assert float(e.max()) < TOL[dtype] and float(e.median()) < TYPICAL[dtype], (float(e.max()), float(e.median()))
 
 
 # ----------------------------------------------------------------------------- the same logits however they are computed
@@ -123,14 +126,13 @@ def test_token_inside_and_outside_the_window_through_the_model(device, dtype, de
     window = 20
     cfg = cases.config([cases.attention(heads=2, kv_heads=1, dim=16, vdim=16, window=window, rot=0, ff=0)], width=32, vocab=16)
     w = cases.weights(cfg, 3)
-    marker = torch.zeros(32)
-    marker[5] = 40.0
-    w["embed"][9] = marker.bfloat16()
-    w["l0.mix.k"].zero_()
-    w["l0.mix.k"][:, 5] = 1.0
-    w["l0.mix.k.norm"].fill_(1.0)
-    w["l0.mix.q.norm"].fill_(6.0)
-    w["l0.mix.q"][:, 0] += 3.0                       # queries lean towards the marker's key
+    # every query is the same vector; the rare token's key points along it, every other key the opposite way
+    w["embed"][:, 0], w["embed"][:, 5] = 2.0, -0.5
+    w["embed"][9, 5] = 3.0
+    for t, col in (("q", 0), ("k", 5)):
+        w["l0.mix." + t].zero_()
+        w["l0.mix." + t][:, col] = 1.0
+        w[f"l0.mix.{t}.norm"].fill_(1.0)
     mc = ModelConfig.from_hf_dict(cfg)
     mc.dtype = dtype
     eng = EngineCore(EngineConfig(model="x", device=device, block_size=64, num_kv_blocks=6, max_num_seqs=2, max_model_len=128),
@@ -143,10 +145,9 @@ def test_token_inside_and_outside_the_window_through_the_model(device, dtype, de
         plan = [[("a", 69)], [("a", 1)]] if decode else [[("a", 70)]]
         got = run(eng, {"a": toks}, plan)["a"]
         want = oracle.forward(cfg, w, toks)
-        assert error(got, want) < TOL[dtype]
-        last.append((got[-1].double(), want[-1]))
-    (gi, wi), (go, wo) = last
-    assert float((wi - wo).norm()) > 5 * TOL[dtype] * float(wi.std()) * len(wi) ** 0.5, "the case does not show the edge"
+        assert error(got, want) < ONE_LAYER[dtype]
+        last.append(want[-1])
+    assert error(last[0][None], last[1][None]) > 3 * ONE_LAYER["bfloat16"], "the case does not show the edge"
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
@@ -157,19 +158,20 @@ def test_far_token_lives_in_the_recurrent_state(device, dtype):
     w = cases.weights(cfg, 5)
     w["l0.mix.A_log"].fill_(-7.0)
     w["l0.mix.dt_bias"].fill_(-2.0)
+    w["embed"][9] *= 6
     mc = ModelConfig.from_hf_dict(cfg)
     mc.dtype = dtype
     eng = EngineCore(EngineConfig(model="x", device=device, block_size=64, num_kv_blocks=10, max_num_seqs=1, max_model_len=512),
                      model_cfg=mc, weights=list(w.items()))
-    a = tokens(300, 16, 1)
-    b = tokens(20, 16, 2) + a[20:]
+    a = [9] * 20 + [t % 8 for t in tokens(280, 16, 1)]      # the first tokens write far more than the others
+    b = tokens(20, 8, 2) + a[20:]
     outs = []
     for toks in (a, b, a):
         got = run(eng, {"a": toks}, [[("a", m)] for m in [200, 64, 2] + [1] * 34])["a"]
         want = oracle.forward(cfg, w, toks)
-        assert error(got, want) < TOL[dtype]
+        assert error(got, want) < ONE_LAYER[dtype]
         outs.append((got, want))
-    assert float((outs[0][1][-1] - outs[1][1][-1]).abs().max()) > 3 * TOL[dtype] * float(outs[0][1].std())
+    assert error(outs[0][1][-1:], outs[1][1][-1:]) > 3 * ONE_LAYER["bfloat16"], "the case does not show the far tokens"
     assert torch.allclose(outs[0][0], outs[2][0], atol=1e-5)
 
 
