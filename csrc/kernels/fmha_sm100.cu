@@ -46,12 +46,19 @@ constexpr int FM_BQ = 128, FM_BK = 64, FM_DV = 128;
 constexpr int FM_QCHUNK = FM_BQ * 128;          // 16 KB
 constexpr int FM_KCHUNK = FM_BK * 128;          // 8 KB
 constexpr int FM_MAXC = 3;                      // up to 192 qk dims
-constexpr int FM_STAGES = 3;
-constexpr int FM_K_STAGE = FM_MAXC * FM_KCHUNK; // 24 KB
 constexpr int FM_V_STAGE = 2 * FM_KCHUNK;       // 16 KB
-constexpr int FM_SMEM = FM_MAXC * FM_QCHUNK + FM_STAGES * (FM_K_STAGE + FM_V_STAGE) + 1024 + 1024;
 constexpr int FM_THREADS = 192;
-constexpr int FT_O = 0, FT_S = 128, FT_P = 256, FT_PLO = 320, FT_COLS = 512;
+// Shared memory and TMEM layout.  MAXC: 64-wide chunks of the qk size that fit.  The paged kernel with two chunks and two
+// stages takes 98 KB and 256 TMEM columns, so that two CTAs share an SM and one's softmax overlaps the other's MMAs; its P
+// (32 columns hi, 32 columns lo) replaces the 64 columns of the S tile that it was computed from, which the next QK^T but
+// one writes again only after the PV that reads P (the MMAs of a CTA complete in order).
+template <bool PAGED, int MAXC, int STAGES>
+struct FmLayout {
+  static constexpr int K_STAGE = MAXC * FM_KCHUNK;
+  static constexpr int SMEM = MAXC * FM_QCHUNK + STAGES * (K_STAGE + FM_V_STAGE) + 1024 + 1024;
+  static constexpr int T_O = 0, T_S = 128, T_P = PAGED ? T_S : 256, T_P_STRIDE = PAGED ? FM_BK : FM_BK / 2;
+  static constexpr int T_COLS = PAGED ? 256 : 512;
+};
 
 __device__ __forceinline__ void fm_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc,
                                            uint32_t accumulate) {
@@ -62,8 +69,8 @@ __device__ __forceinline__ void fm_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uin
       : "memory");
 }
 
-template <bool PAGED>
-__global__ void __launch_bounds__(FM_THREADS, 1)
+template <bool PAGED, int MAXC, int STAGES>
+__global__ void __launch_bounds__(FM_THREADS, (PAGED && MAXC == 2) ? 2 : 1)
 fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                    const __grid_constant__ CUtensorMap tmap_k2, const __grid_constant__ CUtensorMap tmap_v,
                    const FmhaParams p) {
@@ -83,18 +90,19 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const int n = (k_hi + FM_BK - 1) / FM_BK - t_first;
   const int nv = PAGED ? (p.dv + 63) / 64 : 2;         // 64-wide chunks of the value size
 
+  using L = FmLayout<PAGED, MAXC, STAGES>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* sq = smem;
-  uint8_t* sk = smem + FM_MAXC * FM_QCHUNK;
-  uint8_t* sv = sk + FM_STAGES * FM_K_STAGE;
-  uint64_t* bars = (uint64_t*)(sv + FM_STAGES * FM_V_STAGE);
+  uint8_t* sk = smem + MAXC * FM_QCHUNK;
+  uint8_t* sv = sk + STAGES * L::K_STAGE;
+  uint64_t* bars = (uint64_t*)(sv + STAGES * FM_V_STAGE);
   uint64_t* q_full = bars;                       // 1
   uint64_t* k_full = bars + 1;                   // STAGES
-  uint64_t* k_empty = k_full + FM_STAGES;
-  uint64_t* v_full = k_empty + FM_STAGES;
-  uint64_t* v_empty = v_full + FM_STAGES;
-  uint64_t* s_full = v_empty + FM_STAGES;        // 2
+  uint64_t* k_empty = k_full + STAGES;
+  uint64_t* v_full = k_empty + STAGES;
+  uint64_t* v_empty = v_full + STAGES;
+  uint64_t* s_full = v_empty + STAGES;        // 2
   uint64_t* p_full = s_full + 2;                 // 2
   uint64_t* o_done = p_full + 2;                 // 1
   uint64_t* o_final = o_done + 1;                // 1
@@ -104,7 +112,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int s = 0; s < FM_STAGES; ++s) {
+    for (int s = 0; s < STAGES; ++s) {
       mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1);
       mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1);
     }
@@ -115,7 +123,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     mbar_fence_init();
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, FT_COLS);
+    tmem_alloc(tmem_slot, L::T_COLS);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -131,8 +139,8 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         else tma_load_2d(sq + c * FM_QCHUNK, &tmap_q, q_full, h * p.q_head_stride + c * 64, q_begin + q0);
       }
       for (int i = 0; i < n; ++i) {
-        const int st = i % FM_STAGES;
-        const uint32_t ph = (i / FM_STAGES) & 1;
+        const int st = i % STAGES;
+        const uint32_t ph = (i / STAGES) & 1;
         int row = k_begin + i * FM_BK;
         if (PAGED) {
           const int key0 = (t_first + i) * FM_BK;
@@ -141,11 +149,11 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         if (!mbar_wait(&k_empty[st], ph ^ 1, abort_flag, p.status, 11, i)) break;
         mbar_expect_tx(&k_full[st], nc * FM_KCHUNK);
         for (int c = 0; c < p.nk1; ++c) {
-          if (PAGED) tma_load_3d(sk + st * FM_K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], c * 64, hk, row);
-          else tma_load_2d(sk + st * FM_K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], hk * p.k_head_stride + c * 64, row);
+          if (PAGED) tma_load_3d(sk + st * L::K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], c * 64, hk, row);
+          else tma_load_2d(sk + st * L::K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], hk * p.k_head_stride + c * 64, row);
         }
         for (int c = 0; c < p.nk2; ++c)
-          tma_load_2d(sk + st * FM_K_STAGE + (p.nk1 + c) * FM_KCHUNK, &tmap_k2, &k_full[st], p.k2_col0 + c * 64, row);
+          tma_load_2d(sk + st * L::K_STAGE + (p.nk1 + c) * FM_KCHUNK, &tmap_k2, &k_full[st], p.k2_col0 + c * 64, row);
         if (!mbar_wait(&v_empty[st], ph ^ 1, abort_flag, p.status, 12, i)) break;
         mbar_expect_tx(&v_full[st], nv * FM_KCHUNK);
         for (int c = 0; c < nv; ++c) {
@@ -161,14 +169,14 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       const uint32_t idesc_pv = umma_idesc(128, nv * 64, 1, 1, 0, 1);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 13, 0);
       auto issue_qk = [&](int j) -> bool {
-        const int st = j % FM_STAGES;
-        if (!mbar_wait(&k_full[st], (j / FM_STAGES) & 1, abort_flag, p.status, 14, j)) return false;
+        const int st = j % STAGES;
+        if (!mbar_wait(&k_full[st], (j / STAGES) & 1, abort_flag, p.status, 14, j)) return false;
         tc_fence_after();
-        const uint32_t d = tmem_base + FT_S + (j & 1) * FM_BK;
+        const uint32_t d = tmem_base + L::T_S + (j & 1) * FM_BK;
         uint32_t accum = 0;
         for (int c = 0; c < nc; ++c) {
           const uint64_t ad = umma_desc_kmajor_sw128(smem_u32(sq) + c * FM_QCHUNK);
-          const uint64_t bd = umma_desc_kmajor_sw128(smem_u32(sk) + st * FM_K_STAGE + c * FM_KCHUNK);
+          const uint64_t bd = umma_desc_kmajor_sw128(smem_u32(sk) + st * L::K_STAGE + c * FM_KCHUNK);
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
             umma_bf16(d, ad + 2 * k, bd + 2 * k, idesc_qk, accum);
@@ -182,17 +190,17 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       if (ok) ok = issue_qk(0);
       if (ok && n > 1) ok = issue_qk(1);
       for (int i = 0; i < n && ok; ++i) {
-        const int st = i % FM_STAGES;
+        const int st = i % STAGES;
         if (!mbar_wait(&p_full[i & 1], (i >> 1) & 1, abort_flag, p.status, 15, i)) { ok = false; break; }
-        if (!mbar_wait(&v_full[st], (i / FM_STAGES) & 1, abort_flag, p.status, 16, i)) { ok = false; break; }
+        if (!mbar_wait(&v_full[st], (i / STAGES) & 1, abort_flag, p.status, 16, i)) { ok = false; break; }
         tc_fence_after();
         const uint32_t vbase = smem_u32(sv) + st * FM_V_STAGE;
 #pragma unroll
         for (int k = 0; k < FM_BK / 16; ++k) {
           const uint64_t bd = umma_desc_mnmajor_sw128(vbase + k * 2048, FM_KCHUNK, 1024);
-          fm_umma_ts(tmem_base + FT_O, tmem_base + FT_P + (i & 1) * (FM_BK / 2) + k * 8, bd, idesc_pv,
+          fm_umma_ts(tmem_base + L::T_O, tmem_base + L::T_P + (i & 1) * L::T_P_STRIDE + k * 8, bd, idesc_pv,
                      (i > 0 || k > 0) ? 1u : 0u);
-          if (PAGED) fm_umma_ts(tmem_base + FT_O, tmem_base + FT_PLO + (i & 1) * (FM_BK / 2) + k * 8, bd, idesc_pv, 1u);
+          if (PAGED) fm_umma_ts(tmem_base + L::T_O, tmem_base + L::T_P + FM_BK / 2 + (i & 1) * L::T_P_STRIDE + k * 8, bd, idesc_pv, 1u);
         }
         umma_commit(&v_empty[st]);
         umma_commit(o_done);
@@ -220,7 +228,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 #pragma unroll
       for (int c0 = 0; c0 < FM_BK; c0 += 32) {
         uint32_t sv32[32];
-        tmem_ld_x32(lane_addr + FT_S + (i & 1) * FM_BK + c0, sv32);
+        tmem_ld_x32(lane_addr + L::T_S + (i & 1) * FM_BK + c0, sv32);
         tmem_ld_wait();
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
@@ -241,11 +249,11 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 #pragma unroll 1
         for (int c = 0; c < nv * 64; c += 32) {
           uint32_t ov[32];
-          tmem_ld_x32(lane_addr + FT_O + c, ov);
+          tmem_ld_x32(lane_addr + L::T_O + c, ov);
           tmem_ld_wait();
 #pragma unroll
           for (int j = 0; j < 32; ++j) ov[j] = __float_as_uint(__uint_as_float(ov[j]) * f);
-          tmem_st_x32(lane_addr + FT_O + c, ov);
+          tmem_st_x32(lane_addr + L::T_O + c, ov);
         }
         tmem_st_wait();
       }
@@ -265,8 +273,8 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         }
       }
       l += rs;
-      tmem_st_x32(lane_addr + FT_P + (i & 1) * (FM_BK / 2), pk);
-      if (PAGED) tmem_st_x32(lane_addr + FT_PLO + (i & 1) * (FM_BK / 2), pl);
+      tmem_st_x32(lane_addr + L::T_P + (i & 1) * L::T_P_STRIDE, pk);
+      if (PAGED) tmem_st_x32(lane_addr + L::T_P + FM_BK / 2 + (i & 1) * L::T_P_STRIDE, pl);
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
@@ -281,7 +289,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 #pragma unroll 1
       for (int c = 0; c < p.dv; c += 32) {
         uint32_t ov[32];
-        tmem_ld_x32(lane_addr + FT_O + c, ov);
+        tmem_ld_x32(lane_addr + L::T_O + c, ov);
         tmem_ld_wait();
         if (row_ok) {
 #pragma unroll
@@ -306,13 +314,23 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, FT_COLS);
+    tmem_dealloc(tmem_base, L::T_COLS);
   }
 }
 
 }  // namespace omni
 
 using namespace omni;
+
+template <bool PAGED, int MAXC, int STAGES>
+static int launch_fmha(dim3 grid, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tk2, const CUtensorMap& tv,
+                       const FmhaParams& p, cudaStream_t stream) {
+  constexpr int smem = FmLayout<PAGED, MAXC, STAGES>::SMEM;
+  static bool configured[64] = {false};
+  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel<PAGED, MAXC, STAGES>, smem, configured)) return e;
+  fmha_varlen_kernel<PAGED, MAXC, STAGES><<<grid, FM_THREADS, smem, stream>>>(tq, tk, tk2, tv, p);
+  return (int)cudaGetLastError();
+}
 
 // q/k/k2/v are 2-D row-major bf16 matrices given by (pointer, rows, row pitch in elements, columns).
 extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q_cols, const void* k, long long k_rows,
@@ -340,11 +358,7 @@ extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q
   p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = FM_DV; p.out_ld = Hq * FM_DV;
   p.kv_len = nullptr; p.block_table = nullptr; p.bt_ld = 0; p.block_size = 0; p.window = 0;
-  static bool configured[64] = {false};
-  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel<false>, FM_SMEM, configured)) return e;
-  dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
-  fmha_varlen_kernel<false><<<grid, FM_THREADS, FM_SMEM, stream>>>(tq, tk, tk2, tv, p);
-  return (int)cudaGetLastError();
+  return launch_fmha<false, FM_MAXC, 3>(dim3((max_q + FM_BQ - 1) / FM_BQ, B, Hq), tq, tk, tk2, tv, p, stream);
 }
 
 // Ragged queries against the paged cache.  q: rows of pitch q_ld holding Hq heads of d_k; k_cache / v_cache
@@ -370,9 +384,7 @@ extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const 
   p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = d_v; p.out_ld = out_ld; p.kv_len = kv_len; p.block_table = block_table; p.bt_ld = bt_ld;
   p.block_size = block_size; p.window = window;
-  static bool configured[64] = {false};
-  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel<true>, FM_SMEM, configured)) return e;
-  dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
-  fmha_varlen_kernel<true><<<grid, FM_THREADS, FM_SMEM, stream>>>(tq, tk, tk, tv, p);
-  return (int)cudaGetLastError();
+  const dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
+  if (p.nk1 <= 2) return launch_fmha<true, 2, 2>(grid, tq, tk, tk, tv, p, stream);
+  return launch_fmha<true, FM_MAXC, 3>(grid, tq, tk, tk, tv, p, stream);
 }

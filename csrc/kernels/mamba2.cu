@@ -10,11 +10,12 @@
 // State slots: conv [slots, taps - 1, channels] (activation type), ssm [slots, heads, P, N] fp32.  A request whose first
 // token of the call is at position 0 starts from zeros whatever its slot holds; a row with a negative slot is padding.
 //
-// The scan has two forms.
+// The scan has two forms here.
 //   ssm_rows_kernel   token by token, the state in registers: a warp owns a few rows of P, N lies across its lanes.  One
 //                     token per request (decode) makes it a stream over the state; it also is the fp32 path and takes the
 //                     shapes the other form does not.
-//   ssd_chunk_kernel  portions of prompts, bf16: chunks of 64 tokens through the tensor cores,
+//   ssd_chunk_kernel  portions of prompts, bf16, states of more than 128 (up to that size ssd_sm100.cu runs the same scheme
+//                     on tcgen05): chunks of 64 tokens,
 //                       Y = (C B^T o L) (dt x) + exp(cum) C S,   S <- exp(cum_end) S + B^T (exp(cum_end - cum) dt x)
 //                     with L_ij = exp(cum_i - cum_j) for j <= i and cum the running sum of -exp(A_log) dt in the chunk.
 //                     One CTA walks the chunks of one (request, head, 32 columns of P); S stays in fp32 accumulators.
@@ -143,6 +144,7 @@ struct SsmParams {
   void* y;                // [T, y_ld]
   int y_ld;
   int H, P, N, G;
+  int max_rows;           // requests with more rows are left to another kernel (0: none are)
 };
 
 // NV values of N per lane.  VECN: a lane's values are neighbours (N a multiple of NV, 16-byte accesses); otherwise they are
@@ -154,7 +156,7 @@ __global__ void __launch_bounds__(128) ssm_rows_kernel(const SsmParams p) {
   const int p0 = (blockIdx.y * 4 + warp) * R;
   if (p0 >= p.P) return;
   const int row0 = p.cu_q ? p.cu_q[r] : r, row1 = p.cu_q ? p.cu_q[r + 1] : r + 1;
-  if (row1 <= row0) return;
+  if (row1 <= row0 || (p.max_rows > 0 && row1 - row0 > p.max_rows)) return;
   const int slot = p.state_slots[r];
   const int inner = p.H * p.P, g = h / (p.H / p.G);
   const T* xbc = (const T*)p.xbc;
@@ -702,23 +704,20 @@ extern "C" int omni_conv_silu(const void* u, int ld, int C, int taps, const void
   return conv_silu_t<bf16, 1>(u, ld, C, taps, wf, bf, state, positions, q_to_seq, cu_q, state_slots, B, rows, out, out_ld, st);
 }
 
-// cu_q null: one row per request.  by_rows: take the token-by-token form even where the chunked one is possible.
+// cu_q null: one row per request.  max_rows > 0: token by token, requests of up to max_rows rows only; < 0: token by token
+// for all of them.
 extern "C" int omni_ssm_scan(const void* xbc, int xbc_ld, const void* dt, int dt_ld, const void* A_log, const void* dt_bias,
                              const void* D, void* state, const int* cu_q, const int64_t* positions, const int* state_slots,
-                             int B, void* y, int y_ld, int H, int P, int N, int G, int f32, int by_rows, cudaStream_t st) {
+                             int B, void* y, int y_ld, int H, int P, int N, int G, int f32, int max_rows, cudaStream_t st) {
   if (B <= 0) return 0;
   if (H < 1 || P < 1 || N < 1 || G < 1 || H % G != 0 || B > 65535 || H > 65535) return -1;
   SsmParams p;
   p.xbc = xbc; p.xbc_ld = xbc_ld; p.dt = dt; p.dt_ld = dt_ld; p.A_log = (const float*)A_log;
   p.dt_bias = (const float*)dt_bias; p.D = (const float*)D; p.state = (float*)state; p.cu_q = cu_q; p.positions = positions;
-  p.state_slots = state_slots; p.y = y; p.y_ld = y_ld; p.H = H; p.P = P; p.N = N; p.G = G;
-  const bool chunked = cu_q != nullptr && !f32 && !by_rows && P % 8 == 0 && N % 8 == 0 && N <= 256 && xbc_ld % 8 == 0 &&
-                       y_ld % 2 == 0 && (uintptr_t)xbc % 16 == 0 && (uintptr_t)y % 4 == 0;
-  if (chunked) {
-    if (N <= 64) return launch_ssd<64>(p, B, st);
-    if (N <= 128) return launch_ssd<128>(p, B, st);
-    return launch_ssd<256>(p, B, st);
-  }
+  p.state_slots = state_slots; p.y = y; p.y_ld = y_ld; p.H = H; p.P = P; p.N = N; p.G = G; p.max_rows = max_rows > 0 ? max_rows : 0;
+  const bool chunked = cu_q != nullptr && !f32 && max_rows == 0 && P % 8 == 0 && N % 8 == 0 && N > 128 && N <= 256 &&
+                       xbc_ld % 8 == 0 && y_ld % 2 == 0 && (uintptr_t)xbc % 16 == 0 && (uintptr_t)y % 4 == 0;
+  if (chunked) return launch_ssd<256>(p, B, st);
   return f32 ? launch_ssm_rows<float>(p, B, st) : launch_ssm_rows<bf16>(p, B, st);
 }
 

@@ -55,7 +55,7 @@ def _run(cmd, log: Path | None = None) -> None:
 # Kernel sources (stems) that one architecture needs when it is served alone
 ARCH_KERNELS = {
     "Forovik": ("attn_any", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "mamba2", "post_norm_ops",
-                "sampler_misc"),
+                "sampler_misc", "ssd_sm100"),
 }
 
 

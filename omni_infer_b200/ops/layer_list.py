@@ -2,7 +2,7 @@
 paged cache with a q/k norm over the whole projection, and the Mamba-2 layer between its projections.
 
 CUDA tensors run ``csrc/kernels/post_norm_ops.cu``, ``attn_any.cu``, ``fmha_sm100.cu``, ``gqa_decode.cu`` and
-``mamba2.cu``; CPU tensors run the fp32 references here.  Activations are bf16 or fp32.  Rows may be wider than their
+``mamba2.cu`` / ``ssd_sm100.cu``; CPU tensors run the fp32 references here.  Activations are bf16 or fp32.  Rows may be wider than their
 content (a multiple of 8 columns, so that they can be TMA operands); the columns past it are zero.
 
 Ragged batches: the rows of request r are ``cu_q[r]:cu_q[r + 1]``, its rows' positions ascend by one, ``q_to_seq[row] = r``.
@@ -262,21 +262,37 @@ def ssm_scan_ref(xbc, dt, A_log, dt_bias, D, state, positions, state_slots, cu_q
     return out
 
 
-def ssm_scan(xbc, dt, A_log, dt_bias, D, state, *, H, P, N, G, positions, state_slots, cu_q=None, by_rows=False):
+SSD_MIN_ROWS = 8      # portions below this go token by token: a chunk of the tensor-core form costs as much as some tokens
+
+
+def ssm_scan(xbc, dt, A_log, dt_bias, D, state, *, H, P, N, G, positions, state_slots, cu_q=None, min_q=1, by_rows=False):
     """S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x with dt = softplus(dt + dt_bias), per head; ``xbc`` rows are
     x | B | C, ``dt`` [T, H] (rows of any pitch), ``state`` [slots, H, P, N] fp32.  Requests that start at position 0 start
-    from zeros.  ``by_rows``: token by token even where the chunked tensor-core form applies.  -> y [T, pad8(H P)]."""
+    from zeros.  ``min_q``: rows of the shortest request, if known.  ``by_rows``: token by token even where the chunked
+    tensor-core forms apply.  -> y [T, pad8(H P)]."""
     T = xbc.shape[0]
     out = torch.empty(T, pad8(H * P), dtype=xbc.dtype, device=xbc.device)
     if not xbc.is_cuda:
         return ssm_scan_ref(xbc, dt, A_log, dt_bias, D, state, positions, state_slots, cu_q, H, P, N, G, out)
     assert xbc.stride(1) == 1 and dt.dtype == xbc.dtype and dt.stride(1) == 1 and state.dtype == torch.float32
     B = T if cu_q is None else cu_q.shape[0] - 1
+    max_rows = -1 if by_rows else 0
+    if (cu_q is not None and not by_rows and xbc.dtype == torch.bfloat16 and P % 8 == 0 and N % 8 == 0 and N <= 128
+            and xbc.stride(0) % 8 == 0 and xbc.data_ptr() % 16 == 0):
+        rc = nat.lib().omni_ssd_chunks(
+            nat.ptr(xbc), nat.c_int(xbc.stride(0)), nat.c_int64(T), nat.ptr(dt), nat.c_int(dt.stride(0)), nat.ptr(A_log),
+            nat.ptr(dt_bias), nat.ptr(D), nat.ptr(state), nat.ptr(cu_q), nat.ptr(positions), nat.ptr(state_slots),
+            nat.c_int(B), nat.ptr(out), nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N), nat.c_int(G),
+            nat.c_int(SSD_MIN_ROWS), nat.ptr(nat.status_buffer(xbc.device)), nat.stream())
+        nat.check_rc(rc, "omni_ssd_chunks")
+        if min_q >= SSD_MIN_ROWS:
+            return out
+        max_rows = SSD_MIN_ROWS - 1
     rc = nat.lib().omni_ssm_scan(
         nat.ptr(xbc), nat.c_int(xbc.stride(0)), nat.ptr(dt), nat.c_int(dt.stride(0)), nat.ptr(A_log), nat.ptr(dt_bias),
         nat.ptr(D), nat.ptr(state), nat.ptr(cu_q), nat.ptr(positions), nat.ptr(state_slots), nat.c_int(B), nat.ptr(out),
         nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N), nat.c_int(G), nat.c_int(_f32(xbc)),
-        nat.c_int(int(by_rows)), nat.stream())
+        nat.c_int(max_rows), nat.stream())
     nat.check_rc(rc, "omni_ssm_scan")
     return out
 

@@ -303,11 +303,11 @@ SCANS = [(4, 16, 24, 2), (2, 32, 64, 1), (3, 10, 7, 1), (2, 40, 128, 2), (4, 8, 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
 @pytest.mark.parametrize("H,P,N,G", SCANS)
-@pytest.mark.parametrize("sizes", [[400], [2, 1, 3], [65, 2, 64, 1, 1, 63]])
+@pytest.mark.parametrize("sizes", [[700], [2, 1, 3], [65, 2, 64, 1, 1, 63], [257, 8, 7, 128, 129]])
 def test_recurrence_in_portions(device, dtype, H, P, N, G, sizes):
     if device == "cpu" and N > 100:
         pytest.skip("covered by the other sizes")
-    lens = [150, 1, 70, 33] if device == "cuda" else [70, 1, 33]
+    lens = [530, 1, 70, 33] if device == "cuda" else [70, 1, 33]
     inner, C = H * P, H * P + 2 * G * N
     A_log, bias, D = rnd(H, seed=1), rnd(H, seed=2, scale=0.5) - 1, rnd(H, seed=3)
     dev = [t.to(device) for t in (A_log, bias, D)]
@@ -326,7 +326,7 @@ def test_recurrence_in_portions(device, dtype, H, P, N, G, sizes):
         if device == "cuda" and md["cu_q"] is not None:          # the other form, on a copy of the state
             other = state.clone()
             y2 = ll.ssm_scan(x, dt, *dev, other, H=H, P=P, N=N, G=G, by_rows=True, **md)
-        y = ll.ssm_scan(x, dt, *dev, state, H=H, P=P, N=N, G=G, **md)
+        y = ll.ssm_scan(x, dt, *dev, state, H=H, P=P, N=N, G=G, min_q=min(m for _, _, m in batch), **md)
         if device == "cuda" and md["cu_q"] is not None:
             close(y[:, :inner], y2[:, :inner].double().cpu(), TOL[dtype])
             close(state[md["state_slots"].long()], other[md["state_slots"].long()].double().cpu(), 2e-4)
