@@ -11,11 +11,14 @@
 // S lives in fp32 registers (thread = row n).  Every fp32 operand of an MMA is a pair of bf16 values hi + lo (two MMAs), so
 // products keep 16 bits of mantissa on that side; C, B and x are bf16 as stored.
 //
-// One CTA walks the chunks of its request.  Warps: 0 TMA producer (two stages of C, B, x), 1 MMA issue, 2..5 scores -> M and
-// the output rows (thread = token), 6..9 decays, W and the state (thread = token, then thread = state row).  Left of the
-// diagonal block a warp's 32 rows need no exponentials per element: exp(cum_i - cum_j) dt_j = exp(cum_i - cum_b) *
-// (exp(cum_b - cum_j) dt_j) with b the last token of j's block of 32, both factors at most 1 and the second shared by
-// all rows.  Every wait is bounded.
+// A first small kernel turns dt into what both sides need per (chunk, head): cum, cp = cum - log2(dt) (so that
+// exp(cum_i - cum_j) dt_j = 2^(cum_i - cp_j)) and g_j = 2^(cum_b - cp_j) with b the last token of j's block of 32.  Left of the
+// diagonal block a warp's 32 rows then need no exponential per element: 2^(cum_i - cp_j) = 2^(cum_i - cum_b) g_j, both
+// factors at most 1 (times dt) and the second shared by all rows.  All of it is in log2 units.
+//
+// One CTA walks the chunks of its request.  Warps: 0 TMA producer (two stages of C, B, x, cp, g), 1 MMA issue, 2..9 scores ->
+// M and the output rows (thread = token and half of the columns), 10..17 W and the state (thread = token, then state row, and
+// half of the columns).  Every wait is bounded.
 #include "../include/omni_ptx.cuh"
 #include "../include/omni_vec.cuh"
 #include "../include/tma_host.h"
@@ -36,6 +39,7 @@ struct SsdParams {
   int y_ld;
   int H, P, N, G;
   int min_rows;              // requests with fewer rows are left to another kernel
+  float *cum, *cp, *g;       // [chunks, H, 128]; chunk c of request r is row cu_q[r] / 128 + r + c
   OmniStatus* status;
 };
 
@@ -44,12 +48,14 @@ constexpr int SQ_TILE = SQ * 128;              // 128 rows of one 128-byte swizz
 constexpr int SQ_STAGE = 5 * SQ_TILE;          // C (2 tiles), B (2 tiles), x
 constexpr int SQ_W = 2 * SQ_STAGE;             // W hi, W lo
 constexpr int SQ_S = SQ_W + 2 * SQ_TILE;       // S hi, S lo
-constexpr int SQ_F = SQ_S + 2 * SQ_TILE;       // cum, g, dt: 128 floats each
-constexpr int SQ_BAR = SQ_F + 3 * SQ * 4;
+constexpr int SQ_F = SQ_S + 2 * SQ_TILE;       // two stages of cp and g
+constexpr int SQ_FB = SQ * 4;                  // bytes of one such array
+constexpr int SQ_BAR = SQ_F + 4 * SQ_FB;
 constexpr int SQ_SMEM = SQ_BAR + 192;
 static_assert(SQ_SMEM <= 232448, "shared memory of one CTA");
-constexpr int SQ_THREADS = 320;
-// TMEM columns: SC / M two buffers of 128, YO two of 64, YD, ST
+constexpr int SQ_THREADS = 576;
+// TMEM columns: SC / M two buffers of 128, YO two of 64, YD, ST.  M takes the columns of the scores it came from: 16 tokens
+// are 8 columns hi and 8 columns lo.
 constexpr int TC_SC = 0, TC_YO = 256, TC_YD = 384, TC_ST = 448, TC_COLS = 512;
 
 __device__ __forceinline__ void sq_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
@@ -67,14 +73,73 @@ __device__ __forceinline__ void sq_split2(float a, float b, uint32_t& hi, uint32
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 __device__ __forceinline__ float sq_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
-// eight values -> 16-byte chunk `ch` of row `row` of a hi and a lo tile
-__device__ __forceinline__ void sq_store8(uint8_t* hi_tile, uint8_t* lo_tile, int row, int ch, const float (&v)[8]) {
-  uint32_t hi[4], lo[4];
+__device__ __forceinline__ float sq_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void sq_tmem_st_x8(uint32_t taddr, const uint32_t (&r)[8]) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};"
+               ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7])
+               : "memory");
+}
+// 16 columns at each of two addresses.  The wait belongs to the same statement: between a load and its wait the compiler
+// must not touch the destination registers, and it would not know.
+__device__ __forceinline__ void sq_tmem_ld_2x16(uint32_t addr_a, uint32_t addr_b, uint32_t (&a)[16], uint32_t (&b)[16]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%32];\n\t"
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%33];\n\t"
+      "tcgen05.wait::ld.sync.aligned;"
+      : "=&r"(a[0]), "=&r"(a[1]), "=&r"(a[2]), "=&r"(a[3]), "=&r"(a[4]), "=&r"(a[5]), "=&r"(a[6]), "=&r"(a[7]), "=&r"(a[8]), "=&r"(a[9]), "=&r"(a[10]), "=&r"(a[11]), "=&r"(a[12]), "=&r"(a[13]), "=&r"(a[14]), "=&r"(a[15]),
+        "=&r"(b[0]), "=&r"(b[1]), "=&r"(b[2]), "=&r"(b[3]), "=&r"(b[4]), "=&r"(b[5]), "=&r"(b[6]), "=&r"(b[7]), "=&r"(b[8]), "=&r"(b[9]), "=&r"(b[10]), "=&r"(b[11]), "=&r"(b[12]), "=&r"(b[13]), "=&r"(b[14]), "=&r"(b[15])
+      : "r"(addr_a), "r"(addr_b)
+      : "memory");
+}
+__device__ __forceinline__ void sq_bulk_load(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
+}
+// byte offset of 16-byte chunk `ch` of row `row` of a swizzled tile
+__device__ __forceinline__ int sq_off(int row, int ch) { return row * 128 + ((ch ^ (row & 7)) << 4); }
+
+// One CTA per (chunk, request, 8 heads); thread = token of the chunk.
+__global__ void __launch_bounds__(SQ) ssd_decay_kernel(const SsdParams p) {
+  const int c = blockIdx.x, r = blockIdx.y, h0 = blockIdx.z * 8;
+  const int row0 = p.cu_q[r], n_rows = p.cu_q[r + 1] - row0;
+  if (c * SQ >= n_rows || n_rows < p.min_rows) return;
+  const int i = threadIdx.x, warp = i >> 5, lane = i & 31, t = c * SQ + i;
+  __shared__ float tot[4][8];
+  float dt[8], run[8];
 #pragma unroll
-  for (int e = 0; e < 4; ++e) sq_split2(v[2 * e], v[2 * e + 1], hi[e], lo[e]);
-  const int off = row * 128 + ((ch ^ (row & 7)) << 4);
-  *reinterpret_cast<uint4*>(hi_tile + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-  *reinterpret_cast<uint4*>(lo_tile + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  for (int k = 0; k < 8; ++k) {
+    const int h = h0 + k;
+    dt[k] = (h < p.H && t < n_rows) ? sq_softplus(__bfloat162float(p.dt[(size_t)(row0 + t) * p.dt_ld + h]) + p.dt_bias[h]) : 0.f;
+    run[k] = h < p.H ? -expf(p.A_log[h]) * 1.4426950408889634f * dt[k] : 0.f;
+  }
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1)
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const float up = __shfl_up_sync(0xffffffffu, run[k], o);
+      if (lane >= o) run[k] += up;
+    }
+  if (lane == 31)
+#pragma unroll
+    for (int k = 0; k < 8; ++k) tot[warp][k] = run[k];
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < 8; ++k) {
+    const float c31 = __shfl_sync(0xffffffffu, run[k], 31);
+    if (h0 + k >= p.H) break;
+    float off = 0.f;
+    for (int w = 0; w < warp; ++w) off += tot[w][k];
+    const float cum = run[k] + off;
+    const size_t at = ((size_t)(row0 / SQ + r + c) * p.H + h0 + k) * SQ + i;
+    p.cum[at] = cum;
+    p.cp[at] = cum - log2f(dt[k]);               // dt 0 (rows past the end): +inf, i.e. no contribution
+    p.g[at] = exp2f(fminf(c31 - run[k], 0.f)) * dt[k];
+  }
 }
 
 __global__ void __launch_bounds__(SQ_THREADS, 1)
@@ -87,24 +152,23 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
   const int g = h / (p.H / p.G);
   const int n = (n_rows + SQ - 1) / SQ;
   const int nch = (p.N + 63) / 64, ksn = (p.N + 15) / 16;          // 64-wide tiles and 16-wide steps of the state size
+  const size_t arr0 = ((size_t)(row0 / SQ + r) * p.H + h) * SQ, arr_step = (size_t)p.H * SQ;
 
   extern __shared__ __align__(1024) uint8_t sq_smem[];
   uint64_t* bars = (uint64_t*)(sq_smem + SQ_BAR);
   uint64_t *full = bars, *empty = bars + 2, *sc_full = bars + 4;   // two each
-  uint64_t *m_full = bars + 6, *cum_full = bars + 7, *w_full = bars + 8, *st_full = bars + 9, *s_full = bars + 10,
-           *yo_done = bars + 11, *y_full = bars + 12, *y_empty = bars + 13;
-  uint32_t* tmem_slot = (uint32_t*)(bars + 14);
+  uint64_t *m_full = bars + 6, *w_full = bars + 7, *st_full = bars + 8, *s_full = bars + 9, *yo_done = bars + 10,
+           *y_full = bars + 11, *y_empty = bars + 12;
+  uint32_t* tmem_slot = (uint32_t*)(bars + 13);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
-  float* cum = reinterpret_cast<float*>(sq_smem + SQ_F);           // log2 units
-  float* gs = cum + SQ;
-  float* dts = gs + SQ;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool aligned = (smem_u32(sq_smem) & 1023) == 0;            // the swizzled tiles need it
   if (threadIdx.x == 0) {
     for (int s = 0; s < 2; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); mbar_init(&sc_full[s], 1); }
-    mbar_init(m_full, 4); mbar_init(cum_full, 4); mbar_init(w_full, 4); mbar_init(st_full, 1);
-    mbar_init(s_full, 4); mbar_init(yo_done, 1); mbar_init(y_full, 1); mbar_init(y_empty, 4);
-    *abort_flag = (smem_u32(sq_smem) & 1023) ? (0x40000000 | (51 << 16)) : 0;      // swizzled tiles need the alignment
+    mbar_init(m_full, 8); mbar_init(w_full, 8); mbar_init(st_full, 1); mbar_init(s_full, 8);
+    mbar_init(yo_done, 1); mbar_init(y_full, 1); mbar_init(y_empty, 8);
+    *abort_flag = aligned ? 0 : (0x40000000 | (51 << 16));
     mbar_fence_init();
   }
   if (warp == 1) {
@@ -115,7 +179,6 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot;
-  const bool aligned = (smem_u32(sq_smem) & 1023) == 0;
 
   if (!aligned) {
     // nothing runs; reported below
@@ -125,12 +188,14 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
         const int s = c & 1, row = row0 + c * SQ;
         if (!mbar_wait(&empty[s], ((c >> 1) & 1) ^ 1, abort_flag, p.status, 51, c)) break;
         uint8_t* st = sq_smem + s * SQ_STAGE;
-        mbar_expect_tx(&full[s], (2 * nch + 1) * SQ_TILE);
+        mbar_expect_tx(&full[s], (2 * nch + 1) * SQ_TILE + 2 * SQ_FB);
         for (int k = 0; k < nch; ++k) {
           tma_load_3d(st + k * SQ_TILE, &tmap_bc, &full[s], k * 64, p.G + g, row);
           tma_load_3d(st + (2 + k) * SQ_TILE, &tmap_bc, &full[s], k * 64, g, row);
         }
         tma_load_3d(st + 4 * SQ_TILE, &tmap_x, &full[s], p0, h, row);
+        sq_bulk_load(sq_smem + SQ_F + s * 2 * SQ_FB, p.cp + arr0 + c * arr_step, SQ_FB, &full[s]);
+        sq_bulk_load(sq_smem + SQ_F + s * 2 * SQ_FB + SQ_FB, p.g + arr0 + c * arr_step, SQ_FB, &full[s]);
       }
     }
   } else if (warp == 1) {
@@ -139,14 +204,16 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
       constexpr uint32_t id_y = umma_idesc(128, 64, 1, 1, 0, 1);
       constexpr uint32_t id_st = umma_idesc(128, 64, 1, 1, 1, 1);
       const uint32_t sbase = smem_u32(sq_smem);
-      auto mn = [&](uint32_t addr, int k) { return umma_desc_mnmajor_sw128(addr + k * 2048, SQ_TILE, 1024); };
+      // 16-wide step k of a tile pair: along the 128-byte rows (K-major), or 16 rows further down (MN-major)
+      auto kd = [](uint32_t tile, int k) { return umma_desc_kmajor_sw128(tile + (k >> 2) * SQ_TILE + (k & 3) * 32); };
+      auto mn = [](uint32_t tile, int k) { return umma_desc_mnmajor_sw128(tile + k * 2048, SQ_TILE, 1024); };
       auto issue_sc = [&](int c) -> bool {
         if (!mbar_wait(&full[c & 1], (c >> 1) & 1, abort_flag, p.status, 52, c)) return false;
         tc_fence_after();
-        const uint32_t cb = sbase + (c & 1) * SQ_STAGE;
-        for (int k = 0; k < ksn; ++k)
-          umma_bf16(tmem + TC_SC + (c & 1) * 128, umma_desc_kmajor_sw128(cb + (k >> 2) * SQ_TILE) + 2 * (k & 3),
-                    umma_desc_kmajor_sw128(cb + (2 + (k >> 2)) * SQ_TILE) + 2 * (k & 3), id_sc, k > 0);
+        const uint32_t cb = sbase + (c & 1) * SQ_STAGE, d = tmem + TC_SC + (c & 1) * 128;
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          if (k < ksn) umma_bf16(d, kd(cb, k), kd(cb + 2 * SQ_TILE, k), id_sc, k > 0);
         umma_commit(&sc_full[c & 1]);
         return true;
       };
@@ -156,19 +223,23 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
         // ---- YO = C S
         if (!mbar_wait(s_full, ph, abort_flag, p.status, 53, c)) { ok = false; break; }
         tc_fence_after();
-        for (int k = 0; k < ksn; ++k) {
-          const uint64_t ad = umma_desc_kmajor_sw128(cb + (k >> 2) * SQ_TILE) + 2 * (k & 3);
-          umma_bf16(tmem + TC_YO + (c & 1) * 64, ad, mn(sbase + SQ_S, k), id_y, k > 0);
-          umma_bf16(tmem + TC_YO + (c & 1) * 64, ad, mn(sbase + SQ_S + SQ_TILE, k), id_y, 1u);
+        {
+          const uint32_t d = tmem + TC_YO + (c & 1) * 64;
+#pragma unroll
+          for (int k = 0; k < 8; ++k)
+            if (k < ksn) {
+              umma_bf16(d, kd(cb, k), mn(sbase + SQ_S, k), id_y, k > 0);
+              umma_bf16(d, kd(cb, k), mn(sbase + SQ_S + SQ_TILE, k), id_y, 1u);
+            }
         }
         umma_commit(yo_done);
         // ---- ST = B^T W
         if (!mbar_wait(w_full, ph, abort_flag, p.status, 54, c)) { ok = false; break; }
         tc_fence_after();
+#pragma unroll
         for (int k = 0; k < 8; ++k) {
-          const uint64_t ad = mn(cb + 2 * SQ_TILE, k);
-          umma_bf16(tmem + TC_ST, ad, mn(sbase + SQ_W, k), id_st, k > 0);
-          umma_bf16(tmem + TC_ST, ad, mn(sbase + SQ_W + SQ_TILE, k), id_st, 1u);
+          umma_bf16(tmem + TC_ST, mn(cb + 2 * SQ_TILE, k), mn(sbase + SQ_W, k), id_st, k > 0);
+          umma_bf16(tmem + TC_ST, mn(cb + 2 * SQ_TILE, k), mn(sbase + SQ_W + SQ_TILE, k), id_st, 1u);
         }
         umma_commit(st_full);
         // ---- the next chunk's scores, while this one's are worked on
@@ -177,42 +248,47 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
         if (!mbar_wait(m_full, ph, abort_flag, p.status, 55, c)) { ok = false; break; }
         if (c > 0 && !mbar_wait(y_empty, (c - 1) & 1, abort_flag, p.status, 56, c)) { ok = false; break; }
         tc_fence_after();
+#pragma unroll
         for (int k = 0; k < 8; ++k) {
-          const uint32_t m = tmem + TC_SC + (c & 1) * 128 + (k >> 1) * 32 + (k & 1) * 8;
-          const uint64_t xd = mn(cb + 4 * SQ_TILE, k);
-          sq_umma_ts(tmem + TC_YD, m, xd, id_y, k > 0);
-          sq_umma_ts(tmem + TC_YD, m + 16, xd, id_y, 1u);
+          const uint32_t m = tmem + TC_SC + (c & 1) * 128 + k * 16;
+          sq_umma_ts(tmem + TC_YD, m, mn(cb + 4 * SQ_TILE, k), id_y, k > 0);
+          sq_umma_ts(tmem + TC_YD, m + 8, mn(cb + 4 * SQ_TILE, k), id_y, 1u);
         }
         umma_commit(y_full);
         umma_commit(&empty[c & 1]);
       }
     }
-  } else if (warp < 6) {
+  } else if (warp < 10) {
     // ------------------------------------------------------------------ scores -> M, output rows
-    const int qd = warp & 3, i = qd * 32 + lane;
+    const int qd = warp & 3, i = qd * 32 + lane, half = (warp - 2) >> 2;
     const uint32_t la = tmem + ((uint32_t)(qd * 32) << 16);
     const float Dh = p.D[h];
+    const float* cumg = p.cum + arr0;
+    float ci = cumg[i], cb[3];                           // this row's sum and those at the ends of the first three blocks
+#pragma unroll
+    for (int b = 0; b < 3; ++b) cb[b] = cumg[b * 32 + 31];
     float e_prev = 0.f;
-    auto output = [&](int c, float e) -> bool {          // rows of chunk c: YD + e YO
+    auto output = [&](int c, float e) -> bool {          // rows of chunk c: YD + e YO, 32 columns
       if (!mbar_wait(y_full, c & 1, abort_flag, p.status, 57, c)) return false;
       tc_fence_after();
       const int t = c * SQ + i;
       __nv_bfloat16* yr = p.y + (size_t)(row0 + t) * p.y_ld + h * p.P + p0;
-#pragma unroll 1
-      for (int q = 0; q < 64; q += 32) {
-        if (q >= pw) break;
-        uint32_t yd[32], yo[32];
-        tmem_ld_x32(la + TC_YD + q, yd);
-        tmem_ld_x32(la + TC_YO + (c & 1) * 64 + q, yo);
-        tmem_ld_wait();
-        if (t < n_rows) {
 #pragma unroll
-          for (int j = 0; j < 32; j += 8) {
-            if (q + j < pw) {
-              float v[8];
+      for (int q0 = 0; q0 < 32; q0 += 16) {
+        const int q = half * 32 + q0;
+        if (q < pw) {
+          uint32_t yd[16], yo[16];
+          __syncwarp();
+          sq_tmem_ld_2x16(la + TC_YD + q, la + TC_YO + (c & 1) * 64 + q, yd, yo);
+          if (t < n_rows) {
 #pragma unroll
-              for (int k = 0; k < 8; ++k) v[k] = fmaf(e, __uint_as_float(yo[j + k]), __uint_as_float(yd[j + k]));
-              store_vec<8>(yr + q + j, v);
+            for (int j = 0; j < 16; j += 8) {
+              if (q + j < pw) {
+                float v[8];
+#pragma unroll
+                for (int k = 0; k < 8; ++k) v[k] = fmaf(e, __uint_as_float(yo[j + k]), __uint_as_float(yd[j + k]));
+                store_vec<8>(yr + q + j, v);
+              }
             }
           }
         }
@@ -224,148 +300,151 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
     };
     bool ok = true;
     for (int c = 0; c < n; ++c) {
-      if (!mbar_wait(cum_full, c & 1, abort_flag, p.status, 58, c) ||
+      const float my = ci, c0 = cb[0], c1 = cb[1], c2 = cb[2];
+      if (c + 1 < n) {                                   // the next chunk's, on their way while this one is worked on
+        const float* nx = cumg + (c + 1) * arr_step;
+        ci = nx[i];
+#pragma unroll
+        for (int b = 0; b < 3; ++b) cb[b] = nx[b * 32 + 31];
+      }
+      if (!mbar_wait(&full[c & 1], (c >> 1) & 1, abort_flag, p.status, 58, c) ||
           !mbar_wait(&sc_full[c & 1], (c >> 1) & 1, abort_flag, p.status, 59, c)) { ok = false; break; }
       tc_fence_after();
-      const float ci = cum[i];
-#pragma unroll 1
+      const float* cps = reinterpret_cast<const float*>(sq_smem + SQ_F + (c & 1) * 2 * SQ_FB) + half * 16;
+      const float* gs = cps + SQ;
+      const uint32_t col0 = la + TC_SC + (c & 1) * 128 + half * 16;
+      uint32_t s[4][16];
+#pragma unroll
       for (int b = 0; b < 4; ++b) {
-        const uint32_t col = la + TC_SC + (c & 1) * 128 + b * 32;
-        uint32_t hi[16], lo[16];
+        if (b == 0) sq_tmem_ld_2x16(col0, col0 + 32, s[0], s[1]);          // blocks right of the diagonal are not used
+        if (b == 2 && qd >= 2) sq_tmem_ld_2x16(col0 + 64, col0 + 96, s[2], s[3]);
+        uint32_t hi[8], lo[8];
         if (b > qd) {                                    // right of the diagonal
 #pragma unroll
-          for (int j = 0; j < 16; ++j) hi[j] = lo[j] = 0u;
+          for (int j = 0; j < 8; ++j) hi[j] = lo[j] = 0u;
+        } else if (b < qd) {
+          const float f = sq_ex2(my - (b == 0 ? c0 : (b == 1 ? c1 : c2)));
+#pragma unroll
+          for (int j = 0; j < 16; j += 4) {
+            const float4 gj = *reinterpret_cast<const float4*>(gs + b * 32 + j);
+            sq_split2(__uint_as_float(s[b][j]) * (f * gj.x), __uint_as_float(s[b][j + 1]) * (f * gj.y), hi[j / 2], lo[j / 2]);
+            sq_split2(__uint_as_float(s[b][j + 2]) * (f * gj.z), __uint_as_float(s[b][j + 3]) * (f * gj.w), hi[j / 2 + 1],
+                      lo[j / 2 + 1]);
+          }
         } else {
-          uint32_t s[32];
-          tmem_ld_x32(col, s);
-          tmem_ld_wait();
-          if (b < qd) {
-            const float f = exp2f(ci - cum[b * 32 + 31]);
+          const int d = lane - half * 16;                // column of the diagonal among these 16
 #pragma unroll
-            for (int j = 0; j < 32; j += 4) {
-              const float4 gj = *reinterpret_cast<const float4*>(gs + b * 32 + j);
-              sq_split2(__uint_as_float(s[j]) * (f * gj.x), __uint_as_float(s[j + 1]) * (f * gj.y), hi[j / 2], lo[j / 2]);
-              sq_split2(__uint_as_float(s[j + 2]) * (f * gj.z), __uint_as_float(s[j + 3]) * (f * gj.w), hi[j / 2 + 1],
-                        lo[j / 2 + 1]);
-            }
-          } else {
+          for (int j = 0; j < 16; j += 4) {
+            const float4 cj = *reinterpret_cast<const float4*>(cps + b * 32 + j);
+            float m[4] = {cj.x, cj.y, cj.z, cj.w};
 #pragma unroll
-            for (int j = 0; j < 32; j += 2) {
-              const float2 cj = *reinterpret_cast<const float2*>(cum + b * 32 + j);
-              const float2 dj = *reinterpret_cast<const float2*>(dts + b * 32 + j);
-              float m0 = j <= lane ? __uint_as_float(s[j]) * (exp2f(fminf(ci - cj.x, 0.f)) * dj.x) : 0.f;
-              float m1 = j + 1 <= lane ? __uint_as_float(s[j + 1]) * (exp2f(fminf(ci - cj.y, 0.f)) * dj.y) : 0.f;
-              if (j == lane) m0 += Dh;
-              if (j + 1 == lane) m1 += Dh;
-              sq_split2(m0, m1, hi[j / 2], lo[j / 2]);
+            for (int e = 0; e < 4; ++e) {
+              m[e] = j + e <= d ? __uint_as_float(s[b][j + e]) * sq_ex2(my - m[e]) : 0.f;
+              if (j + e == d) m[e] += Dh;
             }
+            sq_split2(m[0], m[1], hi[j / 2], lo[j / 2]);
+            sq_split2(m[2], m[3], hi[j / 2 + 1], lo[j / 2 + 1]);
           }
         }
-        tmem_st_x16(col, hi);
-        tmem_st_x16(col + 16, lo);
+        __syncwarp();
+        sq_tmem_st_x8(col0 + b * 32, hi);
+        sq_tmem_st_x8(col0 + b * 32 + 8, lo);
       }
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(m_full);
       if (c > 0 && !output(c - 1, e_prev)) { ok = false; break; }
-      e_prev = exp2f(ci);
+      e_prev = sq_ex2(my);
     }
     if (ok) output(n - 1, e_prev);
   } else {
-    // ------------------------------------------------------------------ decays, W, state
-    const int qd = warp & 3, i = qd * 32 + lane;         // token of the chunk, and row n of the state
+    // ------------------------------------------------------------------ W, state
+    const int qd = warp & 3, i = qd * 32 + lane, half = (warp - 10) >> 2;      // token of the chunk, and row n of the state
     const uint32_t la = tmem + ((uint32_t)(qd * 32) << 16);
-    const float a2 = -expf(p.A_log[h]) * 1.4426950408889634f, bias = p.dt_bias[h];
-    float* st = p.state + (((size_t)slot * p.H + h) * p.P + p0) * p.N + i;
-    const bool fresh = p.positions[row0] == 0, in_n = i < p.N;
-    float S[64];
+    const int q0 = half * 32, kn = i < p.N ? pw - q0 : 0;                      // columns of this half that exist
+    float* st = p.state + (((size_t)slot * p.H + h) * p.P + p0 + q0) * p.N + i;
+    float S[32];
+    {
+      const bool fresh = p.positions[row0] == 0;
 #pragma unroll
-    for (int k = 0; k < 64; ++k) S[k] = (!fresh && in_n && k < pw) ? st[(size_t)k * p.N] : 0.f;
+      for (int k = 0; k < 32; ++k) S[k] = (!fresh && k < kn) ? st[(size_t)k * p.N] : 0.f;
+    }
     auto write_state = [&]() {
 #pragma unroll
-      for (int ch = 0; ch < 8; ++ch) {
-        float v[8];
+      for (int ch = 0; ch < 4; ++ch) {
+        uint32_t hi[4], lo[4];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = S[ch * 8 + e];
-        sq_store8(sq_smem + SQ_S, sq_smem + SQ_S + SQ_TILE, i, ch, v);
+        for (int e = 0; e < 4; ++e) sq_split2(S[ch * 8 + 2 * e], S[ch * 8 + 2 * e + 1], hi[e], lo[e]);
+        uint8_t* d = sq_smem + SQ_S + sq_off(i, half * 4 + ch);
+        *reinterpret_cast<uint4*>(d) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(d + SQ_TILE) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
       fence_proxy_async_smem();
       __syncwarp();
       if (lane == 0) mbar_arrive(s_full);
     };
     write_state();
-    const __nv_bfloat16* dtp = p.dt + (size_t)row0 * p.dt_ld + h;
-    auto load_dt = [&](int c, float (&d)[4]) {           // every warp sees the whole chunk: it needs all four block sums
+    const float* cend_g = p.cum + arr0 + SQ - 1;
+    float cend = cend_g[0], cend_next = 0.f;
+    uint32_t wh[16], wl[16];                             // this token's W of the coming chunk
+    auto prepare = [&](int c, float ce) -> bool {
+      if (!mbar_wait(&full[c & 1], (c >> 1) & 1, abort_flag, p.status, 61, c)) return false;
+      const uint8_t* xt = sq_smem + (c & 1) * SQ_STAGE + 4 * SQ_TILE;
+      uint4 x[4];
 #pragma unroll
-      for (int b = 0; b < 4; ++b) {
-        const int t = c * SQ + b * 32 + lane;
-        d[b] = t < n_rows ? __bfloat162float(dtp[(size_t)t * p.dt_ld]) : 0.f;
-      }
-    };
-    float raw[4];
-    load_dt(0, raw);
-    for (int c = 0; c < n; ++c) {
-      float off = 0.f, cend = 0.f, ci = 0.f, dt = 0.f;
+      for (int ch = 0; ch < 4; ++ch) x[ch] = *reinterpret_cast<const uint4*>(xt + sq_off(i, half * 4 + ch));
+      const float cp = *(reinterpret_cast<const float*>(sq_smem + SQ_F + (c & 1) * 2 * SQ_FB) + i);
+      const float w = sq_ex2(ce - cp);                   // 0 for rows past the end
 #pragma unroll
-      for (int b = 0; b < 4; ++b) {
-        const float d = c * SQ + b * 32 + lane < n_rows ? sq_softplus(raw[b] + bias) : 0.f;
-        float run = a2 * d;
+      for (int ch = 0; ch < 4; ++ch) {
+        const uint32_t v[4] = {x[ch].x, x[ch].y, x[ch].z, x[ch].w};
 #pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-          const float up = __shfl_up_sync(0xffffffffu, run, o);
-          if (lane >= o) run += up;
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v[e]));
+          sq_split2(f.x * w, f.y * w, wh[ch * 4 + e], wl[ch * 4 + e]);
         }
-        if (b == qd) { dt = d; ci = run; off = cend; }
-        cend += __shfl_sync(0xffffffffu, run, 31);
       }
-      ci += off;
-      if (c + 1 < n) load_dt(c + 1, raw);
-      const float c31 = __shfl_sync(0xffffffffu, ci, 31);
-      if (c > 0 && !mbar_wait(m_full, (c - 1) & 1, abort_flag, p.status, 60, c)) break;    // the arrays have been read
-      cum[i] = ci;
-      gs[i] = exp2f(fminf(c31 - ci, 0.f)) * dt;
-      dts[i] = dt;
-      __syncwarp();
-      if (lane == 0) mbar_arrive(cum_full);
-      // ---- W = exp(cum_end - cum) dt x, this token's row
-      if (!mbar_wait(&full[c & 1], (c >> 1) & 1, abort_flag, p.status, 61, c)) break;
-      const float w = exp2f(fminf(cend - ci, 0.f)) * dt;
-      const uint8_t* xr = sq_smem + (c & 1) * SQ_STAGE + 4 * SQ_TILE + i * 128;
-      const bool live = c * SQ + i < n_rows;             // rows past the end hold another request's values
+      return true;
+    };
+    bool ok = prepare(0, cend);
+    for (int c = 0; c < n && ok; ++c) {
+      // W of the chunk before has been read: its ST was waited for
 #pragma unroll
-      for (int ch = 0; ch < 8; ++ch) {
-        float v[8];
-        load_vec<8>(reinterpret_cast<const __nv_bfloat16*>(xr + ((ch ^ (i & 7)) << 4)), v);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = live ? v[e] * w : 0.f;
-        sq_store8(sq_smem + SQ_W, sq_smem + SQ_W + SQ_TILE, i, ch, v);
+      for (int ch = 0; ch < 4; ++ch) {
+        uint8_t* d = sq_smem + SQ_W + sq_off(i, half * 4 + ch);
+        *reinterpret_cast<uint4*>(d) = make_uint4(wh[4 * ch], wh[4 * ch + 1], wh[4 * ch + 2], wh[4 * ch + 3]);
+        *reinterpret_cast<uint4*>(d + SQ_TILE) = make_uint4(wl[4 * ch], wl[4 * ch + 1], wl[4 * ch + 2], wl[4 * ch + 3]);
       }
       fence_proxy_async_smem();
       __syncwarp();
       if (lane == 0) mbar_arrive(w_full);
+      const float eend = sq_ex2(cend);
+      if (c + 1 < n) {
+        cend_next = cend_g[(c + 1) * arr_step];
+        if (!prepare(c + 1, cend_next)) break;
+      }
       // ---- S <- exp(cum_end) S + ST
       if (!mbar_wait(st_full, c & 1, abort_flag, p.status, 62, c)) break;
       tc_fence_after();
-      const float eend = exp2f(cend);
+      {
+        uint32_t v[2][16];
+        __syncwarp();
+        sq_tmem_ld_2x16(la + TC_ST + q0, la + TC_ST + q0 + 16, v[0], v[1]);
 #pragma unroll
-      for (int q = 0; q < 64; q += 16) {
-        uint32_t v[16];
-        tmem_ld_x16(la + TC_ST + q, v);
-        tmem_ld_wait();
-#pragma unroll
-        for (int j = 0; j < 16; ++j) S[q + j] = fmaf(eend, S[q + j], __uint_as_float(v[j]));
+        for (int j = 0; j < 32; ++j) S[j] = fmaf(eend, S[j], __uint_as_float(v[j >> 4][j & 15]));
       }
       tc_fence_before();
       if (c + 1 < n) {
         if (!mbar_wait(yo_done, c & 1, abort_flag, p.status, 63, c)) break;      // C S has read the old state
         write_state();
       }
+      cend = cend_next;
     }
     if (!*abort_flag) {
 #pragma unroll
-      for (int k = 0; k < 64; ++k)
-        if (in_n && k < pw) st[(size_t)k * p.N] = S[k];
+      for (int k = 0; k < 32; ++k)
+        if (k < kn) st[(size_t)k * p.N] = S[k];
     }
   }
 
@@ -386,12 +465,13 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
 
 using namespace omni;
 
-// Arguments as omni_ssm_scan (mamba2.cu); `rows` rows of xbc in all.  Requests with fewer than min_rows rows are not touched.
+// Arguments as omni_ssm_scan (mamba2.cu); `rows` rows of xbc in all, at most max_q of one request.  Requests with fewer than
+// min_rows rows are not touched.  scratch: 3 * (rows / 128 + B) * H * 128 floats.
 extern "C" int omni_ssd_chunks(const void* xbc, int xbc_ld, long long rows, const void* dt, int dt_ld, const void* A_log,
                                const void* dt_bias, const void* D, void* state, const int* cu_q, const int64_t* positions,
-                               const int* state_slots, int B, void* y, int y_ld, int H, int P, int N, int G, int min_rows,
-                               void* status, cudaStream_t stream) {
-  if (B <= 0 || rows <= 0) return 0;
+                               const int* state_slots, int B, int max_q, void* y, int y_ld, int H, int P, int N, int G,
+                               int min_rows, float* scratch, void* status, cudaStream_t stream) {
+  if (B <= 0 || rows <= 0 || max_q < min_rows) return 0;
   if (H < 1 || G < 1 || H % G != 0 || B > 65535 || H > 65535) return -1;
   if (P < 8 || P % 8 != 0 || N < 8 || N % 8 != 0 || N > 128 || xbc_ld % 8 != 0 || y_ld % 8 != 0) return -2;
   if (((uintptr_t)xbc | (uintptr_t)y) % 16 != 0) return -3;
@@ -405,6 +485,9 @@ extern "C" int omni_ssd_chunks(const void* xbc, int xbc_ld, long long rows, cons
   p.D = (const float*)D; p.state = (float*)state; p.cu_q = cu_q; p.positions = positions; p.state_slots = state_slots;
   p.y = (__nv_bfloat16*)y; p.y_ld = y_ld; p.H = H; p.P = P; p.N = N; p.G = G; p.min_rows = min_rows;
   p.status = (OmniStatus*)status;
+  const size_t arr = (size_t)(rows / SQ + B) * H * SQ;
+  p.cum = scratch; p.cp = scratch + arr; p.g = scratch + 2 * arr;
+  ssd_decay_kernel<<<dim3((max_q + SQ - 1) / SQ, B, (H + 7) / 8), SQ, 0, stream>>>(p);
   static bool configured[64] = {false};
   if (int e = ensure_dyn_smem((const void*)ssd_sm100_kernel, SQ_SMEM, configured)) return e;
   ssd_sm100_kernel<<<dim3((P + 63) / 64, H, B), SQ_THREADS, SQ_SMEM, stream>>>(tbc, tx, p);

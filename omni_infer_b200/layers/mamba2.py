@@ -39,7 +39,7 @@ class Mamba2Mixer(nn.Module):
         dt = u[:, s.inner + s.conv_channels:s.inner + s.conv_channels + s.heads]
         y = ssm_scan(xbc, dt, self.A_log, self.dt_bias, self.D, ssm_state, H=s.heads, P=s.vdim,
                      N=s.state, G=s.groups, positions=md.positions, state_slots=md.state_slots, cu_q=cu_q,
-                     min_q=min(md.query_lens) if md.is_prefill else 1)
+                     min_q=min(md.query_lens) if md.is_prefill else 1, max_q=md.max_q)
         return ops.gemm(gated_group_norm(y, u, self.norm_weight, s.norm_groups, self.eps), self.o_proj.weight)
 
     def checkpoint_targets(self):

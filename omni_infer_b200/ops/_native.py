@@ -41,7 +41,7 @@ def use_library(path) -> None:
 
 
 # kernels launched by one call of each entry point (entry points not listed launch one)
-_KERNELS_PER_CALL = {"omni_moe_align": 2}
+_KERNELS_PER_CALL = {"omni_moe_align": 2, "omni_ssd_chunks": 2}
 
 
 class _CountingLib:

@@ -265,10 +265,10 @@ def ssm_scan_ref(xbc, dt, A_log, dt_bias, D, state, positions, state_slots, cu_q
 SSD_MIN_ROWS = 8      # portions below this go token by token: a chunk of the tensor-core form costs as much as some tokens
 
 
-def ssm_scan(xbc, dt, A_log, dt_bias, D, state, *, H, P, N, G, positions, state_slots, cu_q=None, min_q=1, by_rows=False):
+def ssm_scan(xbc, dt, A_log, dt_bias, D, state, *, H, P, N, G, positions, state_slots, cu_q=None, min_q=1, max_q=0, by_rows=False):
     """S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x with dt = softplus(dt + dt_bias), per head; ``xbc`` rows are
     x | B | C, ``dt`` [T, H] (rows of any pitch), ``state`` [slots, H, P, N] fp32.  Requests that start at position 0 start
-    from zeros.  ``min_q``: rows of the shortest request, if known.  ``by_rows``: token by token even where the chunked
+    from zeros.  ``min_q`` / ``max_q``: rows of the shortest / longest request, if known.  ``by_rows``: token by token even where the chunked
     tensor-core forms apply.  -> y [T, pad8(H P)]."""
     T = xbc.shape[0]
     out = torch.empty(T, pad8(H * P), dtype=xbc.dtype, device=xbc.device)
@@ -279,11 +279,12 @@ def ssm_scan(xbc, dt, A_log, dt_bias, D, state, *, H, P, N, G, positions, state_
     max_rows = -1 if by_rows else 0
     if (cu_q is not None and not by_rows and xbc.dtype == torch.bfloat16 and P % 8 == 0 and N % 8 == 0 and N <= 128
             and xbc.stride(0) % 8 == 0 and xbc.data_ptr() % 16 == 0):
+        scratch = torch.empty(3 * (T // 128 + B) * H * 128, dtype=torch.float32, device=xbc.device)
         rc = nat.lib().omni_ssd_chunks(
             nat.ptr(xbc), nat.c_int(xbc.stride(0)), nat.c_int64(T), nat.ptr(dt), nat.c_int(dt.stride(0)), nat.ptr(A_log),
             nat.ptr(dt_bias), nat.ptr(D), nat.ptr(state), nat.ptr(cu_q), nat.ptr(positions), nat.ptr(state_slots),
-            nat.c_int(B), nat.ptr(out), nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N), nat.c_int(G),
-            nat.c_int(SSD_MIN_ROWS), nat.ptr(nat.status_buffer(xbc.device)), nat.stream())
+            nat.c_int(B), nat.c_int(max_q or T), nat.ptr(out), nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N),
+            nat.c_int(G), nat.c_int(SSD_MIN_ROWS), nat.ptr(scratch), nat.ptr(nat.status_buffer(xbc.device)), nat.stream())
         nat.check_rc(rc, "omni_ssd_chunks")
         if min_q >= SSD_MIN_ROWS:
             return out
