@@ -167,7 +167,8 @@ def kernels(out) -> None:
             fl = T * MH * (chunk * P + 4.0 * N * P) + T * MG * chunk * N if pre else 0
             by = T * (C + inner + MH) * 2 + B * MH * P * N * 4 * (1 if pre else 2)
             row(size, what, "ssm_scan", lambda: ll.ssm_scan(xbc, u[:, inner + C:inner + C + MH], A_log, dtb, Dv, ssm_state, H=MH, P=P,
-                                                            N=N, G=MG, positions=p1, state_slots=st, cu_q=cq), by, fl)
+                                                            N=N, G=MG, positions=p1, state_slots=st, cu_q=cq, min_q=T // B,
+                                                            max_q=T // B), by, fl)
             yy, nw = bf(T, inner), torch.ones(inner, device=dev)
             row(size, what, "gated_group_norm", lambda: ll.gated_group_norm(yy, u, nw, c.get("norm_groups", 1), eps), T * inner * 6)
             del u, xbc, yy, kc, vc

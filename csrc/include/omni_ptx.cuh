@@ -362,7 +362,7 @@ __device__ __forceinline__ float warp_sum(float v) {
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
 // tanh form of gelu: 0.5 x (1 + tanh(u)) = x / (1 + exp(-2 u)), u = sqrt(2/pi) (x + 0.044715 x^3)
 __device__ __forceinline__ float gelu_tanh_f(float x) {
-  return x / (1.0f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
+  return __fdividef(x, 1.0f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
 }
 __device__ __forceinline__ uint8_t f32_to_e4m3(float x) {
   return (uint8_t)__nv_cvt_float_to_fp8(x, __NV_SATFINITE, __NV_E4M3);

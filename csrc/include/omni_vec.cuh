@@ -54,17 +54,21 @@ __device__ __forceinline__ float2 block_sum2(float a, float b) {
   return s;
 }
 
-// silu and the tanh form of gelu: exact exponentials for fp32 activations, the fast ones where the result is rounded to
-// bf16 anyway
+// silu and the tanh form of gelu: exact exponentials and divisions for fp32 activations, the fast ones where the result is
+// rounded to bf16 anyway
 template <typename T>
 __device__ __forceinline__ float exp_for(float x) { return expf(x); }
 template <>
 __device__ __forceinline__ float exp_for<__nv_bfloat16>(float x) { return __expf(x); }
 template <typename T>
-__device__ __forceinline__ float silu_for(float x) { return x / (1.0f + exp_for<T>(-x)); }
+__device__ __forceinline__ float div_for(float a, float b) { return a / b; }
+template <>
+__device__ __forceinline__ float div_for<__nv_bfloat16>(float a, float b) { return __fdividef(a, b); }
+template <typename T>
+__device__ __forceinline__ float silu_for(float x) { return div_for<T>(x, 1.0f + exp_for<T>(-x)); }
 template <typename T>
 __device__ __forceinline__ float gelu_tanh_for(float x) {
-  return x / (1.0f + exp_for<T>(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
+  return div_for<T>(x, 1.0f + exp_for<T>(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
 }
 
 }  // namespace omni

@@ -75,7 +75,51 @@ __global__ void conv_silu_kernel(const T* __restrict__ u, int ld, int C, int tap
   store_vec<V>(out + (size_t)row * out_ld + c, acc);
 }
 
-// after conv_silu_kernel: the last taps - 1 inputs of every request go to its slot
+// The same for up to four taps: a thread walks CONV_ROWS rows with the taps' inputs in registers, so that every input is
+// read once.  blockDim (32, 4).
+constexpr int CONV_ROWS = 16;
+template <typename T, int V, int TAPS>
+__global__ void conv_silu_walk_kernel(const T* __restrict__ u, int ld, int C, const float* __restrict__ w,
+                                      const float* __restrict__ bias, const T* __restrict__ state,
+                                      const int64_t* __restrict__ positions, const int* __restrict__ q_to_seq,
+                                      const int* __restrict__ cu_q, const int* __restrict__ state_slots, T* __restrict__ out,
+                                      int out_ld, int rows) {
+  const int t0 = (blockIdx.x * blockDim.y + threadIdx.y) * CONV_ROWS;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (t0 >= rows || c >= C) return;
+  float g[TAPS][V], b[V], x[TAPS][V];      // x[k]: the input TAPS - 1 - k rows back
+#pragma unroll
+  for (int k = 0; k < TAPS; ++k) load_vec<V>(w + (size_t)k * C + c, g[k]);
+  load_vec<V>(bias + c, b);
+  int next_start = t0;                     // first row of the next request (or of this walk): the window is fetched anew
+#pragma unroll 4
+  for (int e = 0; e < CONV_ROWS; ++e) {
+    const int t = t0 + e;
+    if (t >= rows) break;
+    if (t == next_start) {
+      const int r = q_to_seq[t], row0 = cu_q[r];
+      next_start = cu_q[r + 1];
+      const T* st = state + (size_t)max(state_slots[r], 0) * (TAPS - 1) * C;
+      const long long pos = positions[t];
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; ++k) conv_input<T, V>(u, ld, st, TAPS, C, c, t, pos, row0, TAPS - 1 - k, x[k]);
+    }
+    load_vec<V>(u + (size_t)t * ld + c, x[TAPS - 1]);
+    float acc[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      acc[i] = b[i];
+#pragma unroll
+      for (int k = 0; k < TAPS; ++k) acc[i] = fmaf(g[k][i], x[k][i], acc[i]);
+      acc[i] = silu_for<T>(acc[i]);
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; ++k) x[k][i] = x[k + 1][i];
+    }
+    store_vec<V>(out + (size_t)t * out_ld + c, acc);
+  }
+}
+
+// after the convolution of ragged rows: the last taps - 1 inputs of every request go to its slot
 template <typename T, int V>
 __global__ void conv_state_kernel(const T* __restrict__ u, int ld, int C, int taps, T* __restrict__ state,
                                   const int64_t* __restrict__ positions, const int* __restrict__ cu_q,
@@ -680,8 +724,16 @@ static int conv_silu_t(const void* u, int ld, int C, int taps, const float* w, c
                                                                        state_slots, (T*)out, out_ld);
     return (int)cudaGetLastError();
   }
-  conv_silu_kernel<T, V><<<dim3((rows + 7) / 8, (vecs + 31) / 32), dim3(32, 8), 0, st>>>(
-      (const T*)u, ld, C, taps, w, bias, (const T*)state, positions, q_to_seq, cu_q, state_slots, (T*)out, out_ld, rows);
+#define CONV_WALK(TAPS)                                                                                                   \
+  conv_silu_walk_kernel<T, V, TAPS><<<dim3((rows + 4 * CONV_ROWS - 1) / (4 * CONV_ROWS), (vecs + 31) / 32), dim3(32, 4), 0, st>>>( \
+      (const T*)u, ld, C, w, bias, (const T*)state, positions, q_to_seq, cu_q, state_slots, (T*)out, out_ld, rows)
+  if (taps == 2) CONV_WALK(2);
+  else if (taps == 3) CONV_WALK(3);
+  else if (taps == 4) CONV_WALK(4);
+  else
+    conv_silu_kernel<T, V><<<dim3((rows + 7) / 8, (vecs + 31) / 32), dim3(32, 8), 0, st>>>(
+        (const T*)u, ld, C, taps, w, bias, (const T*)state, positions, q_to_seq, cu_q, state_slots, (T*)out, out_ld, rows);
+#undef CONV_WALK
   if (taps > 1)
     conv_state_kernel<T, V><<<dim3(B, (vecs + 127) / 128), 128, 0, st>>>((const T*)u, ld, C, taps, (T*)state, positions, cu_q,
                                                                         state_slots);

@@ -21,7 +21,7 @@ RUNS = [pytest.param("cpu", "float32", id="cpu-float32"), pytest.param("cuda", "
 # largest row error, typical row error.  Rounding to bf16 alone (the CPU references) gives 0.06 and 0.015 here.
 TOL = {"float32": 2e-5, "bfloat16": 0.15}
 TYPICAL = {"float32": 1e-5, "bfloat16": 0.03}
-ONE_LAYER = {"float32": 1e-5, "bfloat16": 0.03}
+ONE_LAYER = {"float32": 1e-5, "bfloat16": 0.1}      # largest row again, rounding alone gives up to 0.05
 
 
 @pytest.fixture(autouse=True)
