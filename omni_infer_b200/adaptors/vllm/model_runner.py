@@ -256,6 +256,8 @@ class ModelRunner:
             return self.cfg.num_kv_blocks
         if self.device.type != "cuda":
             return 256
+        if self.model_cfg.layers is not None and self.model.kv_bytes_per_token() == 0:
+            return self.cfg.max_num_seqs * self._bt_width + 1      # no layer holds pages: blocks only count tokens
         free, total = torch.cuda.mem_get_info(self.device)
         budget = free - int(total * (1.0 - self.cfg.gpu_memory_utilization))
         if self.has_state:

@@ -119,6 +119,22 @@ def test_small_pages_and_wide_pages(device, dtype):
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("layers", [[cases.attention(ff=0), cases.attention(kv_from=0, window=9, ff=24)],
+                                    [cases.mamba(ff=24), cases.mamba(groups=1, conv=2)]], ids=["attention-only", "mamba-only"])
+def test_stacks_of_one_kind(device, dtype, layers):
+    cfg = cases.config(layers)
+    w = cases.weights(cfg, 8)
+    mc = ModelConfig.from_hf_dict(cfg)
+    mc.dtype = dtype
+    eng = EngineCore(EngineConfig(model="x", device=device, block_size=64, max_num_seqs=2, max_model_len=256), model_cfg=mc,
+                     weights=list(w.items()))      # pool sized by the engine
+    toks = tokens(90, 97, 3)
+    got = run(eng, {"a": toks}, [[("a", m)] for m in (40, 2, 1, 1, 46)])["a"]
+    e = row_errors(got, oracle.forward(cfg, w, toks))
+    assert float(e.max()) < TOL[dtype] and float(e.median()) < TYPICAL[dtype]
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
 @pytest.mark.parametrize("decode", [False, True], ids=["prompt", "decoded"])
 def test_token_inside_and_outside_the_window_through_the_model(device, dtype, decode):
     """One attention layer whose queries look for one rare token: the logits follow it to the last place of the window and
