@@ -364,6 +364,12 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   return __fdividef(x, 1.0f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
 }
+// g sigmoid(1.702 g) (u + 1) with g bounded above and u on both sides
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+}
 __device__ __forceinline__ uint8_t f32_to_e4m3(float x) {
   return (uint8_t)__nv_cvt_float_to_fp8(x, __NV_SATFINITE, __NV_E4M3);
 }

@@ -4,7 +4,8 @@
 //
 //   lane = key     32 scores at a time, each lane reads its key row
 //   lane = column  P V, value rows read coalesced
-// Scores, softmax and the accumulation over the values are fp32.
+// Scores, softmax and the accumulation over the values are fp32.  `sink` (per head, may be null): exp(sink) stands in the
+// softmax denominator; `out_scale` multiplies the result before it is rounded.
 #include "../include/omni_vec.cuh"
 
 namespace omni {
@@ -17,7 +18,7 @@ __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
     const T* __restrict__ q, int q_ld, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
     const int64_t* __restrict__ positions, const int* __restrict__ q_to_seq, const int64_t* __restrict__ slots,
     const int* __restrict__ block_table, int bt_ld, int rows, int Hq, int Hkv, int dk, int dv, int block_size, int window,
-    float scale, T* __restrict__ out, int out_ld) {
+    float scale, const float* __restrict__ sink, float out_scale, T* __restrict__ out, int out_ld) {
   extern __shared__ float aa_q[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * AA_WARPS + warp;
@@ -67,19 +68,21 @@ __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
         if (i * 32 + lane < dv) acc[i] = fmaf(pj, to_f32(vr[i * 32 + lane]), acc[i]);
     }
   }
+  if (sink != nullptr) l += expf(sink[h] - m);      // one more term of the denominator, without a value
 #pragma unroll
   for (int i = 0; i < AA_MAXV; ++i)
-    if (i * 32 + lane < dv) orow[i * 32 + lane] = from_f32<T>(acc[i] / l);
+    if (i * 32 + lane < dv) orow[i * 32 + lane] = from_f32<T>(acc[i] / l * out_scale);
 }
 
 template <typename T>
 static int launch_attn_any(const void* q, int q_ld, const void* k, const void* v, const int64_t* positions,
                            const int* q_to_seq, const int64_t* slots, const int* bt, int bt_ld, int rows, int Hq, int Hkv,
-                           int dk, int dv, int block_size, int window, float scale, void* out, int out_ld, cudaStream_t st) {
+                           int dk, int dv, int block_size, int window, float scale, const float* sink, float out_scale, void* out,
+                           int out_ld, cudaStream_t st) {
   const long long items = (long long)rows * Hq;
   attn_any_kernel<T><<<(unsigned)((items + AA_WARPS - 1) / AA_WARPS), AA_WARPS * 32, AA_WARPS * dk * sizeof(float), st>>>(
       (const T*)q, q_ld, (const T*)k, (const T*)v, positions, q_to_seq, slots, bt, bt_ld, rows, Hq, Hkv, dk, dv, block_size,
-      window, scale, (T*)out, out_ld);
+      window, scale, sink, out_scale, (T*)out, out_ld);
   return (int)cudaGetLastError();
 }
 
@@ -89,13 +92,13 @@ using namespace omni;
 
 extern "C" int omni_attn_any(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int64_t* positions,
                              const int* q_to_seq, const int64_t* slots, const int* block_table, int bt_ld, int rows, int Hq,
-                             int Hkv, int dk, int dv, int block_size, int window, float scale, void* out, int out_ld, int f32,
-                             cudaStream_t st) {
+                             int Hkv, int dk, int dv, int block_size, int window, float scale, const float* sink,
+                             float out_scale, void* out, int out_ld, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (Hkv < 1 || Hq % Hkv != 0 || dk < 1 || dk > 2048 || dv < 1 || dv > 32 * AA_MAXV || block_size < 1 || window < 0) return -1;
   if (f32)
     return launch_attn_any<float>(q, q_ld, k_cache, v_cache, positions, q_to_seq, slots, block_table, bt_ld, rows, Hq, Hkv, dk,
-                                  dv, block_size, window, scale, out, out_ld, st);
+                                  dv, block_size, window, scale, sink, out_scale, out, out_ld, st);
   return launch_attn_any<__nv_bfloat16>(q, q_ld, k_cache, v_cache, positions, q_to_seq, slots, block_table, bt_ld, rows, Hq,
-                                        Hkv, dk, dv, block_size, window, scale, out, out_ld, st);
+                                        Hkv, dk, dv, block_size, window, scale, sink, out_scale, out, out_ld, st);
 }

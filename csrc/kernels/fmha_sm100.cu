@@ -10,7 +10,8 @@
 // omni_fmha_paged: the same kernel reading K and V tiles from the paged cache through the block table (any head sizes
 // up to 192 / 128 that are multiples of 8: the tensor maps are [rows, heads, head size], so a partial 64-wide chunk is
 // zero-filled), with an optional sliding window - key tiles outside every query's window are never loaded - and with the
-// softmax weights carried as a pair of bf16 values (p = hi + lo, two MMAs), i.e. to 16 bits of mantissa.
+// softmax weights carried as a pair of bf16 values (p = hi + lo, two MMAs), i.e. to 16 bits of mantissa; optionally a sink per
+// head in the softmax denominator and a factor on the result.
 // Causal mask is aligned to the end of the key range (query i of a request with Lq queries and Lk keys sees
 // keys <= Lk - Lq + i), which also covers chunked prefill and prefix-cache hits.
 //
@@ -39,6 +40,8 @@ struct FmhaParams {
   const int* block_table;
   int bt_ld, block_size;
   int window;          // a query sees the last `window` keys up to its own; 0 = all
+  const float* sink;   // [Hq] or null: exp(sink) is one more term of the softmax denominator
+  float out_scale;     // multiplies the result before it is rounded
   OmniStatus* status;
 };
 
@@ -284,7 +287,9 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     if (ok) {
       tc_fence_after();
       const bool row_ok = (q0 + row) < Lq;
-      const float inv_l = l > 0.f ? 1.0f / l : 0.f;
+      float den = l;
+      if (PAGED && p.sink != nullptr && m != -INFINITY) den += exp2f(p.sink[h] * 1.4426950408889634f - m);
+      const float inv_l = l > 0.f ? (PAGED ? p.out_scale : 1.0f) / den : 0.f;
       __nv_bfloat16* orow = p.out + (size_t)(q_begin + q0 + row) * p.out_ld + h * p.dv;
 #pragma unroll 1
       for (int c = 0; c < p.dv; c += 32) {
@@ -358,6 +363,7 @@ extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q
   p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = FM_DV; p.out_ld = Hq * FM_DV;
   p.kv_len = nullptr; p.block_table = nullptr; p.bt_ld = 0; p.block_size = 0; p.window = 0;
+  p.sink = nullptr; p.out_scale = 1.0f;
   return launch_fmha<false, FM_MAXC, 3>(dim3((max_q + FM_BQ - 1) / FM_BQ, B, Hq), tq, tk, tk2, tv, p, stream);
 }
 
@@ -366,7 +372,7 @@ extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q
 extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const void* k_cache, const void* v_cache,
                                long long slots, const int* cu_q, const int* kv_len, const int* block_table, int bt_ld, int B,
                                int max_q, int Hq, int Hkv, int d_k, int d_v, int block_size, int window, float scale,
-                               void* out, int out_ld, void* status, cudaStream_t stream) {
+                               const float* sink, float out_scale, void* out, int out_ld, void* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (d_k < 8 || d_v < 8 || d_k % 8 != 0 || d_v % 8 != 0 || d_k > 64 * FM_MAXC || d_v > FM_DV) return -1;
   if (Hkv < 1 || Hq % Hkv != 0 || B > 65535 || Hq > 65535 || window < 0) return -2;
@@ -383,7 +389,7 @@ extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const 
   p.cu_q = cu_q; p.Hq = Hq; p.Hkv = Hkv; p.nk1 = (d_k + 63) / 64; p.nk2 = 0;
   p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = d_v; p.out_ld = out_ld; p.kv_len = kv_len; p.block_table = block_table; p.bt_ld = bt_ld;
-  p.block_size = block_size; p.window = window;
+  p.block_size = block_size; p.window = window; p.sink = sink; p.out_scale = out_scale;
   const dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
   if (p.nk1 <= 2) return launch_fmha<true, 2, 2>(grid, tq, tk, tk, tv, p, stream);
   return launch_fmha<true, FM_MAXC, 3>(grid, tq, tk, tk, tv, p, stream);

@@ -26,6 +26,7 @@
 //   EPI   0 = store (optional per-row multiplier, bf16 or fp32 output)
 //         1 = SwiGLU: silu(gate) * up -> bf16
 //         3 = gelu(gate) * up -> bf16, gelu in its tanh form (bf16 operands only)
+//         4 = clamped gate: g = min(gate, limit), u = clamp(up, +-limit), g sigmoid(1.702 g) (u + 1) -> bf16 (bf16 operands)
 //         2 = SwiGLU then e4m3 quantisation with one scale per (row, 128 output features);
 //             the 128 accumulator lanes of a tile are exactly one quantisation block.
 //
@@ -56,6 +57,7 @@ struct GemmParams {
   float* out_scale;      // EPI 2: [n_out/128, out_scale_ld]
   int out_scale_ld;
   const float* row_scale;  // optional [rows]
+  float glu_limit;         // EPI 4: bound of gate and up
   int x_group_col;       // head-batched mode: group g reads X columns [g*x_group_col, +K) ...
   int out_group_col;     // ... and writes out columns [g*out_group_col, +n_out)
   int k_splits;          // > 1: the K range is cut into k_splits parts that different CTAs accumulate into a
@@ -457,13 +459,14 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const float g = __uint_as_float(vg[j]);
-              act[j] = (EPI == 3 ? gelu_tanh_f(g) : silu_f(g)) * __uint_as_float(vu[j]);
+              const float u = __uint_as_float(vu[j]);
+              act[j] = EPI == 4 ? clamped_glu_f(g, u, p.glu_limit) : (EPI == 3 ? gelu_tanh_f(g) : silu_f(g)) * u;
             }
           } else {
 #pragma unroll
             for (int j = 0; j < 16; ++j) act[j] = silu_f(accv(0, c0 + j)) * accv(NACC - 1, c0 + j);
           }
-          if (EPI == 1 || EPI == 3) {
+          if (EPI == 1 || EPI == 3 || EPI == 4) {
             if (c_lo + c0 < rows && n_ok) {
 #pragma unroll
               for (int j = 0; j < 16; ++j)
@@ -556,7 +559,7 @@ static int launch_gemm(const CUtensorMap& tw, const CUtensorMap& tx, const GemmP
 using namespace omni;
 
 
-// kind: 0 bf16, 1 fp8 block-scaled.  epi: 0 store, 1 swiglu->bf16, 2 swiglu->fp8+scales, 3 geglu->bf16.
+// kind: 0 bf16, 1 fp8 block-scaled.  epi: 0 store, 1 swiglu->bf16, 2 swiglu->fp8+scales, 3 geglu->bf16, 4 clamped glu->bf16 (bound glu_limit).
 // bn: token tile (16, 32, 64, 128, 256); 0 picks from `t_hint` (expected rows per group).
 // x_rows: number of addressable rows of X (and of `out`); rows beyond it read as zero.
 // Returns 0 on success, a negative value for bad arguments, a positive CUDA error otherwise.
@@ -564,7 +567,7 @@ extern "C" int omni_gemm(int kind, int epi, const void* w, const void* x, void* 
                          int x_rows, int T, const int* seg_start, const int* seg_len, const float* w_scale,
                          const float* x_scale, int x_scale_ld, int out_ld, int out_f32, float* out_scale,
                          int out_scale_ld, const float* row_scale, int x_group_col, int out_group_col, int x_ld,
-                         int bn, int t_hint, void* status, cudaStream_t stream) {
+                         int bn, int t_hint, float glu_limit, void* status, cudaStream_t stream) {
   if (G < 1 || G > MAX_GROUPS || n_out < 1 || K < 1) return -1;
   const int nacc = (epi == 0) ? 1 : 2;
   const int esz = (kind == 0) ? 2 : 1;
@@ -607,7 +610,7 @@ extern "C" int omni_gemm(int kind, int epi, const void* w, const void* x, void* 
   p.w_rows_per_group = n_out * nacc; p.w_scale = w_scale; p.x_scale = x_scale; p.x_scale_ld = x_scale_ld;
   p.out = out; p.out_ld = out_ld; p.out_f32 = out_f32; p.out_scale = out_scale; p.out_scale_ld = out_scale_ld;
   p.row_scale = row_scale; p.x_group_col = x_group_col; p.out_group_col = out_group_col;
-  p.status = (OmniStatus*)status;
+  p.status = (OmniStatus*)status; p.glu_limit = glu_limit;
   if (x_ld <= 0) x_ld = K;
   const uint64_t x_cols = x_group_col > 0 ? (uint64_t)x_ld : (uint64_t)K;
 
@@ -622,6 +625,7 @@ extern "C" int omni_gemm(int kind, int epi, const void* w, const void* x, void* 
   if (kind == KIND_ && bn == BN_ && epi == EPI_) return launch_gemm<KIND_, BN_, NACC_, EPI_>(tw, tx, p, grid, stream);
   OMNI_GEMM_CASE(0, 32, 1, 0) OMNI_GEMM_CASE(0, 64, 1, 0) OMNI_GEMM_CASE(0, 128, 1, 0) OMNI_GEMM_CASE(0, 256, 1, 0)
   OMNI_GEMM_CASE(0, 32, 2, 1) OMNI_GEMM_CASE(0, 64, 2, 1) OMNI_GEMM_CASE(0, 128, 2, 1)
+  OMNI_GEMM_CASE(0, 32, 2, 4) OMNI_GEMM_CASE(0, 64, 2, 4) OMNI_GEMM_CASE(0, 128, 2, 4)
   OMNI_GEMM_CASE(0, 32, 2, 3) OMNI_GEMM_CASE(0, 64, 2, 3) OMNI_GEMM_CASE(0, 128, 2, 3)
   OMNI_GEMM_CASE(1, 32, 1, 0) OMNI_GEMM_CASE(1, 64, 1, 0) OMNI_GEMM_CASE(1, 128, 1, 0)
   OMNI_GEMM_CASE(1, 32, 2, 1) OMNI_GEMM_CASE(1, 64, 2, 1)

@@ -25,7 +25,7 @@
 // The 256 weight rows of a tile are two blocks of 128 (each with its own weight scale).  EPI 0 = store: the
 // blocks are consecutive output features (bf16 or fp32 output, optional per-row multiplier).  EPI 1 / 2 =
 // SwiGLU: W holds n_out gate rows, then n_out up rows, per group; block 0 is 128 gate rows, block 1 the
-// matching up rows, and the tile produces 128 output features: EPI 1 -> bf16 (EPI 3: the same with gelu), EPI 2 -> e4m3 with one scale
+// matching up rows, and the tile produces 128 output features: EPI 1 -> bf16 (EPI 3: the same with gelu, EPI 4: the clamped gate), EPI 2 -> e4m3 with one scale
 // per token and 128 output features (exactly one tile).
 //
 // KIND 0 = bf16 operands: the whole K range accumulates in TMEM and the epilogue runs once per tile.
@@ -68,6 +68,7 @@ struct TmGemmParams {
   float* out_scale;      // EPI 2: [n_out/128, out_scale_ld]
   int out_scale_ld;
   const float* row_scale;  // optional [rows]
+  float glu_limit;         // EPI 4: bound of gate and up
   int x_group_col;       // head-batched mode: group g reads X columns [g*x_group_col, +K) ...
   int out_group_col;     // ... and writes out columns [g*out_group_col, +n_out)
   // reduce-scatter epilogue (rs_world > 1): out is ignored, rows go to rs_out[row / rs_rows_per_rank]
@@ -489,11 +490,13 @@ gemm_tokmajor_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_co
         float amax = 0.f;
 #pragma unroll
         for (int j = 0; j < TM_CW / 2; ++j) {
-          acc[0][j].x = (EPI == 3 ? gelu_tanh_f(acc[0][j].x) : silu_f(acc[0][j].x)) * acc[NB - 1][j].x;
-          acc[0][j].y = (EPI == 3 ? gelu_tanh_f(acc[0][j].y) : silu_f(acc[0][j].y)) * acc[NB - 1][j].y;
+          acc[0][j].x = EPI == 4 ? clamped_glu_f(acc[0][j].x, acc[NB - 1][j].x, p.glu_limit)
+                                  : (EPI == 3 ? gelu_tanh_f(acc[0][j].x) : silu_f(acc[0][j].x)) * acc[NB - 1][j].x;
+          acc[0][j].y = EPI == 4 ? clamped_glu_f(acc[0][j].y, acc[NB - 1][j].y, p.glu_limit)
+                                  : (EPI == 3 ? gelu_tanh_f(acc[0][j].y) : silu_f(acc[0][j].y)) * acc[NB - 1][j].y;
           amax = fmaxf(amax, fmaxf(fabsf(acc[0][j].x), fabsf(acc[0][j].y)));
         }
-        if (EPI == 1 || EPI == 3) {
+        if (EPI == 1 || EPI == 3 || EPI == 4) {
           if (row_ok) {
             __nv_bfloat16* o = (__nv_bfloat16*)p.out + row * p.out_ld + n0;
             const bool wide = ((uintptr_t)o & 31) == 0;
@@ -622,7 +625,7 @@ extern "C" int omni_gemm_tm2(int kind, int epi, const void* w, const void* x, vo
                              int T, const int* seg_start, const int* seg_len, const float* w_scale, const float* x_scale,
                              int x_scale_ld, int out_ld, int out_f32, float* out_scale, int out_scale_ld,
                              const float* row_scale, int x_group_col, int out_group_col, int x_ld,
-                             const OmniTmCollective* coll, void* status, cudaStream_t stream) {
+                             float glu_limit, const OmniTmCollective* coll, void* status, cudaStream_t stream) {
   if (G < 1 || G > TM_MAX_GROUPS || n_out < 1 || K < 1) return -1;
   if (kind != 0 && kind != 1) return -1;
   const int nb = (epi == 0) ? 1 : 2;
@@ -633,14 +636,14 @@ extern "C" int omni_gemm_tm2(int kind, int epi, const void* w, const void* x, vo
   if (kind == 1 && ((x_scale_ld % 4) != 0 || ((uintptr_t)x_scale % 16) != 0)) return -7;
   if (epi == 2 && (out_scale == nullptr || kind != 1)) return -5;
   if ((n_out % 8) != 0 || (out_ld % 8) != 0 || (out_group_col % 8) != 0) return -8;
-  if (epi < 0 || epi > 3 || (epi == 3 && kind != 0)) return -9;
+  if (epi < 0 || epi > 4 || (epi >= 3 && kind != 0)) return -9;
   TmGemmParams p;
   memset(&p, 0, sizeof(p));
   p.G = G; p.n_out = n_out; p.K = K; p.T = T; p.seg_start = seg_start; p.seg_len = seg_len;
   p.w_rows_per_group = n_out * nb; p.w_scale = w_scale; p.x_scale = x_scale; p.x_scale_ld = x_scale_ld;
   p.out = out; p.out_ld = out_ld; p.out_f32 = out_f32; p.out_scale = out_scale; p.out_scale_ld = out_scale_ld;
   p.row_scale = row_scale; p.x_group_col = x_group_col; p.out_group_col = out_group_col; p.status = (OmniStatus*)status;
-  p.rs_world = 1; p.ag_world = 1;
+  p.rs_world = 1; p.ag_world = 1; p.glu_limit = glu_limit;
   if (coll != nullptr) {
     if (coll->rs_world > 1) {
       if (coll->rs_world > 8 || epi != 0 || out_f32 || G != 1 || seg_len != nullptr || coll->rs_rows_per_rank < 1) return -12;
@@ -673,6 +676,7 @@ extern "C" int omni_gemm_tm2(int kind, int epi, const void* w, const void* x, vo
     if (epi == 0) return launch_tm<0, 0>(tx, tw, p, grid, stream);
     if (epi == 1) return launch_tm<0, 1>(tx, tw, p, grid, stream);
     if (epi == 3) return launch_tm<0, 3>(tx, tw, p, grid, stream);
+    if (epi == 4) return launch_tm<0, 4>(tx, tw, p, grid, stream);
     return -9;
   }
   if (epi == 0) return launch_tm<1, 0>(tx, tw, p, grid, stream);

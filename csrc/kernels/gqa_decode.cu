@@ -49,6 +49,8 @@ struct GqSmem {
 
 struct GqShape {           // used by the general form only
   int q_ld, out_ld, dk, dv, window;
+  const float* sink;       // [Hq] or null: exp(sink) is one more term of the softmax denominator
+  float out_scale;         // multiplies the result before it is rounded
 };
 
 __device__ __forceinline__ uint32_t gq_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -284,7 +286,9 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
     }
     const int hq = hk * Gall + g0 + g;
     if (splits == 1) {
-      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+      float den = ll;
+      if (GEN && sh.sink != nullptr && ll > 0.f) den += exp2f(sh.sink[hq] * 1.4426950408889634f - mm);
+      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / den * (GEN ? sh.out_scale : 1.f) : 0.f);
     } else {
       o_part[(((size_t)b * splits + split) * Hq + hq) * dv + d] = ll > 0.f ? acc / ll : 0.f;
       if (d == 0) lse_part[((size_t)b * splits + split) * Hq + hq] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
@@ -293,7 +297,8 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 }
 
 __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part, int splits,
-                                   int Hq, int dv, int out_ld, __nv_bfloat16* out) {
+                                   int Hq, int dv, int out_ld, const float* __restrict__ sink, float out_scale,
+                                   __nv_bfloat16* out) {
   const int bh = blockIdx.x;
   const int b = bh / Hq, h = bh - b * Hq;
   const int d = threadIdx.x;
@@ -308,7 +313,8 @@ __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float
     den += w;
     acc += w * o_part[(((size_t)b * splits + s) * Hq + h) * dv + d];
   }
-  out[(size_t)b * out_ld + h * dv + d] = __float2bfloat16(den > 0.f ? acc / den : 0.f);
+  if (sink != nullptr && den > 0.f) den += exp2f(sink[h] * 1.4426950408889634f - mx);
+  out[(size_t)b * out_ld + h * dv + d] = __float2bfloat16(den > 0.f ? acc / den * out_scale : 0.f);
 }
 
 }  // namespace omni
@@ -334,8 +340,8 @@ static int launch_gqa(dim3 grid, const void* q, const void* k_cache, const void*
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   if (splits > 1) {
-    gqa_combine_kernel<<<B * Hq, (dv + 31) / 32 * 32, 0, stream>>>(o_part, lse_part, splits, Hq, dv, out_ld,
-                                                                   (__nv_bfloat16*)out);
+    gqa_combine_kernel<<<B * Hq, (dv + 31) / 32 * 32, 0, stream>>>(o_part, lse_part, splits, Hq, dv, out_ld, sh.sink,
+                                                                   sh.out_scale, (__nv_bfloat16*)out);
     e = cudaGetLastError();
   }
   return (int)e;
@@ -349,6 +355,7 @@ extern "C" int omni_gqa_paged_decode(const void* q, const void* k_cache, const v
   if (D != GQ_D || Hq % Hkv != 0 || Hq / Hkv > 16 || splits < 1) return -1;
   if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;
   GqShape sh = {};
+  sh.out_scale = 1.f;
   return launch_gqa<GQ_D, false>(dim3(Hkv, splits, B), q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq,
                                  Hkv, scale, splits, o_part, lse_part, out, sh, GQ_D, Hq * GQ_D, stream);
 }
@@ -356,14 +363,14 @@ extern "C" int omni_gqa_paged_decode(const void* q, const void* k_cache, const v
 // General form: q rows of pitch q_ld, key size dk, value size dv, out rows of pitch out_ld, window 0 = all keys.
 extern "C" int omni_gqa_paged_decode_window(const void* q, int q_ld, const void* k_cache, const void* v_cache,
                                             const int* block_table, int bt_ld, const int* seq_lens, int B, int Hq, int Hkv,
-                                            int dk, int dv, int block_size, int window, float scale, int splits,
-                                            float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
+                                            int dk, int dv, int block_size, int window, float scale, const float* sink,
+                                            float out_scale, int splits, float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (Hkv < 1 || Hq % Hkv != 0 || splits < 1 || splits > 65535 || B > 65535 || window < 0) return -1;
   if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;
   if (dk < 8 || dv < 8 || dk % 8 != 0 || dv % 8 != 0 || dk > 256 || dv > 256) return -3;
   if (q_ld % 8 != 0 || ((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16 != 0) return -4;
-  const GqShape sh = {q_ld, out_ld, dk, dv, window};
+  const GqShape sh = {q_ld, out_ld, dk, dv, window, sink, out_scale};
   const dim3 grid(Hkv * ((Hq / Hkv + 15) / 16), splits, B);
   const int d = dk > dv ? dk : dv;
 #define GQA_CASE(DP)                                                                                                     \

@@ -10,6 +10,7 @@
 // planner remap (omni/accelerators/placement/omni_planner/omni_planner.py:244-274) and the
 // init_routing / finalize_routing pair (fused_moe.py:109-186).
 #include "../include/omni_ptx.cuh"
+#include "../include/omni_vec.cuh"
 
 namespace omni {
 
@@ -72,7 +73,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const RouterParams p) 
 #pragma unroll
     for (int i = 0; i < ROUTER_MAX_PER_LANE; ++i) {
       const int e = i * 32 + lane;
-      score[i] = (i < per_lane && e < p.E) ? __expf(score[i] - mx) : 0.f;
+      score[i] = (i < per_lane && e < p.E) ? expf(score[i] - mx) : 0.f;
       s += score[i];
     }
     s = warp_sum(s);
@@ -201,6 +202,28 @@ __global__ void moe_prefix_kernel(const int* __restrict__ counts, int e_local, i
     }
     *total_rows = acc;
   }
+}
+
+// fp32 rows: one warp per (t,k)
+__global__ void moe_scatter_f32_kernel(const float* __restrict__ x, int H, const int* __restrict__ ids,
+                                       const float* __restrict__ w, const int* __restrict__ pos, int n, int top_k, int e_lo,
+                                       const int* __restrict__ seg_start, const int* __restrict__ seg_len, float* xp,
+                                       int* row_of, float* row_w) {
+  const int i = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  const int lane = threadIdx.x & 31;
+  if (i >= n) return;
+  const int ps = pos[i];
+  const int e = ids[i] - e_lo;
+  if (ps < 0 || ps >= seg_len[e]) {
+    if (lane == 0) row_of[i] = -1;
+    return;
+  }
+  const int row = seg_start[e] + ps;
+  if (lane == 0) {
+    row_of[i] = row;
+    row_w[row] = w[i];
+  }
+  for (int c = lane; c < H; c += 32) xp[(size_t)row * H + c] = x[(size_t)(i / top_k) * H + c];
 }
 
 // one warp per (t,k): copy / quantise the token row into its expert-sorted slot
@@ -362,6 +385,16 @@ extern "C" int omni_moe_scatter(const void* x, int H, const int* ids, const floa
   moe_scatter_kernel<<<(int)((threads + 255) / 256), 256, 0, stream>>>(
       (const __nv_bfloat16*)x, H, ids, w, pos, n, top_k, e_lo, seg_start, seg_len, (__nv_bfloat16*)xp, (uint8_t*)xq,
       xs, xs_ld, row_of, row_w, src_of);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_moe_scatter_f32(const void* x, int H, const int* ids, const float* w, const int* pos, int n, int top_k, int e_lo,
+                                    const int* seg_start, const int* seg_len, void* xp, int* row_of, float* row_w,
+                                    cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const long long threads = (long long)n * 32;
+  moe_scatter_f32_kernel<<<(int)((threads + 255) / 256), 256, 0, stream>>>(
+      (const float*)x, H, ids, w, pos, n, top_k, e_lo, seg_start, seg_len, (float*)xp, row_of, row_w);
   return (int)cudaGetLastError();
 }
 

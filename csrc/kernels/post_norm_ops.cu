@@ -2,10 +2,10 @@
 //   omni_embed_residual      embedding gather -> fp32 residual and its activation copy (the first sublayer's input)
 //   omni_post_norm_add       residual += rmsnorm(sublayer output) * w, and the activation copy for the next sublayer
 //   omni_rmsnorm_residual    final norm: fp32 residual -> activations
-//   omni_qk_norm_rope_cache  RMSNorm over the whole q and the whole k projection, rotate-half RoPE on the first
+//   omni_qk_norm_rope_cache  optional RMSNorm over the whole q and the whole k projection, rotate-half RoPE on the first
 //                            dimensions of every head, K/V scatter into the paged cache
-//   omni_gelu_mul            gelu(gate) * up for widths the GEMM epilogue does not take
-//   omni_gemm_f32            plain fp32 matrix product (fp32 runs of a model)
+//   omni_gated_mul           gelu(gate) * up, or the clamped form, for widths the GEMM epilogue does not take
+//   omni_gemm_f32            plain fp32 matrix products: dense, by row segments, or by column groups (fp32 runs of a model)
 // Activations are bf16 or fp32 (`f32` argument).  Rows have a pitch (`ld`, elements) that may exceed their width: the
 // padding columns of an output are written as zeros so that it can be a TMA operand of the next GEMM.  Norm weights are
 // fp32.  Every value between two roundings to the activation type is fp32.
@@ -103,7 +103,7 @@ __global__ void rmsnorm_residual_kernel(const float* __restrict__ x, const float
   for (int c = H + threadIdx.x; c < ld; c += blockDim.x) out[(size_t)t * ld + c] = from_f32<T>(0.f);
 }
 
-// One CTA per token, one warp per head.  q rows are normed and rotated in place, k rows go to the cache the same way,
+// One CTA per token, one warp per head.  q rows are normed (qw null: not) and rotated in place, k rows go to the cache the same way,
 // v rows are copied.  Hkv = 0: the layer reads another layer's cache and has q rows only.
 template <typename T, int V>
 __global__ void qk_norm_rope_cache_kernel(T* __restrict__ qkv, int ld, int Hq, int Hkv, int D, int DV,
@@ -115,8 +115,9 @@ __global__ void qk_norm_rope_cache_kernel(T* __restrict__ qkv, int ld, int Hq, i
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
   T* row = qkv + (size_t)t * ld;
   const int nq = Hq * D, nk = Hkv * D;
+  const bool normed = qw != nullptr;
   float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+  for (int c = threadIdx.x * V; normed && c < nq + nk; c += blockDim.x * V) {
     float v[V];
     load_vec<V>(row + c, v);
     float s = 0.f;
@@ -124,9 +125,12 @@ __global__ void qk_norm_rope_cache_kernel(T* __restrict__ qkv, int ld, int Hq, i
     for (int i = 0; i < V; ++i) s += v[i] * v[i];
     if (c < nq) sq += s; else sk += s;
   }
-  const float2 tot = block_sum2(sq, sk);
-  const float rq = 1.0f / sqrtf(tot.x / (float)nq + eps);
-  const float rk = nk > 0 ? 1.0f / sqrtf(tot.y / (float)nk + eps) : 0.f;
+  float rq = 1.0f, rk = 1.0f;
+  if (normed) {
+    const float2 tot = block_sum2(sq, sk);
+    rq = 1.0f / sqrtf(tot.x / (float)nq + eps);
+    rk = nk > 0 ? 1.0f / sqrtf(tot.y / (float)nk + eps) : 0.f;
+  }
   const int64_t slot = slots[t];
   const int half = rot >> 1;
   const float* cs = cos_sin + (size_t)positions[t] * rot;
@@ -135,24 +139,29 @@ __global__ void qk_norm_rope_cache_kernel(T* __restrict__ qkv, int ld, int Hq, i
     const T* src = row + (size_t)hd * D;
     T* dst = is_q ? row + (size_t)hd * D : k_cache + ((size_t)slot * Hkv + (hd - Hq)) * D;
     if (!is_q && slot < 0) continue;
-    const float* w = is_q ? qw + (size_t)hd * D : kw + (size_t)(hd - Hq) * D;
+    const float* w = !normed ? nullptr : (is_q ? qw + (size_t)hd * D : kw + (size_t)(hd - Hq) * D);
     const float r = is_q ? rq : rk;
     for (int c = lane * V; c < D; c += 32 * V) {
       if (c >= half && c < rot) continue;      // written together with its partner
       float a[V], wa[V];
       load_vec<V>(src + c, a);
-      load_vec<V>(w + c, wa);
+      if (normed) {
+        load_vec<V>(w + c, wa);
 #pragma unroll
-      for (int i = 0; i < V; ++i) a[i] = a[i] * r * wa[i];
+        for (int i = 0; i < V; ++i) a[i] = a[i] * r * wa[i];
+      }
       if (c < half) {
         float b[V], wb[V], co[V], si[V];
         load_vec<V>(src + c + half, b);
-        load_vec<V>(w + c + half, wb);
+        if (normed) {
+          load_vec<V>(w + c + half, wb);
+#pragma unroll
+          for (int i = 0; i < V; ++i) b[i] = b[i] * r * wb[i];
+        }
         load_vec<V>(cs + c, co);
         load_vec<V>(cs + half + c, si);
 #pragma unroll
         for (int i = 0; i < V; ++i) {
-          b[i] = b[i] * r * wb[i];
           const float u = a[i];
           a[i] = u * co[i] - b[i] * si[i];
           b[i] = b[i] * co[i] + u * si[i];
@@ -170,9 +179,10 @@ __global__ void qk_norm_rope_cache_kernel(T* __restrict__ qkv, int ld, int Hq, i
   }
 }
 
-template <typename T, int V>
-__global__ void gelu_mul_kernel(const T* __restrict__ x, int x_ld, int up_off, T* __restrict__ out, int out_ld, int T_rows,
-                                int I) {
+// KIND 0: gelu(g) u, 1: min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1)
+template <typename T, int V, int KIND>
+__global__ void gated_mul_kernel(const T* __restrict__ x, int x_ld, int up_off, T* __restrict__ out, int out_ld, int T_rows,
+                                 int I, float limit) {
   const int row = blockIdx.y;
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (c >= out_ld) return;
@@ -184,26 +194,46 @@ __global__ void gelu_mul_kernel(const T* __restrict__ x, int x_ld, int up_off, T
     load_vec<V>(x + (size_t)row * x_ld + c, g);
     load_vec<V>(x + (size_t)row * x_ld + up_off + c, u);
 #pragma unroll
-    for (int i = 0; i < V; ++i) o[i] = gelu_tanh_for<T>(g[i]) * u[i];
+    for (int i = 0; i < V; ++i) {
+      if (KIND == 0) {
+        o[i] = gelu_tanh_for<T>(g[i]) * u[i];
+      } else {
+        const float gc = fminf(g[i], limit);
+        o[i] = div_for<T>(gc, 1.0f + exp_for<T>(-1.702f * gc)) * (fminf(fmaxf(u[i], -limit), limit) + 1.0f);
+      }
+    }
   }
   store_vec<V>(out + (size_t)row * out_ld + c, o);
 }
 
-// out[t, n] = sum_k x[t, k] w[n, k].  64 x 64 tile per CTA, 16 k per step, 4 x 4 outputs per thread.
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w,
-                                                       float* __restrict__ out, int T, int N, int K, int x_ld, int w_ld,
-                                                       int out_ld) {
-  __shared__ float xs[16][68], ws[16][68];
+struct GemmF32Params {
+  const float *x, *w;
+  float* out;
+  int T, N, K, x_ld, out_ld;
+  const int *seg_start, *seg_len;      // [G] row segment of every group, or null: all rows
+  const float* row_scale;              // [T] or null
+  int x_group_col, out_group_col;      // first column of a group's x and out rows is group * this
+};
+
+// out[t, n] = sum_k x[t, k] w[g, n, k].  64 x 64 tile per CTA, 16 k per step, 4 x 4 outputs per thread; blockIdx.z = group.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
+  const int g = blockIdx.z;
+  const int first = p.seg_len ? p.seg_start[g] : 0, rows = p.seg_len ? p.seg_len[g] : p.T;
   const int t0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  if (t0 >= rows) return;
+  const float* x = p.x + (size_t)first * p.x_ld + (size_t)g * p.x_group_col;
+  const float* w = p.w + (size_t)g * p.N * p.K;
+  float* out = p.out + (size_t)first * p.out_ld + (size_t)g * p.out_group_col;
+  __shared__ float xs[16][68], ws[16][68];
   const int tr = (threadIdx.x >> 4) * 4, tc = (threadIdx.x & 15) * 4;
   const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
   float acc[4][4] = {};
-  for (int k0 = 0; k0 < K; k0 += 16) {
+  for (int k0 = 0; k0 < p.K; k0 += 16) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int k = k0 + lk + i;
-      xs[lk + i][lr] = (t0 + lr < T && k < K) ? x[(size_t)(t0 + lr) * x_ld + k] : 0.f;
-      ws[lk + i][lr] = (n0 + lr < N && k < K) ? w[(size_t)(n0 + lr) * w_ld + k] : 0.f;
+      xs[lk + i][lr] = (t0 + lr < rows && k < p.K) ? x[(size_t)(t0 + lr) * p.x_ld + k] : 0.f;
+      ws[lk + i][lr] = (n0 + lr < p.N && k < p.K) ? w[(size_t)(n0 + lr) * p.K + k] : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -219,10 +249,13 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
+  for (int i = 0; i < 4; ++i) {
+    if (t0 + tr + i >= rows) break;
+    const float s = p.row_scale ? p.row_scale[first + t0 + tr + i] : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (t0 + tr + i < T && n0 + tc + j < N) out[(size_t)(t0 + tr + i) * out_ld + n0 + tc + j] = acc[i][j];
+      if (n0 + tc + j < p.N) out[(size_t)(t0 + tr + i) * p.out_ld + n0 + tc + j] = acc[i][j] * s;
+  }
 }
 
 static inline int row_threads(int n, int v) {
@@ -280,7 +313,7 @@ extern "C" int omni_qk_norm_rope_cache(void* qkv, int ld, int Hq, int Hkv, int D
                                        cudaStream_t st) {
   if (T_rows <= 0) return 0;
   if (Hq < 1 || D < 1 || rot < 0 || rot > D || rot % 2 != 0 || (rot > 0 && cos_sin == nullptr)) return -1;
-  if (Hkv > 0 && (k_cache == nullptr || v_cache == nullptr || kw == nullptr)) return -2;
+  if (Hkv > 0 && (k_cache == nullptr || v_cache == nullptr || (qw != nullptr && kw == nullptr))) return -2;
   if (D % 4 == 0 && DV % 4 == 0 && (rot / 2) % 4 == 0 && ld % 4 == 0) {
     FOR_TYPE((qk_norm_rope_cache_kernel<T, 4><<<T_rows, 256, 0, st>>>(
                   (T*)qkv, ld, Hq, Hkv, D, DV, (const float*)qw, (const float*)kw, eps, (const float*)cos_sin, rot, positions,
@@ -293,32 +326,38 @@ extern "C" int omni_qk_norm_rope_cache(void* qkv, int ld, int Hq, int Hkv, int D
   return (int)cudaGetLastError();
 }
 
-extern "C" int omni_gelu_mul(const void* x, int x_ld, int up_off, void* out, int out_ld, int T_rows, int I, int f32,
-                             cudaStream_t st) {
+extern "C" int omni_gated_mul(const void* x, int x_ld, int up_off, void* out, int out_ld, int T_rows, int I, int kind, float limit,
+                              int f32, cudaStream_t st) {
   if (T_rows <= 0) return 0;
-  if (I < 1 || out_ld < I || T_rows > 65535 * 16) return -1;
+  if (I < 1 || out_ld < I || T_rows > 65535 * 16 || kind < 0 || kind > 1) return -1;
   const int vec = (I % 8 == 0 && x_ld % 8 == 0 && up_off % 8 == 0 && out_ld % 8 == 0) ? 8 : 1;
+#define GATED(V, KIND)                                                                                                        \
+  FOR_TYPE((gated_mul_kernel<T, V, KIND><<<grid, 128, 0, st>>>((const T*)x + (size_t)r0 * x_ld, x_ld, up_off,                 \
+                                                               (T*)out + (size_t)r0 * out_ld, out_ld, n, I, limit));)
   for (int r0 = 0; r0 < T_rows; r0 += 65535) {      // grid.y limit
     const int n = T_rows - r0 < 65535 ? T_rows - r0 : 65535;
     const dim3 grid((out_ld / vec + 127) / 128 + (out_ld % vec ? 1 : 0), n);
-    if (vec == 8) {
-      FOR_TYPE((gelu_mul_kernel<T, 8><<<grid, 128, 0, st>>>((const T*)x + (size_t)r0 * x_ld, x_ld, up_off,
-                                                            (T*)out + (size_t)r0 * out_ld, out_ld, n, I));)
-    } else {
-      FOR_TYPE((gelu_mul_kernel<T, 1><<<grid, 128, 0, st>>>((const T*)x + (size_t)r0 * x_ld, x_ld, up_off,
-                                                            (T*)out + (size_t)r0 * out_ld, out_ld, n, I));)
-    }
+    if (vec == 8 && kind == 0) { GATED(8, 0) }
+    else if (vec == 8) { GATED(8, 1) }
+    else if (kind == 0) { GATED(1, 0) }
+    else { GATED(1, 1) }
   }
+#undef GATED
   return (int)cudaGetLastError();
 }
 
-extern "C" int omni_gemm_f32(const void* x, const void* w, void* out, int T_rows, int N, int K, int x_ld, int w_ld, int out_ld,
-                             cudaStream_t st) {
+// w [G, N, K] contiguous.  Groups by row segments (seg_start / seg_len), by columns (x_group_col / out_group_col), or one.
+extern "C" int omni_gemm_f32(const void* x, const void* w, void* out, int T_rows, int N, int K, int x_ld, int out_ld, int G,
+                             const int* seg_start, const int* seg_len, const float* row_scale, int x_group_col,
+                             int out_group_col, cudaStream_t st) {
   if (T_rows <= 0) return 0;
-  if (N < 1 || K < 1 || x_ld < K || w_ld < K || out_ld < N) return -1;
-  const dim3 grid((N + 63) / 64, (T_rows + 63) / 64);
+  if (N < 1 || K < 1 || G < 1 || G > 65535 || x_ld < K || out_ld < N) return -1;
+  if ((seg_len == nullptr) != (seg_start == nullptr)) return -3;
+  const dim3 grid((N + 63) / 64, (T_rows + 63) / 64, G);
   if (grid.y > 65535) return -2;
-  gemm_f32_kernel<<<grid, 256, 0, st>>>((const float*)x, (const float*)w, (float*)out, T_rows, N, K, x_ld, w_ld, out_ld);
+  const GemmF32Params p = {(const float*)x, (const float*)w, (float*)out, T_rows, N, K, x_ld, out_ld, seg_start, seg_len,
+                           row_scale, x_group_col, out_group_col};
+  gemm_f32_kernel<<<grid, 256, 0, st>>>(p);
   return (int)cudaGetLastError();
 }
 #undef FOR_TYPE

@@ -84,6 +84,9 @@ class ModelRunner:
                 raise ValueError("layer-list models run whole on every rank (data parallel)")
             if self.kv_connector is not None and self.has_state:
                 raise ValueError("KV hand-over between instances does not carry recurrent state")
+            if weights is not None and cfg.unresolved_sizes():
+                weights = list(weights)
+                cfg.resolve_sizes({k: tuple(v.shape) for k, v in weights})
             # positions are unbounded by design: the rotation tables cover what this engine may reach
             cfg.max_position_embeddings = max(cfg.max_position_embeddings, self.cfg.max_model_len + 64)
         self.model = build_model(cfg, device=self.device, planner=self.planner,
@@ -289,8 +292,7 @@ class ModelRunner:
                 num_blocks, bs, self.cfg.max_num_seqs, lambda *shape, dtype: torch.zeros(*shape, dtype=dtype, device=self.device))
             self.drafter_kv = []
             if self.kv_connector is not None:
-                self.kv_connector.register_kv_caches([c for c, s in zip(self.kv_caches, cfg.layers)
-                                                      if s.attention is not None and s.attention.owns_kv])
+                self.kv_connector.register_kv_caches(self.model.paged_caches(self.kv_caches))
             return
         self.kv_caches = [one() for _ in range(self.model.num_kv_layers)]
         self.drafter_kv = [[one()] for _ in self.drafters]

@@ -108,10 +108,11 @@ class PaddedLinear(Linear):
 class GeGLUMLP(nn.Module):
     """gate_up (merged, gate rows first, each block padded to a multiple of 8) -> gelu (tanh form) of the gate times up,
     in the GEMM epilogue where the width allows -> down."""
+    epi = "geglu"
 
     def __init__(self, hidden: int, inter: int, *, dtype=torch.bfloat16, device=None):
         super().__init__()
-        self.inter, self.block = inter, (inter + 7) // 8 * 8
+        self.inter, self.block, self.limit = inter, (inter + 7) // 8 * 8, 0.0
         self.gate_up_proj = PaddedLinear(hidden, 2 * self.block, dtype=dtype, device=device)
         self.down_proj = PaddedLinear(inter, hidden, dtype=dtype, device=device)
 
@@ -121,7 +122,21 @@ class GeGLUMLP(nn.Module):
         w[self.block + self.inter:] = 0
 
     def forward(self, x):
-        return ops.gemm(ops.gemm(x, self.gate_up_proj.weight, epi="geglu"), self.down_proj.weight)
+        return ops.gemm(ops.gemm(x, self.gate_up_proj.weight, epi=self.epi, glu_limit=self.limit), self.down_proj.weight)
+
+    def checkpoint_targets(self):
+        """{checkpoint suffix: (parameter, first row, rows, columns)}."""
+        w, h = self.gate_up_proj.weight, self.gate_up_proj.real_in
+        return {"gate": (w, 0, self.inter, h), "up": (w, self.block, self.inter, h), "down": (self.down_proj.weight, 0, h, self.inter)}
+
+
+class ClampedGLUMLP(GeGLUMLP):
+    """The same with g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1)."""
+    epi = "clamped_glu"
+
+    def __init__(self, hidden: int, inter: int, limit: float, *, dtype=torch.bfloat16, device=None):
+        super().__init__(hidden, inter, dtype=dtype, device=device)
+        self.limit = limit
 
 
 class PostNorm(nn.Module):

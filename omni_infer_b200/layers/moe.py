@@ -25,7 +25,9 @@ from torch import nn
 from .. import ops
 from ..ops import FP8
 from ..parallel import get_parallel_state
-from .common import Linear, SwiGLUMLP
+from ..ops.layer_list import pad8
+from ..ops.streams import ExpertSum
+from .common import ClampedGLUMLP, Linear, PaddedLinear, SwiGLUMLP
 
 
 import os as _os
@@ -40,6 +42,23 @@ def _side_stream(device):
     if st is None:
         st = _SIDE_STREAMS[key] = torch.cuda.Stream(device=device)
     return st
+
+
+def run_beside(fn, device):
+    """Shared experts only depend on the layer input, so they run on a second stream beside the router, the permutation and the
+    dispatch (small kernels that leave most SMs idle); the routed path joins before it adds their output.  Under CUDA-graph
+    capture this becomes a parallel branch of the graph (the reference overlaps the same work with its multi-stream option,
+    omni/models/deepseek/deepseek_moe.py).  Returns (result, event to wait for)."""
+    main, side = torch.cuda.current_stream(), _side_stream(device)
+    ready = torch.cuda.Event()
+    ready.record(main)
+    side.wait_event(ready)
+    with torch.cuda.stream(side):
+        out = fn()
+        done = torch.cuda.Event()
+        done.record(side)
+    out.record_stream(main)
+    return out, done
 
 
 class MoEGate(nn.Module):
@@ -195,21 +214,7 @@ class MoELayer(nn.Module):
         return ops.gemm(act, self.w2, seg_start=seg_start, seg_len=seg_len, row_scale=row_w, t_hint=t_hint)
 
     def _shared_on_side_stream(self, x, xq):
-        """The shared experts only depend on the layer input, so they run on a second stream beside the router,
-        the permutation and the dispatch (small kernels that leave most SMs idle); the routed path joins before it
-        adds their output.  Under CUDA-graph capture this becomes a parallel branch of the graph
-        (the reference overlaps the same work with its multi-stream option, omni/models/deepseek/deepseek_moe.py)."""
-        main = torch.cuda.current_stream()
-        side = _side_stream(x.device)
-        ready = torch.cuda.Event()
-        ready.record(main)
-        side.wait_event(ready)
-        with torch.cuda.stream(side):
-            shared = self.shared_experts(x, xq=xq)
-            done = torch.cuda.Event()
-            done.record(side)
-        shared.record_stream(main)
-        self._shared_done = done
+        shared, self._shared_done = run_beside(lambda: self.shared_experts(x, xq=xq), x.device)
         return shared
 
     def join_shared(self):
@@ -241,3 +246,60 @@ class MoELayer(nn.Module):
             return self.ep_ctx.moe_forward(self, x, ids, w, shared, xq=xq)
         from ..parallel.ep_nccl import moe_forward_nccl
         return moe_forward_nccl(self, x, ids, w, shared)
+
+
+class ExpertMixture(nn.Module):
+    """Mixture of clamped gated experts of a layer-list model: softmax scores over the experts and the identity experts (whose
+    output is the input), the choice by score + correction, weights = scores * scale without renormalising, and a shared
+    expert.  Every rank holds all experts.  The parts are returned unsummed; the residual kernel adds them up."""
+
+    def __init__(self, spec, hidden: int, *, dtype, device=None):
+        super().__init__()
+        self.spec, self.hidden = spec, hidden
+        s, W = spec, pad8(hidden)
+        self.block = pad8(s.ff)
+        zeros = lambda *n, dt=dtype: nn.Parameter(torch.zeros(*n, dtype=dt, device=device), requires_grad=False)  # noqa: E731
+        self.router = zeros(s.experts + s.identity, W)
+        self.correction = zeros(s.experts + s.identity, dt=torch.float32)
+        self.correction.init_value = 0.0
+        self.w13, self.w2 = zeros(s.experts, 2 * self.block, W), zeros(s.experts, W, self.block)
+        self.shared = ClampedGLUMLP(hidden, s.shared_ff, s.shared_limit, dtype=dtype, device=device) if s.shared_ff else None
+
+    def zero_padding(self):
+        H, ff, b = self.hidden, self.spec.ff, self.block
+        for w in (self.router.data, self.w13.data):
+            w[..., H:] = 0
+        self.w13.data[:, ff:b] = 0
+        self.w13.data[:, b + ff:] = 0
+        self.w2.data[:, H:] = 0
+        self.w2.data[:, :, ff:] = 0
+
+    def forward(self, x, num_valid=None):
+        s, T = self.spec, x.shape[0]
+        shared = done = None
+        if self.shared is not None:
+            if x.is_cuda and MULTI_STREAM:
+                shared, done = run_beside(lambda: self.shared(x), x.device)
+            else:
+                shared = self.shared(x)
+        logits = ops.gemm(x, self.router, out_dtype=torch.float32)
+        ids, w = ops.router_topk(logits, s.top, mode="softmax", bias=self.correction, scale=s.scale, num_valid=num_valid)
+        perm = ops.moe_permute(x, ids, w, 0, s.experts)
+        kw = dict(seg_start=perm.seg_start, seg_len=perm.seg_len, t_hint=max(16, (T * s.top + s.experts - 1) // s.experts))
+        act = ops.gemm(perm.x, self.w13, epi="clamped_glu", glu_limit=s.limit, **kw)
+        y = ops.gemm(act, self.w2, row_scale=perm.row_w, **kw)
+        if done is not None:
+            torch.cuda.current_stream().wait_event(done)
+        return ExpertSum(y, perm.row_of, ids, w, s.experts, x, shared)
+
+    def checkpoint_targets(self):
+        """{checkpoint suffix: (parameter or a view of one, first row, rows, columns)}; columns None: a vector."""
+        s, H, b = self.spec, self.hidden, self.block
+        n = s.experts + s.identity
+        t = {"router": (self.router, 0, n, H), "correction": (self.correction, 0, n, None)}
+        for e in range(s.experts):
+            t[f"e{e}.gate"], t[f"e{e}.up"] = (self.w13.data[e], 0, s.ff, H), (self.w13.data[e], b, s.ff, H)
+            t[f"e{e}.down"] = (self.w2.data[e], 0, H, s.ff)
+        if self.shared is not None:
+            t.update({"shared." + k: v for k, v in self.shared.checkpoint_targets().items()})
+        return t

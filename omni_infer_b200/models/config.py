@@ -2,6 +2,7 @@
 Qwen2 dense GQA, Qwen3-MoE GQA, layer-list models) plus the named configurations used by the benchmarks."""
 from __future__ import annotations
 
+import dataclasses
 import json
 import re
 from dataclasses import asdict, dataclass, field
@@ -22,6 +23,9 @@ class AttentionSpec:
     rot_base: float = 10000.0
     rot_factor: float = 1.0                  # linear scaling: every frequency is divided by it
     kv_from: Optional[int] = None            # attends to the cached keys and values of this earlier layer
+    qk_norm: bool = True                     # RMSNorm over the whole q and the whole k projection
+    sink: bool = False                       # a learned term per head in the softmax denominator
+    rot_scaling: Optional[dict] = None       # other scalings, as ``ops.rope_cos_sin_table`` takes them
 
     @property
     def owns_kv(self) -> bool:
@@ -51,18 +55,82 @@ class Mamba2Spec:
 
 
 @dataclass
+class MLSTMSpec:
+    """Matrix memory (xLSTM) of one layer of a layer-list model."""
+    heads: int
+    dim: int                                 # query / key size per head
+    vdim: int                                # value size per head
+    gate_cap: float                          # both log gates are bounded softly by it
+
+
+@dataclass
+class WkvSpec:
+    """WKV time mixing of one layer of a layer-list model."""
+    heads: int
+    dim: int                                 # key and value size per head
+    rank: int = 0                            # of the decay's projection; 0 = as the checkpoint has it
+
+
+@dataclass
+class ParallelSpec:
+    """Attention and a matrix memory side by side on the same input."""
+    left: AttentionSpec
+    right: MLSTMSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass
+class ExpertsSpec:
+    """Mixture of clamped gated experts of one layer of a layer-list model."""
+    experts: int
+    top: int
+    ff: int
+    limit: float
+    identity: int = 0                        # router outputs after the experts' whose expert is the identity
+    scale: float = 1.0                       # of the routing weights
+    shared_ff: int = 0                       # expert that runs for every token, 0 = none
+    shared_limit: float = 0.0
+
+
+@dataclass
 class LayerSpec:
-    """One entry of a layer-list model: a mixer and an optional gated dense feed-forward."""
+    """One entry of a layer-list model: a mixer and an optional feed-forward (gated dense, or a mixture of experts)."""
     attention: Optional[AttentionSpec] = None
     mamba2: Optional[Mamba2Spec] = None
-    ff: int = 0                              # width of the feed-forward, 0 = the layer has none
+    ff: int = 0                              # width of the dense feed-forward
+    parallel: Optional[ParallelSpec] = None
+    wkv: Optional[WkvSpec] = None
+    experts: Optional[ExpertsSpec] = None
+    weights_of: Optional[int] = None         # the layer runs with this layer's weights and a cache or state of its own
+
+    @property
+    def paged(self) -> Optional[AttentionSpec]:
+        """The attention that reads (and, unless it shares them, fills) cache pages."""
+        return self.parallel.left if self.parallel is not None else self.attention
+
+    @property
+    def recurrent(self) -> bool:
+        return self.mamba2 is not None or self.parallel is not None or self.wkv is not None
+
+    @staticmethod
+    def _pre_norm_attention(i: int, m: dict) -> AttentionSpec:
+        """Attention without q/k norms, with a sink per head and Llama-3.1 frequency scaling."""
+        rot = m.get("rot") or {}
+        a = AttentionSpec(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]),
+                          rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)), qk_norm=False, sink=True)
+        if rot.get("scaling"):
+            s = rot["scaling"]
+            a.rot_scaling = {"type": "llama3", "factor": s["factor"], "low_freq_factor": s["low"], "high_freq_factor": s["high"],
+                             "original_max_position_embeddings": s["original"]}
+        return a
 
     @classmethod
     def from_dict(cls, i: int, d: dict) -> "LayerSpec":
         """Entry ``i`` of the ``layers`` list of a config.json.  The type may carry a running number (several mixers of
         one kind with sizes of their own)."""
         kind, m = re.sub(r"_\d+$", "", d["type"]), d["mixer"]
-        s = cls()
+        s = cls(weights_of=d.get("weights_of"))
         if kind == "attention":
             rot = m.get("rot") or {}
             s.attention = AttentionSpec(
@@ -70,21 +138,40 @@ class LayerSpec:
                 window=int((m.get("mask") or {}).get("size") or 0), rot_dims=int(rot.get("dims", 0)),
                 rot_base=float(rot.get("base", 10000.0)),
                 rot_factor=float((rot.get("scaling") or {}).get("factor", 1.0)), kv_from=m.get("kv_from"))
-            if s.attention.heads % s.attention.kv_heads or s.attention.rot_dims % 2 or s.attention.rot_dims > s.attention.dim:
-                raise ValueError(f"layer {i}: heads must divide over the key/value heads, rotated dimensions be even and "
-                                 "fit the head")
         elif kind == "mamba2":
             s.mamba2 = Mamba2Spec(heads=m["heads"], vdim=m["vdim"], state=m["state"], groups=m["groups"], conv=m["conv"],
                                   norm_groups=m["norm_groups"])
             if s.mamba2.heads % s.mamba2.groups or s.mamba2.inner % s.mamba2.norm_groups:
                 raise ValueError(f"layer {i}: heads must divide over the groups, the inner width over the norm groups")
+        elif kind == "parallel":
+            r = m["right"]
+            s.parallel = ParallelSpec(cls._pre_norm_attention(i, m["left"]),
+                                      MLSTMSpec(heads=r["heads"], dim=r["dim"], vdim=r["vdim"], gate_cap=float(r["gate_cap"])),
+                                      float(m["left_scale"]), float(m["right_scale"]))
+        elif kind == "wkv":
+            s.wkv = WkvSpec(heads=m["heads"], dim=m["dim"])
         else:
             raise ValueError(f"layer {i}: unknown mixer type {d['type']!r}")
+        a = s.paged
+        if a is not None and (a.heads % a.kv_heads or a.rot_dims % 2 or a.rot_dims > a.dim):
+            raise ValueError(f"layer {i}: heads must divide over the key/value heads, rotated dimensions be even and fit the head")
         mlp = d.get("mlp")
         if mlp:
-            if mlp.get("kind", "dense") != "dense":
-                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
-            s.ff = int(mlp["ff"])
+            fkind = mlp.get("kind", "dense")
+            if fkind == "dense":
+                s.ff = int(mlp["ff"])
+            elif fkind == "moe":
+                if not mlp.get("router") or not mlp.get("expert"):
+                    raise ValueError(f"layer {i}: a feed-forward of kind 'moe' needs a router and an expert")
+                r, e, sh = mlp["router"], mlp["expert"], mlp.get("shared") or {}
+                s.experts = ExpertsSpec(experts=r["experts"], top=r["top"], ff=e["ff"], limit=float(e["limit"]),
+                                        identity=int(r.get("identity") or 0), scale=float(r.get("scale", 1.0)),
+                                        shared_ff=int(sh.get("ff", 0)), shared_limit=float(sh.get("limit", 0.0)))
+                n = s.experts.experts + s.experts.identity
+                if not 0 < s.experts.top <= min(n, 32) or n > 512:
+                    raise ValueError(f"layer {i}: {s.experts.top} of {n} experts (at most 32 of 512)")
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {fkind!r}")
         return s
 
 
@@ -93,6 +180,9 @@ class ModelConfig:
     architecture: str = "DeepseekV3ForCausalLM"
     # layer-list models: one LayerSpec per layer; None = the uniform stacks described by the fields below
     layers: Optional[list] = None
+    # residual streams of a layer-list model with layer norms ahead of its sublayers; 0 = one residual, norms on the outputs
+    streams: int = 0
+    embedding_scale: float = 1.0
     # tensor-parallel attention: heads sharded over attn_tp_size ranks, hidden states sharded by token rows between
     # layers (set by the model runner; 1 = every rank runs whole attention layers on its own requests)
     attn_tp_size: int = 1
@@ -180,11 +270,11 @@ class ModelConfig:
     @property
     def has_recurrent_state(self) -> bool:
         """Does a request hold state besides its cached tokens (one slot per live request)?"""
-        return any(s.mamba2 is not None for s in self.layers or ())
+        return any(s.recurrent for s in self.layers or ())
 
     def kv_bytes_per_token(self, elem_bytes: int = 2) -> int:
         if self.layers is not None:     # mean over the layers that hold a cache
-            per = [s.attention.cache_elems_per_token() for s in self.layers if s.attention is not None and s.attention.owns_kv]
+            per = [s.paged.cache_elems_per_token() for s in self.layers if s.paged is not None and s.paged.owns_kv]
             return sum(per) * elem_bytes // max(1, len(per))
         if self.use_mla:
             return (self.kv_lora_rank + self.qk_rope_head_dim) * elem_bytes
@@ -244,13 +334,47 @@ class ModelConfig:
                 raise ValueError(f"layer {i} takes its keys from layer {a.kv_from}, which holds none")
             if (src.kv_heads, src.dim, src.vdim) != (a.kv_heads, a.dim, a.vdim):
                 raise ValueError(f"layers {i} and {a.kv_from} share keys but differ in their head sizes")
+        streams = int(d.get("streams", 0))
+        if any((s.parallel or s.wkv or s.experts) is not None if not streams else (s.attention or s.mamba2) is not None or s.ff for s in layers):
+            raise ValueError("attention, mamba2 and dense layers run on one residual with norms on the outputs, parallel, wkv and "
+                             "mixture-of-experts layers on residual streams with norms ahead")
+        for i, s in enumerate(layers):
+            seen = {i}
+            while s.weights_of is not None:
+                j = s.weights_of
+                if not 0 <= j < len(layers) or j in seen:
+                    raise ValueError(f"layer {i} takes its weights from layer {j}, which has none")
+                seen.add(j)
+                s = layers[j]
+            if len(seen) > 1:
+                if dataclasses.replace(layers[i], weights_of=None) != s:
+                    raise ValueError(f"layers {i} and {layers[i].weights_of} share weights but differ in their sizes")
+                layers[i].weights_of = next(j for j, o in enumerate(layers) if o is s)
         return cls(architecture=arch, layers=layers, vocab_size=d["vocab"], hidden_size=d["width"],
                    num_hidden_layers=len(layers), rms_norm_eps=float(d["norm"]["eps"]), use_mla=False,
-                   tie_word_embeddings=True, n_routed_experts=0, name=arch)
+                   tie_word_embeddings=True, n_routed_experts=0, name=arch, streams=streams,
+                   embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
 
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
-        return cls.from_hf_dict(json.loads((Path(path) / "config.json").read_text()))
+        c = cls.from_hf_dict(json.loads((Path(path) / "config.json").read_text()))
+        if c.unresolved_sizes():
+            from ..quantization.loader import safetensors_shapes
+            c.resolve_sizes(safetensors_shapes(path))
+        return c
+
+    def unresolved_sizes(self) -> bool:
+        """Are there sizes that only the checkpoint's tensors tell?"""
+        return any(s.wkv is not None and s.wkv.rank == 0 for s in self.layers or ())
+
+    def resolve_sizes(self, shapes: dict) -> None:
+        """``shapes``: checkpoint tensor name -> shape."""
+        for i, s in enumerate(self.layers or ()):
+            if s.wkv is not None and s.wkv.rank == 0:
+                name = f"l{i if s.weights_of is None else s.weights_of}.mix.w1"
+                if name not in shapes:
+                    raise KeyError(f"checkpoint lacks {name}")
+                s.wkv.rank = int(shapes[name][0])
 
 
 # ------------------------------------------------------------------------------------------------
@@ -368,6 +492,38 @@ def forovik(width=2048, layers=12, vocab=32768, heads=16, kv_heads=4, dim=128, w
     return c
 
 
+def fimudra(width=2048, layers=12, vocab=32768, streams=2, heads=16, kv_heads=4, dim=128, m_heads=16, m_dim=64, m_vdim=128,
+            w_heads=32, w_dim=64, w_rank=64, experts=32, identity=4, top=4, ff=768, shared_ff=1536, loop=True, **kw) -> ModelConfig:
+    """Layer-list model with residual streams: attention beside a matrix memory in two of three layers, WKV in the third, a
+    mixture of experts in each; with ``loop`` the last layer runs with the weights of the first of its kind."""
+    ffn = lambda: ExpertsSpec(experts, top, ff, 7.0, identity, 2.5, shared_ff, 7.0)        # noqa: E731
+    specs = []
+    for i in range(layers):
+        if i % 3 == 2:
+            specs.append(LayerSpec(wkv=WkvSpec(w_heads, w_dim, w_rank), experts=ffn()))
+        else:
+            att = AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, rot_dims=dim, rot_base=5e5, qk_norm=False, sink=True,
+                                rot_scaling={"type": "llama3", "factor": 8.0, "low_freq_factor": 1.0, "high_freq_factor": 4.0,
+                                             "original_max_position_embeddings": 8192})
+            specs.append(LayerSpec(parallel=ParallelSpec(att, MLSTMSpec(m_heads, m_dim, m_vdim, 15.0), 0.7, 0.7), experts=ffn()))
+    if loop and layers > 3:
+        specs[-1].weights_of = (layers - 1) % 3
+    c = ModelConfig(architecture="Fimudra", name="fimudra", layers=specs, vocab_size=vocab, hidden_size=width,
+                    num_hidden_layers=layers, use_mla=False, tie_word_embeddings=True, rms_norm_eps=1e-5, streams=streams,
+                    embedding_scale=width ** 0.5)
+    for k, v in kw.items():
+        setattr(c, k, v)
+    return c
+
+
+def tiny_fimudra(**kw) -> ModelConfig:
+    """CPU-sized layer-list model with residual streams."""
+    kw.setdefault("dtype", "float32")
+    kw.setdefault("name", "tiny-fimudra")
+    return fimudra(width=64, layers=6, vocab=512, streams=3, heads=4, kv_heads=2, dim=16, m_heads=3, m_dim=8, m_vdim=16, w_heads=4,
+                   w_dim=12, w_rank=5, experts=6, identity=2, top=2, ff=24, shared_ff=40, **kw)
+
+
 def tiny_forovik(**kw) -> ModelConfig:
     """CPU-sized layer-list model."""
     kw.setdefault("dtype", "float32")
@@ -379,6 +535,8 @@ def tiny_forovik(**kw) -> ModelConfig:
 PRESETS = {
     "forovik": forovik,
     "tiny-forovik": tiny_forovik,
+    "fimudra": fimudra,
+    "tiny-fimudra": tiny_fimudra,
     "tiny-deepseek-v3": tiny_deepseek_v3,
     "tiny-qwen3-moe": tiny_qwen3_moe,
     "small-deepseek": small_deepseek_gpu,

@@ -1,12 +1,19 @@
-"""Models described layer by layer: ``ModelConfig.layers`` lists a mixer (windowed attention or Mamba-2) and an optional
-gated feed-forward per layer, each with sizes of its own.
+"""Models described layer by layer: ``ModelConfig.layers`` lists a mixer and an optional feed-forward per layer, each with sizes
+of its own.  Two ways to connect them:
 
-Sublayers read the residual stream itself and their outputs are normed before they are added to it:
-``x <- x + norm1(mixer(x))``, ``x <- x + norm2(ff(x))``.  The residual is fp32; every addition, its norm and the activation
-copy for the next sublayer are one kernel.  The embedding table is also the LM head.
+One residual, norms on the outputs (``cfg.streams == 0``; windowed attention, Mamba-2, gated dense feed-forward): sublayers read
+the residual stream itself, ``x <- x + norm1(mixer(x))``, ``x <- x + norm2(ff(x))``.  Every addition, its norm and the activation
+copy for the next sublayer are one kernel.
 
-A layer's entry in ``kv_caches`` is what its mixer reads: the (k, v) page pools of an attention layer - the same tensors
-for a layer that attends to another layer's keys - or the (convolution, recurrence) slot tensors of a Mamba-2 layer."""
+Residual streams, norms ahead (attention beside a matrix memory, WKV, mixture of experts): a sublayer reads the layer norm of a
+learned sum of the streams, and every stream becomes a learned sum of all of them and the sublayer's output.  Update, sum and
+norm for the next sublayer are one kernel.  A layer may run with another layer's weights (``weights_of``) on a cache or state
+of its own.
+
+The residual is fp32 either way, and the embedding table is also the LM head.
+
+A layer's entry in ``kv_caches`` is what its mixer reads: the (k, v) page pools of an attention layer - the same tensors for a
+layer that attends to another layer's keys - or the slot tensors of a recurrent one, or both."""
 from __future__ import annotations
 
 import torch
@@ -15,20 +22,33 @@ from torch import nn
 from .. import ops
 from ..layers.common import GeGLUMLP, PaddedLinear, PostNorm, _dtype
 from ..layers.mamba2 import Mamba2Mixer
+from ..layers.matrix_state import ParallelMixer, WkvMixer
+from ..layers.moe import ExpertMixture
 from ..layers.vocab_parallel import lm_logits
 from ..layers.windowed_attention import WindowedAttention
 from ..ops.layer_list import embed_residual, pad8, rmsnorm_residual
+from ..ops.streams import embed_streams, stream_step
 from .config import ModelConfig
 
 
+def _mixer(s, width, eps, **kw):
+    cos_sin = kw.pop("cos_sin")
+    if s.attention is not None:
+        return WindowedAttention(s.attention, width, eps, cos_sin=cos_sin, **kw)
+    if s.parallel is not None:
+        return ParallelMixer(s.parallel, width, eps, cos_sin=cos_sin, **kw)
+    if s.wkv is not None:
+        return WkvMixer(s.wkv, width, eps, **kw)
+    return Mamba2Mixer(s.mamba2, width, eps, **kw)
+
+
 class LayerListLayer(nn.Module):
+    """One residual, norms on the outputs."""
+
     def __init__(self, cfg: ModelConfig, i: int, *, dtype, device=None, cos_sin=None):
         super().__init__()
         s, width, eps = cfg.layers[i], cfg.hidden_size, cfg.rms_norm_eps
-        if s.attention is not None:
-            self.mixer = WindowedAttention(s.attention, width, eps, dtype=dtype, device=device, cos_sin=cos_sin)
-        else:
-            self.mixer = Mamba2Mixer(s.mamba2, width, eps, dtype=dtype, device=device)
+        self.mixer = _mixer(s, width, eps, dtype=dtype, device=device, cos_sin=cos_sin)
         self.norm1 = PostNorm(width, eps, device)
         self.mlp = GeGLUMLP(width, s.ff, dtype=dtype, device=device) if s.ff else None
         self.norm2 = PostNorm(width, eps, device) if s.ff else None
@@ -37,6 +57,52 @@ class LayerListLayer(nn.Module):
         """x: fp32 residual (updated in place), xa: the same as activations; returns the new activations."""
         xa = self.norm1(self.mixer(xa, md, cache), x)
         return self.norm2(self.mlp(xa), x) if self.mlp is not None else xa
+
+    def checkpoint_targets(self):
+        H = self.norm1.weight.shape[0]
+        out = {"norm1": (self.norm1.weight, 0, H, None)}
+        out.update({"mix." + k: v for k, v in self.mixer.checkpoint_targets().items()})
+        if self.mlp is not None:
+            out["norm2"] = (self.norm2.weight, 0, H, None)
+            out.update({"mlp." + k: v for k, v in self.mlp.checkpoint_targets().items()})
+        return out
+
+
+class StreamLink(nn.Module):
+    """How a sublayer hangs on the streams: weights of its input sum and norm, and of the update with its output."""
+
+    def __init__(self, streams: int, width: int, device=None):
+        super().__init__()
+        par = lambda v: nn.Parameter(v.to(torch.float32).to(device or "cpu"), requires_grad=False)      # noqa: E731
+        self.inw, self.out, self.mix = par(torch.full((streams,), 1.0 / streams)), par(torch.ones(streams)), par(torch.eye(streams))
+        self.norm = par(torch.ones(width))
+        for p in (self.inw, self.out, self.mix):
+            p.init_value = p.data.clone()
+
+    def checkpoint_targets(self, q: int):
+        n = self.inw.shape[0]
+        return {f"norm{q}": (self.norm, 0, self.norm.shape[0], None), f"hc{q}.in": (self.inw, 0, n, None),
+                f"hc{q}.out": (self.out, 0, n, None), f"hc{q}.mix": (self.mix, 0, n, n)}
+
+
+class StreamLayer(nn.Module):
+    """Residual streams, norms ahead.  The model runs the sublayers; this holds their weights."""
+
+    def __init__(self, cfg: ModelConfig, i: int, *, dtype, device=None, cos_sin=None):
+        super().__init__()
+        s, width = cfg.layers[i], cfg.hidden_size
+        self.mixer = _mixer(s, width, cfg.rms_norm_eps, dtype=dtype, device=device, cos_sin=cos_sin)
+        self.link1 = StreamLink(cfg.streams, width, device)
+        self.mlp = ExpertMixture(s.experts, width, dtype=dtype, device=device) if s.experts is not None else None
+        self.link2 = StreamLink(cfg.streams, width, device) if s.experts is not None else None
+
+    def checkpoint_targets(self):
+        out = self.link1.checkpoint_targets(1)
+        out.update({"mix." + k: v for k, v in self.mixer.checkpoint_targets().items()})
+        if self.mlp is not None:
+            out.update(self.link2.checkpoint_targets(2))
+            out.update({"mlp." + k: v for k, v in self.mlp.checkpoint_targets().items()})
+        return out
 
 
 class LayerListModel(nn.Module):
@@ -48,24 +114,49 @@ class LayerListModel(nn.Module):
         def cos_sin(a):
             if a is None or a.rot_dims == 0:
                 return None
-            key = (a.rot_dims, a.rot_base, a.rot_factor)
+            scaling = a.rot_scaling or {"type": "linear", "factor": a.rot_factor}
+            key = (a.rot_dims, a.rot_base, tuple(sorted(scaling.items())))
             if key not in tables:
-                tables[key] = ops.rope_cos_sin_table(a.rot_dims, cfg.max_position_embeddings, a.rot_base,
-                                                     {"type": "linear", "factor": a.rot_factor}, device=device or "cpu")
+                tables[key] = ops.rope_cos_sin_table(a.rot_dims, cfg.max_position_embeddings, a.rot_base, scaling,
+                                                     device=device or "cpu")
             return tables[key]
 
         self.embed_tokens = nn.Embedding(cfg.vocab_size, pad8(cfg.hidden_size), dtype=self.dtype, device=device)
         self.embed_tokens.weight.requires_grad_(False)
-        self.layers = nn.ModuleList([LayerListLayer(cfg, i, dtype=self.dtype, device=device, cos_sin=cos_sin(s.attention))
-                                     for i, s in enumerate(cfg.layers)])
+        kind = StreamLayer if cfg.streams else LayerListLayer
+        built: list = []
+        for i, s in enumerate(cfg.layers):      # a layer with another's weights is that layer's module
+            built.append(None if s.weights_of is not None else
+                         kind(cfg, i, dtype=self.dtype, device=device, cos_sin=cos_sin(s.paged)))
+        self.layers = nn.ModuleList([built[i if s.weights_of is None else s.weights_of] for i, s in enumerate(cfg.layers)])
         self.norm = nn.Parameter(torch.ones(cfg.hidden_size, dtype=torch.float32, device=device), requires_grad=False)
+        if cfg.streams:
+            self.register_buffer("every_stream", torch.ones(cfg.streams, dtype=torch.float32, device=device), persistent=False)
 
     def forward(self, input_ids, md, kv_caches, inputs_embeds=None):
         assert inputs_embeds is None
+        if self.cfg.streams:
+            return self._forward_streams(input_ids, md, kv_caches)
         x, xa = embed_residual(input_ids, self.embed_tokens.weight)
         for layer, cache in zip(self.layers, kv_caches):
             xa = layer(x, xa, md, cache)
         return rmsnorm_residual(x, self.norm, self.cfg.rms_norm_eps, self.dtype)
+
+    def _forward_streams(self, input_ids, md, kv_caches):
+        eps = self.cfg.rms_norm_eps
+        subs = []
+        for layer, cache in zip(self.layers, kv_caches):
+            subs.append((layer.link1, lambda h, m=layer.mixer, c=cache: m(h, md, c)))
+            if layer.mlp is not None:
+                subs.append((layer.link2, lambda h, m=layer.mlp: m(h, md.num_valid)))
+        first = subs[0][0]
+        x, h = embed_streams(input_ids, self.embed_tokens.weight, self.cfg.hidden_size, self.cfg.embedding_scale, first.inw,
+                             first.norm, eps)
+        for k, (link, run) in enumerate(subs):
+            last = k + 1 == len(subs)
+            inw, norm = (self.every_stream, self.norm) if last else (subs[k + 1][0].inw, subs[k + 1][0].norm)
+            h = stream_step(x, run(h), link.mix, link.out, inw, norm, eps, self.dtype, last=last)
+        return h
 
 
 class LayerListForCausalLM(nn.Module):
@@ -83,31 +174,36 @@ class LayerListForCausalLM(nn.Module):
     @property
     def num_kv_layers(self):
         """Layers that hold pages of their own."""
-        return sum(s.attention is not None and s.attention.owns_kv for s in self.cfg.layers)
+        return sum(s.paged is not None and s.paged.owns_kv for s in self.cfg.layers)
 
     def allocate_caches(self, num_blocks: int, block_size: int, state_slots: int, zeros) -> list:
         """One entry per layer (see the module text).  ``zeros(*shape, dtype=)`` allocates."""
         caches: list = []
         for s, layer in zip(self.cfg.layers, self.model.layers):
-            a = s.attention
-            if a is None:
-                caches.append(tuple(zeros(*shape, dtype=dt) for shape, dt in layer.mixer.state_shapes(state_slots, self.model.dtype)))
-            elif a.owns_kv:
-                caches.append((zeros(num_blocks, block_size, a.kv_heads, a.dim, dtype=self.model.dtype),
-                               zeros(num_blocks, block_size, a.kv_heads, a.vdim, dtype=self.model.dtype)))
-            else:
-                caches.append(caches[a.kv_from])
+            a, pages, state = s.paged, None, None
+            if a is not None and not a.owns_kv:
+                pages = caches[a.kv_from]
+            elif a is not None:
+                pages = (zeros(num_blocks, block_size, a.kv_heads, a.dim, dtype=self.model.dtype),
+                         zeros(num_blocks, block_size, a.kv_heads, a.vdim, dtype=self.model.dtype))
+            if s.recurrent:
+                state = tuple(zeros(*shape, dtype=dt) for shape, dt in layer.mixer.state_shapes(state_slots, self.model.dtype))
+            caches.append(pages if state is None else (state if pages is None else (pages, state)))
         return caches
+
+    def paged_caches(self, caches: list) -> list:
+        """The (k, v) pools among ``caches`` that belong to a layer of their own."""
+        return [c[0] if s.recurrent else c for c, s in zip(caches, self.cfg.layers) if s.paged is not None and s.paged.owns_kv]
 
     def kv_bytes_per_token(self) -> int:
         esz = torch.empty(0, dtype=self.model.dtype).element_size()
-        return esz * sum(s.attention.cache_elems_per_token() for s in self.cfg.layers if s.attention is not None)
+        return esz * sum(s.paged.cache_elems_per_token() for s in self.cfg.layers if s.paged is not None)
 
     def state_bytes(self, slots: int) -> int:
         """Bytes of recurrent state for ``slots`` requests."""
         total = 0
-        for layer in self.model.layers:
-            if isinstance(layer.mixer, Mamba2Mixer):
+        for s, layer in zip(self.cfg.layers, self.model.layers):
+            if s.recurrent:
                 for shape, dt in layer.mixer.state_shapes(slots, self.model.dtype):
                     total += torch.Size(shape).numel() * torch.empty(0, dtype=dt).element_size()
         return total
@@ -121,12 +217,9 @@ class LayerListForCausalLM(nn.Module):
     def process_weights_after_loading(self):
         """Padding rows and columns hold zeros whatever the loader or the random initialisation put there."""
         self.model.embed_tokens.weight.data[:, self.cfg.hidden_size:] = 0
-        for m in self.modules():
-            if isinstance(m, PaddedLinear):
-                m.zero_padding()
-        for m in self.modules():
-            if isinstance(m, GeGLUMLP):
-                m.zero_padding()
+        mods = [m for m in self.modules() if hasattr(m, "zero_padding")]
+        for m in sorted(mods, key=lambda m: not isinstance(m, PaddedLinear)):      # single layers first, then what is made of them
+            m.zero_padding()
 
     def should_use_eager_mode(self, md):
         return md.is_prefill
@@ -137,14 +230,8 @@ class LayerListForCausalLM(nn.Module):
         H = self.cfg.hidden_size
         out = {"embed": (self.model.embed_tokens.weight, 0, self.cfg.vocab_size, H), "final.norm": (self.model.norm, 0, H, None)}
         for i, layer in enumerate(self.model.layers):
-            p = f"l{i}."
-            out[p + "norm1"] = (layer.norm1.weight, 0, H, None)
-            out.update({p + "mix." + k: v for k, v in layer.mixer.checkpoint_targets().items()})
-            if layer.mlp is not None:
-                m, w = layer.mlp, layer.mlp.gate_up_proj.weight
-                out[p + "norm2"] = (layer.norm2.weight, 0, H, None)
-                out[p + "mlp.gate"], out[p + "mlp.up"] = (w, 0, m.inter, H), (w, m.block, m.inter, H)
-                out[p + "mlp.down"] = (m.down_proj.weight, 0, H, m.inter)
+            if self.cfg.layers[i].weights_of is None:
+                out.update({f"l{i}." + k: v for k, v in layer.checkpoint_targets().items()})
         return out
 
     def load_weights(self, weights, planner=None) -> set:

@@ -13,7 +13,7 @@ from . import _native as nat
 
 FP8 = torch.float8_e4m3fn
 FP8_MAX = 448.0
-_EPI = {"store": 0, "swiglu": 1, "swiglu_quant": 2, "geglu": 3}
+_EPI = {"store": 0, "swiglu": 1, "swiglu_quant": 2, "geglu": 3, "clamped_glu": 4}
 
 
 def quant_fp8_block_ref(x: torch.Tensor, block: int = 128, ld: int | None = None):
@@ -59,8 +59,13 @@ def dequant_act_ref(xq: torch.Tensor, scale_t: torch.Tensor, block: int = 128) -
     return xq.float() * s
 
 
+def clamped_glu_ref(gate, up, limit):
+    g = gate.clamp(max=limit)
+    return g * torch.sigmoid(1.702 * g) * (up.clamp(-limit, limit) + 1)
+
+
 def gemm_ref(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi="store",
-             row_scale=None, out_dtype=torch.bfloat16, out_scale_ld=None):
+             row_scale=None, out_dtype=torch.bfloat16, out_scale_ld=None, glu_limit=0.0):
     """fp32 reference of :func:`gemm` with identical argument conventions."""
     if w.dim() == 2:
         w = w.unsqueeze(0)
@@ -84,6 +89,9 @@ def gemm_ref(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, 
         acc = xf[s:s + l] @ wf[g].t()
         if epi != "store":
             gate = acc[:, :n_out]
+            if epi == "clamped_glu":
+                y[s:s + l] = clamped_glu_ref(gate, acc[:, n_out:], glu_limit)
+                continue
             act = torch.nn.functional.gelu(gate, approximate="tanh") if epi == "geglu" else torch.nn.functional.silu(gate)
             acc = act * acc[:, n_out:]
         y[s:s + l] = acc
@@ -105,7 +113,7 @@ class TmCollective(nat.ctypes.Structure):
 
 
 def _tm2(kind, e, w, x, out, G, n_out, K, T, seg_start, seg_len, w_scale, x_scale, out_f32, out_scale, row_scale,
-         x_group_col=0, out_group_col=0, out_ld=None, x_ld=None, coll=None):
+         x_group_col=0, out_group_col=0, out_ld=None, x_ld=None, coll=None, glu_limit=0.0):
     rc = nat.lib().omni_gemm_tm2(
         nat.c_int(kind), nat.c_int(e), nat.ptr(w), nat.ptr(x), nat.ptr(out), nat.c_int(G), nat.c_int(n_out), nat.c_int(K),
         nat.c_int(T), nat.c_int(T), nat.ptr(seg_start), nat.ptr(seg_len), nat.ptr(w_scale), nat.ptr(x_scale),
@@ -113,30 +121,31 @@ def _tm2(kind, e, w, x, out, G, n_out, K, T, seg_start, seg_len, w_scale, x_scal
         nat.c_int(out_ld if out_ld is not None else out.stride(0)), nat.c_int(out_f32), nat.ptr(out_scale),
         nat.c_int(out_scale.shape[1] if out_scale is not None else 0), nat.ptr(row_scale),
         nat.c_int(x_group_col), nat.c_int(out_group_col), nat.c_int(x_ld if x_ld is not None else x.stride(0)),
-        nat.ctypes.byref(coll) if coll is not None else None,
+        nat.c_float(glu_limit), nat.ctypes.byref(coll) if coll is not None else None,
         nat.ptr(nat.status_buffer(x.device)), nat.stream())
     nat.check_rc(rc, "omni_gemm_tm2")
 
 
 def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi="store",
-         row_scale=None, out_dtype=None, out=None, out_scale=None, bn=0, t_hint=0):
+         row_scale=None, out_dtype=None, out=None, out_scale=None, bn=0, t_hint=0, glu_limit=0.0):
     """``out[t] = epi(x[t] @ w[g(t)].T)``.
 
     x: [T, K] bf16 or e4m3 (then ``x_scale`` is [K/128, ld] fp32, K-block major).
     w: [N, K] or [G, N, K]; e4m3 weights carry ``w_scale`` [G, N/128, K/128].
     seg_start/seg_len: int32 [G] row segments per group (grouped GEMM).
     epi: "store" | "swiglu" (w holds gate rows then up rows) | "geglu" (the same with the tanh form of gelu) |
+    "clamped_glu" (gate bounded above and up on both sides by ``glu_limit``: g sigmoid(1.702 g) (u + 1)) |
     "swiglu_quant" (returns (q, scale_t)).
-    fp32 operands run a plain fp32 kernel (dense, "store" and "geglu" only).
+    fp32 operands run a plain fp32 kernel ("store", "geglu" and "clamped_glu").
     """
     if out_dtype is None:
         out_dtype = torch.bfloat16 if (x.dtype == FP8 or x.is_cuda) else x.dtype
     if not x.is_cuda:
         return gemm_ref(x, w, w_scale=w_scale, x_scale=x_scale, seg_start=seg_start, seg_len=seg_len,
-                        epi=epi, row_scale=row_scale, out_dtype=out_dtype)
+                        epi=epi, row_scale=row_scale, out_dtype=out_dtype, glu_limit=glu_limit)
     L = nat.lib()
     if x.dtype == torch.float32:
-        return _gemm_f32(x, w, epi, seg_len, row_scale, out)
+        return _gemm_f32(x, w, epi, seg_start, seg_len, row_scale, out, glu_limit)
     if w.dim() == 2:
         w = w.unsqueeze(0)
     G, n_w, K = w.shape
@@ -148,9 +157,10 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
         assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     e = _EPI[epi]
     n_out = n_w if e == 0 else n_w // 2
-    if e == 3 and n_out % 128 != 0:
-        from .layer_list import gelu_mul
-        return gelu_mul(gemm(x, w, seg_start=seg_start, seg_len=seg_len, row_scale=row_scale, bn=bn, t_hint=t_hint), n_out, n_out)
+    if e in (3, 4) and n_out % 128 != 0:
+        from .layer_list import gated_mul
+        return gated_mul(gemm(x, w, seg_start=seg_start, seg_len=seg_len, row_scale=row_scale, bn=bn, t_hint=t_hint), n_out, n_out,
+                         epi, glu_limit)
     if e == 1 and n_out % 128 != 0:
         # the fused SwiGLU epilogue pairs 128-row gate and up blocks; odd widths (e.g. 10944) take the plain GEMM
         # and a separate activation kernel
@@ -173,7 +183,7 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
     # group on (vector stores, N = 256 tiles); below that, and for the split-K fp32 router GEMM, tokens stay on N.
     rows_hint = t_hint if (seg_len is not None and t_hint > 0) else T
     if tm_ok and e != 2 and kind == 0 and rows_hint >= 64 and not out_f32 and bn == 0:
-        _tm2(0, e, w, x, out, G, n_out, K, T, seg_start, seg_len, None, None, 0, None, row_scale)
+        _tm2(0, e, w, x, out, G, n_out, K, T, seg_start, seg_len, None, None, 0, None, row_scale, glu_limit=glu_limit)
         return out
     if tm_ok and kind == 1:
         _tm2(1, e, w, x, out, G, n_out, K, T, seg_start, seg_len, w_scale, x_scale, out_f32, out_scale, row_scale)
@@ -186,25 +196,31 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
         nat.ptr(x_scale), nat.c_int(x_scale.shape[1] if x_scale is not None else 0),
         nat.c_int(out.stride(0)), nat.c_int(out_f32), nat.ptr(out_scale),
         nat.c_int(out_scale.shape[1] if out_scale is not None else 0), nat.ptr(row_scale),
-        nat.c_int(0), nat.c_int(0), nat.c_int(x.stride(0)), nat.c_int(bn), nat.c_int(t_hint), nat.ptr(nat.status_buffer(x.device)), nat.stream())
+        nat.c_int(0), nat.c_int(0), nat.c_int(x.stride(0)), nat.c_int(bn), nat.c_int(t_hint), nat.c_float(glu_limit),
+        nat.ptr(nat.status_buffer(x.device)), nat.stream())
     nat.check_rc(rc, "omni_gemm")
     if e == 2:
         return out, out_scale
     return out
 
 
-def _gemm_f32(x, w, epi, seg_len, row_scale, out):
-    assert w.dtype == torch.float32 and w.dim() == 2 and seg_len is None and row_scale is None and epi in ("store", "geglu")
-    assert x.shape[1] == w.shape[1] and x.stride(1) == 1 and w.stride(1) == 1
-    T, n = x.shape[0], w.shape[0]
+def _gemm_f32(x, w, epi, seg_start, seg_len, row_scale, out, glu_limit):
+    assert w.dtype == torch.float32 and epi in ("store", "geglu", "clamped_glu") and w.is_contiguous()
+    assert x.shape[1] == w.shape[-1] and x.stride(1) == 1 and (w.dim() == 2 or seg_len is not None)
+    T, n = x.shape[0], w.shape[-2]
     y = out if out is not None and epi == "store" else torch.empty(T, n, dtype=torch.float32, device=x.device)
-    rc = nat.lib().omni_gemm_f32(nat.ptr(x), nat.ptr(w), nat.ptr(y), nat.c_int(T), nat.c_int(n), nat.c_int(x.shape[1]),
-                                 nat.c_int(x.stride(0)), nat.c_int(w.stride(0)), nat.c_int(y.stride(0)), nat.stream())
-    nat.check_rc(rc, "omni_gemm_f32")
-    if epi == "geglu":
-        from .layer_list import gelu_mul
-        return gelu_mul(y, n // 2, n // 2)
+    _f32_call(x, w, y, T, n, x.shape[1], 1 if w.dim() == 2 else w.shape[0], seg_start, seg_len, row_scale, 0, 0)
+    if epi != "store":
+        from .layer_list import gated_mul
+        return gated_mul(y, n // 2, n // 2, epi, glu_limit)
     return y
+
+
+def _f32_call(x, w, y, T, n, K, G, seg_start, seg_len, row_scale, x_group_col, out_group_col):
+    rc = nat.lib().omni_gemm_f32(nat.ptr(x), nat.ptr(w), nat.ptr(y), nat.c_int(T), nat.c_int(n), nat.c_int(K), nat.c_int(x.stride(0)),
+                                 nat.c_int(y.stride(0)), nat.c_int(G), nat.ptr(seg_start), nat.ptr(seg_len), nat.ptr(row_scale),
+                                 nat.c_int(x_group_col), nat.c_int(out_group_col), nat.stream())
+    nat.check_rc(rc, "omni_gemm_f32")
 
 
 def bmm_heads_ref(x, w):
@@ -227,11 +243,15 @@ def bmm_heads(x, w, out=None, out_col_offset=0):
             return y
         out[:, :, out_col_offset:out_col_offset + N] = y
         return out
-    assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous()
-    assert x.stride(2) == 1 and x.stride(0) == H * x.stride(1), "x must be a [T, H, Dx] buffer view"
+    assert x.dtype == w.dtype and w.is_contiguous()
+    assert x.stride(2) == 1 and x.stride(0) >= H * x.stride(1), "x must be a [T, H, Dx] buffer view"
     if out is None:
         out = torch.empty(T, H, N, dtype=x.dtype, device=x.device)
     assert out.stride(2) == 1 and out.stride(0) == H * out.stride(1)
+    if x.dtype == torch.float32:
+        _f32_call(x, w, out[:, :, out_col_offset:], T, N, K, H, None, None, None, x.stride(1), out.stride(1))
+        return out
+    assert x.dtype == torch.bfloat16
     base_out = out[:, :, out_col_offset:] if out_col_offset else out
     if (T >= 64 and N % 8 == 0 and out.stride(0) % 8 == 0 and out.stride(1) % 8 == 0 and base_out.data_ptr() % 16 == 0):
         _tm2(0, 0, w, x, base_out, H, N, K, T, None, None, None, None, 0, None, None,
@@ -241,7 +261,7 @@ def bmm_heads(x, w, out=None, out_col_offset=0):
         nat.c_int(0), nat.c_int(0), nat.ptr(w), nat.ptr(x), nat.ptr(base_out), nat.c_int(H), nat.c_int(N), nat.c_int(K),
         nat.c_int(T), nat.c_int(T), nat.ptr(None), nat.ptr(None), nat.ptr(None), nat.ptr(None), nat.c_int(0),
         nat.c_int(out.stride(0)), nat.c_int(0), nat.ptr(None), nat.c_int(0), nat.ptr(None),
-        nat.c_int(x.stride(1)), nat.c_int(out.stride(1)), nat.c_int(x.stride(0)), nat.c_int(0), nat.c_int(T),
+        nat.c_int(x.stride(1)), nat.c_int(out.stride(1)), nat.c_int(x.stride(0)), nat.c_int(0), nat.c_int(T), nat.c_float(0.0),
         nat.ptr(nat.status_buffer(x.device)), nat.stream())
     nat.check_rc(rc, "omni_gemm(bmm_heads)")
     return out

@@ -13,6 +13,7 @@ import torch
 import torch.nn.functional as F
 
 from . import _native as nat
+from .gemm import clamped_glu_ref
 
 
 def pad8(n: int) -> int:
@@ -94,14 +95,15 @@ def _rotate_half_ref(x, cos_sin, positions, rot):
 
 def qk_norm_rope_cache(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, positions, slots, k_cache, v_cache):
     """``qkv`` rows are q heads | k heads | v heads (``hkv=0``: q only).  RMSNorm over the whole q and the whole k
-    projection, rotate-half RoPE on the first ``rot`` dimensions of every head; q in place, k and v into the caches
+    projection (``q_w=None``: none), rotate-half RoPE on the first ``rot`` dimensions of every head; q in place, k and v into the caches
     [blocks, block, hkv, d] at ``slots`` (-1: not stored)."""
     T, nq, nk = qkv.shape[0], hq * dk, hkv * dk
     if not qkv.is_cuda:
-        q = rms_ref(qkv[:, :nq].float(), q_w, eps).view(T, hq, dk)
+        norm = (lambda x, w: x) if q_w is None else (lambda x, w: rms_ref(x, w, eps))
+        q = norm(qkv[:, :nq].float(), q_w).view(T, hq, dk)
         qkv[:, :nq] = _rotate_half_ref(q, cos_sin, positions, rot).reshape(T, nq).to(qkv.dtype)
         if hkv:
-            k = rms_ref(qkv[:, nq:nq + nk].float(), k_w, eps).view(T, hkv, dk)
+            k = norm(qkv[:, nq:nq + nk].float(), k_w).view(T, hkv, dk)
             k = _rotate_half_ref(k, cos_sin, positions, rot)
             ok = slots >= 0
             k_cache.view(-1, hkv, dk)[slots[ok]] = k[ok].to(k_cache.dtype)
@@ -116,7 +118,7 @@ def qk_norm_rope_cache(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, positi
 
 
 # ----------------------------------------------------------------------------- windowed attention over the paged cache
-def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, out):
+def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out):
     hq, dk = q.shape[1], q.shape[2]
     bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     kf, vf = k_cache.view(-1, hkv, dk), v_cache.view(-1, hkv, dv)
@@ -131,36 +133,40 @@ def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_t
         k = kf[rows].float().repeat_interleave(rep, 1)
         v = vf[rows].float().repeat_interleave(rep, 1)
         s = torch.einsum("hd,lhd->hl", q[t].float(), k) * scale
-        o = torch.einsum("hl,lhd->hd", torch.softmax(s, -1), v)
+        if sink is not None:
+            s = torch.cat([s, sink[:, None]], 1)
+        o = torch.einsum("hl,lhd->hd", torch.softmax(s, -1)[:, :len(pos)], v) * out_scale
         out[t, :hq * dv] = o.reshape(-1).to(out.dtype)
     return out
 
 
 def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_table, seq_lens, scale, window=0, cu_q=None,
-                    max_q=1, max_seq_len=0, any_shape=False):
+                    max_q=1, max_seq_len=0, sink=None, out_scale=1.0, out=None, any_shape=False):
     """q [T, hq, dk] (rows of any pitch) against the cached keys of the rows' requests, each row seeing the ``window``
-    positions up to its own (0: all of them).  Returns [T, pad8(hq * dv)].
+    positions up to its own (0: all of them).  ``sink`` [hq] fp32: exp(sink) is one more term of the head's softmax
+    denominator; ``out_scale`` multiplies the result.  Returns [T, pad8(hq * dv)], or writes the first columns of ``out``.
 
     bf16 portions of prompts run on tcgen05 (``omni_fmha_paged``), bf16 single tokens on the split-KV decode kernel; fp32
     and head shapes those two do not take - or ``any_shape`` - go to ``omni_attn_any``."""
     T, hq, dk = q.shape
     bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
-    ld = pad8(hq * dv)
-    alloc = torch.empty if ld == hq * dv else torch.zeros
-    out = alloc(T, ld, dtype=q.dtype, device=q.device)
+    if out is None:
+        ld = pad8(hq * dv)
+        out = (torch.empty if ld == hq * dv else torch.zeros)(T, ld, dtype=q.dtype, device=q.device)
+    ld = out.stride(0)
     if not q.is_cuda:
-        return paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, out)
+        return paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out)
     assert q.stride(2) == 1 and q.stride(1) == dk and k_cache.dtype == q.dtype and block_table.stride(1) == 1
     f32 = _f32(q)
     lib = nat.lib()
-    tc = not any_shape and not f32 and dk % 8 == 0 and dv % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+    tc = not any_shape and not f32 and ld % 8 == 0 and out.data_ptr() % 16 == 0 and dk % 8 == 0 and dv % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
     if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0:
         rc = lib.omni_fmha_paged(
             nat.ptr(q), nat.c_int64(T), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache),
             nat.c_int64(k_cache.shape[0] * bs), nat.ptr(cu_q), nat.ptr(seq_lens), nat.ptr(block_table),
             nat.c_int(block_table.stride(0)), nat.c_int(cu_q.shape[0] - 1), nat.c_int(max_q), nat.c_int(hq), nat.c_int(hkv),
-            nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(out), nat.c_int(ld),
-            nat.ptr(nat.status_buffer(q.device)), nat.stream())
+            nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(sink), nat.c_float(out_scale),
+            nat.ptr(out), nat.c_int(ld), nat.ptr(nat.status_buffer(q.device)), nat.stream())
         nat.check_rc(rc, "omni_fmha_paged")
         return out
     if tc and cu_q is None and dk <= 256 and dv <= 256:
@@ -175,30 +181,32 @@ def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_ta
         rc = lib.omni_gqa_paged_decode_window(
             nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.ptr(block_table),
             nat.c_int(block_table.stride(0)), nat.ptr(seq_lens), nat.c_int(T), nat.c_int(hq), nat.c_int(hkv), nat.c_int(dk),
-            nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.c_int(splits), nat.ptr(o_part),
-            nat.ptr(lse), nat.ptr(out), nat.c_int(ld), nat.stream())
+            nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(sink), nat.c_float(out_scale),
+            nat.c_int(splits), nat.ptr(o_part), nat.ptr(lse), nat.ptr(out), nat.c_int(ld), nat.stream())
         nat.check_rc(rc, "omni_gqa_paged_decode_window")
         return out
     rc = lib.omni_attn_any(
         nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.ptr(positions), nat.ptr(q_to_seq),
         nat.ptr(slots), nat.ptr(block_table), nat.c_int(block_table.stride(0)), nat.c_int(T), nat.c_int(hq), nat.c_int(hkv),
-        nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(out), nat.c_int(ld),
-        nat.c_int(f32), nat.stream())
+        nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(sink), nat.c_float(out_scale),
+        nat.ptr(out), nat.c_int(ld), nat.c_int(f32), nat.stream())
     nat.check_rc(rc, "omni_attn_any")
     return out
 
 
 # ----------------------------------------------------------------------------- gated feed-forward
-def gelu_mul(x, inter, up_off):
-    """gelu(x[:, :inter]) * x[:, up_off:up_off + inter] -> [T, pad8(inter)]."""
+def gated_mul(x, inter, up_off, kind="geglu", limit=0.0):
+    """act(x[:, :inter], x[:, up_off:up_off + inter]) -> [T, pad8(inter)]; kinds as the gated epilogues of ``ops.gemm``."""
     T, ld = x.shape[0], pad8(inter)
     if not x.is_cuda:
         g, u = x[:, :inter].float(), x[:, up_off:up_off + inter].float()
-        return F.pad(F.gelu(g, approximate="tanh") * u, (0, ld - inter)).to(x.dtype)
+        y = F.gelu(g, approximate="tanh") * u if kind == "geglu" else clamped_glu_ref(g, u, limit)
+        return F.pad(y, (0, ld - inter)).to(x.dtype)
     out = torch.empty(T, ld, dtype=x.dtype, device=x.device)
-    rc = nat.lib().omni_gelu_mul(nat.ptr(x), nat.c_int(x.stride(0)), nat.c_int(up_off), nat.ptr(out), nat.c_int(ld),
-                                 nat.c_int(T), nat.c_int(inter), nat.c_int(_f32(x)), nat.stream())
-    nat.check_rc(rc, "omni_gelu_mul")
+    rc = nat.lib().omni_gated_mul(nat.ptr(x), nat.c_int(x.stride(0)), nat.c_int(up_off), nat.ptr(out), nat.c_int(ld),
+                                  nat.c_int(T), nat.c_int(inter), nat.c_int({"geglu": 0, "clamped_glu": 1}[kind]),
+                                  nat.c_float(limit), nat.c_int(_f32(x)), nat.stream())
+    nat.check_rc(rc, "omni_gated_mul")
     return out
 
 

@@ -149,6 +149,12 @@ def moe_permute(x, ids, w, e_lo, e_local, quant=False, align=16, capacity=None, 
                                    nat.ptr(row_of), nat.ptr(row_w), nat.ptr(None), nat.stream())
         nat.check_rc(rc, "omni_moe_scatter_q8")
         return MoePermutation(xq, xs, seg_start, seg_len, row_of, row_w, total)
+    if x.dtype == torch.float32:
+        rc = L.omni_moe_scatter_f32(nat.ptr(x), nat.c_int(H), nat.ptr(ids), nat.ptr(w), nat.ptr(pos), nat.c_int(n), nat.c_int(k),
+                                    nat.c_int(e_lo), nat.ptr(seg_start), nat.ptr(seg_len), nat.ptr(xp), nat.ptr(row_of),
+                                    nat.ptr(row_w), nat.stream())
+        nat.check_rc(rc, "omni_moe_scatter_f32")
+        return MoePermutation(xp, None, seg_start, seg_len, row_of, row_w, total)
     rc = L.omni_moe_scatter(nat.ptr(x), nat.c_int(H), nat.ptr(ids), nat.ptr(w), nat.ptr(pos), nat.c_int(n),
                             nat.c_int(k), nat.c_int(e_lo), nat.ptr(seg_start), nat.ptr(seg_len), nat.ptr(xp),
                             nat.ptr(xq), nat.ptr(xs), nat.c_int(capacity), nat.ptr(row_of), nat.ptr(row_w),

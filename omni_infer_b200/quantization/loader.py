@@ -292,6 +292,16 @@ def iter_safetensors(model_dir: str):
                 yield k, sf.get_tensor(k)
 
 
+def safetensors_shapes(model_dir: str) -> dict:
+    """{tensor: shape} of every *.safetensors shard, from the headers."""
+    out: dict = {}
+    for f in sorted(Path(model_dir).glob("*.safetensors")):
+        with open(f, "rb") as fh:
+            head = json.loads(fh.read(int.from_bytes(fh.read(8), "little")))
+        out.update({k: tuple(v["shape"]) for k, v in head.items() if k != "__metadata__"})
+    return out
+
+
 def load_quant_description(model_dir: str) -> dict:
     """``quant_model_description.json`` of the int8 compressed-tensors layout
     (omni/quantization/compressed_tensors/compressed_tensors.py:66)."""
@@ -398,7 +408,9 @@ def init_random_weights(model, seed: int = 0, std: float = 0.02) -> None:
                 fill(p[slot], sp[slot] if sp is not None else None, g)
             continue
         g = gen(p.device, name)
-        if "norm" in name and p.dim() == 1:
+        if getattr(p, "init_value", None) is not None:
+            p.copy_(torch.as_tensor(p.init_value, dtype=p.dtype))
+        elif "norm" in name and p.dim() == 1:
             p.fill_(1.0)
         elif name.endswith("bias") and p.dim() == 1 and "e_score" not in name:
             p.zero_()
