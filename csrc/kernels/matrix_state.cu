@@ -213,7 +213,10 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
       if (p.vec) {
         done = true;
 #pragma unroll
-        for (int j = 0; j < NV; ++j) k.a[j] = k.b[j] = 0.f;
+        for (int j = 0; j < NV; ++j) {
+          k.a[j] = k.b[j] = 0.f;
+          if constexpr (WKV) k.z[j] = 0.f;
+        }
         if (lane * NV < p.N) {
           load_vec<NV>(ar + lane * NV, k.a);
           load_vec<NV>(br + lane * NV, k.b);

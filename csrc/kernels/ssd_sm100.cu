@@ -16,6 +16,13 @@
 // diagonal block a warp's 32 rows then need no exponential per element: 2^(cum_i - cp_j) = 2^(cum_i - cum_b) g_j, both
 // factors at most 1 (times dt) and the second shared by all rows.  All of it is in log2 units.
 //
+// The matrix memory of xLSTM (MEM) is the same scheme with C = q, B = k, x = v, and its own pre-pass (matrix_state.cu: gates):
+// with b the running sum of the log forget gates, i the log input gate and m the running maximum,
+//   M = SC o exp(b_i - m_i + i_j - b_j) N^-1/2,   y = YD + exp(b_i + m_in - m_i) N^-1/2 YO,   S <- exp(b_end + m_in - m_end) S + ST
+// so `cum` holds b - m, cp = b - i, the factor of YO and S has m_in (m before the chunk) added, and blocks left of the diagonal
+// take the largest i - b of the block as the reference between their two factors.  The CTA of the first 64 columns also moves
+// the normaliser n (the last state row) and adds up n . q: row sums of M beside the dot products of q with n, in fp32.
+//
 // One CTA walks the chunks of its request.  Warps: 0 TMA producer (two stages of C, B, x, cp, g), 1 MMA issue, 2..9 scores ->
 // M and the output rows (thread = token and half of the columns), 10..17 W and the state (thread = token, then state row, and
 // half of the columns).  Every wait is bounded.
@@ -40,6 +47,9 @@ struct SsdParams {
   int H, P, N, G;
   int min_rows;              // requests with fewer rows are left to another kernel
   float *cum, *cp, *g;       // [chunks, H, 128]; chunk c of request r is row cu_q[r] / 128 + r + c
+  const float *gmax, *m_in;  // MEM: [chunks, H, 4], [chunks, H]
+  float* den;                // MEM: [T, H], zeroed: n . q
+  float log2_scale;          // MEM: of the factor on q
   OmniStatus* status;
 };
 
@@ -51,7 +61,8 @@ constexpr int SQ_S = SQ_W + 2 * SQ_TILE;       // S hi, S lo
 constexpr int SQ_F = SQ_S + 2 * SQ_TILE;       // two stages of cp and g
 constexpr int SQ_FB = SQ * 4;                  // bytes of one such array
 constexpr int SQ_BAR = SQ_F + 4 * SQ_FB;
-constexpr int SQ_SMEM = SQ_BAR + 192;
+constexpr int SQ_N = SQ_BAR + 192;             // MEM: n
+constexpr int SQ_SMEM = SQ_N + SQ_FB;
 static_assert(SQ_SMEM <= 232448, "shared memory of one CTA");
 constexpr int SQ_THREADS = 576;
 // TMEM columns: SC / M two buffers of 128, YO two of 64, YD, ST.  M takes the columns of the scores it came from: 16 tokens
@@ -142,14 +153,17 @@ __global__ void __launch_bounds__(SQ) ssd_decay_kernel(const SsdParams p) {
   }
 }
 
+template <bool MEM>
 __global__ void __launch_bounds__(SQ_THREADS, 1)
-ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_constant__ CUtensorMap tmap_x, const SsdParams p) {
+ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid_constant__ CUtensorMap tmap_b,
+                 const __grid_constant__ CUtensorMap tmap_x, const SsdParams p) {
   const int pt = blockIdx.x, h = blockIdx.y, r = blockIdx.z;
   const int row0 = p.cu_q[r], n_rows = p.cu_q[r + 1] - row0;
   const int slot = p.state_slots[r];
   if (n_rows <= 0 || n_rows < p.min_rows || slot < 0) return;      // uniform, before any barrier / TMEM use
   const int p0 = pt * 64, pw = min(64, p.P - p0);
-  const int g = h / (p.H / p.G);
+  const int g = MEM ? h : h / (p.H / p.G);
+  const bool own_n = MEM && pt == 0;
   const int n = (n_rows + SQ - 1) / SQ;
   const int nch = (p.N + 63) / 64, ksn = (p.N + 15) / 16;          // 64-wide tiles and 16-wide steps of the state size
   const size_t arr0 = ((size_t)(row0 / SQ + r) * p.H + h) * SQ, arr_step = (size_t)p.H * SQ;
@@ -158,8 +172,8 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
   uint64_t* bars = (uint64_t*)(sq_smem + SQ_BAR);
   uint64_t *full = bars, *empty = bars + 2, *sc_full = bars + 4;   // two each
   uint64_t *m_full = bars + 6, *w_full = bars + 7, *st_full = bars + 8, *s_full = bars + 9, *yo_done = bars + 10,
-           *y_full = bars + 11, *y_empty = bars + 12;
-  uint32_t* tmem_slot = (uint32_t*)(bars + 13);
+           *y_full = bars + 11, *y_empty = bars + 12, *n_full = bars + 13;
+  uint32_t* tmem_slot = (uint32_t*)(bars + 14);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -168,6 +182,7 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
     for (int s = 0; s < 2; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); mbar_init(&sc_full[s], 1); }
     mbar_init(m_full, 8); mbar_init(w_full, 8); mbar_init(st_full, 1); mbar_init(s_full, 8);
     mbar_init(yo_done, 1); mbar_init(y_full, 1); mbar_init(y_empty, 8);
+    if (MEM) mbar_init(n_full, 8);
     *abort_flag = aligned ? 0 : (0x40000000 | (51 << 16));
     mbar_fence_init();
   }
@@ -190,8 +205,8 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
         uint8_t* st = sq_smem + s * SQ_STAGE;
         mbar_expect_tx(&full[s], (2 * nch + 1) * SQ_TILE + 2 * SQ_FB);
         for (int k = 0; k < nch; ++k) {
-          tma_load_3d(st + k * SQ_TILE, &tmap_bc, &full[s], k * 64, p.G + g, row);
-          tma_load_3d(st + (2 + k) * SQ_TILE, &tmap_bc, &full[s], k * 64, g, row);
+          tma_load_3d(st + k * SQ_TILE, &tmap_c, &full[s], k * 64, MEM ? h : p.G + g, row);
+          tma_load_3d(st + (2 + k) * SQ_TILE, &tmap_b, &full[s], k * 64, g, row);
         }
         tma_load_3d(st + 4 * SQ_TILE, &tmap_x, &full[s], p0, h, row);
         sq_bulk_load(sq_smem + SQ_F + s * 2 * SQ_FB, p.cp + arr0 + c * arr_step, SQ_FB, &full[s]);
@@ -262,11 +277,14 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
     // ------------------------------------------------------------------ scores -> M, output rows
     const int qd = warp & 3, i = qd * 32 + lane, half = (warp - 2) >> 2;
     const uint32_t la = tmem + ((uint32_t)(qd * 32) << 16);
-    const float Dh = p.D[h];
+    const float Dh = MEM ? 0.f : p.D[h];
     const float* cumg = p.cum + arr0;
-    float ci = cumg[i], cb[3];                           // this row's sum and those at the ends of the first three blocks
+    const float* gm = MEM ? p.gmax + ((size_t)(row0 / SQ + r) * p.H + h) * 4 : nullptr;
+    const float* min_g = MEM ? p.m_in + (size_t)(row0 / SQ + r) * p.H + h : nullptr;
+    // this row's sum and the references of the first three blocks: the sums at their ends, or minus their largest i - b
+    float ci = cumg[i], cb[3], mi = MEM ? min_g[0] : 0.f;
 #pragma unroll
-    for (int b = 0; b < 3; ++b) cb[b] = cumg[b * 32 + 31];
+    for (int b = 0; b < 3; ++b) cb[b] = MEM ? -gm[b] : cumg[b * 32 + 31];
     float e_prev = 0.f;
     auto output = [&](int c, float e) -> bool {          // rows of chunk c: YD + e YO, 32 columns
       if (!mbar_wait(y_full, c & 1, abort_flag, p.status, 57, c)) return false;
@@ -300,12 +318,14 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
     };
     bool ok = true;
     for (int c = 0; c < n; ++c) {
-      const float my = ci, c0 = cb[0], c1 = cb[1], c2 = cb[2];
+      const float my = MEM ? ci + p.log2_scale : ci, c0 = cb[0], c1 = cb[1], c2 = cb[2];
+      const float my_in = MEM ? my + mi : my;
       if (c + 1 < n) {                                   // the next chunk's, on their way while this one is worked on
         const float* nx = cumg + (c + 1) * arr_step;
         ci = nx[i];
 #pragma unroll
-        for (int b = 0; b < 3; ++b) cb[b] = nx[b * 32 + 31];
+        for (int b = 0; b < 3; ++b) cb[b] = MEM ? -gm[(size_t)(c + 1) * p.H * 4 + b] : nx[b * 32 + 31];
+        if (MEM) mi = min_g[(size_t)(c + 1) * p.H];
       }
       if (!mbar_wait(&full[c & 1], (c >> 1) & 1, abort_flag, p.status, 58, c) ||
           !mbar_wait(&sc_full[c & 1], (c >> 1) & 1, abort_flag, p.status, 59, c)) { ok = false; break; }
@@ -314,6 +334,7 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
       const float* gs = cps + SQ;
       const uint32_t col0 = la + TC_SC + (c & 1) * 128 + half * 16;
       uint32_t s[4][16];
+      float rs = 0.f;                                    // MEM: sum of this thread's part of the row of M
 #pragma unroll
       for (int b = 0; b < 4; ++b) {
         if (b == 0) sq_tmem_ld_2x16(col0, col0 + 32, s[0], s[1]);          // blocks right of the diagonal are not used
@@ -327,9 +348,11 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
 #pragma unroll
           for (int j = 0; j < 16; j += 4) {
             const float4 gj = *reinterpret_cast<const float4*>(gs + b * 32 + j);
-            sq_split2(__uint_as_float(s[b][j]) * (f * gj.x), __uint_as_float(s[b][j + 1]) * (f * gj.y), hi[j / 2], lo[j / 2]);
-            sq_split2(__uint_as_float(s[b][j + 2]) * (f * gj.z), __uint_as_float(s[b][j + 3]) * (f * gj.w), hi[j / 2 + 1],
-                      lo[j / 2 + 1]);
+            const float m0 = __uint_as_float(s[b][j]) * (f * gj.x), m1 = __uint_as_float(s[b][j + 1]) * (f * gj.y);
+            const float m2 = __uint_as_float(s[b][j + 2]) * (f * gj.z), m3 = __uint_as_float(s[b][j + 3]) * (f * gj.w);
+            if (MEM) rs += (m0 + m1) + (m2 + m3);
+            sq_split2(m0, m1, hi[j / 2], lo[j / 2]);
+            sq_split2(m2, m3, hi[j / 2 + 1], lo[j / 2 + 1]);
           }
         } else {
           const int d = lane - half * 16;                // column of the diagonal among these 16
@@ -340,8 +363,9 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               m[e] = j + e <= d ? __uint_as_float(s[b][j + e]) * sq_ex2(my - m[e]) : 0.f;
-              if (j + e == d) m[e] += Dh;
+              if (!MEM && j + e == d) m[e] += Dh;
             }
+            if (MEM) rs += (m[0] + m[1]) + (m[2] + m[3]);
             sq_split2(m[0], m[1], hi[j / 2], lo[j / 2]);
             sq_split2(m[2], m[3], hi[j / 2 + 1], lo[j / 2 + 1]);
           }
@@ -352,10 +376,27 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
       }
       tmem_st_wait();
       tc_fence_before();
+      if (own_n) {                                       // n . q of this row: before m_full, which lets go of the chunk's tiles
+        if (!mbar_wait(n_full, c & 1, abort_flag, p.status, 64, c)) { ok = false; break; }
+        const float* sn = reinterpret_cast<const float*>(sq_smem + SQ_N);
+        float dot = 0.f;
+        for (int k8 = half; k8 * 8 < p.N; k8 += 2) {
+          const uint4 q8 = *reinterpret_cast<const uint4*>(sq_smem + (c & 1) * SQ_STAGE + (k8 >> 3) * SQ_TILE + sq_off(i, k8 & 7));
+          const float4 na = *reinterpret_cast<const float4*>(sn + k8 * 8), nb = *reinterpret_cast<const float4*>(sn + k8 * 8 + 4);
+          const uint32_t v[4] = {q8.x, q8.y, q8.z, q8.w};
+          float2 f[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) f[e] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v[e]));
+          dot += (f[0].x * na.x + f[0].y * na.y) + (f[1].x * na.z + f[1].y * na.w) + (f[2].x * nb.x + f[2].y * nb.y) +
+                 (f[3].x * nb.z + f[3].y * nb.w);
+        }
+        const int t = c * SQ + i;
+        if (t < n_rows) atomicAdd(p.den + (size_t)(row0 + t) * p.H + h, fmaf(sq_ex2(my_in), dot, rs));      // two addends: order-free
+      }
       __syncwarp();
       if (lane == 0) mbar_arrive(m_full);
       if (c > 0 && !output(c - 1, e_prev)) { ok = false; break; }
-      e_prev = sq_ex2(my);
+      e_prev = sq_ex2(my_in);
     }
     if (ok) output(n - 1, e_prev);
   } else {
@@ -363,10 +404,24 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
     const int qd = warp & 3, i = qd * 32 + lane, half = (warp - 10) >> 2;      // token of the chunk, and row n of the state
     const uint32_t la = tmem + ((uint32_t)(qd * 32) << 16);
     const int q0 = half * 32, kn = i < p.N ? pw - q0 : 0;                      // columns of this half that exist
-    float* st = p.state + (((size_t)slot * p.H + h) * p.P + p0 + q0) * p.N + i;
+    const int PR = MEM ? p.P + 1 : p.P;
+    float* st = p.state + (((size_t)slot * p.H + h) * PR + p0 + q0) * p.N + i;
+    const bool fresh = p.positions[row0] == 0;
+    // MEM: a lane owns channel nc of n for half of the tokens (those with bit 2 of their number set or not)
+    const int nc = (warp - 10) * 16 + (lane & 15), nth = lane >> 4;
+    float* st_n = p.state + (((size_t)slot * p.H + h) * PR + p.P) * p.N + nc;
+    float n_now = 0.f, n_part = 0.f;
+    auto write_n = [&]() {
+      if (nth == 0) reinterpret_cast<float*>(sq_smem + SQ_N)[nc] = n_now;
+      __syncwarp();
+      if (lane == 0) mbar_arrive(n_full);
+    };
+    if (own_n) {
+      if (!fresh && nc < p.N) n_now = *st_n;
+      write_n();
+    }
     float S[32];
     {
-      const bool fresh = p.positions[row0] == 0;
 #pragma unroll
       for (int k = 0; k < 32; ++k) S[k] = (!fresh && k < kn) ? st[(size_t)k * p.N] : 0.f;
     }
@@ -387,6 +442,8 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
     write_state();
     const float* cend_g = p.cum + arr0 + SQ - 1;
     float cend = cend_g[0], cend_next = 0.f;
+    const float* min_g = MEM ? p.m_in + (size_t)(row0 / SQ + r) * p.H + h : nullptr;
+    const float* gm = MEM ? p.gmax + ((size_t)(row0 / SQ + r) * p.H + h) * 4 : nullptr;
     uint32_t wh[16], wl[16];                             // this token's W of the coming chunk
     auto prepare = [&](int c, float ce) -> bool {
       if (!mbar_wait(&full[c & 1], (c >> 1) & 1, abort_flag, p.status, 61, c)) return false;
@@ -405,6 +462,28 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
           sq_split2(f.x * w, f.y * w, wh[ch * 4 + e], wl[ch * 4 + e]);
         }
       }
+      if (own_n) {                                       // sum of w_j k_j; before w_full, which lets go of the chunk's tiles
+        n_part = 0.f;
+        if (nc < p.N) {
+          const uint8_t* kt = sq_smem + (c & 1) * SQ_STAGE + (2 + (nc >> 6)) * SQ_TILE + (nc & 7) * 2;
+          const float* gs = reinterpret_cast<const float*>(sq_smem + SQ_F + (c & 1) * 2 * SQ_FB) + SQ;
+#pragma unroll
+          for (int b = 0; b < 4; ++b) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j4 = 0; j4 < 32; j4 += 8) {
+              const int j = b * 32 + j4 + nth * 4;
+              const float4 gj = *reinterpret_cast<const float4*>(gs + j);
+              const float gv[4] = {gj.x, gj.y, gj.z, gj.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e)
+                acc = fmaf(gv[e], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(kt + sq_off(j + e, (nc >> 3) & 7))), acc);
+            }
+            n_part = fmaf(sq_ex2(ce + gm[(size_t)c * p.H * 4 + b]), acc, n_part);
+          }
+        }
+        n_part += __shfl_xor_sync(0xffffffffu, n_part, 16);
+      }
       return true;
     };
     bool ok = prepare(0, cend);
@@ -419,7 +498,8 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
       fence_proxy_async_smem();
       __syncwarp();
       if (lane == 0) mbar_arrive(w_full);
-      const float eend = sq_ex2(cend);
+      const float eend = sq_ex2(MEM ? cend + min_g[(size_t)c * p.H] : cend);
+      if (own_n) n_now = fmaf(eend, n_now, n_part);      // n after this chunk; the next prepare overwrites n_part
       if (c + 1 < n) {
         cend_next = cend_g[(c + 1) * arr_step];
         if (!prepare(c + 1, cend_next)) break;
@@ -438,6 +518,10 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
       if (c + 1 < n) {
         if (!mbar_wait(yo_done, c & 1, abort_flag, p.status, 63, c)) break;      // C S has read the old state
         write_state();
+        if (own_n) {
+          if (!mbar_wait(y_full, c & 1, abort_flag, p.status, 65, c)) break;     // every row has read the old n
+          write_n();
+        }
       }
       cend = cend_next;
     }
@@ -445,6 +529,7 @@ ssd_sm100_kernel(const __grid_constant__ CUtensorMap tmap_bc, const __grid_const
 #pragma unroll
       for (int k = 0; k < 32; ++k)
         if (k < kn) st[(size_t)k * p.N] = S[k];
+      if (own_n && nth == 0 && nc < p.N) *st_n = n_now;
     }
   }
 
@@ -489,7 +574,35 @@ extern "C" int omni_ssd_chunks(const void* xbc, int xbc_ld, long long rows, cons
   p.cum = scratch; p.cp = scratch + arr; p.g = scratch + 2 * arr;
   ssd_decay_kernel<<<dim3((max_q + SQ - 1) / SQ, B, (H + 7) / 8), SQ, 0, stream>>>(p);
   static bool configured[64] = {false};
-  if (int e = ensure_dyn_smem((const void*)ssd_sm100_kernel, SQ_SMEM, configured)) return e;
-  ssd_sm100_kernel<<<dim3((P + 63) / 64, H, B), SQ_THREADS, SQ_SMEM, stream>>>(tbc, tx, p);
+  if (int e = ensure_dyn_smem((const void*)ssd_sm100_kernel<false>, SQ_SMEM, configured)) return e;
+  ssd_sm100_kernel<false><<<dim3((P + 63) / 64, H, B), SQ_THREADS, SQ_SMEM, stream>>>(tbc, tbc, tx, p);
+  return (int)cudaGetLastError();
+}
+
+// Matrix memory over portions of prompts.  q, k, v [rows, ld] with head h at column h N / h N / h P; chunks: what omni_mlstm_gates
+// left (n_chunks = rows / 128 + B of them); state [slots, H, P + 1, N]; den [rows, H] zeroed; y = S^T q N^-1/2.
+extern "C" int omni_mlstm_chunks(const void* q, int q_ld, const void* k, int k_ld, const void* v, int v_ld, long long rows,
+                                 const float* chunks, int n_chunks, float* den, float scale, void* state, const int* cu_q,
+                                 const int64_t* positions, const int* state_slots, int B, int max_q, void* y, int y_ld, int H, int P,
+                                 int N, int min_rows, void* status, cudaStream_t stream) {
+  if (B <= 0 || rows <= 0 || max_q < min_rows) return 0;
+  if (H < 1 || B > 65535 || H > 65535 || !(scale > 0.f) || chunks == nullptr || n_chunks < rows / SQ + B) return -1;
+  if (P < 8 || P % 8 != 0 || N < 8 || N % 8 != 0 || N > 128 || (q_ld | k_ld | v_ld | y_ld) % 8 != 0) return -2;
+  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)y | (uintptr_t)chunks) % 16 != 0) return -3;
+  CUtensorMap tq, tk, tv;
+  if (make_tmap_3d(&tq, q, 2, N, H, (uint64_t)rows, (uint64_t)N * 2, (uint64_t)q_ld * 2, 64, 1, SQ, true)) return -10;
+  if (make_tmap_3d(&tk, k, 2, N, H, (uint64_t)rows, (uint64_t)N * 2, (uint64_t)k_ld * 2, 64, 1, SQ, true)) return -11;
+  if (make_tmap_3d(&tv, v, 2, P, H, (uint64_t)rows, (uint64_t)P * 2, (uint64_t)v_ld * 2, 64, 1, SQ, true)) return -12;
+  SsdParams p;
+  memset(&p, 0, sizeof(p));
+  const size_t arr = (size_t)n_chunks * H * SQ;
+  p.cum = const_cast<float*>(chunks); p.cp = p.cum + arr; p.g = p.cum + 2 * arr; p.gmax = p.cum + 3 * arr;
+  p.m_in = p.gmax + (size_t)n_chunks * H * 4; p.den = den; p.log2_scale = log2f(scale);
+  p.state = (float*)state; p.cu_q = cu_q; p.positions = positions; p.state_slots = state_slots;
+  p.y = (__nv_bfloat16*)y; p.y_ld = y_ld; p.H = H; p.P = P; p.N = N; p.G = H; p.min_rows = min_rows;
+  p.status = (OmniStatus*)status;
+  static bool configured[64] = {false};
+  if (int e = ensure_dyn_smem((const void*)ssd_sm100_kernel<true>, SQ_SMEM, configured)) return e;
+  ssd_sm100_kernel<true><<<dim3((P + 63) / 64, H, B), SQ_THREADS, SQ_SMEM, stream>>>(tq, tk, tv, p);
   return (int)cudaGetLastError();
 }

@@ -8,7 +8,7 @@ from torch import nn
 from .. import ops
 from ..models.config import MLSTMSpec, ParallelSpec, WkvSpec
 from ..ops.layer_list import pad8
-from ..ops.matrix_state import head_norm, mlstm_gates, mlstm_scan, wkv_scan
+from ..ops.matrix_state import CHUNK_MIN_ROWS, head_norm, mlstm_chunked, mlstm_gates, mlstm_scan, wkv_scan
 from ..ops.streams import tanh_split, token_shift
 from .common import AttnMetadata, PaddedLinear
 from .windowed_attention import WindowedAttention
@@ -58,7 +58,7 @@ class MLSTM(nn.Module):
         """u: this mixer's part of the projected rows, z: gates before their biases (fp32).  Writes scale * (o W_norm gate)."""
         s, where = self.spec, _ragged(md)
         S, m = state
-        chunks = False
+        chunks = u.is_cuda and md.is_prefill and mlstm_chunked(u.dtype, s.dim, s.vdim) and md.max_q >= CHUNK_MIN_ROWS
         gates = mlstm_gates(z, self.f_col, self.i_bias, self.f_bias, s.gate_cap, m, chunks=chunks, **where)
         y = mlstm_scan(u[:, :self.nk], u[:, self.k0:self.k0 + self.nk], u[:, self.v0:self.v0 + self.nv], gates, S, H=s.heads,
                        P=s.vdim, N=s.dim, **where, **_rows_of(md))

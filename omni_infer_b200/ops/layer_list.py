@@ -123,7 +123,7 @@ def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_t
     bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     kf, vf = k_cache.view(-1, hkv, dk), v_cache.view(-1, hkv, dv)
     rep = hq // hkv
-    out.zero_()
+    out[:, :hq * dv] = 0
     for t in range(q.shape[0]):
         if int(slots[t]) < 0:
             continue

@@ -62,6 +62,15 @@ def mlstm_gates(z, f_col, i_bias, f_bias, cap, m_state, *, positions, state_slot
     return MlstmGates(ka, m, den, buf, n_chunks)
 
 
+def mlstm_chunked(dtype, N: int, P: int) -> bool:
+    """Do portions of prompts run on tensor cores at these sizes?"""
+    return dtype == torch.bfloat16 and N % 8 == 0 and N <= 128 and P % 8 == 0
+
+
+def _tma(*ts) -> bool:
+    return all(t.stride(1) == 1 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in ts)
+
+
 def _rows(kind, a, a_scale, b, v, gates, z, w0, u, state, out, H, P, N, positions, state_slots, cu_q, max_rows):
     B = a.shape[0] if cu_q is None else cu_q.shape[0] - 1
     rc = nat.lib().omni_state_rows(
@@ -92,9 +101,18 @@ def mlstm_scan(q, k, v, gates, state, *, H, P, N, positions, state_slots, cu_q=N
                 out[t], gates.den[t] = y[:, :P].reshape(-1).to(out.dtype), y[:, P]
             state[slot] = S
         return out
-    max_rows = -1 if by_rows else 0
-    if cu_q is not None and not by_rows and gates.chunks is not None:
-        raise NotImplementedError
+    max_rows = 0
+    if cu_q is not None and not by_rows and gates.chunks is not None and mlstm_chunked(q.dtype, N, P) and _tma(q, k, v):
+        rc = nat.lib().omni_mlstm_chunks(
+            nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k), nat.c_int(k.stride(0)), nat.ptr(v), nat.c_int(v.stride(0)), nat.c_int64(T),
+            nat.ptr(gates.chunks), nat.c_int(gates.n_chunks), nat.ptr(gates.den), nat.c_float(scale), nat.ptr(state), nat.ptr(cu_q),
+            nat.ptr(positions), nat.ptr(state_slots), nat.c_int(cu_q.shape[0] - 1), nat.c_int(max_q or T), nat.ptr(out),
+            nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N), nat.c_int(CHUNK_MIN_ROWS),
+            nat.ptr(nat.status_buffer(q.device)), nat.stream())
+        nat.check_rc(rc, "omni_mlstm_chunks")
+        if min_q >= CHUNK_MIN_ROWS:
+            return out
+        max_rows = CHUNK_MIN_ROWS - 1
     _rows(0, q, scale, k, v, gates, None, None, None, state, out, H, P, N, positions, state_slots, cu_q, max_rows)
     return out
 
