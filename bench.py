@@ -44,9 +44,11 @@ def parse():
     ap.add_argument("--decode-ctx", type=int, default=-1,
                     help="context length at the middle of the timed steps; -1 = the config's mean decode context "
                          "(input + output / 2), 0 = time right after the prefill")
-    ap.add_argument("--layer-list", default=None, choices=["kernels", "model", "all"],
-                    help="instead of the headline: layer-list models (windowed attention + Mamba-2) beside the GQA model at equal "
-                         "sizes, per kernel and whole, one JSON line each")
+    ap.add_argument("--layer-list", default=None, 
+                    choices=["kernels", "model", "all", "fimudra-kernels", "fimudra-model", "fimudra"],
+                    help="instead of the headline: layer-list models (windowed attention + Mamba-2; fimudra: attention beside a "
+                         "matrix memory, WKV, expert mixtures) beside the closest models at equal sizes, per kernel and whole, one "
+                         "JSON line each")
     ap.add_argument("--no-breakdown", action="store_true", help="skip the untimed per-module timing step")
     ap.add_argument("--no-nccl-arm", action="store_true", help="skip the untimed NCCL all-to-all comparison steps (N > 1)")
     return ap.parse_args()
@@ -205,7 +207,10 @@ def main():
     if args.impl == "reference":
         return reference_arm(args)
     if args.layer_list:
-        from benchmarks.layer_list_bench import main as layer_list_main
+        if args.layer_list.startswith("fimudra"):
+            from benchmarks.fimudra_bench import main as layer_list_main
+        else:
+            from benchmarks.layer_list_bench import main as layer_list_main
         return layer_list_main(args.layer_list)
     import torch
     import torch.distributed as dist

@@ -57,7 +57,7 @@ ARCH_KERNELS = {
     "Forovik": ("attn_any", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "mamba2", "post_norm_ops",
                 "sampler_misc", "ssd_sm100"),
     "Fimudra": ("attn_any", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "matrix_state", "moe_route",
-                "post_norm_ops", "sampler_misc", "ssd_sm100", "stream_ops"),
+                "post_norm_ops", "sampler_misc", "ssd_sm100", "stream_ops", "wkv_chunk"),
 }
 
 

@@ -120,7 +120,7 @@ def _site_kernel(site: int) -> str:
     """Which kernel family a wait-site id belongs to (each family numbers its sites in its own decade)."""
     for lo, hi, name in ((1, 9, "weight-major GEMM"), (11, 19, "prefill attention"), (21, 29, "token-major GEMM"),
                          (31, 39, "MLA decode"), (41, 49, "TP collectives"),
-                         (51, 69, "Mamba-2 chunked scan"), (200, 299, "EP dispatch/combine")):
+                         (51, 69, "chunked scan (Mamba-2, matrix memory)"), (71, 79, "chunked WKV scan"), (200, 299, "EP dispatch/combine")):
         if lo <= site <= hi:
             return name
     return "an unnamed kernel"

@@ -1,7 +1,7 @@
 """Mixers whose state is a matrix per head, between their projections: the matrix memory of xLSTM (mLSTM) and WKV.
 
-CUDA tensors run ``csrc/kernels/matrix_state.cu`` (gates, token by token, norm) and ``ssd_sm100.cu`` (mLSTM portions of
-prompts on tcgen05); CPU tensors the fp32 references here.  Ragged batches as in :mod:`.layer_list`.
+CUDA tensors run ``csrc/kernels/matrix_state.cu`` (gates, token by token, norm), ``ssd_sm100.cu`` (mLSTM portions of prompts on
+tcgen05) and ``wkv_chunk.cu`` (WKV portions); CPU tensors the fp32 references here.  Ragged batches as in :mod:`.layer_list`.
 
 State: [slots, H, P, N] fp32 (N key size, P value size; the mLSTM's has one more row, its normaliser) and for the mLSTM
 m [slots, H], the running maximum of its log gates.  A request that starts at position 0 starts from zeros."""
@@ -136,7 +136,18 @@ def wkv_scan(r, k, v, z, w0, u, state, *, H, N, positions, state_slots, cu_q=Non
             state[slot] = S
         return out
     assert z.dtype == torch.float32
-    _rows(1, r, 1.0, k, v, None, z, w0, u, state, out, H, N, N, positions, state_slots, cu_q, 0)
+    max_rows = 0
+    if cu_q is not None and not by_rows and r.dtype == torch.bfloat16 and N % 8 == 0 and N <= 128 and _tma(v):
+        rc = nat.lib().omni_wkv_chunks(
+            nat.ptr(r), nat.c_int(r.stride(0)), nat.ptr(k), nat.c_int(k.stride(0)), nat.ptr(v), nat.c_int(v.stride(0)), nat.ptr(z),
+            nat.c_int(z.stride(0)), nat.ptr(w0), nat.ptr(u), nat.ptr(state), nat.ptr(cu_q), nat.ptr(positions), nat.ptr(state_slots),
+            nat.c_int(cu_q.shape[0] - 1), nat.c_int(max_q or T), nat.ptr(out), nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(N),
+            nat.c_int(CHUNK_MIN_ROWS), nat.ptr(nat.status_buffer(r.device)), nat.stream())
+        nat.check_rc(rc, "omni_wkv_chunks")
+        if min_q >= CHUNK_MIN_ROWS:
+            return out
+        max_rows = CHUNK_MIN_ROWS - 1
+    _rows(1, r, 1.0, k, v, None, z, w0, u, state, out, H, N, N, positions, state_slots, cu_q, max_rows)
     return out
 
 
