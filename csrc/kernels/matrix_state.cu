@@ -346,37 +346,52 @@ static int launch_state_rows(StateParams p, int B, cudaStream_t stream) {
 }
 
 // ------------------------------------------------------------------------------------------------ norm and gate
-// One warp per (token, head).  ACT 0: sigmoid gate, 1: silu gate.
-template <typename T, int V, int ACT>
+// LANES lanes per (token, head).  ACT 0: sigmoid gate, 1: silu gate.
+template <typename T, int V, int LANES, int ACT>
 __global__ void __launch_bounds__(256) head_norm_kernel(const T* __restrict__ y, int y_ld, const float* __restrict__ den,
                                                         const float* __restrict__ m, const T* __restrict__ gate, int gate_ld,
                                                         const float* __restrict__ w, float scale, T* __restrict__ out, int out_ld,
                                                         int rows, int H, int P, float eps) {
-  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-  const int lane = threadIdx.x & 31;
-  if (item >= (long long)rows * H) return;
-  const int t = (int)(item / H), h = (int)(item % H);
+  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / LANES;
+  const int lane = threadIdx.x & (LANES - 1);
+  const bool ok = item < (long long)rows * H;            // every lane takes part in the sums
+  const int t = ok ? (int)(item / H) : 0, h = ok ? (int)(item % H) : 0;
   const T* yr = y + (size_t)t * y_ld + h * P;
   const T* gr = gate + (size_t)t * gate_ld + h * P;
   T* o = out + (size_t)t * out_ld + h * P;
-  const float div = den ? 1.0f / (fmaxf(fabsf(den[item]), expf(-m[item])) + 1e-6f) : 1.0f;
-  float ss = 0.f;
-  for (int c = lane * V; c < P; c += 32 * V) {
+  const float div = (ok && den) ? 1.0f / (fmaxf(fabsf(den[item]), expf(-m[item])) + 1e-6f) : 1.0f;
+  float first[V], ss = 0.f;                              // the first vector stays in registers
+#pragma unroll
+  for (int i = 0; i < V; ++i) first[i] = 0.f;
+  if (ok && lane * V < P) load_vec<V>(yr + lane * V, first);
+#pragma unroll
+  for (int i = 0; i < V; ++i) { first[i] *= div; ss += first[i] * first[i]; }
+  for (int c = (LANES + lane) * V; ok && c < P; c += LANES * V) {
     float v[V];
     load_vec<V>(yr + c, v);
 #pragma unroll
     for (int i = 0; i < V; ++i) { v[i] *= div; ss += v[i] * v[i]; }
   }
-  const float r = 1.0f / sqrtf(warp_sum32(ss) / (float)P + eps) * div * scale;
-  for (int c = lane * V; c < P; c += 32 * V) {
-    float v[V], g[V], g2[V];
-    load_vec<V>(yr + c, v);
+#pragma unroll
+  for (int s = LANES / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  if (!ok) return;
+  const float r = 1.0f / sqrtf(ss / (float)P + eps) * scale;
+  auto finish = [&](int c, const float (&v)[V]) {
+    float g[V], g2[V], a[V];
     load_vec<V>(gr + c, g);
     load_vec<V>(w + h * P + c, g2);
 #pragma unroll
     for (int i = 0; i < V; ++i)
-      v[i] = v[i] * r * g2[i] * (ACT == 0 ? div_for<T>(1.0f, 1.0f + exp_for<T>(-g[i])) : silu_for<T>(g[i]));
-    store_vec<V>(o + c, v);
+      a[i] = v[i] * r * g2[i] * (ACT == 0 ? div_for<T>(1.0f, 1.0f + exp_for<T>(-g[i])) : silu_for<T>(g[i]));
+    store_vec<V>(o + c, a);
+  };
+  if (lane * V < P) finish(lane * V, first);
+  for (int c = (LANES + lane) * V; c < P; c += LANES * V) {
+    float v[V];
+    load_vec<V>(yr + c, v);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] *= div;
+    finish(c, v);
   }
 }
 
@@ -422,14 +437,19 @@ extern "C" int omni_head_norm(const void* y, int y_ld, const float* den, const f
                               cudaStream_t st) {
   if (rows <= 0) return 0;
   if (H < 1 || P < 1 || act < 0 || act > 1) return -1;
-  const long long blocks = ((long long)rows * H + 7) / 8;
   const size_t esz = f32 ? 4 : 2;
-  const bool v4 = P % 4 == 0 && y_ld % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 &&
-                  (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)out) & (4 * esz - 1)) == 0;
-#define HEAD_NORM(T, V, ACT)                                                                                                   \
-  head_norm_kernel<T, V, ACT><<<(unsigned)blocks, 256, 0, st>>>((const T*)y, y_ld, den, m, (const T*)gate, gate_ld,            \
-                                                                (const float*)w, scale, (T*)out, out_ld, rows, H, P, eps)
-#define HEAD_NORM_V(T, ACT) do { if (v4) HEAD_NORM(T, 4, ACT); else HEAD_NORM(T, 1, ACT); } while (0)
+  const bool v8 = P % 8 == 0 && y_ld % 8 == 0 && gate_ld % 8 == 0 && out_ld % 8 == 0 &&
+                  (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)out) & (esz == 4 ? 15 : 8 * esz - 1)) == 0;
+#define HEAD_NORM(T, V, LANES, ACT)                                                                                            \
+  head_norm_kernel<T, V, LANES, ACT><<<(unsigned)(((long long)rows * H * LANES + 255) / 256), 256, 0, st>>>(                   \
+      (const T*)y, y_ld, den, m, (const T*)gate, gate_ld, (const float*)w, scale, (T*)out, out_ld, rows, H, P, eps)
+#define HEAD_NORM_V(T, ACT)                            \
+  do {                                                 \
+    if (!v8) HEAD_NORM(T, 1, 32, ACT);                 \
+    else if (P <= 64) HEAD_NORM(T, 8, 8, ACT);         \
+    else if (P <= 128) HEAD_NORM(T, 8, 16, ACT);       \
+    else HEAD_NORM(T, 8, 32, ACT);                     \
+  } while (0)
   if (f32) { if (act == 0) HEAD_NORM_V(float, 0); else HEAD_NORM_V(float, 1); }
   else { if (act == 0) HEAD_NORM_V(bf16, 0); else HEAD_NORM_V(bf16, 1); }
 #undef HEAD_NORM_V

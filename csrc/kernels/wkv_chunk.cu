@@ -9,8 +9,8 @@
 // exponent that is taken here is a difference whose sign makes it at most zero.  A is made of 4 x 4 tiles: below the diagonal
 // tiles both sides refer to the tile's first row (8 exponentials for 16 products), on it every pair has its own.
 //
-// One CTA walks the chunks of one (request, head); two kinds of warps, two stages between them:
-//   prep   (4 warps) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
+// One CTA walks the chunks of one (request, head); two kinds of warps, four stages between them:
+//   prep   (two groups of 4 warps, alternate chunks) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
 //          the tiles of A with lanes over channels
 //   state  (one warp per 16 value columns) S^T in fp32 accumulators; O^T = S^T R^T + V^T A^T and S^T += V^T K on mma.sync, S^T being
 //          its own A operand.  A chunk of 16 tokens is too short for tcgen05: the chain from S to S would go through tensor memory
@@ -40,7 +40,9 @@ struct WkvParams {
 };
 
 constexpr int WK_L = 16;                           // tokens per chunk
-constexpr int WK_PREP = 4;                         // prep warps
+constexpr int WK_GROUPS = 2;                       // prep groups
+constexpr int WK_PREP = 4;                         // warps of one
+constexpr int WK_STAGES = 2 * WK_GROUPS;
 constexpr int WK_TP = 20;                          // floats per channel of the arrays [channel][token]
 constexpr int WK_APITCH = 48;                      // bytes per row of A
 template <int DP>
@@ -50,13 +52,13 @@ struct WkLayout {
   static constexpr int A_OFF = 5 * TILE;           // after R hi, R lo, K hi, K lo, V
   static constexpr int DS_OFF = A_OFF + 2 * WK_L * WK_APITCH;
   static constexpr int STAGE = DS_OFF + DP * 4;
-  static constexpr int T_OFF = 2 * STAGE;          // two buffers of r, k, c: [DP][WK_TP] floats each
+  static constexpr int T_OFF = WK_STAGES * STAGE;  // per group r, k, c: [DP][WK_TP] floats each
   static constexpr int T_ARR = DP * WK_TP * 4;
-  static constexpr int U_OFF = T_OFF + 6 * T_ARR;
+  static constexpr int U_OFF = T_OFF + WK_GROUPS * 3 * T_ARR;
   static constexpr int BAR_OFF = U_OFF + DP * 4;
-  static constexpr int SMEM = BAR_OFF + 64;
+  static constexpr int SMEM = BAR_OFF + 128;
   static constexpr int STATE_WARPS = DP / 16;
-  static constexpr int THREADS = 32 * (WK_PREP + STATE_WARPS);
+  static constexpr int THREADS = 32 * (WK_GROUPS * WK_PREP + STATE_WARPS);
 };
 
 __device__ __forceinline__ void wk_ldsm4(uint32_t addr, uint32_t (&r)[4]) {
@@ -117,12 +119,12 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
   const int n = (n_rows + WK_L - 1) / WK_L, D = p.D;
   extern __shared__ __align__(16) uint8_t wk_smem[];
   uint64_t* bars = reinterpret_cast<uint64_t*>(wk_smem + L::BAR_OFF);
-  uint64_t *full = bars, *empty = bars + 2, *tiles = bars + 4;
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 5);
+  uint64_t *full = bars, *empty = bars + WK_STAGES, *tiles = bars + 2 * WK_STAGES;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 2 * WK_STAGES + WK_GROUPS);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int s = 0; s < 2; ++s) { mbar_init(&full[s], WK_PREP); mbar_init(&empty[s], L::STATE_WARPS); }
-    mbar_init(tiles, WK_PREP);
+    for (int s = 0; s < WK_STAGES; ++s) { mbar_init(&full[s], WK_PREP); mbar_init(&empty[s], L::STATE_WARPS); }
+    for (int g = 0; g < WK_GROUPS; ++g) mbar_init(&tiles[g], WK_PREP);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -132,9 +134,10 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
   for (int c = threadIdx.x; c < D; c += L::THREADS) reinterpret_cast<float*>(wk_smem + L::U_OFF)[c] = p.u[h * D + c];
   __syncthreads();
 
-  if (warp < WK_PREP) {
+  if (warp < WK_GROUPS * WK_PREP) {
     // ------------------------------------------------------------------ prep
     constexpr int PASS = (DP + 63) / 64;
+    const int grp = warp / WK_PREP, gw = warp % WK_PREP, tid = threadIdx.x % (32 * WK_PREP);
     const int half = lane >> 4;                          // tokens 8 half .. 8 half + 7
     const float* us = reinterpret_cast<const float*>(wk_smem + L::U_OFF);
     __nv_bfloat16 rn[PASS][8], kn[PASS][8];              // the coming chunk
@@ -142,29 +145,32 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
     const __nv_bfloat16 zero = __float2bfloat16(0.f);
 #pragma unroll
     for (int a = 0; a < PASS; ++a) {
-      const int c = a * 64 + warp * 16 + (lane & 15);
+      const int c = a * 64 + gw * 16 + (lane & 15);
       w0[a] = c < D ? p.w0[h * D + c] : 0.f;
     }
     auto fetch = [&](int ch) {
 #pragma unroll
       for (int a = 0; a < PASS; ++a) {
-        const int c = a * 64 + warp * 16 + (lane & 15);
+        const int c = a * 64 + gw * 16 + (lane & 15), t0 = ch * WK_L + half * 8;
+        const size_t row = (size_t)(row0 + t0);
+        const __nv_bfloat16 *rp = p.r + row * p.r_ld + h * D + c, *kp = p.k + row * p.k_ld + h * D + c;
+        const float* zp = p.z + row * p.z_ld + h * D + c;
+        const int left = c < D ? n_rows - t0 : 0;
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-          const int t = ch * WK_L + half * 8 + e;
-          const bool ok = t < n_rows && c < D;
-          const size_t row = (size_t)(row0 + t);
-          rn[a][e] = ok ? p.r[row * p.r_ld + h * D + c] : zero;
-          kn[a][e] = ok ? p.k[row * p.k_ld + h * D + c] : zero;
-          zn[a][e] = ok ? p.z[row * p.z_ld + h * D + c] : -INFINITY;      // no decay
+          const bool ok = e < left;
+          rn[a][e] = ok ? *rp : zero;
+          kn[a][e] = ok ? *kp : zero;
+          zn[a][e] = ok ? *zp : -INFINITY;               // no decay
+          rp += p.r_ld; kp += p.k_ld; zp += p.z_ld;
         }
       }
     };
-    fetch(0);
-    for (int ch = 0; ch < n; ++ch) {
-      const int s = ch & 1;
+    if (grp < n) fetch(grp);
+    for (int ch = grp; ch < n; ch += WK_GROUPS) {
+      const int s = ch % WK_STAGES, ph = (ch / WK_STAGES) & 1;
       uint8_t* st = wk_smem + s * L::STAGE;
-      float* rT = reinterpret_cast<float*>(wk_smem + L::T_OFF + s * 3 * L::T_ARR);
+      float* rT = reinterpret_cast<float*>(wk_smem + L::T_OFF + grp * 3 * L::T_ARR);
       float* kT = rT + DP * WK_TP;
       float* cT = kT + DP * WK_TP;                       // cT[channel][t] = c_t-1, t = 0 .. 16
       float w2[PASS][8];
@@ -172,9 +178,9 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
       for (int a = 0; a < PASS; ++a)
 #pragma unroll
         for (int e = 0; e < 8; ++e) w2[a][e] = fmaxf(-1.4426950408889634f * expf(zn[a][e] + w0[a]), -256.f);   // log2 w; 2^-256 is 0
-      if (!mbar_wait(&empty[s], ((ch >> 1) & 1) ^ 1, abort_flag, p.status, 71, ch)) break;
+      if (!mbar_wait(&empty[s], ph ^ 1, abort_flag, p.status, 71, ch)) break;
       // ---- v rows
-      for (int i = threadIdx.x; i < WK_L * (D / 8); i += 32 * WK_PREP) {
+      for (int i = tid; i < WK_L * (D / 8); i += 32 * WK_PREP) {
         const int t = i / (D / 8), c8 = i % (D / 8);
         const bool ok = ch * WK_L + t < n_rows;
         const __nv_bfloat16* src = p.v + (size_t)(row0 + (ok ? ch * WK_L + t : 0)) * p.v_ld + h * D + c8 * 8;
@@ -182,10 +188,11 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;"
                      ::"r"(smem_u32(st + 4 * L::TILE + t * L::PITCH + c8 * 16)), "l"(src), "r"(bytes) : "memory");
       }
-      // ---- elementwise
+      // ---- elementwise; the arrays are free once the whole group has handed over its chunk before
+      if (ch >= WK_GROUPS && !mbar_wait(&full[(ch - WK_GROUPS) % WK_STAGES], ((ch - WK_GROUPS) / WK_STAGES) & 1, abort_flag, p.status, 74, ch)) break;
 #pragma unroll
       for (int a = 0; a < PASS; ++a) {
-        const int c = a * 64 + warp * 16 + (lane & 15);
+        const int c = a * 64 + gw * 16 + (lane & 15);
         float cum[8], run = 0.f;
 #pragma unroll
         for (int e = 0; e < 8; ++e) { run += w2[a][e]; cum[e] = run; }
@@ -219,10 +226,10 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           }
         }
       }
-      if (ch + 1 < n) fetch(ch + 1);
+      if (ch + WK_GROUPS < n) fetch(ch + WK_GROUPS);
       __syncwarp();
-      if (lane == 0) mbar_arrive(tiles);
-      if (!mbar_wait(tiles, ch & 1, abort_flag, p.status, 72, ch)) break;
+      if (lane == 0) mbar_arrive(&tiles[grp]);
+      if (!mbar_wait(&tiles[grp], (ch / WK_GROUPS) & 1, abort_flag, p.status, 72, ch)) break;
       // ---- A
       float acc[16];
 #pragma unroll
@@ -233,9 +240,11 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
         *reinterpret_cast<__nv_bfloat16*>(At + i * WK_APITCH + j * 2) = hi;
         *reinterpret_cast<__nv_bfloat16*>(At + WK_L * WK_APITCH + i * WK_APITCH + j * 2) = __float2bfloat16(x - __bfloat162float(hi));
       };
-      if (warp == 0) {                                   // the four diagonal tiles, eight lanes each
+      if (gw == 0) {                                     // the four diagonal tiles, eight lanes each
         const int b = (lane >> 3) * 4;
-        for (int c = lane & 7; c < DP; c += 8) {
+#pragma unroll 4
+        for (int cc = 0; cc < DP; cc += 8) {
+          const int c = cc + (lane & 7);
           const float4 r4 = *reinterpret_cast<const float4*>(rT + c * WK_TP + b), k4 = *reinterpret_cast<const float4*>(kT + c * WK_TP + b);
           const float4 p4 = *reinterpret_cast<const float4*>(cT + c * WK_TP + b);
           const float rv[4] = {r4.x, r4.y, r4.z, r4.w}, kv[4] = {k4.x, k4.y, k4.z, k4.w}, cv[4] = {p4.x, p4.y, p4.z, p4.w};
@@ -255,9 +264,11 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           if (j <= i) put(b + i, b + j, acc[e]);
         }
       } else {                                           // two tiles below it per warp, sixteen lanes each
-        const int tile = (warp - 1) * 2 + (lane >> 4);   // (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
+        const int tile = (gw - 1) * 2 + (lane >> 4);   // (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
         const int I = tile == 0 ? 1 : (tile < 3 ? 2 : 3), J = tile == 0 ? 0 : (tile < 3 ? tile - 1 : tile - 3);
-        for (int c = lane & 15; c < DP; c += 16) {
+#pragma unroll 4
+        for (int cc = 0; cc < DP; cc += 16) {
+          const int c = cc + (lane & 15);
           const float4 r4 = *reinterpret_cast<const float4*>(rT + c * WK_TP + I * 4), k4 = *reinterpret_cast<const float4*>(kT + c * WK_TP + J * 4);
           const float4 pi = *reinterpret_cast<const float4*>(cT + c * WK_TP + I * 4), pj = *reinterpret_cast<const float4*>(cT + c * WK_TP + J * 4);
           const float ref = pi.x, pj4 = cT[c * WK_TP + J * 4 + 4];
@@ -279,7 +290,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
     }
   } else {
     // ------------------------------------------------------------------ state
-    const int p0 = (warp - WK_PREP) * 16, g = lane >> 2, t2 = (lane & 3) * 2;
+    const int p0 = (warp - WK_GROUPS * WK_PREP) * 16, g = lane >> 2, t2 = (lane & 3) * 2;
     float S[DP / 8][4];                                  // rows p0 + g (+ 8) of S^T, channels nt * 8 + t2 (+ 1)
     float* gs = p.state + ((size_t)slot * p.H + h) * D * D;
     const bool fresh = p.positions[row0] == 0;
@@ -297,13 +308,15 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
     const uint32_t sb = smem_u32(wk_smem);
     bool ok = true;
     for (int ch = 0; ch < n; ++ch) {
-      const int s = ch & 1;
-      if (!mbar_wait(&full[s], (ch >> 1) & 1, abort_flag, p.status, 73, ch)) { ok = false; break; }
+      const int s = ch % WK_STAGES;
+      if (!mbar_wait(&full[s], (ch / WK_STAGES) & 1, abort_flag, p.status, 73, ch)) { ok = false; break; }
       __syncwarp();
       const uint32_t st = sb + s * L::STAGE;
-      float o[2][4];
+      float o[2][4], o2[2][4], o3[2][4];               // sums of their own: short chains of dependent MMAs
 #pragma unroll
-      for (int i = 0; i < 2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[i][e] = o2[i][e] = o3[i][e] = 0.f;
       // ---- O^T = S^T R^T
 #pragma unroll
       for (int ks = 0; ks < DP / 16; ++ks) {
@@ -318,8 +331,8 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           wk_mma(o[i], ah, bh[2 * i], bh[2 * i + 1]);
-          wk_mma(o[i], ah, bl[2 * i], bl[2 * i + 1]);
-          wk_mma(o[i], al, bh[2 * i], bh[2 * i + 1]);
+          wk_mma(o2[i], ah, bl[2 * i], bl[2 * i + 1]);
+          wk_mma(o3[i], al, bh[2 * i], bh[2 * i + 1]);
         }
       }
       // ---- + V^T A^T
@@ -332,8 +345,8 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
         wk_ldsm4(at + WK_L * WK_APITCH, bl);
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-          wk_mma(o[i], va, bh[2 * i], bh[2 * i + 1]);
-          wk_mma(o[i], va, bl[2 * i], bl[2 * i + 1]);
+          wk_mma(o2[i], va, bh[2 * i], bh[2 * i + 1]);
+          wk_mma(o3[i], va, bl[2 * i], bl[2 * i + 1]);
         }
       }
       // ---- S^T <- 2^c_15 S^T + V^T K
@@ -362,7 +375,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t = ch * WK_L + i * 8 + t2 + (e & 1), pr = p0 + g + (e >> 1) * 8;
-          if (t < n_rows && pr < D) p.y[(size_t)(row0 + t) * p.y_ld + h * D + pr] = __float2bfloat16(o[i][e]);
+          if (t < n_rows && pr < D) p.y[(size_t)(row0 + t) * p.y_ld + h * D + pr] = __float2bfloat16(o[i][e] + (o2[i][e] + o3[i][e]));
         }
     }
     if (ok) {
