@@ -9,8 +9,8 @@
 // exponent that is taken here is a difference whose sign makes it at most zero.  A is made of 4 x 4 tiles: below the diagonal
 // tiles both sides refer to the tile's first row (8 exponentials for 16 products), on it every pair has its own.
 //
-// One CTA walks the chunks of one (request, head); two kinds of warps, four stages between them:
-//   prep   (two groups of 4 warps, alternate chunks) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
+// One CTA walks the chunks of one (request, head); two kinds of warps, stages of shared memory between them:
+//   prep   (two or three groups of 4 warps that take turns) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
 //          the tiles of A with lanes over channels
 //   state  (one warp per 16 value columns) S^T in fp32 accumulators; O^T = S^T R^T + V^T A^T and S^T += V^T K on mma.sync, S^T being
 //          its own A operand.  A chunk of 16 tokens is too short for tcgen05: the chain from S to S would go through tensor memory
@@ -40,25 +40,25 @@ struct WkvParams {
 };
 
 constexpr int WK_L = 16;                           // tokens per chunk
-constexpr int WK_GROUPS = 2;                       // prep groups
-constexpr int WK_PREP = 4;                         // warps of one
-constexpr int WK_STAGES = 2 * WK_GROUPS;
+constexpr int WK_PREP = 4;                         // warps of a prep group
 constexpr int WK_TP = 20;                          // floats per channel of the arrays [channel][token]
 constexpr int WK_APITCH = 48;                      // bytes per row of A
 template <int DP>
 struct WkLayout {
+  static constexpr int GROUPS = DP > 64 ? 2 : 3;   // prep groups, as many as fit
+  static constexpr int STAGES = 2 * GROUPS;
   static constexpr int PITCH = DP * 2 + 16;        // bytes per token row; ldmatrix rows fall into different banks
   static constexpr int TILE = WK_L * PITCH;
   static constexpr int A_OFF = 5 * TILE;           // after R hi, R lo, K hi, K lo, V
   static constexpr int DS_OFF = A_OFF + 2 * WK_L * WK_APITCH;
   static constexpr int STAGE = DS_OFF + DP * 4;
-  static constexpr int T_OFF = WK_STAGES * STAGE;  // per group r, k, c: [DP][WK_TP] floats each
+  static constexpr int T_OFF = STAGES * STAGE;  // per group r, k, c: [DP][WK_TP] floats each
   static constexpr int T_ARR = DP * WK_TP * 4;
-  static constexpr int U_OFF = T_OFF + WK_GROUPS * 3 * T_ARR;
+  static constexpr int U_OFF = T_OFF + GROUPS * 3 * T_ARR;
   static constexpr int BAR_OFF = U_OFF + DP * 4;
   static constexpr int SMEM = BAR_OFF + 128;
   static constexpr int STATE_WARPS = DP / 16;
-  static constexpr int THREADS = 32 * (WK_GROUPS * WK_PREP + STATE_WARPS);
+  static constexpr int THREADS = 32 * (GROUPS * WK_PREP + STATE_WARPS);
 };
 
 __device__ __forceinline__ void wk_ldsm4(uint32_t addr, uint32_t (&r)[4]) {
@@ -119,12 +119,12 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
   const int n = (n_rows + WK_L - 1) / WK_L, D = p.D;
   extern __shared__ __align__(16) uint8_t wk_smem[];
   uint64_t* bars = reinterpret_cast<uint64_t*>(wk_smem + L::BAR_OFF);
-  uint64_t *full = bars, *empty = bars + WK_STAGES, *tiles = bars + 2 * WK_STAGES;
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 2 * WK_STAGES + WK_GROUPS);
+  uint64_t *full = bars, *empty = bars + L::STAGES, *tiles = bars + 2 * L::STAGES;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 2 * L::STAGES + L::GROUPS);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int s = 0; s < WK_STAGES; ++s) { mbar_init(&full[s], WK_PREP); mbar_init(&empty[s], L::STATE_WARPS); }
-    for (int g = 0; g < WK_GROUPS; ++g) mbar_init(&tiles[g], WK_PREP);
+    for (int s = 0; s < L::STAGES; ++s) { mbar_init(&full[s], WK_PREP); mbar_init(&empty[s], L::STATE_WARPS); }
+    for (int g = 0; g < L::GROUPS; ++g) mbar_init(&tiles[g], WK_PREP);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -134,7 +134,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
   for (int c = threadIdx.x; c < D; c += L::THREADS) reinterpret_cast<float*>(wk_smem + L::U_OFF)[c] = p.u[h * D + c];
   __syncthreads();
 
-  if (warp < WK_GROUPS * WK_PREP) {
+  if (warp < L::GROUPS * WK_PREP) {
     // ------------------------------------------------------------------ prep
     constexpr int PASS = (DP + 63) / 64;
     const int grp = warp / WK_PREP, gw = warp % WK_PREP, tid = threadIdx.x % (32 * WK_PREP);
@@ -167,8 +167,8 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
       }
     };
     if (grp < n) fetch(grp);
-    for (int ch = grp; ch < n; ch += WK_GROUPS) {
-      const int s = ch % WK_STAGES, ph = (ch / WK_STAGES) & 1;
+    for (int ch = grp; ch < n; ch += L::GROUPS) {
+      const int s = ch % L::STAGES, ph = (ch / L::STAGES) & 1;
       uint8_t* st = wk_smem + s * L::STAGE;
       float* rT = reinterpret_cast<float*>(wk_smem + L::T_OFF + grp * 3 * L::T_ARR);
       float* kT = rT + DP * WK_TP;
@@ -189,7 +189,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
                      ::"r"(smem_u32(st + 4 * L::TILE + t * L::PITCH + c8 * 16)), "l"(src), "r"(bytes) : "memory");
       }
       // ---- elementwise; the arrays are free once the whole group has handed over its chunk before
-      if (ch >= WK_GROUPS && !mbar_wait(&full[(ch - WK_GROUPS) % WK_STAGES], ((ch - WK_GROUPS) / WK_STAGES) & 1, abort_flag, p.status, 74, ch)) break;
+      if (ch >= L::GROUPS && !mbar_wait(&full[(ch - L::GROUPS) % L::STAGES], ((ch - L::GROUPS) / L::STAGES) & 1, abort_flag, p.status, 74, ch)) break;
 #pragma unroll
       for (int a = 0; a < PASS; ++a) {
         const int c = a * 64 + gw * 16 + (lane & 15);
@@ -226,10 +226,10 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           }
         }
       }
-      if (ch + WK_GROUPS < n) fetch(ch + WK_GROUPS);
+      if (ch + L::GROUPS < n) fetch(ch + L::GROUPS);
       __syncwarp();
       if (lane == 0) mbar_arrive(&tiles[grp]);
-      if (!mbar_wait(&tiles[grp], (ch / WK_GROUPS) & 1, abort_flag, p.status, 72, ch)) break;
+      if (!mbar_wait(&tiles[grp], (ch / L::GROUPS) & 1, abort_flag, p.status, 72, ch)) break;
       // ---- A
       float acc[16];
 #pragma unroll
@@ -290,7 +290,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
     }
   } else {
     // ------------------------------------------------------------------ state
-    const int p0 = (warp - WK_GROUPS * WK_PREP) * 16, g = lane >> 2, t2 = (lane & 3) * 2;
+    const int p0 = (warp - L::GROUPS * WK_PREP) * 16, g = lane >> 2, t2 = (lane & 3) * 2;
     float S[DP / 8][4];                                  // rows p0 + g (+ 8) of S^T, channels nt * 8 + t2 (+ 1)
     float* gs = p.state + ((size_t)slot * p.H + h) * D * D;
     const bool fresh = p.positions[row0] == 0;
@@ -308,8 +308,8 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
     const uint32_t sb = smem_u32(wk_smem);
     bool ok = true;
     for (int ch = 0; ch < n; ++ch) {
-      const int s = ch % WK_STAGES;
-      if (!mbar_wait(&full[s], (ch / WK_STAGES) & 1, abort_flag, p.status, 73, ch)) { ok = false; break; }
+      const int s = ch % L::STAGES;
+      if (!mbar_wait(&full[s], (ch / L::STAGES) & 1, abort_flag, p.status, 73, ch)) { ok = false; break; }
       __syncwarp();
       const uint32_t st = sb + s * L::STAGE;
       float o[2][4], o2[2][4], o3[2][4];               // sums of their own: short chains of dependent MMAs

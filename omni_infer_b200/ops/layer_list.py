@@ -101,7 +101,7 @@ def qk_norm_rope_cache(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, positi
     if not qkv.is_cuda:
         norm = (lambda x, w: x) if q_w is None else (lambda x, w: rms_ref(x, w, eps))
         q = norm(qkv[:, :nq].float(), q_w).view(T, hq, dk)
-        qkv[:, :nq] = _rotate_half_ref(q, cos_sin, positions, rot).reshape(T, nq).to(qkv.dtype)
+        qkv[:, :nq] = _rotate_half_ref(q, cos_sin, positions, rot).reshape(T, nq).to(qkv.dtype, copy=True)
         if hkv:
             k = norm(qkv[:, nq:nq + nk].float(), k_w).view(T, hkv, dk)
             k = _rotate_half_ref(k, cos_sin, positions, rot)
