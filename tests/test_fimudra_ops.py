@@ -229,7 +229,7 @@ def by_cuts(cuts, call):
     return [torch.cat(g) for g in got]
 
 
-MEM_SIZES = [(2, 8, 8), (3, 32, 48), (2, 64, 128), (1, 128, 72), (2, 13, 9), (1, 160, 40), (2, 72, 64)]
+MEM_SIZES = [(2, 8, 8), (3, 40, 56), (2, 64, 128), (1, 128, 72), (2, 13, 9), (1, 160, 40), (2, 72, 64)]
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
