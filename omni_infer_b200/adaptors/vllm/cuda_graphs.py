@@ -7,6 +7,8 @@ static input buffers: a step copies its inputs into the buffers and replays; the
 slots and the expert selector from device memory, so one graph serves every batch of that bucket."""
 from __future__ import annotations
 
+import gc
+
 import torch
 
 from ...layers.common import AttnMetadata
@@ -56,9 +58,18 @@ class DecodeGraphs:
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
         before = nat.launch_count()
-        with torch.cuda.graph(g, pool=self.pool):
-            hidden = r.model(ids, md, r.kv_caches)
-            logits = r.model.compute_logits(hidden)
+        # a garbage collection during the capture could destroy CUDA objects of an engine that has gone (graphs, events), and
+        # such a call invalidates the capture: collect now, and not again before it is over
+        gc.collect()
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(g, pool=self.pool):
+                hidden = r.model(ids, md, r.kv_caches)
+                logits = r.model.compute_logits(hidden)
+        finally:
+            if collecting:
+                gc.enable()
         captured = nat.launch_count() - before
         nat.add_launches(-captured)          # capture itself runs nothing
         if self.pool is None:
