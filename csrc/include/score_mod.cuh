@@ -1,0 +1,41 @@
+// What may happen to an attention score between q k^T and the softmax, and which keys a query sees.
+#pragma once
+#include <cuda_runtime.h>
+
+namespace omni {
+
+// score = cap tanh(raw scale / cap) - slope distance (each part optional), in units of log 2
+struct ScoreMod {
+  float scale_log2;        // scale * log2(e)
+  float cap_in;            // 2 log2(e) scale / cap
+  float cap_log2;          // cap * log2(e); 0 = no cap
+  const float* slopes;     // [heads] or null
+};
+
+inline ScoreMod make_score_mod(float scale, float cap, const float* slopes) {
+  constexpr float kLog2e = 1.4426950408889634f;
+  return {scale * kLog2e, cap > 0.f ? 2.f * kLog2e * scale / cap : 0.f, cap > 0.f ? cap * kLog2e : 0.f, slopes};
+}
+
+__device__ __forceinline__ float ex2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// tanh(z) = 1 - 2 / (1 + e^2z): absolute error of some 1e-7, which the cap multiplies
+__device__ __forceinline__ float cap_score(const ScoreMod& m, float raw) {
+  return m.cap_log2 > 0.f ? m.cap_log2 - __fdividef(2.f * m.cap_log2, 1.f + ex2_fast(raw * m.cap_in)) : raw * m.scale_log2;
+}
+
+// First key that a query at `pos` sees through its window (of `window` keys) and in its chunk (of `chunk` positions); 0 = none.
+// Kept first keys come on top.
+__host__ __device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+  int lo = window > 0 ? pos - window + 1 : 0;
+  if (chunk > 0 && pos >= 0) {
+    const int c = pos / chunk * chunk;
+    lo = c > lo ? c : lo;
+  }
+  return lo > 0 ? lo : 0;
+}
+
+}  // namespace omni

@@ -11,7 +11,10 @@
 // up to 192 / 128 that are multiples of 8: the tensor maps are [rows, heads, head size], so a partial 64-wide chunk is
 // zero-filled), with an optional sliding window - key tiles outside every query's window are never loaded - and with the
 // softmax weights carried as a pair of bf16 values (p = hi + lo, two MMAs), i.e. to 16 bits of mantissa; optionally a sink per
-// head in the softmax denominator and a factor on the result.
+// head in the softmax denominator and a factor on the result, kept first keys beside the window (their tiles come first), chunks
+// instead of it, and capped or biased scores (an instantiation of its own).
+// omni_fmha_latent: contiguous key rows as in the first form, but with any head sizes, the window, the pair of bf16 weights and a
+// gate per row and head as in the second: latent attention over keys and values that were projected from their latents.
 // Causal mask is aligned to the end of the key range (query i of a request with Lq queries and Lk keys sees
 // keys <= Lk - Lq + i), which also covers chunked prefill and prefix-cache hits.
 //
@@ -20,13 +23,18 @@
 // Reference call sites: npu_fused_infer_attention_score / npu_fusion_attention
 // (omni/models/common/layers/attention/deepseek_mla.py:386-400, omni/models/common/layers/attention/backend/attention.py:590-666).
 #include "../include/omni_ptx.cuh"
+#include "../include/score_mod.cuh"
 #include "../include/tma_host.h"
 
 namespace omni {
 
+enum { FM_DENSE = 0, FM_PAGED = 1, FM_PAGED_MOD = 2, FM_LATENT = 3 };
+
 struct FmhaParams {
-  const int* cu_q;   // [B+1]
-  const int* cu_k;   // [B+1]
+  const int* cu_q;   // [B] first row of each request
+  const int* end_q;  // [B] and the row after its last: cu_q + 1 where requests follow one another
+  const int* cu_k;
+  const int* end_k;
   int Hq, Hkv;
   int q_head_stride, k_head_stride, v_head_stride;  // in elements (column offset per head)
   int v_col0, k2_col0;
@@ -40,6 +48,10 @@ struct FmhaParams {
   const int* block_table;
   int bt_ld, block_size;
   int window;          // a query sees the last `window` keys up to its own; 0 = all
+  int chunk, keep;     // see first_key; the first `keep` keys are visible in any case
+  ScoreMod score;      // FM_PAGED_MOD
+  const __nv_bfloat16* gate;   // [Tq, gate_ld] or null: the result of head h is multiplied by sigmoid(gate[t, h])
+  int gate_ld;
   const float* sink;   // [Hq] or null: exp(sink) is one more term of the softmax denominator
   float out_scale;     // multiplies the result before it is rounded
   OmniStatus* status;
@@ -55,12 +67,13 @@ constexpr int FM_THREADS = 192;
 // stages takes 98 KB and 256 TMEM columns, so that two CTAs share an SM and one's softmax overlaps the other's MMAs; its P
 // (32 columns hi, 32 columns lo) replaces the 64 columns of the S tile that it was computed from, which the next QK^T but
 // one writes again only after the PV that reads P (the MMAs of a CTA complete in order).
-template <bool PAGED, int MAXC, int STAGES>
+template <int MODE, int MAXC, int STAGES>
 struct FmLayout {
+  static constexpr bool EXACT = MODE != FM_DENSE;
   static constexpr int K_STAGE = MAXC * FM_KCHUNK;
   static constexpr int SMEM = MAXC * FM_QCHUNK + STAGES * (K_STAGE + FM_V_STAGE) + 1024 + 1024;
-  static constexpr int T_O = 0, T_S = 128, T_P = PAGED ? T_S : 256, T_P_STRIDE = PAGED ? FM_BK : FM_BK / 2;
-  static constexpr int T_COLS = PAGED ? 256 : 512;
+  static constexpr int T_O = 0, T_S = 128, T_P = EXACT ? T_S : 256, T_P_STRIDE = EXACT ? FM_BK : FM_BK / 2;
+  static constexpr int T_COLS = EXACT ? 256 : 512;
 };
 
 __device__ __forceinline__ void fm_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc,
@@ -72,15 +85,17 @@ __device__ __forceinline__ void fm_umma_ts(uint32_t d_tmem, uint32_t a_tmem, uin
       : "memory");
 }
 
-template <bool PAGED, int MAXC, int STAGES>
-__global__ void __launch_bounds__(FM_THREADS, (PAGED && MAXC == 2) ? 2 : 1)
-fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                   const __grid_constant__ CUtensorMap tmap_k2, const __grid_constant__ CUtensorMap tmap_v,
-                   const FmhaParams p) {
+template <int MODE, int MAXC, int STAGES>
+__global__ void __launch_bounds__(FM_THREADS, (MODE != FM_DENSE && MAXC == 2) ? 2 : 1)
+fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_q2,
+                   const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_k2,
+                   const __grid_constant__ CUtensorMap tmap_v, const FmhaParams p) {
+  constexpr bool PAGED = MODE == FM_PAGED || MODE == FM_PAGED_MOD;      // keys through the block table
+  constexpr bool EXACT = MODE != FM_DENSE;                              // any head sizes, masks, softmax weights as hi + lo
   const int b = blockIdx.y, h = blockIdx.z;
-  const int q_begin = p.cu_q[b], q_end = p.cu_q[b + 1];
+  const int q_begin = p.cu_q[b], q_end = p.end_q[b];
   const int k_begin = PAGED ? 0 : p.cu_k[b];
-  const int Lq = q_end - q_begin, Lk = PAGED ? p.kv_len[b] : p.cu_k[b + 1] - k_begin;
+  const int Lq = q_end - q_begin, Lk = PAGED ? p.kv_len[b] : p.end_k[b] - k_begin;
   const int q0 = blockIdx.x * FM_BQ;
   if (q0 >= Lq) return;  // uniform for the whole CTA, before any barrier / TMEM use
   const int ctx = Lk - Lq;
@@ -88,12 +103,14 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const int nc = p.nk1 + p.nk2;
   // keys this tile can see
   int k_hi = p.causal ? min(Lk, ctx + q0 + FM_BQ) : Lk;
-  int t_first = 0;                                     // first key tile inside the window of the tile's first query
-  if (PAGED && p.window > 0) t_first = max(0, ctx + q0 - p.window + 1) / FM_BK;
-  const int n = (k_hi + FM_BK - 1) / FM_BK - t_first;
-  const int nv = PAGED ? (p.dv + 63) / 64 : 2;         // 64-wide chunks of the value size
+  // first key tile that the tile's first query sees, but for those of kept keys, which come ahead of it
+  const int t_first = EXACT ? first_key(ctx + q0, p.window, p.chunk) / FM_BK : 0;
+  const int n_keep = PAGED ? min((p.keep + FM_BK - 1) / FM_BK, t_first) : 0;
+  const int n = n_keep + (k_hi + FM_BK - 1) / FM_BK - t_first;
+  auto first_of_tile = [&](int i) { return (PAGED && i < n_keep ? i : t_first - n_keep + i) * FM_BK; };
+  const int nv = EXACT ? (p.dv + 63) / 64 : 2;         // 64-wide chunks of the value size
 
-  using L = FmLayout<PAGED, MAXC, STAGES>;
+  using L = FmLayout<MODE, MAXC, STAGES>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* sq = smem;
@@ -138,21 +155,22 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     if (lane == 0) {
       mbar_expect_tx(q_full, nc * FM_QCHUNK);
       for (int c = 0; c < nc; ++c) {
-        if (PAGED) tma_load_3d(sq + c * FM_QCHUNK, &tmap_q, q_full, c * 64, h, q_begin + q0);
+        if (EXACT && c < p.nk1) tma_load_3d(sq + c * FM_QCHUNK, &tmap_q, q_full, c * 64, h, q_begin + q0);
+        else if (EXACT) tma_load_3d(sq + c * FM_QCHUNK, &tmap_q2, q_full, (c - p.nk1) * 64, h, q_begin + q0);
         else tma_load_2d(sq + c * FM_QCHUNK, &tmap_q, q_full, h * p.q_head_stride + c * 64, q_begin + q0);
       }
       for (int i = 0; i < n; ++i) {
         const int st = i % STAGES;
         const uint32_t ph = (i / STAGES) & 1;
-        int row = k_begin + i * FM_BK;
+        const int key0 = first_of_tile(i);
+        int row = k_begin + key0;
         if (PAGED) {
-          const int key0 = (t_first + i) * FM_BK;
           row = p.block_table[(size_t)b * p.bt_ld + key0 / p.block_size] * p.block_size + key0 % p.block_size;
         }
         if (!mbar_wait(&k_empty[st], ph ^ 1, abort_flag, p.status, 11, i)) break;
         mbar_expect_tx(&k_full[st], nc * FM_KCHUNK);
         for (int c = 0; c < p.nk1; ++c) {
-          if (PAGED) tma_load_3d(sk + st * L::K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], c * 64, hk, row);
+          if (EXACT) tma_load_3d(sk + st * L::K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], c * 64, hk, row);
           else tma_load_2d(sk + st * L::K_STAGE + c * FM_KCHUNK, &tmap_k, &k_full[st], hk * p.k_head_stride + c * 64, row);
         }
         for (int c = 0; c < p.nk2; ++c)
@@ -160,7 +178,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         if (!mbar_wait(&v_empty[st], ph ^ 1, abort_flag, p.status, 12, i)) break;
         mbar_expect_tx(&v_full[st], nv * FM_KCHUNK);
         for (int c = 0; c < nv; ++c) {
-          if (PAGED) tma_load_3d(sv + st * FM_V_STAGE + c * FM_KCHUNK, &tmap_v, &v_full[st], c * 64, hk, row);
+          if (EXACT) tma_load_3d(sv + st * FM_V_STAGE + c * FM_KCHUNK, &tmap_v, &v_full[st], c * 64, hk, row);
           else tma_load_2d(sv + st * FM_V_STAGE + c * FM_KCHUNK, &tmap_v, &v_full[st],
                            hk * p.v_head_stride + p.v_col0 + c * 64, row);
         }
@@ -203,7 +221,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
           const uint64_t bd = umma_desc_mnmajor_sw128(vbase + k * 2048, FM_KCHUNK, 1024);
           fm_umma_ts(tmem_base + L::T_O, tmem_base + L::T_P + (i & 1) * L::T_P_STRIDE + k * 8, bd, idesc_pv,
                      (i > 0 || k > 0) ? 1u : 0u);
-          if (PAGED) fm_umma_ts(tmem_base + L::T_O, tmem_base + L::T_P + FM_BK / 2 + (i & 1) * L::T_P_STRIDE + k * 8, bd, idesc_pv, 1u);
+          if (EXACT) fm_umma_ts(tmem_base + L::T_O, tmem_base + L::T_P + FM_BK / 2 + (i & 1) * L::T_P_STRIDE + k * 8, bd, idesc_pv, 1u);
         }
         umma_commit(&v_empty[st]);
         umma_commit(o_done);
@@ -216,16 +234,21 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     const int row = qd * 32 + lane;          // query row inside the tile
     const uint32_t lane_addr = tmem_base + ((uint32_t)(qd * 32) << 16);
     const int q_pos = ctx + q0 + row;        // last key index this row may see (causal)
+    const int first = EXACT ? first_key(q_pos, p.window, p.chunk) : 0;
+    float slope = 0.f;
+    if (MODE == FM_PAGED_MOD && p.score.slopes != nullptr) slope = p.score.slopes[h] * 1.4426950408889634f;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int i = 0; i < n; ++i) {
       if (!mbar_wait(&s_full[i & 1], (i >> 1) & 1, abort_flag, p.status, 17, i)) { ok = false; break; }
       tc_fence_after();
-      const int kbase = (t_first + i) * FM_BK;
+      const int kbase = first_of_tile(i);
       int lim = Lk - kbase;                        // keys beyond the request end are masked
       if (p.causal) lim = min(lim, q_pos - kbase + 1);
-      int low = 0;                                 // and those before the window
-      if (PAGED && p.window > 0) low = q_pos - p.window + 1 - kbase;
+      const int low = first - kbase;               // and those before the window, but for the kept ones
+      const int kept = p.keep - kbase;
+      float dist_bias = 0.f;                       // of column 0
+      if (MODE == FM_PAGED_MOD) dist_bias = slope * (float)(q_pos - kbase);
       float s[FM_BK];
       float mx = -INFINITY;
 #pragma unroll
@@ -235,7 +258,10 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         tmem_ld_wait();
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
-          s[c0 + j] = (c0 + j < lim && (!PAGED || c0 + j >= low)) ? __uint_as_float(sv32[j]) * p.scale_log2 : -INFINITY;
+          float v = __uint_as_float(sv32[j]);
+          if (MODE == FM_PAGED_MOD) v = cap_score(p.score, v) - (dist_bias - slope * (float)(c0 + j));
+          else v *= p.scale_log2;
+          s[c0 + j] = (c0 + j < lim && (!EXACT || c0 + j >= low || (PAGED && c0 + j < kept))) ? v : -INFINITY;
           mx = fmaxf(mx, s[c0 + j]);
         }
       }
@@ -269,7 +295,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         rs += p0 + p1;
         __nv_bfloat162 h2 = __floats2bfloat162_rn(p0, p1);
         pk[j] = *reinterpret_cast<uint32_t*>(&h2);
-        if (PAGED) {      // what the rounding to bf16 left over
+        if (EXACT) {      // what the rounding to bf16 left over
           const float2 hf = __bfloat1622float2(h2);
           h2 = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
           pl[j] = *reinterpret_cast<uint32_t*>(&h2);
@@ -277,7 +303,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       }
       l += rs;
       tmem_st_x32(lane_addr + L::T_P + (i & 1) * L::T_P_STRIDE, pk);
-      if (PAGED) tmem_st_x32(lane_addr + L::T_P + FM_BK / 2 + (i & 1) * L::T_P_STRIDE, pl);
+      if (EXACT) tmem_st_x32(lane_addr + L::T_P + FM_BK / 2 + (i & 1) * L::T_P_STRIDE, pl);
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
@@ -289,7 +315,9 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       const bool row_ok = (q0 + row) < Lq;
       float den = l;
       if (PAGED && p.sink != nullptr && m != -INFINITY) den += exp2f(p.sink[h] * 1.4426950408889634f - m);
-      const float inv_l = l > 0.f ? (PAGED ? p.out_scale : 1.0f) / den : 0.f;
+      float inv_l = l > 0.f ? (EXACT ? p.out_scale : 1.0f) / den : 0.f;
+      if (MODE == FM_LATENT && p.gate != nullptr && row_ok)
+        inv_l /= 1.f + __expf(-__bfloat162float(p.gate[(size_t)(q_begin + q0 + row) * p.gate_ld + h]));
       __nv_bfloat16* orow = p.out + (size_t)(q_begin + q0 + row) * p.out_ld + h * p.dv;
 #pragma unroll 1
       for (int c = 0; c < p.dv; c += 32) {
@@ -299,7 +327,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         if (row_ok) {
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
-            if (PAGED && c + j >= p.dv) break;
+            if (EXACT && c + j >= p.dv) break;
             __nv_bfloat16 o8[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) o8[e] = __float2bfloat16(__uint_as_float(ov[j + e]) * inv_l);
@@ -327,13 +355,13 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 
 using namespace omni;
 
-template <bool PAGED, int MAXC, int STAGES>
-static int launch_fmha(dim3 grid, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tk2, const CUtensorMap& tv,
-                       const FmhaParams& p, cudaStream_t stream) {
-  constexpr int smem = FmLayout<PAGED, MAXC, STAGES>::SMEM;
+template <int MODE, int MAXC, int STAGES>
+static int launch_fmha(dim3 grid, const CUtensorMap& tq, const CUtensorMap& tq2, const CUtensorMap& tk, const CUtensorMap& tk2,
+                       const CUtensorMap& tv, const FmhaParams& p, cudaStream_t stream) {
+  constexpr int smem = FmLayout<MODE, MAXC, STAGES>::SMEM;
   static bool configured[64] = {false};
-  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel<PAGED, MAXC, STAGES>, smem, configured)) return e;
-  fmha_varlen_kernel<PAGED, MAXC, STAGES><<<grid, FM_THREADS, smem, stream>>>(tq, tk, tk2, tv, p);
+  if (int e = ensure_dyn_smem((const void*)fmha_varlen_kernel<MODE, MAXC, STAGES>, smem, configured)) return e;
+  fmha_varlen_kernel<MODE, MAXC, STAGES><<<grid, FM_THREADS, smem, stream>>>(tq, tq2, tk, tk2, tv, p);
   return (int)cudaGetLastError();
 }
 
@@ -357,25 +385,25 @@ extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q
   }
   if (make_tmap_2d(&tv, v, 2, (uint64_t)k_rows, v_cols, v_ld, FM_BK, 64, true)) return -13;
   FmhaParams p;
-  p.cu_q = cu_q; p.cu_k = cu_k; p.Hq = Hq; p.Hkv = Hkv; p.q_head_stride = q_head_stride;
+  memset(&p, 0, sizeof(p));
+  p.cu_q = cu_q; p.end_q = cu_q + 1; p.cu_k = cu_k; p.end_k = cu_k + 1; p.Hq = Hq; p.Hkv = Hkv; p.q_head_stride = q_head_stride;
   p.k_head_stride = k_head_stride; p.v_head_stride = v_head_stride; p.v_col0 = v_col0; p.k2_col0 = k2_col0;
   p.nk1 = d_k1 / 64; p.nk2 = d_k2 / 64; p.scale_log2 = scale * 1.4426950408889634f; p.causal = causal;
   p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = FM_DV; p.out_ld = Hq * FM_DV;
-  p.kv_len = nullptr; p.block_table = nullptr; p.bt_ld = 0; p.block_size = 0; p.window = 0;
-  p.sink = nullptr; p.out_scale = 1.0f;
-  return launch_fmha<false, FM_MAXC, 3>(dim3((max_q + FM_BQ - 1) / FM_BQ, B, Hq), tq, tk, tk2, tv, p, stream);
+  p.out_scale = 1.0f;
+  return launch_fmha<FM_DENSE, FM_MAXC, 3>(dim3((max_q + FM_BQ - 1) / FM_BQ, B, Hq), tq, tq, tk, tk2, tv, p, stream);
 }
 
 // Ragged queries against the paged cache.  q: rows of pitch q_ld holding Hq heads of d_k; k_cache / v_cache
 // [slots, Hkv, d_k / d_v]; kv_len[b] keys of request b, of which its cu_q segment is the end; out rows of pitch out_ld.
 extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const void* k_cache, const void* v_cache,
                                long long slots, const int* cu_q, const int* kv_len, const int* block_table, int bt_ld, int B,
-                               int max_q, int Hq, int Hkv, int d_k, int d_v, int block_size, int window, float scale,
-                               const float* sink, float out_scale, void* out, int out_ld, void* status, cudaStream_t stream) {
+                               int max_q, int Hq, int Hkv, int d_k, int d_v, int block_size, int window, int chunk, int keep,
+                               float scale, float softcap, const float* slopes, const float* sink, float out_scale, void* out, int out_ld, void* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (d_k < 8 || d_v < 8 || d_k % 8 != 0 || d_v % 8 != 0 || d_k > 64 * FM_MAXC || d_v > FM_DV) return -1;
-  if (Hkv < 1 || Hq % Hkv != 0 || B > 65535 || Hq > 65535 || window < 0) return -2;
+  if (Hkv < 1 || Hq % Hkv != 0 || B > 65535 || Hq > 65535 || window < 0 || chunk < 0 || keep < 0) return -2;
   if (block_size < FM_BK || block_size % FM_BK != 0 || q_ld % 8 != 0 || out_ld % 8 != 0) return -3;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % 16 != 0) return -4;
   CUtensorMap tq, tk, tv;
@@ -386,11 +414,47 @@ extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const 
     return -13;
   FmhaParams p;
   memset(&p, 0, sizeof(p));
-  p.cu_q = cu_q; p.Hq = Hq; p.Hkv = Hkv; p.nk1 = (d_k + 63) / 64; p.nk2 = 0;
+  p.cu_q = cu_q; p.end_q = cu_q + 1; p.Hq = Hq; p.Hkv = Hkv; p.nk1 = (d_k + 63) / 64; p.nk2 = 0;
   p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = d_v; p.out_ld = out_ld; p.kv_len = kv_len; p.block_table = block_table; p.bt_ld = bt_ld;
-  p.block_size = block_size; p.window = window; p.sink = sink; p.out_scale = out_scale;
+  p.block_size = block_size; p.window = window; p.chunk = chunk; p.keep = keep; p.sink = sink; p.out_scale = out_scale;
+  p.score = make_score_mod(scale, softcap, slopes);
   const dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
-  if (p.nk1 <= 2) return launch_fmha<true, 2, 2>(grid, tq, tk, tk, tv, p, stream);
-  return launch_fmha<true, FM_MAXC, 3>(grid, tq, tk, tk, tv, p, stream);
+  if (softcap > 0.f || slopes != nullptr) {
+    if (p.nk1 <= 2) return launch_fmha<FM_PAGED_MOD, 2, 2>(grid, tq, tq, tk, tk, tv, p, stream);
+    return launch_fmha<FM_PAGED_MOD, FM_MAXC, 3>(grid, tq, tq, tk, tk, tv, p, stream);
+  }
+  if (p.nk1 <= 2) return launch_fmha<FM_PAGED, 2, 2>(grid, tq, tq, tk, tk, tv, p, stream);
+  return launch_fmha<FM_PAGED, FM_MAXC, 3>(grid, tq, tq, tk, tk, tv, p, stream);
+}
+
+// Latent attention of ragged queries over projected keys.  q rows of pitch q_ld: per head d1 unrotated | d2 rotated; kv rows of
+// pitch kv_ld: per head d1 keys | d_v values; k2 rows of pitch k2_ld: the d2 rotated key columns that all heads share.  Request
+// b has query rows q_start[b] .. q_end[b] and key rows k_start[b] .. k_end[b], whose last ones belong to its queries.
+extern "C" int omni_fmha_latent(const void* q, long long q_rows, int q_ld, const void* kv, long long k_rows, int kv_ld,
+                                const void* k2, int k2_ld, const int* q_start, const int* q_end, const int* k_start,
+                                const int* k_end, int B, int max_q, int H, int d1, int d2, int d_v, int window, float scale,
+                                const void* gate, int gate_ld, void* out, int out_ld, void* status, cudaStream_t stream) {
+  if (B <= 0 || max_q <= 0) return 0;
+  const int nk1 = (d1 + 63) / 64, nk2 = (d2 + 63) / 64;
+  if (d1 < 8 || d2 < 8 || d_v < 8 || d1 % 8 != 0 || d2 % 8 != 0 || d_v % 8 != 0 || nk1 + nk2 > FM_MAXC || d_v > FM_DV) return -1;
+  if (H < 1 || B > 65535 || H > 65535 || window < 0 || q_rows < 1 || k_rows < 1) return -2;
+  if (q_ld % 8 != 0 || kv_ld % 8 != 0 || k2_ld % 8 != 0 || out_ld % 8 != 0 || q_ld < H * (d1 + d2) || kv_ld < H * (d1 + d_v)) return -3;
+  if (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)k2 | (uintptr_t)out) % 16 != 0) return -4;
+  CUtensorMap tq, tq2, tk, tk2, tv;
+  const __nv_bfloat16 *qb = (const __nv_bfloat16*)q, *kb = (const __nv_bfloat16*)kv;
+  const uint64_t q_head = (uint64_t)(d1 + d2) * 2, k_head = (uint64_t)(d1 + d_v) * 2;
+  if (make_tmap_3d(&tq, qb, 2, d1, H, (uint64_t)q_rows, q_head, (uint64_t)q_ld * 2, 64, 1, FM_BQ, true)) return -10;
+  if (make_tmap_3d(&tq2, qb + d1, 2, d2, H, (uint64_t)q_rows, q_head, (uint64_t)q_ld * 2, 64, 1, FM_BQ, true)) return -11;
+  if (make_tmap_3d(&tk, kb, 2, d1, H, (uint64_t)k_rows, k_head, (uint64_t)kv_ld * 2, 64, 1, FM_BK, true)) return -12;
+  if (make_tmap_2d(&tk2, k2, 2, (uint64_t)k_rows, d2, k2_ld, FM_BK, 64, true)) return -13;
+  if (make_tmap_3d(&tv, kb + d1, 2, d_v, H, (uint64_t)k_rows, k_head, (uint64_t)kv_ld * 2, 64, 1, FM_BK, true)) return -14;
+  FmhaParams p;
+  memset(&p, 0, sizeof(p));
+  p.cu_q = q_start; p.end_q = q_end; p.cu_k = k_start; p.end_k = k_end; p.Hq = H; p.Hkv = H; p.nk1 = nk1; p.nk2 = nk2;
+  p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
+  p.dv = d_v; p.out_ld = out_ld; p.window = window; p.out_scale = 1.0f; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
+  const dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, H);
+  if (nk1 + nk2 <= 2) return launch_fmha<FM_LATENT, 2, 2>(grid, tq, tq2, tk, tk2, tv, p, stream);
+  return launch_fmha<FM_LATENT, FM_MAXC, 3>(grid, tq, tq2, tk, tk2, tv, p, stream);
 }

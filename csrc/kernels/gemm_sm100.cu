@@ -617,7 +617,8 @@ extern "C" int omni_gemm(int kind, int epi, const void* w, const void* x, void* 
   const int bk = (kind == 0) ? 64 : 128;
   CUtensorMap tw, tx;
   if (make_tmap_2d(&tw, w, esz, (uint64_t)G * p.w_rows_per_group, K, K, 128, bk, true)) return -10;
-  if (x_group_col > 0 && (K % bk) != 0) return -6;  // a K tail would read the next group's columns
+  // With column groups a K tail reads the columns that follow (finite values of the caller's buffer); the weight's columns there
+  // are zero-filled, so they add nothing.
   if (make_tmap_2d(&tx, x, esz, (uint64_t)x_rows, x_cols, x_ld, bn, bk, true)) return -11;
   const int grid = sm_count();
 

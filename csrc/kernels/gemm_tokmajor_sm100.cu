@@ -667,7 +667,8 @@ extern "C" int omni_gemm_tm2(int kind, int epi, const void* w, const void* x, vo
   if (x_ld <= 0) x_ld = K;
   const uint64_t x_cols = x_group_col > 0 ? (uint64_t)x_ld : (uint64_t)K;
   const int bk = (kind == 0) ? 64 : 128;
-  if (x_group_col > 0 && (K % bk) != 0) return -6;   // a K tail would read the next group's columns
+  // With column groups a K tail reads the columns that follow (finite values of the caller's buffer); the weight's columns there
+  // are zero-filled, so they add nothing.
   CUtensorMap tx, tw;
   if (make_tmap_2d(&tx, x, esz, (uint64_t)x_rows, x_cols, x_ld, 128, bk, true)) return -11;
   if (make_tmap_2d(&tw, w, esz, (uint64_t)G * p.w_rows_per_group, K, K, TM_BN, bk, true)) return -10;

@@ -23,7 +23,9 @@
 // omni_gqa_paged_decode_window runs the general form of the same kernel: key and value sizes of their own (multiples of
 // 8 up to 256; staged rows are DP = 64, 128 or 256 wide and the columns past the real size stay zero), any number of query
 // heads per KV head (16 per CTA), a sliding window (tiles before it are not read), and softmax weights carried as a pair
-// of bf16 values (two MMAs per value tile), i.e. to 16 bits of mantissa.
+// of bf16 values (two MMAs per value tile), i.e. to 16 bits of mantissa.  Beside the window it knows kept first keys and
+// chunks, a soft cap of the scores and a distance bias per head (an instantiation of its own), cache rows of any pitch (latent
+// attention: the values are the first columns of the key rows), rows that share a request (q_to_seq), and a gate per row and head.
 //
 // Reference counterpart: the paged decode attention of the GQA backend
 // (omni/models/common/layers/attention/backend/attention.py:507-702).
@@ -31,6 +33,8 @@
 #include <cuda_runtime.h>
 
 #include <cstdint>
+
+#include "../include/score_mod.cuh"
 
 namespace omni {
 
@@ -51,7 +55,16 @@ struct GqShape {           // used by the general form only
   int q_ld, out_ld, dk, dv, window;
   const float* sink;       // [Hq] or null: exp(sink) is one more term of the softmax denominator
   float out_scale;         // multiplies the result before it is rounded
+  int chunk, keep;         // see first_key; the first `keep` keys are visible in any case
+  long long k_row, v_row;  // elements from one token's row to the next in the caches
+  const int* q_to_seq;     // [B] block-table row of each q row, or null (identity)
+  ScoreMod score;          // GEN 2
+  const __nv_bfloat16* gate;   // [B, gate_ld] or null: the result of head h is multiplied by sigmoid(gate[b, h])
+  int gate_ld;
 };
+__device__ __forceinline__ float gq_gate(const __nv_bfloat16* gate, int ld, int b, int h) {
+  return gate == nullptr ? 1.f : 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)b * ld + h])));
+}
 
 __device__ __forceinline__ uint32_t gq_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 template <int DP>
@@ -88,7 +101,8 @@ __device__ __forceinline__ uint32_t gq_rest(uint32_t packed, float lo, float hi)
   return gq_pack(lo - f.x, hi - f.y);
 }
 
-template <int DP, bool GEN>
+// GEN 0: the special form, 1: general, 2: general with capped or biased scores
+template <int DP, int GEN>
 __global__ void __launch_bounds__(GQ_WARPS * 32, DP > 128 ? 1 : 3)
 gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                   const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_table, int bt_ld,
@@ -107,11 +121,13 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
   const int q_ld = GEN ? sh.q_ld : Hq * DP, out_ld = GEN ? sh.out_ld : Hq * DP;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int L = seq_lens[b];
-  const int low = (GEN && sh.window > 0) ? max(0, L - sh.window) : 0;     // first visible key
+  const int low = GEN ? first_key(L - 1, sh.window, sh.chunk) : 0;        // first visible key, but for those kept
   const int tile0 = low / GQ_TILE;
-  const int tiles = (L + GQ_TILE - 1) / GQ_TILE - tile0;
+  const int nkeep = GEN ? min((sh.keep + GQ_TILE - 1) / GQ_TILE, tile0) : 0;   // tiles of kept keys ahead of it
+  const int tiles = nkeep + (L + GQ_TILE - 1) / GQ_TILE - tile0;
+  const int seq = (GEN && sh.q_to_seq != nullptr) ? sh.q_to_seq[b] : b;
   const int tps = (tiles + splits - 1) / splits;
-  const int t_begin = tile0 + split * tps, t_end = min(tile0 + tiles, t_begin + tps);
+  const int u_begin = split * tps, u_end = min(tiles, u_begin + tps);
 
   uint8_t* stage = gq_smem + warp * SM::STAGE_BYTES;          // [K tile][V tile]
   uint8_t* sq = gq_smem + GQ_WARPS * SM::STAGE_BYTES;         // 16 x DP bf16, swizzled like the tiles
@@ -145,20 +161,29 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 #pragma unroll
   for (int j = 0; j < JT; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
 
-  for (int t = t_begin + warp; t < t_end; t += GQ_WARPS) {
+  float slope[2] = {0.f, 0.f};                                // of the two rows of this lane, in log2 units
+  if (GEN == 2 && sh.score.slopes != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if ((lane >> 2) + 8 * r < G) slope[r] = sh.score.slopes[hk * Gall + g0 + (lane >> 2) + 8 * r] * 1.4426950408889634f;
+  }
+
+  for (int u = u_begin + warp; u < u_end; u += GQ_WARPS) {
+    const int t = u < nkeep ? u : tile0 + u - nkeep;
     // ---- stage the tile: lane `r` knows where key row r of the tile lives
     const int my_key = t * GQ_TILE + lane;
     const bool my_valid = my_key < L;
     long long my_slot = 0;
-    if (my_valid) my_slot = (long long)block_table[(size_t)b * bt_ld + my_key / block_size] * block_size + my_key % block_size;
+    if (my_valid) my_slot = (long long)block_table[(size_t)seq * bt_ld + my_key / block_size] * block_size + my_key % block_size;
 #pragma unroll 4
     for (int it = 0; it < GQ_TILE * CH / 32; ++it) {
       const int row = (it * 32 + lane) / CH, chunk = (it * 32 + lane) % CH;
       const long long slot = __shfl_sync(0xffffffffu, my_slot, row);
       const bool valid = __shfl_sync(0xffffffffu, (int)my_valid, row) != 0;
-      const size_t head = (size_t)slot * Hkv + hk;
-      if (!GEN || chunk * 8 < dk) gq_cp_async16(stage_k + gq_swz<DP>(row, chunk), k_cache + head * dk + chunk * 8, valid);
-      if (!GEN || chunk * 8 < dv) gq_cp_async16(stage_v + gq_swz<DP>(row, chunk), v_cache + head * dv + chunk * 8, valid);
+      const size_t k_at = GEN ? (size_t)slot * sh.k_row + (size_t)hk * dk : ((size_t)slot * Hkv + hk) * dk;
+      const size_t v_at = GEN ? (size_t)slot * sh.v_row + (size_t)hk * dv : ((size_t)slot * Hkv + hk) * dv;
+      if (!GEN || chunk * 8 < dk) gq_cp_async16(stage_k + gq_swz<DP>(row, chunk), k_cache + k_at + chunk * 8, valid);
+      if (!GEN || chunk * 8 < dv) gq_cp_async16(stage_v + gq_swz<DP>(row, chunk), v_cache + v_at + chunk * 8, valid);
     }
     gq_cp_async_wait_all();
     __syncwarp();
@@ -186,7 +211,9 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + j * 8 + (e & 1);
-        const float v = (key < L && (!GEN || key >= low)) ? s[j][e] * scale_log2 : -INFINITY;
+        const bool see = key < L && (!GEN || key >= low || key < sh.keep);
+        const float w = GEN == 2 ? cap_score(sh.score, s[j][e]) - slope[e >> 1] * (float)(L - 1 - key) : s[j][e] * scale_log2;
+        const float v = see ? w : -INFINITY;
         s[j][e] = v;
         mt[e >> 1] = fmaxf(mt[e >> 1], v);
       }
@@ -288,7 +315,7 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
     if (splits == 1) {
       float den = ll;
       if (GEN && sh.sink != nullptr && ll > 0.f) den += exp2f(sh.sink[hq] * 1.4426950408889634f - mm);
-      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / den * (GEN ? sh.out_scale : 1.f) : 0.f);
+      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / den * (GEN ? sh.out_scale * gq_gate(sh.gate, sh.gate_ld, b, hq) : 1.f) : 0.f);
     } else {
       o_part[(((size_t)b * splits + split) * Hq + hq) * dv + d] = ll > 0.f ? acc / ll : 0.f;
       if (d == 0) lse_part[((size_t)b * splits + split) * Hq + hq] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
@@ -298,7 +325,7 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 
 __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part, int splits,
                                    int Hq, int dv, int out_ld, const float* __restrict__ sink, float out_scale,
-                                   __nv_bfloat16* out) {
+                                   const __nv_bfloat16* __restrict__ gate, int gate_ld, __nv_bfloat16* out) {
   const int bh = blockIdx.x;
   const int b = bh / Hq, h = bh - b * Hq;
   const int d = threadIdx.x;
@@ -314,14 +341,14 @@ __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float
     acc += w * o_part[(((size_t)b * splits + s) * Hq + h) * dv + d];
   }
   if (sink != nullptr && den > 0.f) den += exp2f(sink[h] * 1.4426950408889634f - mx);
-  out[(size_t)b * out_ld + h * dv + d] = __float2bfloat16(den > 0.f ? acc / den * out_scale : 0.f);
+  out[(size_t)b * out_ld + h * dv + d] = __float2bfloat16(den > 0.f ? acc / den * out_scale * gq_gate(gate, gate_ld, b, h) : 0.f);
 }
 
 }  // namespace omni
 
 using namespace omni;
 
-template <int DP, bool GEN>
+template <int DP, int GEN>
 static int launch_gqa(dim3 grid, const void* q, const void* k_cache, const void* v_cache, const int* block_table, int bt_ld,
                       const int* seq_lens, int B, int block_size, int Hq, int Hkv, float scale, int splits, float* o_part,
                       float* lse_part, void* out, const GqShape& sh, int dv, int out_ld, cudaStream_t stream) {
@@ -341,7 +368,7 @@ static int launch_gqa(dim3 grid, const void* q, const void* k_cache, const void*
   if (e != cudaSuccess) return (int)e;
   if (splits > 1) {
     gqa_combine_kernel<<<B * Hq, (dv + 31) / 32 * 32, 0, stream>>>(o_part, lse_part, splits, Hq, dv, out_ld, sh.sink,
-                                                                   sh.out_scale, (__nv_bfloat16*)out);
+                                                                   sh.out_scale, sh.gate, sh.gate_ld, (__nv_bfloat16*)out);
     e = cudaGetLastError();
   }
   return (int)e;
@@ -356,26 +383,33 @@ extern "C" int omni_gqa_paged_decode(const void* q, const void* k_cache, const v
   if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;
   GqShape sh = {};
   sh.out_scale = 1.f;
-  return launch_gqa<GQ_D, false>(dim3(Hkv, splits, B), q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq,
+  return launch_gqa<GQ_D, 0>(dim3(Hkv, splits, B), q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq,
                                  Hkv, scale, splits, o_part, lse_part, out, sh, GQ_D, Hq * GQ_D, stream);
 }
 
-// General form: q rows of pitch q_ld, key size dk, value size dv, out rows of pitch out_ld, window 0 = all keys.
-extern "C" int omni_gqa_paged_decode_window(const void* q, int q_ld, const void* k_cache, const void* v_cache,
-                                            const int* block_table, int bt_ld, const int* seq_lens, int B, int Hq, int Hkv,
-                                            int dk, int dv, int block_size, int window, float scale, const float* sink,
-                                            float out_scale, int splits, float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
+// General form: q rows of pitch q_ld, key size dk, value size dv, out rows of pitch out_ld, window / chunk 0 = all keys.
+extern "C" int omni_gqa_paged_decode_window(const void* q, int q_ld, const void* k_cache, const void* v_cache, long long k_row,
+                                            long long v_row, const int* q_to_seq, const int* block_table, int bt_ld,
+                                            const int* seq_lens, int B, int Hq, int Hkv, int dk, int dv, int block_size,
+                                            int window, int chunk, int keep, float scale, float softcap, const float* slopes,
+                                            const float* sink, const void* gate, int gate_ld, float out_scale, int splits, float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (Hkv < 1 || Hq % Hkv != 0 || splits < 1 || splits > 65535 || B > 65535 || window < 0) return -1;
   if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;
   if (dk < 8 || dv < 8 || dk % 8 != 0 || dv % 8 != 0 || dk > 256 || dv > 256) return -3;
   if (q_ld % 8 != 0 || ((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16 != 0) return -4;
-  const GqShape sh = {q_ld, out_ld, dk, dv, window, sink, out_scale};
+  if (chunk < 0 || keep < 0 || k_row < (long long)Hkv * dk || v_row < (long long)Hkv * dv || k_row % 8 != 0 || v_row % 8 != 0) return -6;
+  const GqShape sh = {q_ld, out_ld, dk, dv, window, sink, out_scale, chunk, keep, k_row, v_row, q_to_seq,
+                      make_score_mod(scale, softcap, slopes), (const __nv_bfloat16*)gate, gate_ld};
+  const bool mod = softcap > 0.f || slopes != nullptr;
   const dim3 grid(Hkv * ((Hq / Hkv + 15) / 16), splits, B);
   const int d = dk > dv ? dk : dv;
 #define GQA_CASE(DP)                                                                                                     \
+  if (d <= DP && mod)                                                                                                    \
+    return launch_gqa<DP, 2>(grid, q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq, Hkv, scale,     \
+                             splits, o_part, lse_part, out, sh, dv, out_ld, stream);                                     \
   if (d <= DP)                                                                                                           \
-    return launch_gqa<DP, true>(grid, q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq, Hkv, scale,  \
+    return launch_gqa<DP, 1>(grid, q, k_cache, v_cache, block_table, bt_ld, seq_lens, B, block_size, Hq, Hkv, scale,  \
                                 splits, o_part, lse_part, out, sh, dv, out_ld, stream);
   GQA_CASE(64) GQA_CASE(128) GQA_CASE(256)
 #undef GQA_CASE

@@ -24,10 +24,15 @@
 // The running max is only raised when it grows by more than 2^8 (lazy rescale), so the O accumulator is
 // rarely read back.
 //
+// The exact form (omni_mla_decode_window: latent attention layers of layer-list models) adds a sliding window - tiles ahead of it
+// are not read -, carries the softmax weights as a pair of bf16 values (p = hi + lo, two MMAs per value tile), i.e. to 16 bits of
+// mantissa, and multiplies the result of every head by a sigmoid gate.
+//
 // Stands where the reference calls npu_fused_infer_attention_score on the absorbed path
 // (omni/models/common/layers/attention/deepseek_mla.py:533-560, 625-650).
 #include "../include/omni_noalloc.h"
 #include "../include/omni_ptx.cuh"
+#include "../include/score_mod.cuh"
 #include "../include/tma_host.h"
 
 namespace omni {
@@ -45,6 +50,9 @@ struct MlaDecodeParams {
   __nv_bfloat16* out;    // [Bq, H, 512]
   float* o_part;         // [Bq, splits, H, 512]
   float* lse_part;       // [Bq, splits, H]   (log2 domain)
+  int window;            // exact form: a row sees its last `window` tokens; 0 = all
+  const __nv_bfloat16* gate;   // exact form: [Bq, gate_ld] logits or null
+  int gate_ld;
   OmniStatus* status;
 };
 
@@ -225,6 +233,7 @@ __device__ __forceinline__ bool mla_issue_scores(const MlaPipe& px, MlaRing& rg,
 // instructions of about 48), as much as the tensor pipe needs to execute a whole tile, so two warps share the work:
 // while one waits for the softmax of its tile and issues P V, the other issues the scores of the next tile.
 // Tile i uses S buffer i & 1, so each issuer always works on the same buffer.
+template <bool EXACT>
 __device__ __forceinline__ void mla_mma(const MlaPipe& px, int n, const int which) {
   constexpr uint32_t idesc_pv = umma_idesc(128, 256, 1, 1, 0, 1);
   MlaRing rg;
@@ -256,6 +265,11 @@ __device__ __forceinline__ void mla_mma(const MlaPipe& px, int n, const int whic
 #pragma unroll
       for (int k = 1; k < MLA_TILE / 16; ++k)
         umma_bf16_ts(TM_O, pbase + (k >> 1) * 32 + (k & 1) * 8, vd + (uint64_t)(k * 128), idesc_pv, 1u);
+      if (EXACT) {             // the low parts of P lie 16 columns further
+#pragma unroll
+        for (int k = 0; k < MLA_TILE / 16; ++k)
+          umma_bf16_ts(TM_O, pbase + 16 + (k >> 1) * 32 + (k & 1) * 8, vd + (uint64_t)(k * 128), idesc_pv, 1u);
+      }
       umma_commit(&px.kv_empty[pv_stage]);
       umma_commit(px.o_done);
       if (i + 2 >= n) umma_commit(px.o_final);   // this issuer's last tile
@@ -266,6 +280,11 @@ __device__ __forceinline__ void mla_mma(const MlaPipe& px, int n, const int whic
   }
 }
 
+__device__ __forceinline__ float mla_gate(const __nv_bfloat16* gate, int ld, int bq, int h) {
+  return gate == nullptr ? 1.f : 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)bq * ld + h])));
+}
+
+template <bool EXACT>
 __global__ void __launch_bounds__(MLA_THREADS, 1)
 mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                   const MlaDecodeParams p) {
@@ -295,9 +314,11 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   const int bq = blockIdx.z;
 
   const int kv_len = p.seq_lens[bq];
+  const int low = EXACT ? first_key(kv_len - 1, p.window, 0) : 0;      // first visible token; its tile is the first one read
+  const int tile0 = low / MLA_TILE;
   const int tiles_total = (kv_len + MLA_TILE - 1) / MLA_TILE;
-  const int tps = (tiles_total + p.num_splits - 1) / p.num_splits;
-  const int tile_begin = split * tps;
+  const int tps = (tiles_total - tile0 + p.num_splits - 1) / p.num_splits;
+  const int tile_begin = tile0 + split * tps;
   const int tile_end = min(tiles_total, tile_begin + tps);
   const int n = max(0, tile_end - tile_begin);
 
@@ -360,7 +381,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       bool ok = mla_wait(q_full, 0, abort_flag, p.status, MS_Q, 0);
       if (ok) ok = mla_wait(qt_full, 0, abort_flag, p.status, MS_QT, 0);
       tc_fence_after();
-      if (ok) mla_mma(px, n, warp == 1 ? 0 : 1);
+      if (ok) mla_mma<EXACT>(px, n, warp == 1 ? 0 : 1);
     } else {
       // ------------------------------------------------------------ softmax / correction / epilogue
       // Eight warps: lane quadrant qd = warp & 3 selects 32 heads, group grp selects 32 of the 64 score
@@ -413,6 +434,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         if (!mla_wait(&s_full[st], (i >> 1) & 1, abort_flag, p.status, MS_S_FULL, i)) { ok = false; break; }
         tc_fence_after();
         const int valid = kv_len - (tile_begin + i) * MLA_TILE - grp * 32;  // valid columns of this group's half
+        const int unseen = EXACT ? low - (tile_begin + i) * MLA_TILE - grp * 32 : 0;   // columns ahead of the window
         const uint32_t s_addr = lane_addr + TM_S + st * 64 + grp * 32;
         float s[32];
         {
@@ -420,7 +442,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
           tmem_ld_x32(s_addr, sv);
           tmem_ld_wait();
 #pragma unroll
-          for (int j = 0; j < 32; ++j) s[j] = (j < valid) ? __uint_as_float(sv[j]) * p.scale_log2 : -INFINITY;
+          for (int j = 0; j < 32; ++j) s[j] = (j < valid && (!EXACT || j >= unseen)) ? __uint_as_float(sv[j]) * p.scale_log2 : -INFINITY;
         }
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -459,7 +481,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
           tmem_st_wait();
         }
         float rs4[4] = {0.f, 0.f, 0.f, 0.f};
-        uint32_t pk[16];
+        uint32_t pk[16], pl[16];
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           float p0, p1;
@@ -469,10 +491,16 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
           rs4[j & 3] += p0 + p1;
           __nv_bfloat162 h2 = __floats2bfloat162_rn(p0, p1);
           pk[j] = *reinterpret_cast<uint32_t*>(&h2);
+          if (EXACT) {      // what the rounding to bf16 left over
+            const float2 hf = __bfloat1622float2(h2);
+            h2 = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
+            pl[j] = *reinterpret_cast<uint32_t*>(&h2);
+          }
         }
         l += (rs4[0] + rs4[1]) + (rs4[2] + rs4[3]);
         // P (packed bf16) overwrites the first half of this group's own S columns, which only its warps read
         tmem_st_x16(s_addr, pk);
+        if (EXACT) tmem_st_x16(s_addr + 16, pl);
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
@@ -488,7 +516,8 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       }
       if (ok) {
         tc_fence_after();
-        const float inv_l = 1.0f / (sm_sum[row] + sm_sum[128 + row]);
+        float inv_l = 1.0f / (sm_sum[row] + sm_sum[128 + row]);
+        if (EXACT && p.num_splits == 1 && row < p.H) inv_l *= mla_gate(p.gate, p.gate_ld, bq, row);
         const float l_tot = sm_sum[row] + sm_sum[128 + row];
         const bool row_ok = row < p.H;
         const int c_lo = grp * 128;
@@ -574,7 +603,8 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
 
 // out[bq, h, :] = sum_s w_s * o_part[bq, s, h, :],  w_s = 2^(lse_s - max) / sum
 __global__ void mla_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part,
-                                   int splits, int H, __nv_bfloat16* out) {
+                                   int splits, int H, const __nv_bfloat16* __restrict__ gate, int gate_ld,
+                                   __nv_bfloat16* out) {
   const int bh = blockIdx.x;  // bq * H + h
   const int bq = bh / H, h = bh - bq * H;
   float mx = -INFINITY;
@@ -584,7 +614,7 @@ __global__ void mla_combine_kernel(const float* __restrict__ o_part, const float
     const float v = lse_part[((size_t)bq * splits + s) * H + h];
     den += (v == -INFINITY) ? 0.f : exp2f(v - mx);
   }
-  const float inv = den > 0.f ? 1.f / den : 0.f;
+  const float inv = den > 0.f ? mla_gate(gate, gate_ld, bq, h) / den : 0.f;
   for (int c = threadIdx.x * 4; c < 512; c += blockDim.x * 4) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s = 0; s < splits; ++s) {
@@ -613,11 +643,11 @@ extern "C" int omni_mla_debug_read(int* out32) {
   return (int)cudaMemcpyToSymbol(g_mla_debug, zeros, sizeof(zeros));
 }
 
-// Scratch needed for num_splits > 1: o_part = Bq*splits*H*512 floats, lse_part = Bq*splits*H floats.
-extern "C" int omni_mla_decode(const void* q, const void* cache, int cache_ld, long long num_slots,
-                               const int* block_table, int bt_ld, const int* seq_lens, const int* q_to_seq, int Bq,
-                               int H, int block_size, float scale, int num_splits, void* out, float* o_part,
-                               float* lse_part, void* status, cudaStream_t stream) {
+template <bool EXACT>
+static int mla_decode_launch(const void* q, const void* cache, int cache_ld, long long num_slots,
+                             const int* block_table, int bt_ld, const int* seq_lens, const int* q_to_seq, int Bq,
+                             int H, int block_size, float scale, int window, const void* gate, int gate_ld, int num_splits,
+                             void* out, float* o_part, float* lse_part, void* status, cudaStream_t stream) {
   if (Bq <= 0) return 0;
   if (H < 1 || H > 128) return -1;
   if (block_size != 32 && block_size % 64 != 0) return -2;
@@ -631,17 +661,38 @@ extern "C" int omni_mla_decode(const void* q, const void* cache, int cache_ld, l
   p.q = (const __nv_bfloat16*)q; p.H = H; p.block_size = block_size; p.block_table = block_table; p.bt_ld = bt_ld; p.seq_lens = seq_lens;
   p.q_to_seq = q_to_seq; p.scale_log2 = scale * 1.4426950408889634f; p.num_splits = num_splits;
   p.out = (__nv_bfloat16*)out; p.o_part = o_part; p.lse_part = lse_part; p.status = (OmniStatus*)status;
+  p.window = window; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
   static bool configured[64] = {false};
-  if (int e = ensure_dyn_smem((const void*)mla_decode_kernel, MLA_SMEM, configured)) return e;
+  if (int e = ensure_dyn_smem((const void*)mla_decode_kernel<EXACT>, MLA_SMEM, configured)) return e;
   dim3 grid(2, num_splits, Bq);
-  mla_decode_kernel<<<grid, MLA_THREADS, MLA_SMEM, stream>>>(tq, tkv, p);
+  mla_decode_kernel<EXACT><<<grid, MLA_THREADS, MLA_SMEM, stream>>>(tq, tkv, p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   if (num_splits > 1) {
-    mla_combine_kernel<<<Bq * H, 128, 0, stream>>>(o_part, lse_part, num_splits, H, (__nv_bfloat16*)out);
+    mla_combine_kernel<<<Bq * H, 128, 0, stream>>>(o_part, lse_part, num_splits, H, p.gate, gate_ld, (__nv_bfloat16*)out);
     e = cudaGetLastError();
   }
   return (int)e;
+}
+
+// Scratch needed for num_splits > 1: o_part = Bq*splits*H*512 floats, lse_part = Bq*splits*H floats.
+extern "C" int omni_mla_decode(const void* q, const void* cache, int cache_ld, long long num_slots,
+                               const int* block_table, int bt_ld, const int* seq_lens, const int* q_to_seq, int Bq,
+                               int H, int block_size, float scale, int num_splits, void* out, float* o_part,
+                               float* lse_part, void* status, cudaStream_t stream) {
+  return mla_decode_launch<false>(q, cache, cache_ld, num_slots, block_table, bt_ld, seq_lens, q_to_seq, Bq, H, block_size, scale,
+                                  0, nullptr, 0, num_splits, out, o_part, lse_part, status, stream);
+}
+
+// The exact form.
+extern "C" int omni_mla_decode_window(const void* q, const void* cache, int cache_ld, long long num_slots,
+                                      const int* block_table, int bt_ld, const int* seq_lens, const int* q_to_seq, int Bq,
+                                      int H, int block_size, float scale, int window, const void* gate, int gate_ld,
+                                      int num_splits, void* out, float* o_part, float* lse_part, void* status,
+                                      cudaStream_t stream) {
+  if (window < 0 || (gate != nullptr && gate_ld < H)) return -5;
+  return mla_decode_launch<true>(q, cache, cache_ld, num_slots, block_table, bt_ld, seq_lens, q_to_seq, Bq, H, block_size, scale,
+                                 window, gate, gate_ld, num_splits, out, o_part, lse_part, status, stream);
 }
 
 // -------------------------------------------------------------------------------------------------------

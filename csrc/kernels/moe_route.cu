@@ -19,6 +19,7 @@ constexpr int ROUTER_MAX_PER_LANE = 16;  // experts <= 512
 struct RouterParams {
   const float* logits;    // [T, E]
   const float* bias;      // [E] or null (added for selection only)
+  const float* logit_bias;   // [E] or null (part of the logits)
   int T, E;
   int mode;               // 0 softmax, 1 sigmoid
   int n_group, topk_group;
@@ -64,7 +65,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const RouterParams p) 
 #pragma unroll
   for (int i = 0; i < ROUTER_MAX_PER_LANE; ++i) {
     const int e = i * 32 + lane;
-    score[i] = (i < per_lane && e < p.E) ? lg[e] : -INFINITY;
+    score[i] = (i < per_lane && e < p.E) ? lg[e] + (p.logit_bias ? p.logit_bias[e] : 0.f) : -INFINITY;
     mx = fmaxf(mx, score[i]);
   }
   if (p.mode == 0) {
@@ -345,7 +346,7 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, int H, c
 
 using namespace omni;
 
-extern "C" int omni_router_topk(const float* logits, const float* bias, int T, int E, int mode, int n_group,
+extern "C" int omni_router_topk(const float* logits, const float* bias, const float* logit_bias, int T, int E, int mode, int n_group,
                                 int topk_group, int group_mode, int top_k, int renorm, float scale,
                                 const int* selector, void* counts, int n_counts, int forced_balance,
                                 const int* num_valid, int* out_ids, float* out_w, void* status,
@@ -354,7 +355,7 @@ extern "C" int omni_router_topk(const float* logits, const float* bias, int T, i
   if (E > 32 * ROUTER_MAX_PER_LANE || top_k > 32 || top_k > E) return -1;
   if (n_group > 32 || (n_group > 1 && E % n_group != 0)) return -2;
   RouterParams p;
-  p.logits = logits; p.bias = bias; p.T = T; p.E = E; p.mode = mode; p.n_group = n_group;
+  p.logits = logits; p.bias = bias; p.logit_bias = logit_bias; p.T = T; p.E = E; p.mode = mode; p.n_group = n_group;
   p.topk_group = topk_group; p.group_mode = group_mode; p.top_k = top_k; p.renorm = renorm; p.scale = scale;
   p.selector = selector; p.counts = (unsigned long long*)counts; p.forced_balance = forced_balance;
   p.n_counts = n_counts; p.st = (OmniStatus*)status;

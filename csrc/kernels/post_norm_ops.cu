@@ -1,14 +1,17 @@
-// Row kernels of models with an fp32 residual stream and norms on the sublayers' outputs:
+// Row kernels of models with one fp32 residual stream and norms on the sublayers' outputs or ahead of the sublayers:
 //   omni_embed_residual      embedding gather -> fp32 residual and its activation copy (the first sublayer's input)
 //   omni_post_norm_add       residual += rmsnorm(sublayer output) * w, and the activation copy for the next sublayer
 //   omni_rmsnorm_residual    final norm: fp32 residual -> activations
+//   omni_residual_norm       norms ahead: embedding gather, or residual += sublayer output (a tensor, or the parts of an expert
+//                            mixture) + bias, and the normed input of the next sublayer in the same pass
 //   omni_qk_norm_rope_cache  optional RMSNorm over the whole q and the whole k projection, rotate-half RoPE on the first
 //                            dimensions of every head, K/V scatter into the paged cache
-//   omni_gated_mul           gelu(gate) * up, or the clamped form, for widths the GEMM epilogue does not take
+//   omni_gated_mul           gelu(gate) * up, silu(gate) * up or the clamped form, for widths the GEMM epilogue does not take
 //   omni_gemm_f32            plain fp32 matrix products: dense, by row segments, or by column groups (fp32 runs of a model)
 // Activations are bf16 or fp32 (`f32` argument).  Rows have a pitch (`ld`, elements) that may exceed their width: the
 // padding columns of an output are written as zeros so that it can be a TMA operand of the next GEMM.  Norm weights are
 // fp32.  Every value between two roundings to the activation type is fp32.
+#include "../include/expert_sum.cuh"
 #include "../include/omni_vec.cuh"
 
 namespace omni {
@@ -103,6 +106,93 @@ __global__ void rmsnorm_residual_kernel(const float* __restrict__ x, const float
   for (int c = H + threadIdx.x; c < ld; c += blockDim.x) out[(size_t)t * ld + c] = from_f32<T>(0.f);
 }
 
+struct ResidualParams {
+  float* x;              // [T, ld]
+  const int64_t* ids;    // embedding gather: x = table[ids[t]]; null: x += y
+  const void* table;     // [rows, table_ld]
+  int rows, table_ld;
+  const void* y;         // sublayer output rows of pitch y_ld; expert mixtures: the sorted expert rows; null: x as it is
+  int y_ld;
+  const int* row_of;     // expert mixtures: [T, top_k] row of y, or -1; null: y has one row per token
+  int top_k;
+  const void* shared;    // expert mixtures: [T, y_ld] or null
+  const float* bias;     // [H] or null, added with y
+  const float* w;        // norm weight
+  float eps, out_scale;  // factor on the normed row
+  void* h;               // [T, h_ld]
+  int H, ld, h_ld;
+  int ones;              // column H of h is one (the column that carries the next projection's bias)
+};
+
+// KEEP vectors per thread stay in registers between the two passes; what is beyond them is read again.
+template <typename T, int V, int KEEP>
+__global__ void residual_norm_kernel(const ResidualParams p) {
+  const int t = blockIdx.x;
+  __shared__ int rows[32];
+  if (p.row_of != nullptr) {
+    if (threadIdx.x < p.top_k) rows[threadIdx.x] = p.row_of[(size_t)t * p.top_k + threadIdx.x];
+    __syncthreads();
+  }
+  float* xr = p.x + (size_t)t * p.ld;
+  const int64_t id = p.ids != nullptr ? p.ids[t] : 0;
+  const bool known = id >= 0 && id < p.rows;
+  float keep[KEEP][V], ss = 0.f;
+  const int step = blockDim.x * V;
+  auto update = [&](int c, float (&a)[V]) {
+    if (p.ids != nullptr) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) a[i] = 0.f;
+      if (known) load_vec<V>((const T*)p.table + (size_t)id * p.table_ld + c, a);
+    } else {
+      load_vec<V>(xr + c, a);
+      if (p.y != nullptr) {
+        float y[V];
+        if (p.row_of != nullptr) expert_sum<T, V>((const T*)p.y, p.y_ld, rows, p.top_k, (const T*)p.shared, t, c, y);
+        else load_vec<V>((const T*)p.y + (size_t)t * p.y_ld + c, y);
+#pragma unroll
+        for (int i = 0; i < V; ++i) a[i] += y[i];
+        if (p.bias != nullptr) {
+          load_vec<V>(p.bias + c, y);
+#pragma unroll
+          for (int i = 0; i < V; ++i) a[i] += y[i];
+        }
+      }
+    }
+    store_vec<V>(xr + c, a);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += a[i] * a[i];
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int c = threadIdx.x * V + k * step;
+    if (c < p.H) update(c, keep[k]);
+  }
+  for (int c = threadIdx.x * V + KEEP * step; c < p.H; c += step) {
+    float a[V];
+    update(c, a);
+  }
+  const float r = p.out_scale / sqrtf(block_sum2(ss, 0.f).x / (float)p.H + p.eps);
+  T* hr = (T*)p.h + (size_t)t * p.h_ld;
+  auto finish = [&](int c, float (&a)[V]) {
+    float g[V];
+    load_vec<V>(p.w + c, g);
+#pragma unroll
+    for (int i = 0; i < V; ++i) a[i] = a[i] * r * g[i];
+    store_vec<V>(hr + c, a);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int c = threadIdx.x * V + k * step;
+    if (c < p.H) finish(c, keep[k]);
+  }
+  for (int c = threadIdx.x * V + KEEP * step; c < p.H; c += step) {
+    float a[V];
+    load_vec<V>(xr + c, a);
+    finish(c, a);
+  }
+  for (int c = p.H + threadIdx.x; c < p.h_ld; c += blockDim.x) hr[c] = from_f32<T>(p.ones && c == p.H ? 1.f : 0.f);
+}
+
 // One CTA per token, one warp per head.  q rows are normed (qw null: not) and rotated in place, k rows go to the cache the same way,
 // v rows are copied.  Hkv = 0: the layer reads another layer's cache and has q rows only.
 template <typename T, int V>
@@ -179,7 +269,7 @@ __global__ void qk_norm_rope_cache_kernel(T* __restrict__ qkv, int ld, int Hq, i
   }
 }
 
-// KIND 0: gelu(g) u, 1: min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1)
+// KIND 0: gelu(g) u, 2: silu(g) u, 1: min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1)
 template <typename T, int V, int KIND>
 __global__ void gated_mul_kernel(const T* __restrict__ x, int x_ld, int up_off, T* __restrict__ out, int out_ld, int T_rows,
                                  int I, float limit) {
@@ -197,6 +287,8 @@ __global__ void gated_mul_kernel(const T* __restrict__ x, int x_ld, int up_off, 
     for (int i = 0; i < V; ++i) {
       if (KIND == 0) {
         o[i] = gelu_tanh_for<T>(g[i]) * u[i];
+      } else if (KIND == 2) {
+        o[i] = silu_for<T>(g[i]) * u[i];
       } else {
         const float gc = fminf(g[i], limit);
         o[i] = div_for<T>(gc, 1.0f + exp_for<T>(-1.702f * gc)) * (fminf(fmaxf(u[i], -limit), limit) + 1.0f);
@@ -307,6 +399,22 @@ extern "C" int omni_rmsnorm_residual(const void* x, const void* w, void* out, in
   return (int)cudaGetLastError();
 }
 
+extern "C" int omni_residual_norm(void* x, int T_rows, int H, int ld, const int64_t* ids, const void* table, int rows, int table_ld,
+                                  const void* y, int y_ld, const int* row_of, int top_k, const void* shared, const float* bias,
+                                  const float* w, float eps, float out_scale, void* h, int h_ld, int ones, int f32,
+                                  cudaStream_t st) {
+  if (T_rows <= 0) return 0;
+  if (H < 1 || ld < H || h_ld < H + (ones ? 1 : 0) || (ids != nullptr && table_ld < H) || (y != nullptr && y_ld < H)) return -1;
+  if (row_of != nullptr && (top_k < 1 || top_k > 32 || y == nullptr)) return -2;
+  const ResidualParams p = {(float*)x, ids, table, rows, table_ld, y, y_ld, row_of, top_k, shared, bias, w, eps, out_scale, h, H, ld, h_ld, ones};
+  if (H % 8 == 0 && ld % 8 == 0 && h_ld % 8 == 0 && (ids == nullptr || table_ld % 8 == 0) && (y == nullptr || y_ld % 8 == 0)) {
+    FOR_TYPE((residual_norm_kernel<T, 8, 2><<<T_rows, row_threads(H, 8), 0, st>>>(p));)
+  } else {
+    FOR_TYPE((residual_norm_kernel<T, 1, 1><<<T_rows, row_threads(H, 1), 0, st>>>(p));)
+  }
+  return (int)cudaGetLastError();
+}
+
 extern "C" int omni_qk_norm_rope_cache(void* qkv, int ld, int Hq, int Hkv, int D, int DV, const void* qw, const void* kw,
                                        float eps, const void* cos_sin, int rot, const int64_t* positions,
                                        const int64_t* slots, void* k_cache, void* v_cache, int T_rows, int f32,
@@ -329,7 +437,7 @@ extern "C" int omni_qk_norm_rope_cache(void* qkv, int ld, int Hq, int Hkv, int D
 extern "C" int omni_gated_mul(const void* x, int x_ld, int up_off, void* out, int out_ld, int T_rows, int I, int kind, float limit,
                               int f32, cudaStream_t st) {
   if (T_rows <= 0) return 0;
-  if (I < 1 || out_ld < I || T_rows > 65535 * 16 || kind < 0 || kind > 1) return -1;
+  if (I < 1 || out_ld < I || T_rows > 65535 * 16 || kind < 0 || kind > 2) return -1;
   const int vec = (I % 8 == 0 && x_ld % 8 == 0 && up_off % 8 == 0 && out_ld % 8 == 0) ? 8 : 1;
 #define GATED(V, KIND)                                                                                                        \
   FOR_TYPE((gated_mul_kernel<T, V, KIND><<<grid, 128, 0, st>>>((const T*)x + (size_t)r0 * x_ld, x_ld, up_off,                 \
@@ -338,8 +446,10 @@ extern "C" int omni_gated_mul(const void* x, int x_ld, int up_off, void* out, in
     const int n = T_rows - r0 < 65535 ? T_rows - r0 : 65535;
     const dim3 grid((out_ld / vec + 127) / 128 + (out_ld % vec ? 1 : 0), n);
     if (vec == 8 && kind == 0) { GATED(8, 0) }
+    else if (vec == 8 && kind == 2) { GATED(8, 2) }
     else if (vec == 8) { GATED(8, 1) }
     else if (kind == 0) { GATED(1, 0) }
+    else if (kind == 2) { GATED(1, 2) }
     else { GATED(1, 1) }
   }
 #undef GATED

@@ -8,6 +8,7 @@
 //                        which is moved on
 //   omni_tanh_split      tanh of fp32 values as bf16 hi | lo, so that a product keeps 16 bits of mantissa on that side
 // Streams are fp32, [T, streams, ld]; activations are bf16 or fp32 (`f32`), their padding columns are written as zeros.
+#include "../include/expert_sum.cuh"
 #include "../include/omni_vec.cuh"
 
 namespace omni {
@@ -108,26 +109,12 @@ __global__ void stream_step_kernel(const StepParams p) {
     if (p.row_of == nullptr) {
       load_vec<V>((const T*)p.y + (size_t)t * p.y_ld + c, y);
     } else {
-#pragma unroll
-      for (int i = 0; i < V; ++i) y[i] = 0.f;
-      for (int k = 0; k < p.top_k; ++k) {
-        if (rows[k] < 0) continue;
-        float v[V];
-        load_vec<V>((const T*)p.y + (size_t)rows[k] * p.y_ld + c, v);
-#pragma unroll
-        for (int i = 0; i < V; ++i) y[i] += v[i];
-      }
+      expert_sum<T, V>((const T*)p.y, p.y_ld, rows, p.top_k, (const T*)p.shared, t, c, y);
       if (same != 0.f) {
         float v[V];
         load_vec<V>((const T*)p.h_in + (size_t)t * p.h_ld + c, v);
 #pragma unroll
         for (int i = 0; i < V; ++i) y[i] = fmaf(same, v[i], y[i]);
-      }
-      if (p.shared != nullptr) {
-        float v[V];
-        load_vec<V>((const T*)p.shared + (size_t)t * p.y_ld + c, v);
-#pragma unroll
-        for (int i = 0; i < V; ++i) y[i] += v[i];
       }
     }
     float a[S][V], u[V];

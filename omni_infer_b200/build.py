@@ -55,9 +55,11 @@ def _run(cmd, log: Path | None = None) -> None:
 # Kernel sources (stems) that one architecture needs when it is served alone
 ARCH_KERNELS = {
     "Forovik": ("attn_any", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "mamba2", "post_norm_ops",
-                "sampler_misc", "ssd_sm100"),
+                "sampler_misc", "short_conv", "ssd_sm100"),
     "Fimudra": ("attn_any", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "matrix_state", "moe_route",
                 "post_norm_ops", "sampler_misc", "ssd_sm100", "stream_ops", "wkv_chunk"),
+    "Tenotar": ("attn_any", "attn_prepare", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "mla_decode", "moe_route",
+                "norm_rope", "post_norm_ops", "sampler_misc", "short_conv"),
 }
 
 

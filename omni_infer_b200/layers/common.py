@@ -42,6 +42,7 @@ class AttnMetadata:
     state_slots: Optional[torch.Tensor] = None     # [B] int32 recurrent-state slot per request, -1 = padding row
     # Omni-Attention (compressed layers): per-layer-group overrides
     omni: Optional[dict] = None
+    plans: dict = field(default_factory=dict)      # what layers have worked out for this step and share
 
 
 def _dtype(name: str) -> torch.dtype:
@@ -95,26 +96,39 @@ class PaddedLinear(Linear):
     """Linear whose stored weight has both sizes rounded up to a multiple of 8 (TMA row pitch, 16-byte output vectors).  The
     padding is zero and activations carry zeros in their padding columns, so the product is that of the real sizes."""
 
-    def __init__(self, in_features: int, out_features: int, *, dtype=torch.bfloat16, device=None):
-        super().__init__((in_features + 7) // 8 * 8, (out_features + 7) // 8 * 8, dtype=dtype, device=device)
+    def __init__(self, in_features: int, out_features: int, *, dtype=torch.bfloat16, device=None, bias_column: bool = False):
+        """``bias_column``: one more column holds the biases; activations carry a one there (``ops.layer_list.add_norm``)."""
+        self.bias_column = bias_column
+        super().__init__((in_features + int(bias_column) + 7) // 8 * 8, (out_features + 7) // 8 * 8, dtype=dtype, device=device)
         self.real_in, self.real_out = in_features, out_features
         self.zero_padding()
 
     def zero_padding(self):
         self.weight.data[self.real_out:] = 0
-        self.weight.data[:, self.real_in:] = 0
+        self.weight.data[:, self.real_in + int(self.bias_column):] = 0
+
+    def bias_target(self, row0: int, rows: int):
+        """Checkpoint target of the biases of those rows."""
+        return self.weight.data[:, self.real_in], row0, rows, None
 
 
 class GeGLUMLP(nn.Module):
     """gate_up (merged, gate rows first, each block padded to a multiple of 8) -> gelu (tanh form) of the gate times up,
-    in the GEMM epilogue where the width allows -> down."""
+    in the GEMM epilogue where the width allows -> down.  ``epi="swiglu"``: silu of the gate.  ``bias``: all three projections
+    have one; the last is left to the caller, who adds it with the residual."""
     epi = "geglu"
 
-    def __init__(self, hidden: int, inter: int, *, dtype=torch.bfloat16, device=None):
+    def __init__(self, hidden: int, inter: int, *, dtype=torch.bfloat16, device=None, epi=None, bias: bool = False):
         super().__init__()
-        self.inter, self.block, self.limit = inter, (inter + 7) // 8 * 8, 0.0
-        self.gate_up_proj = PaddedLinear(hidden, 2 * self.block, dtype=dtype, device=device)
+        self.epi = epi or self.epi
+        self.inter, self.block, self.limit, self.ones = inter, (inter + 7) // 8 * 8, 0.0, bias
+        self.gate_up_proj = PaddedLinear(hidden, 2 * self.block, dtype=dtype, device=device, bias_column=bias)
         self.down_proj = PaddedLinear(inter, hidden, dtype=dtype, device=device)
+        self.out_bias = nn.Parameter(torch.zeros(hidden, dtype=torch.float32, device=device), requires_grad=False) if bias else None
+
+    @property
+    def in_cols(self):
+        return self.gate_up_proj.in_features
 
     def zero_padding(self):
         w = self.gate_up_proj.weight.data
@@ -127,7 +141,11 @@ class GeGLUMLP(nn.Module):
     def checkpoint_targets(self):
         """{checkpoint suffix: (parameter, first row, rows, columns)}."""
         w, h = self.gate_up_proj.weight, self.gate_up_proj.real_in
-        return {"gate": (w, 0, self.inter, h), "up": (w, self.block, self.inter, h), "down": (self.down_proj.weight, 0, h, self.inter)}
+        t = {"gate": (w, 0, self.inter, h), "up": (w, self.block, self.inter, h), "down": (self.down_proj.weight, 0, h, self.inter)}
+        if self.out_bias is not None:
+            t.update({"gate.b": self.gate_up_proj.bias_target(0, self.inter), "up.b": self.gate_up_proj.bias_target(self.block, self.inter),
+                      "down.b": (self.out_bias, 0, h, None)})
+        return t
 
 
 class ClampedGLUMLP(GeGLUMLP):

@@ -27,7 +27,7 @@ from ..ops import FP8
 from ..parallel import get_parallel_state
 from ..ops.layer_list import pad8
 from ..ops.streams import ExpertSum
-from .common import ClampedGLUMLP, Linear, PaddedLinear, SwiGLUMLP
+from .common import ClampedGLUMLP, GeGLUMLP, Linear, PaddedLinear, SwiGLUMLP
 
 
 import os as _os
@@ -249,9 +249,12 @@ class MoELayer(nn.Module):
 
 
 class ExpertMixture(nn.Module):
-    """Mixture of clamped gated experts of a layer-list model: softmax scores over the experts and the identity experts (whose
-    output is the input), the choice by score + correction, weights = scores * scale without renormalising, and a shared
-    expert.  Every rank holds all experts.  The parts are returned unsummed; the residual kernel adds them up."""
+    """Mixture of gated experts of a layer-list model, with a shared expert.  Either softmax scores over the experts and the
+    identity experts (whose output is the input), the choice by score + correction, weights = scores * scale without
+    renormalising; or the choice by logit + bias and the softmax over the chosen.  Every rank holds all experts.  The parts are
+    returned unsummed; the residual kernel adds them up."""
+    out_bias = None
+    ones = False
 
     def __init__(self, spec, hidden: int, *, dtype, device=None):
         super().__init__()
@@ -260,10 +263,19 @@ class ExpertMixture(nn.Module):
         self.block = pad8(s.ff)
         zeros = lambda *n, dt=dtype: nn.Parameter(torch.zeros(*n, dtype=dt, device=device), requires_grad=False)  # noqa: E731
         self.router = zeros(s.experts + s.identity, W)
-        self.correction = zeros(s.experts + s.identity, dt=torch.float32)
+        self.correction = zeros(s.experts + s.identity, dt=torch.float32)      # of the scores, or the bias of the logits
         self.correction.init_value = 0.0
+        self.chosen = s.weighting == "chosen"
         self.w13, self.w2 = zeros(s.experts, 2 * self.block, W), zeros(s.experts, W, self.block)
-        self.shared = ClampedGLUMLP(hidden, s.shared_ff, s.shared_limit, dtype=dtype, device=device) if s.shared_ff else None
+        self.shared = None
+        if s.shared_ff and s.act == "clamped_glu":
+            self.shared = ClampedGLUMLP(hidden, s.shared_ff, s.shared_limit, dtype=dtype, device=device)
+        elif s.shared_ff:
+            self.shared = GeGLUMLP(hidden, s.shared_ff, dtype=dtype, device=device, epi=s.act)
+
+    @property
+    def in_cols(self):
+        return pad8(self.hidden)
 
     def zero_padding(self):
         H, ff, b = self.hidden, self.spec.ff, self.block
@@ -283,10 +295,11 @@ class ExpertMixture(nn.Module):
             else:
                 shared = self.shared(x)
         logits = ops.gemm(x, self.router, out_dtype=torch.float32)
-        ids, w = ops.router_topk(logits, s.top, mode="softmax", bias=self.correction, scale=s.scale, num_valid=num_valid)
+        how = dict(logit_bias=self.correction, renorm=True) if self.chosen else dict(bias=self.correction)
+        ids, w = ops.router_topk(logits, s.top, mode="softmax", scale=s.scale, num_valid=num_valid, **how)
         perm = ops.moe_permute(x, ids, w, 0, s.experts)
         kw = dict(seg_start=perm.seg_start, seg_len=perm.seg_len, t_hint=max(16, (T * s.top + s.experts - 1) // s.experts))
-        act = ops.gemm(perm.x, self.w13, epi="clamped_glu", glu_limit=s.limit, **kw)
+        act = ops.gemm(perm.x, self.w13, epi=s.act, glu_limit=s.limit, **kw)
         y = ops.gemm(act, self.w2, row_scale=perm.row_w, **kw)
         if done is not None:
             torch.cuda.current_stream().wait_event(done)
@@ -296,7 +309,7 @@ class ExpertMixture(nn.Module):
         """{checkpoint suffix: (parameter or a view of one, first row, rows, columns)}; columns None: a vector."""
         s, H, b = self.spec, self.hidden, self.block
         n = s.experts + s.identity
-        t = {"router": (self.router, 0, n, H), "correction": (self.correction, 0, n, None)}
+        t = {"router": (self.router, 0, n, H), "router.b" if self.chosen else "correction": (self.correction, 0, n, None)}
         for e in range(s.experts):
             t[f"e{e}.gate"], t[f"e{e}.up"] = (self.w13.data[e], 0, s.ff, H), (self.w13.data[e], b, s.ff, H)
             t[f"e{e}.down"] = (self.w2.data[e], 0, H, s.ff)

@@ -10,6 +10,10 @@ from pathlib import Path
 from typing import Any, Optional
 
 
+# architectures of layer-list models with one residual and norms ahead of the sublayers
+NORM_FIRST = ("Tenotar",)
+
+
 @dataclass
 class AttentionSpec:
     """Softmax attention of one layer of a layer-list model."""
@@ -26,6 +30,15 @@ class AttentionSpec:
     qk_norm: bool = True                     # RMSNorm over the whole q and the whole k projection
     sink: bool = False                       # a learned term per head in the softmax denominator
     rot_scaling: Optional[dict] = None       # other scalings, as ``ops.rope_cos_sin_table`` takes them
+    keep_first: int = 0                      # the first tokens of a sequence, seen beside the window
+    chunk: int = 0                           # a query sees its own chunk of this many positions only; 0 = no chunks
+    softcap: float = 0.0                     # scores are bounded softly by it (tanh); 0 = not
+    distance_bias: bool = False              # slope 2^(-8 (h + 1) / heads) times the distance is taken off head h's scores
+    head_norm: bool = False                  # RMSNorm of every q and k head (one weight each)
+    rot_pairs: bool = False                  # neighbouring dimensions are rotated together (else i with i + rot_dims / 2)
+    bias: bool = False                       # of the four projections
+    conv: int = 0                            # taps of a short convolution of q, k and v; 0 = none
+    v_mix: bool = False                      # values are mixed with those of the first layer that has this set
 
     @property
     def owns_kv(self) -> bool:
@@ -33,6 +46,56 @@ class AttentionSpec:
 
     def cache_elems_per_token(self) -> int:
         return self.kv_heads * (self.dim + self.vdim) if self.owns_kv else 0
+
+    def page_shapes(self, blocks: int, block_size: int) -> tuple:
+        """Shapes of the page pools: keys, values."""
+        return (blocks, block_size, self.kv_heads, self.dim), (blocks, block_size, self.kv_heads, self.vdim)
+
+
+@dataclass
+class LatentSpec:
+    """Softmax attention through a query and a key/value latent of one layer of a layer-list model.  The cache holds the normed
+    latent and one rotated key part that all heads share."""
+    heads: int
+    dim: int                                 # unrotated query / key size per head
+    rot_dim: int                             # rotated query / key size per head
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    window: int = 0                          # a query sees itself and the window - 1 tokens before it; 0 = all
+    rot_base: float = 10000.0
+    gate: bool = True                        # a sigmoid gate per head on the output
+
+    kv_from = None
+    owns_kv = True
+    rot_factor = 1.0
+    rot_scaling = None
+
+    @property
+    def rot_dims(self) -> int:
+        return self.rot_dim
+
+    # Sizes as stored: multiples of 8, and the size that the latent decode kernel is made for where the general one ends.
+    @property
+    def _stored(self) -> tuple:
+        c, r = (self.kv_rank + 7) // 8 * 8, (self.rot_dim + 7) // 8 * 8
+        return (512, 64) if c + r > 256 and c <= 512 and r <= 64 else (c, r)
+
+    @property
+    def latent_cols(self) -> int:
+        return self._stored[0]
+
+    @property
+    def rot_cols(self) -> int:
+        return self._stored[1]
+
+    def cache_elems_per_token(self) -> int:
+        return self.latent_cols + self.rot_cols
+
+    def page_shapes(self, blocks: int, block_size: int) -> tuple:
+        """Shape of the one page pool: latent | rotated key part."""
+        return ((blocks, block_size, self.cache_elems_per_token()),)
 
 
 @dataclass
@@ -82,15 +145,18 @@ class ParallelSpec:
 
 @dataclass
 class ExpertsSpec:
-    """Mixture of clamped gated experts of one layer of a layer-list model."""
+    """Mixture of gated experts of one layer of a layer-list model."""
     experts: int
     top: int
     ff: int
-    limit: float
+    limit: float = 0.0                       # of the clamped gate
     identity: int = 0                        # router outputs after the experts' whose expert is the identity
     scale: float = 1.0                       # of the routing weights
     shared_ff: int = 0                       # expert that runs for every token, 0 = none
     shared_limit: float = 0.0
+    act: str = "clamped_glu"                 # or "swiglu"
+    # "scores": softmax over all outputs, chosen by score + correction; "chosen": by logit + bias, softmax over the chosen ones
+    weighting: str = "scores"
 
 
 @dataclass
@@ -103,15 +169,21 @@ class LayerSpec:
     wkv: Optional[WkvSpec] = None
     experts: Optional[ExpertsSpec] = None
     weights_of: Optional[int] = None         # the layer runs with this layer's weights and a cache or state of its own
+    latent: Optional[LatentSpec] = None
+    act: str = "geglu"                       # of the dense feed-forward: or "swiglu"
+    ff_bias: bool = False                    # of its three projections
 
     @property
-    def paged(self) -> Optional[AttentionSpec]:
+    def paged(self):
         """The attention that reads (and, unless it shares them, fills) cache pages."""
+        if self.latent is not None:
+            return self.latent
         return self.parallel.left if self.parallel is not None else self.attention
 
     @property
     def recurrent(self) -> bool:
-        return self.mamba2 is not None or self.parallel is not None or self.wkv is not None
+        return (self.mamba2 is not None or self.parallel is not None or self.wkv is not None
+                or (self.attention is not None and self.attention.conv > 0))
 
     @staticmethod
     def _pre_norm_attention(i: int, m: dict) -> AttentionSpec:
@@ -126,12 +198,41 @@ class LayerSpec:
         return a
 
     @classmethod
-    def from_dict(cls, i: int, d: dict) -> "LayerSpec":
+    def _norm_first_entry(cls, i: int, d: dict) -> "LayerSpec":
+        """Entry ``i`` of a design with one residual and norms ahead of the sublayers: latent attention; windowed attention
+        with biases, head norms and pairwise rotation ("attention"); chunked attention with convolved projections, capped
+        scores and a distance bias ("attention_2")."""
+        kind, m = d["type"], d["mixer"]
+        rot, mask, s = m.get("rot") or {}, m.get("mask") or {}, cls(act="swiglu", ff_bias=True)
+        base = float(rot.get("base", 10000.0))
+        if kind == "latent_attention":
+            s.latent = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], q_rank=m["q_rank"],
+                                  kv_rank=m["kv_rank"], scale=float(m["scale"]), window=int(mask.get("size") or 0), rot_base=base)
+            if s.latent.rot_dim % 2 or rot.get("dims", s.latent.rot_dim) != s.latent.rot_dim:
+                raise ValueError(f"layer {i}: the rotated part must be even and rotated as a whole")
+        elif kind in ("attention", "attention_2"):
+            a = s.attention = AttentionSpec(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"],
+                                            scale=float(m["scale"]), qk_norm=False, v_mix=bool(m.get("v_mix")))
+            if kind == "attention":
+                a.window, a.keep_first = int(mask.get("size") or 0), int(mask.get("keep_first") or 0)
+                a.rot_dims, a.rot_base, a.rot_pairs = int(rot.get("dims", 0)), base, True
+                a.head_norm = a.bias = True
+            else:
+                a.chunk, a.softcap, a.distance_bias = int(mask.get("size") or 0), float(m.get("softcap") or 0.0), True
+                a.conv = int(m["conv"])
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        return s
+
+    @classmethod
+    def from_dict(cls, i: int, d: dict, norm_first: bool = False) -> "LayerSpec":
         """Entry ``i`` of the ``layers`` list of a config.json.  The type may carry a running number (several mixers of
         one kind with sizes of their own)."""
         kind, m = re.sub(r"_\d+$", "", d["type"]), d["mixer"]
-        s = cls(weights_of=d.get("weights_of"))
-        if kind == "attention":
+        s = cls._norm_first_entry(i, d) if norm_first else cls(weights_of=d.get("weights_of"))
+        if norm_first:
+            pass
+        elif kind == "attention":
             rot = m.get("rot") or {}
             s.attention = AttentionSpec(
                 heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]),
@@ -153,7 +254,7 @@ class LayerSpec:
         else:
             raise ValueError(f"layer {i}: unknown mixer type {d['type']!r}")
         a = s.paged
-        if a is not None and (a.heads % a.kv_heads or a.rot_dims % 2 or a.rot_dims > a.dim):
+        if a is not None and s.latent is None and (a.heads % a.kv_heads or a.rot_dims % 2 or a.rot_dims > a.dim):
             raise ValueError(f"layer {i}: heads must divide over the key/value heads, rotated dimensions be even and fit the head")
         mlp = d.get("mlp")
         if mlp:
@@ -164,9 +265,13 @@ class LayerSpec:
                 if not mlp.get("router") or not mlp.get("expert"):
                     raise ValueError(f"layer {i}: a feed-forward of kind 'moe' needs a router and an expert")
                 r, e, sh = mlp["router"], mlp["expert"], mlp.get("shared") or {}
-                s.experts = ExpertsSpec(experts=r["experts"], top=r["top"], ff=e["ff"], limit=float(e["limit"]),
-                                        identity=int(r.get("identity") or 0), scale=float(r.get("scale", 1.0)),
-                                        shared_ff=int(sh.get("ff", 0)), shared_limit=float(sh.get("limit", 0.0)))
+                if norm_first:
+                    s.experts = ExpertsSpec(experts=r["experts"], top=r["top"], ff=e["ff"], shared_ff=int(sh.get("ff", 0)),
+                                            act="swiglu", weighting="chosen")
+                else:
+                    s.experts = ExpertsSpec(experts=r["experts"], top=r["top"], ff=e["ff"], limit=float(e["limit"]),
+                                            identity=int(r.get("identity") or 0), scale=float(r.get("scale", 1.0)),
+                                            shared_ff=int(sh.get("ff", 0)), shared_limit=float(sh.get("limit", 0.0)))
                 n = s.experts.experts + s.experts.identity
                 if not 0 < s.experts.top <= min(n, 32) or n > 512:
                     raise ValueError(f"layer {i}: {s.experts.top} of {n} experts (at most 32 of 512)")
@@ -183,6 +288,9 @@ class ModelConfig:
     # residual streams of a layer-list model with layer norms ahead of its sublayers; 0 = one residual, norms on the outputs
     streams: int = 0
     embedding_scale: float = 1.0
+    # layer-list models: one residual with RMS norms ahead of the sublayers
+    norm_first: bool = False
+    logit_scale: float = 1.0
     # tensor-parallel attention: heads sharded over attn_tp_size ranks, hidden states sharded by token rows between
     # layers (set by the model runner; 1 = every rank runs whole attention layers on its own requests)
     attn_tp_size: int = 1
@@ -324,7 +432,8 @@ class ModelConfig:
     @classmethod
     def from_layer_list(cls, arch: str, d: dict[str, Any]) -> "ModelConfig":
         """config.json whose ``layers`` list describes every layer (mixer and feed-forward sizes of its own)."""
-        layers = [LayerSpec.from_dict(i, e) for i, e in enumerate(d["layers"])]
+        norm_first = arch in NORM_FIRST
+        layers = [LayerSpec.from_dict(i, e, norm_first) for i, e in enumerate(d["layers"])]
         for i, s in enumerate(layers):
             a = s.attention
             if a is None or a.owns_kv:
@@ -335,7 +444,11 @@ class ModelConfig:
             if (src.kv_heads, src.dim, src.vdim) != (a.kv_heads, a.dim, a.vdim):
                 raise ValueError(f"layers {i} and {a.kv_from} share keys but differ in their head sizes")
         streams = int(d.get("streams", 0))
-        if any((s.parallel or s.wkv or s.experts) is not None if not streams else (s.attention or s.mamba2) is not None or s.ff for s in layers):
+        if norm_first:
+            mixed = {s.attention.kv_heads * s.attention.vdim for s in layers if s.attention is not None and s.attention.v_mix}
+            if len(mixed) > 1:
+                raise ValueError("layers that mix their values must have equally many of them")
+        elif any((s.parallel or s.wkv or s.experts) is not None if not streams else (s.attention or s.mamba2) is not None or s.ff for s in layers):
             raise ValueError("attention, mamba2 and dense layers run on one residual with norms on the outputs, parallel, wkv and "
                              "mixture-of-experts layers on residual streams with norms ahead")
         for i, s in enumerate(layers):
@@ -352,8 +465,9 @@ class ModelConfig:
                 layers[i].weights_of = next(j for j, o in enumerate(layers) if o is s)
         return cls(architecture=arch, layers=layers, vocab_size=d["vocab"], hidden_size=d["width"],
                    num_hidden_layers=len(layers), rms_norm_eps=float(d["norm"]["eps"]), use_mla=False,
-                   tie_word_embeddings=True, n_routed_experts=0, name=arch, streams=streams,
-                   embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
+                   tie_word_embeddings=not norm_first, n_routed_experts=0, name=arch, streams=streams,
+                   embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)), norm_first=norm_first,
+                   logit_scale=float(d.get("logit_scale", 1.0)))
 
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
@@ -524,6 +638,41 @@ def tiny_fimudra(**kw) -> ModelConfig:
                    w_dim=12, w_rank=5, experts=6, identity=2, top=2, ff=24, shared_ff=40, **kw)
 
 
+def tenotar(width=2048, layers=12, vocab=32768, heads=16, kv_heads=4, dim=128, q_rank=768, kv_rank=512, rot_dim=64, window=1024,
+            keep_first=4, chunk=1024, conv=4, ff=5632, experts=32, top=4, expert_ff=768, shared_ff=1536, **kw) -> ModelConfig:
+    """Layer-list model with norms ahead of its sublayers: latent, windowed and chunked attention in turn, the first layer with a
+    dense feed-forward and the others with a mixture of experts."""
+    specs = []
+    for i in range(layers):
+        if i % 3 == 0:
+            s = LayerSpec(latent=LatentSpec(heads, dim, rot_dim, dim, q_rank, kv_rank, (dim + rot_dim) ** -0.5, window))
+        elif i % 3 == 1:
+            s = LayerSpec(AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window, dim, 5e5, qk_norm=False, keep_first=keep_first,
+                                        head_norm=True, rot_pairs=True, bias=True, v_mix=True))
+        else:
+            s = LayerSpec(AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, qk_norm=False, chunk=chunk, softcap=30.0,
+                                        distance_bias=True, conv=conv, v_mix=True))
+        if i == 0:
+            s.ff, s.act, s.ff_bias = ff, "swiglu", True
+        else:
+            s.experts = ExpertsSpec(experts, top, expert_ff, shared_ff=shared_ff, act="swiglu", weighting="chosen")
+        specs.append(s)
+    c = ModelConfig(architecture="Tenotar", name="tenotar", layers=specs, vocab_size=vocab, hidden_size=width,
+                    num_hidden_layers=layers, use_mla=False, tie_word_embeddings=False, rms_norm_eps=1e-5, norm_first=True,
+                    logit_scale=0.5)
+    for k, v in kw.items():
+        setattr(c, k, v)
+    return c
+
+
+def tiny_tenotar(**kw) -> ModelConfig:
+    """CPU-sized layer-list model with norms ahead of its sublayers."""
+    kw.setdefault("dtype", "float32")
+    kw.setdefault("name", "tiny-tenotar")
+    return tenotar(width=64, layers=6, vocab=512, heads=4, kv_heads=2, dim=16, q_rank=24, kv_rank=40, rot_dim=8, window=40, keep_first=3,
+                   chunk=48, conv=3, ff=96, experts=6, top=2, expert_ff=24, shared_ff=40, **kw)
+
+
 def tiny_forovik(**kw) -> ModelConfig:
     """CPU-sized layer-list model."""
     kw.setdefault("dtype", "float32")
@@ -535,6 +684,8 @@ def tiny_forovik(**kw) -> ModelConfig:
 PRESETS = {
     "forovik": forovik,
     "tiny-forovik": tiny_forovik,
+    "tenotar": tenotar,
+    "tiny-tenotar": tiny_tenotar,
     "fimudra": fimudra,
     "tiny-fimudra": tiny_fimudra,
     "tiny-deepseek-v3": tiny_deepseek_v3,

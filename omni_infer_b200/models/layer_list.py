@@ -1,5 +1,5 @@
 """Models described layer by layer: ``ModelConfig.layers`` lists a mixer and an optional feed-forward per layer, each with sizes
-of its own.  Two ways to connect them:
+of its own.  Three ways to connect them:
 
 One residual, norms on the outputs (``cfg.streams == 0``; windowed attention, Mamba-2, gated dense feed-forward): sublayers read
 the residual stream itself, ``x <- x + norm1(mixer(x))``, ``x <- x + norm2(ff(x))``.  Every addition, its norm and the activation
@@ -10,10 +10,14 @@ learned sum of the streams, and every stream becomes a learned sum of all of the
 norm for the next sublayer are one kernel.  A layer may run with another layer's weights (``weights_of``) on a cache or state
 of its own.
 
-The residual is fp32 either way, and the embedding table is also the LM head.
+One residual, norms ahead (``cfg.norm_first``; latent, windowed and chunked attention, dense feed-forwards and mixtures of
+experts): ``x <- x + mixer(norm1(x))``, ``x <- x + ff(norm2(x))``.  Addition, output bias and the norm for the next sublayer are
+one kernel.  The head is a matrix of its own; its factor enters with the last norm.
+
+The residual is fp32 in all of them, and the embedding table is also the LM head in the first two.
 
 A layer's entry in ``kv_caches`` is what its mixer reads: the (k, v) page pools of an attention layer - the same tensors for a
-layer that attends to another layer's keys - or the slot tensors of a recurrent one, or both."""
+layer that attends to another layer's keys, one pool for latent attention - or the slot tensors of a recurrent one, or both."""
 from __future__ import annotations
 
 import torch
@@ -21,18 +25,21 @@ from torch import nn
 
 from .. import ops
 from ..layers.common import GeGLUMLP, PaddedLinear, PostNorm, _dtype
+from ..layers.latent_attention import LatentAttention
 from ..layers.mamba2 import Mamba2Mixer
 from ..layers.matrix_state import ParallelMixer, WkvMixer
 from ..layers.moe import ExpertMixture
 from ..layers.vocab_parallel import lm_logits
 from ..layers.windowed_attention import WindowedAttention
-from ..ops.layer_list import embed_residual, pad8, rmsnorm_residual
+from ..ops.layer_list import add_norm, embed_norm, embed_residual, pad8, rmsnorm_residual
 from ..ops.streams import embed_streams, stream_step
 from .config import ModelConfig
 
 
 def _mixer(s, width, eps, **kw):
     cos_sin = kw.pop("cos_sin")
+    if s.latent is not None:
+        return LatentAttention(s.latent, width, eps, cos_sin=cos_sin, **kw)
     if s.attention is not None:
         return WindowedAttention(s.attention, width, eps, cos_sin=cos_sin, **kw)
     if s.parallel is not None:
@@ -105,6 +112,30 @@ class StreamLayer(nn.Module):
         return out
 
 
+class NormFirstLayer(nn.Module):
+    """One residual, norms ahead.  The model runs the sublayers; this holds their weights."""
+
+    def __init__(self, cfg: ModelConfig, i: int, *, dtype, device=None, cos_sin=None):
+        super().__init__()
+        s, width = cfg.layers[i], cfg.hidden_size
+        norm = lambda: nn.Parameter(torch.ones(width, dtype=torch.float32, device=device), requires_grad=False)      # noqa: E731
+        self.mixer, self.norm1 = _mixer(s, width, cfg.rms_norm_eps, dtype=dtype, device=device, cos_sin=cos_sin), norm()
+        self.mlp, self.norm2 = None, None
+        if s.experts is not None:
+            self.mlp, self.norm2 = ExpertMixture(s.experts, width, dtype=dtype, device=device), norm()
+        elif s.ff:
+            self.mlp, self.norm2 = GeGLUMLP(width, s.ff, dtype=dtype, device=device, epi=s.act, bias=s.ff_bias), norm()
+
+    def checkpoint_targets(self):
+        H = self.norm1.shape[0]
+        out = {"norm1": (self.norm1, 0, H, None)}
+        out.update({"mix." + k: v for k, v in self.mixer.checkpoint_targets().items()})
+        if self.mlp is not None:
+            out["norm2"] = (self.norm2, 0, H, None)
+            out.update({"mlp." + k: v for k, v in self.mlp.checkpoint_targets().items()})
+        return out
+
+
 class LayerListModel(nn.Module):
     def __init__(self, cfg: ModelConfig, *, device=None):
         super().__init__()
@@ -123,7 +154,7 @@ class LayerListModel(nn.Module):
 
         self.embed_tokens = nn.Embedding(cfg.vocab_size, pad8(cfg.hidden_size), dtype=self.dtype, device=device)
         self.embed_tokens.weight.requires_grad_(False)
-        kind = StreamLayer if cfg.streams else LayerListLayer
+        kind = StreamLayer if cfg.streams else (NormFirstLayer if cfg.norm_first else LayerListLayer)
         built: list = []
         for i, s in enumerate(cfg.layers):      # a layer with another's weights is that layer's module
             built.append(None if s.weights_of is not None else
@@ -137,6 +168,8 @@ class LayerListModel(nn.Module):
         assert inputs_embeds is None
         if self.cfg.streams:
             return self._forward_streams(input_ids, md, kv_caches)
+        if self.cfg.norm_first:
+            return self._forward_norm_first(input_ids, md, kv_caches)
         x, xa = embed_residual(input_ids, self.embed_tokens.weight)
         for layer, cache in zip(self.layers, kv_caches):
             xa = layer(x, xa, md, cache)
@@ -159,6 +192,25 @@ class LayerListModel(nn.Module):
         return h
 
 
+    def _forward_norm_first(self, input_ids, md, kv_caches):
+        eps, width, shared, subs = self.cfg.rms_norm_eps, pad8(self.cfg.hidden_size), {}, []
+        for layer, cache in zip(self.layers, kv_caches):
+            subs.append((layer.norm1, layer.mixer, lambda h, m=layer.mixer, c=cache: m(h, md, c, shared)))
+            if isinstance(layer.mlp, ExpertMixture):
+                subs.append((layer.norm2, layer.mlp, lambda h, m=layer.mlp: m(h, md.num_valid)))
+            elif layer.mlp is not None:
+                subs.append((layer.norm2, layer.mlp, layer.mlp))
+        norm, sub, _ = subs[0]
+        x, h = embed_norm(input_ids, self.embed_tokens.weight, norm, eps, ld=sub.in_cols, ones=sub.ones)
+        for k, (_, sub, run) in enumerate(subs):
+            if k + 1 < len(subs):
+                norm, nxt, _ = subs[k + 1]
+                h = add_norm(x, run(h), norm, eps, self.dtype, ld=nxt.in_cols, ones=nxt.ones, bias=sub.out_bias)
+            else:
+                h = add_norm(x, run(h), self.norm, eps, self.dtype, ld=width, bias=sub.out_bias, scale=self.cfg.logit_scale)
+        return h
+
+
 class LayerListForCausalLM(nn.Module):
     is_mla = False
 
@@ -170,6 +222,10 @@ class LayerListForCausalLM(nn.Module):
             raise ValueError(f"{cfg.architecture} runs in bfloat16 or float32, not quantised")
         self.cfg = cfg
         self.model = LayerListModel(cfg, device=device)
+        self.lm_head = None
+        if not cfg.tie_word_embeddings:
+            self.lm_head = nn.Parameter(torch.zeros(cfg.vocab_size, pad8(cfg.hidden_size), dtype=self.model.dtype, device=device),
+                                        requires_grad=False)
 
     @property
     def num_kv_layers(self):
@@ -184,15 +240,15 @@ class LayerListForCausalLM(nn.Module):
             if a is not None and not a.owns_kv:
                 pages = caches[a.kv_from]
             elif a is not None:
-                pages = (zeros(num_blocks, block_size, a.kv_heads, a.dim, dtype=self.model.dtype),
-                         zeros(num_blocks, block_size, a.kv_heads, a.vdim, dtype=self.model.dtype))
+                pages = tuple(zeros(*shape, dtype=self.model.dtype) for shape in a.page_shapes(num_blocks, block_size))
+                pages = pages if len(pages) > 1 else pages[0]
             if s.recurrent:
                 state = tuple(zeros(*shape, dtype=dt) for shape, dt in layer.mixer.state_shapes(state_slots, self.model.dtype))
             caches.append(pages if state is None else (state if pages is None else (pages, state)))
         return caches
 
     def paged_caches(self, caches: list) -> list:
-        """The (k, v) pools among ``caches`` that belong to a layer of their own."""
+        """The pools among ``caches`` - (k, v), or one - that belong to a layer of their own."""
         return [c[0] if s.recurrent else c for c, s in zip(caches, self.cfg.layers) if s.paged is not None and s.paged.owns_kv]
 
     def kv_bytes_per_token(self) -> int:
@@ -212,11 +268,13 @@ class LayerListForCausalLM(nn.Module):
         return self.model(input_ids, md, kv_caches, inputs_embeds)
 
     def compute_logits(self, hidden):
-        return lm_logits(hidden, self.model.embed_tokens.weight)
+        return lm_logits(hidden, self.model.embed_tokens.weight if self.lm_head is None else self.lm_head)
 
     def process_weights_after_loading(self):
         """Padding rows and columns hold zeros whatever the loader or the random initialisation put there."""
         self.model.embed_tokens.weight.data[:, self.cfg.hidden_size:] = 0
+        if self.lm_head is not None:
+            self.lm_head.data[:, self.cfg.hidden_size:] = 0
         mods = [m for m in self.modules() if hasattr(m, "zero_padding")]
         for m in sorted(mods, key=lambda m: not isinstance(m, PaddedLinear)):      # single layers first, then what is made of them
             m.zero_padding()
@@ -229,6 +287,8 @@ class LayerListForCausalLM(nn.Module):
         """{checkpoint tensor: (parameter, first row, rows, columns)} for the weight loader."""
         H = self.cfg.hidden_size
         out = {"embed": (self.model.embed_tokens.weight, 0, self.cfg.vocab_size, H), "final.norm": (self.model.norm, 0, H, None)}
+        if self.lm_head is not None:
+            out["head"] = (self.lm_head, 0, self.cfg.vocab_size, H)
         for i, layer in enumerate(self.model.layers):
             if self.cfg.layers[i].weights_of is None:
                 out.update({f"l{i}." + k: v for k, v in layer.checkpoint_targets().items()})

@@ -29,6 +29,7 @@ def _lazy():
         "Qwen3MoeForCausalLM": Qwen3MoeForCausalLM,
         "Forovik": LayerListForCausalLM,
         "Fimudra": LayerListForCausalLM,
+        "Tenotar": LayerListForCausalLM,
     }
     if any(os.environ.get(k) == "1" for k in ("RANDOM_MODE", "CAPTURE_MODE", "REPLAY_MODE")):
         from .mock import mock_model_class_factory

@@ -41,10 +41,13 @@ def _mla_scratch(dev, n_o, n_l):
     return buf
 
 
-def mla_decode(q, cache, block_table, seq_lens, scale, q_to_seq=None, num_splits=0, max_seq_len=None, kv_lora=512):
+def mla_decode(q, cache, block_table, seq_lens, scale, q_to_seq=None, num_splits=0, max_seq_len=None, kv_lora=512, exact=False,
+               window=0, gate=None):
     """Absorbed MLA decode attention.  ``seq_lens[b]`` is the number of cache tokens q row b attends to
-    (MTP rows of one request get consecutive lengths); ``q_to_seq`` maps q rows to block-table rows."""
+    (MTP rows of one request get consecutive lengths); ``q_to_seq`` maps q rows to block-table rows.  ``exact`` (GPU only): softmax
+    weights to 16 bits of mantissa, optionally a sliding ``window`` and a factor sigmoid(``gate`` [Bq, H]) on the heads."""
     if not q.is_cuda:
+        assert not exact
         return mla_decode_ref(q, cache, block_table, seq_lens, scale, q_to_seq, kv_lora)
     Bq, H, D = q.shape
     assert D == 576 and kv_lora == 512, "the sm_100a kernel is specialised for kv_lora 512 + rope 64"
@@ -56,16 +59,18 @@ def mla_decode(q, cache, block_table, seq_lens, scale, q_to_seq=None, num_splits
         num_splits = 1
         if max_seq_len is not None and Bq * 2 < 148:
             want = max(1, 296 // (Bq * 2))
-            tiles = (max_seq_len + 31) // 32
+            tiles = (min(max_seq_len, window + 32 if window else max_seq_len) + 31) // 32
             num_splits = max(1, min(want, tiles // 4 if tiles >= 4 else 1, 32))
     out = torch.empty(Bq, H, 512, dtype=q.dtype, device=q.device)
     o_part = lse = None
     if num_splits > 1:
         o_part, lse = _mla_scratch(q.device, Bq * num_splits * H * 512, Bq * num_splits * H)
-    rc = nat.lib().omni_mla_decode(
+    assert exact or (window == 0 and gate is None)
+    extra = (nat.c_int(window), nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0)) if exact else ()
+    rc = (nat.lib().omni_mla_decode_window if exact else nat.lib().omni_mla_decode)(
         nat.ptr(q), nat.ptr(cache2), nat.c_int(cache2.stride(0)), nat.ctypes.c_longlong(cache2.shape[0]),
         nat.ptr(block_table), nat.c_int(block_table.stride(0)), nat.ptr(seq_lens), nat.ptr(q_to_seq), nat.c_int(Bq),
-        nat.c_int(H), nat.c_int(bs), nat.c_float(scale), nat.c_int(num_splits), nat.ptr(out), nat.ptr(o_part),
+        nat.c_int(H), nat.c_int(bs), nat.c_float(scale), *extra, nat.c_int(num_splits), nat.ptr(out), nat.ptr(o_part),
         nat.ptr(lse), nat.ptr(nat.status_buffer(q.device)), nat.stream())
     nat.check_rc(rc, "omni_mla_decode")
     return out

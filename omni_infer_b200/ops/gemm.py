@@ -136,7 +136,7 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
     epi: "store" | "swiglu" (w holds gate rows then up rows) | "geglu" (the same with the tanh form of gelu) |
     "clamped_glu" (gate bounded above and up on both sides by ``glu_limit``: g sigmoid(1.702 g) (u + 1)) |
     "swiglu_quant" (returns (q, scale_t)).
-    fp32 operands run a plain fp32 kernel ("store", "geglu" and "clamped_glu").
+    fp32 operands run a plain fp32 kernel (all but "swiglu_quant").
     """
     if out_dtype is None:
         out_dtype = torch.bfloat16 if (x.dtype == FP8 or x.is_cuda) else x.dtype
@@ -205,7 +205,7 @@ def gemm(x, w, *, w_scale=None, x_scale=None, seg_start=None, seg_len=None, epi=
 
 
 def _gemm_f32(x, w, epi, seg_start, seg_len, row_scale, out, glu_limit):
-    assert w.dtype == torch.float32 and epi in ("store", "geglu", "clamped_glu") and w.is_contiguous()
+    assert w.dtype == torch.float32 and epi in ("store", "swiglu", "geglu", "clamped_glu") and w.is_contiguous()
     assert x.shape[1] == w.shape[-1] and x.stride(1) == 1 and (w.dim() == 2 or seg_len is not None)
     T, n = x.shape[0], w.shape[-2]
     y = out if out is not None and epi == "store" else torch.empty(T, n, dtype=torch.float32, device=x.device)

@@ -1,7 +1,8 @@
-"""Ops of the layer-list models: the fp32 residual stream with norms on the sublayers' outputs, windowed attention over the
-paged cache with a q/k norm over the whole projection, and the Mamba-2 layer between its projections.
+"""Ops of the layer-list models: the fp32 residual stream with norms on the sublayers' outputs or ahead of the sublayers, attention
+over the paged cache (windows, kept first tokens, chunks, capped and biased scores) with a q/k norm over the whole projection, the
+short convolution, and the Mamba-2 layer between its projections.
 
-CUDA tensors run ``csrc/kernels/post_norm_ops.cu``, ``attn_any.cu``, ``fmha_sm100.cu``, ``gqa_decode.cu`` and
+CUDA tensors run ``csrc/kernels/post_norm_ops.cu``, ``attn_any.cu``, ``fmha_sm100.cu``, ``gqa_decode.cu``, ``short_conv.cu`` and
 ``mamba2.cu`` / ``ssd_sm100.cu``; CPU tensors run the fp32 references here.  Activations are bf16 or fp32.  Rows may be wider than their
 content (a multiple of 8 columns, so that they can be TMA operands); the columns past it are zero.
 
@@ -82,6 +83,56 @@ def rmsnorm_residual(x, w, eps, dtype):
     return out
 
 
+def _normed_rows(x, w, eps, scale, ld, ones, dtype):
+    H = w.shape[0]
+    h = torch.zeros(x.shape[0], ld, dtype=dtype)
+    h[:, :H] = (rms_ref(x[:, :H], w, eps) * scale).to(dtype)
+    if ones:
+        h[:, H] = 1
+    return h
+
+
+def _residual_call(x, w, eps, scale, ld, ones, dtype, ids=None, table=None, y=None, bias=None):
+    """``y``: rows, or the parts of an expert mixture (``streams.ExpertSum`` without identity experts)."""
+    parts = y is not None and not torch.is_tensor(y)
+    rows = y.y if parts else y
+    if parts:
+        assert y.shared is None or y.shared.stride(0) == rows.stride(0)
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.is_contiguous() and (rows is None or (rows.dtype == dtype and rows.stride(1) == 1))
+    T, H = x.shape[0], w.shape[0]
+    h = torch.empty(T, ld, dtype=dtype, device=x.device)
+    rc = nat.lib().omni_residual_norm(
+        nat.ptr(x), nat.c_int(T), nat.c_int(H), nat.c_int(x.shape[1]), nat.ptr(ids), nat.ptr(table),
+        nat.c_int(table.shape[0] if table is not None else 0), nat.c_int(table.stride(0) if table is not None else 0), nat.ptr(rows),
+        nat.c_int(rows.stride(0) if rows is not None else 0), nat.ptr(y.row_of if parts else None),
+        nat.c_int(y.ids.shape[1] if parts else 0), nat.ptr(y.shared if parts else None), nat.ptr(bias), nat.ptr(w), nat.c_float(eps),
+        nat.c_float(scale), nat.ptr(h), nat.c_int(ld), nat.c_int(int(ones)), nat.c_int(int(dtype == torch.float32)), nat.stream())
+    nat.check_rc(rc, "omni_residual_norm")
+    return h
+
+
+def embed_norm(ids, table, w, eps, *, ld, ones=False):
+    """Embedding rows -> (fp32 residual, rmsnorm of it times ``w`` as activations [T, ld]).  Columns past the width are zeros, but
+    for the first of them with ``ones`` (it meets the column of the next weight that holds the biases)."""
+    T, H = ids.shape[0], w.shape[0]
+    x = torch.empty(T, pad8(H), dtype=torch.float32, device=table.device)
+    if not table.is_cuda:
+        x[:, :H] = table[ids][:, :H].float()
+        return x, _normed_rows(x, w, eps, 1.0, ld, ones, table.dtype)
+    return x, _residual_call(x, w, eps, 1.0, ld, ones, table.dtype, ids=ids, table=table)
+
+
+def add_norm(x, y, w, eps, dtype, *, ld, ones=False, bias=None, scale=1.0):
+    """x (fp32, in place) += y + bias, then as :func:`embed_norm`; ``scale`` multiplies the normed rows."""
+    if not x.is_cuda:
+        H = w.shape[0]
+        x[:, :H] += (y.float() if torch.is_tensor(y) else y.total())[:, :H]
+        if bias is not None:
+            x[:, :H] += bias
+        return _normed_rows(x, w, eps, scale, ld, ones, dtype)
+    return _residual_call(x, w, eps, scale, ld, ones, dtype, y=y, bias=bias)
+
+
 # ----------------------------------------------------------------------------- q/k norm, rotation, cache write
 def _rotate_half_ref(x, cos_sin, positions, rot):
     """x [T, heads, D] fp32; rotates the first ``rot`` entries of every head."""
@@ -118,36 +169,61 @@ def qk_norm_rope_cache(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, positi
 
 
 # ----------------------------------------------------------------------------- windowed attention over the paged cache
-def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out):
+def first_visible(pos: int, window: int, chunk: int) -> int:
+    """First key that a query at ``pos`` sees through its window and in its chunk (0: none)."""
+    return max(0, pos - window + 1 if window else 0, pos // chunk * chunk if chunk else 0)
+
+
+def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out, keep_first=0,
+                        chunk=0, softcap=0.0, slopes=None, gate=None):
     hq, dk = q.shape[1], q.shape[2]
     bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
-    kf, vf = k_cache.view(-1, hkv, dk), v_cache.view(-1, hkv, dv)
+    kf, vf = k_cache.flatten(0, 1), v_cache.flatten(0, 1)
     rep = hq // hkv
     out[:, :hq * dv] = 0
     for t in range(q.shape[0]):
         if int(slots[t]) < 0:
             continue
         p = int(positions[t])
-        pos = torch.arange(max(0, p - window + 1) if window else 0, p + 1)
+        lo = first_visible(p, window, chunk)
+        pos = torch.cat([torch.arange(min(keep_first, lo)), torch.arange(lo, p + 1)])
         rows = block_table[int(q_to_seq[t]), pos // bs].long() * bs + pos % bs
         k = kf[rows].float().repeat_interleave(rep, 1)
         v = vf[rows].float().repeat_interleave(rep, 1)
         s = torch.einsum("hd,lhd->hl", q[t].float(), k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        if slopes is not None:
+            s = s - slopes[:, None] * (p - pos)
         if sink is not None:
             s = torch.cat([s, sink[:, None]], 1)
         o = torch.einsum("hl,lhd->hd", torch.softmax(s, -1)[:, :len(pos)], v) * out_scale
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t].float())[:, None]
         out[t, :hq * dv] = o.reshape(-1).to(out.dtype)
     return out
 
 
+def _splits(ctas: int, keys: int) -> int:
+    """Parts of the key range of a decode launch with that many blocks: three of them fit an SM, and a part should have several
+    tiles of 32 keys per warp."""
+    tiles = (keys + 31) // 32 + 1
+    return max(1, min((444 + ctas - 1) // ctas, tiles // 8, 32)) if ctas < 444 else 1
+
+
 def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_table, seq_lens, scale, window=0, cu_q=None,
-                    max_q=1, max_seq_len=0, sink=None, out_scale=1.0, out=None, any_shape=False):
+                    max_q=1, max_seq_len=0, sink=None, out_scale=1.0, out=None, any_shape=False, keep_first=0, chunk=0, softcap=0.0,
+                    slopes=None, gate=None, rows_share=False):
     """q [T, hq, dk] (rows of any pitch) against the cached keys of the rows' requests, each row seeing the ``window``
-    positions up to its own (0: all of them).  ``sink`` [hq] fp32: exp(sink) is one more term of the head's softmax
-    denominator; ``out_scale`` multiplies the result.  Returns [T, pad8(hq * dv)], or writes the first columns of ``out``.
+    positions up to its own (0: all of them), only those of its own ``chunk`` of positions (0: no chunks), and the ``keep_first``
+    first ones in any case.  A score is ``softcap tanh(q k scale / softcap) - slopes[head] distance`` (each part optional).  ``sink``
+    [hq] fp32: exp(sink) is one more term of the head's softmax denominator; ``out_scale`` multiplies the result, and so does the
+    sigmoid of ``gate`` [T, hq].  Returns [T, pad8(hq * dv)], or writes the first columns of ``out``.  The value cache may be a
+    column slice of the key cache (one key/value head).
 
     bf16 portions of prompts run on tcgen05 (``omni_fmha_paged``), bf16 single tokens on the split-KV decode kernel; fp32
-    and head shapes those two do not take - or ``any_shape`` - go to ``omni_attn_any``."""
+    and head shapes those two do not take - or ``any_shape`` - go to ``omni_attn_any``.  ``cu_q=None``: every row stands alone;
+    with ``rows_share`` they belong to the requests ``q_to_seq`` (else row i to request i) and see ``seq_lens`` keys each."""
     T, hq, dk = q.shape
     bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     if out is None:
@@ -155,40 +231,44 @@ def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_ta
         out = (torch.empty if ld == hq * dv else torch.zeros)(T, ld, dtype=q.dtype, device=q.device)
     ld = out.stride(0)
     if not q.is_cuda:
-        return paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out)
+        return paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out,
+                                   keep_first, chunk, softcap, slopes, gate)
     assert q.stride(2) == 1 and q.stride(1) == dk and k_cache.dtype == q.dtype and block_table.stride(1) == 1
+    k_row, v_row = k_cache.stride(1), v_cache.stride(1)
+    assert k_cache.stride(0) == bs * k_row and v_cache.stride(0) == bs * v_row and (gate is None or gate.stride(1) == 1)
+    packed = k_row == hkv * dk and v_row == hkv * dv
     f32 = _f32(q)
     lib = nat.lib()
+    gate_args = (nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0))
+    mod = (nat.c_int(window), nat.c_int(chunk), nat.c_int(keep_first), nat.c_float(scale), nat.c_float(softcap), nat.ptr(slopes), nat.ptr(sink))
     tc = not any_shape and not f32 and ld % 8 == 0 and out.data_ptr() % 16 == 0 and dk % 8 == 0 and dv % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
-    if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0:
+    if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0 and packed and gate is None:
         rc = lib.omni_fmha_paged(
             nat.ptr(q), nat.c_int64(T), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache),
             nat.c_int64(k_cache.shape[0] * bs), nat.ptr(cu_q), nat.ptr(seq_lens), nat.ptr(block_table),
             nat.c_int(block_table.stride(0)), nat.c_int(cu_q.shape[0] - 1), nat.c_int(max_q), nat.c_int(hq), nat.c_int(hkv),
-            nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(sink), nat.c_float(out_scale),
-            nat.ptr(out), nat.c_int(ld), nat.ptr(nat.status_buffer(q.device)), nat.stream())
+            nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), *mod, nat.c_float(out_scale), nat.ptr(out), nat.c_int(ld),
+            nat.ptr(nat.status_buffer(q.device)), nat.stream())
         nat.check_rc(rc, "omni_fmha_paged")
         return out
-    if tc and cu_q is None and dk <= 256 and dv <= 256:
-        ctas = T * hkv * ((hq // hkv + 15) // 16)
-        span = min(max_seq_len, window) if window else max_seq_len
-        tiles = (span + 31) // 32 + 1
-        splits = max(1, min((444 + ctas - 1) // ctas, tiles // 8, 32)) if ctas < 444 else 1
+    if tc and cu_q is None and dk <= 256 and dv <= 256 and k_row % 8 == 0 and v_row % 8 == 0:
+        span = min(max_seq_len, window + keep_first if window else max_seq_len, chunk + keep_first if chunk else max_seq_len)
+        splits = _splits(T * hkv * ((hq // hkv + 15) // 16), span)
         o_part = lse = None
         if splits > 1:
             o_part = torch.empty(T * splits * hq * dv, dtype=torch.float32, device=q.device)
             lse = torch.empty(T * splits * hq, dtype=torch.float32, device=q.device)
         rc = lib.omni_gqa_paged_decode_window(
-            nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.ptr(block_table),
-            nat.c_int(block_table.stride(0)), nat.ptr(seq_lens), nat.c_int(T), nat.c_int(hq), nat.c_int(hkv), nat.c_int(dk),
-            nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(sink), nat.c_float(out_scale),
-            nat.c_int(splits), nat.ptr(o_part), nat.ptr(lse), nat.ptr(out), nat.c_int(ld), nat.stream())
+            nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.c_int64(k_row), nat.c_int64(v_row),
+            nat.ptr(q_to_seq if rows_share else None), nat.ptr(block_table), nat.c_int(block_table.stride(0)), nat.ptr(seq_lens),
+            nat.c_int(T), nat.c_int(hq), nat.c_int(hkv), nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), *mod, *gate_args,
+            nat.c_float(out_scale), nat.c_int(splits), nat.ptr(o_part), nat.ptr(lse), nat.ptr(out), nat.c_int(ld), nat.stream())
         nat.check_rc(rc, "omni_gqa_paged_decode_window")
         return out
     rc = lib.omni_attn_any(
-        nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.ptr(positions), nat.ptr(q_to_seq),
-        nat.ptr(slots), nat.ptr(block_table), nat.c_int(block_table.stride(0)), nat.c_int(T), nat.c_int(hq), nat.c_int(hkv),
-        nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), nat.c_int(window), nat.c_float(scale), nat.ptr(sink), nat.c_float(out_scale),
+        nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache), nat.c_int64(k_row), nat.c_int64(v_row),
+        nat.ptr(positions), nat.ptr(q_to_seq), nat.ptr(slots), nat.ptr(block_table), nat.c_int(block_table.stride(0)), nat.c_int(T),
+        nat.c_int(hq), nat.c_int(hkv), nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), *mod, *gate_args, nat.c_float(out_scale),
         nat.ptr(out), nat.c_int(ld), nat.c_int(f32), nat.stream())
     nat.check_rc(rc, "omni_attn_any")
     return out
@@ -200,18 +280,18 @@ def gated_mul(x, inter, up_off, kind="geglu", limit=0.0):
     T, ld = x.shape[0], pad8(inter)
     if not x.is_cuda:
         g, u = x[:, :inter].float(), x[:, up_off:up_off + inter].float()
-        y = F.gelu(g, approximate="tanh") * u if kind == "geglu" else clamped_glu_ref(g, u, limit)
+        y = clamped_glu_ref(g, u, limit) if kind == "clamped_glu" else (F.silu(g) if kind == "swiglu" else F.gelu(g, approximate="tanh")) * u
         return F.pad(y, (0, ld - inter)).to(x.dtype)
     out = torch.empty(T, ld, dtype=x.dtype, device=x.device)
     rc = nat.lib().omni_gated_mul(nat.ptr(x), nat.c_int(x.stride(0)), nat.c_int(up_off), nat.ptr(out), nat.c_int(ld),
-                                  nat.c_int(T), nat.c_int(inter), nat.c_int({"geglu": 0, "clamped_glu": 1}[kind]),
+                                  nat.c_int(T), nat.c_int(inter), nat.c_int({"geglu": 0, "clamped_glu": 1, "swiglu": 2}[kind]),
                                   nat.c_float(limit), nat.c_int(_f32(x)), nat.stream())
     nat.check_rc(rc, "omni_gated_mul")
     return out
 
 
-# ----------------------------------------------------------------------------- Mamba-2
-def conv_silu_ref(u, w, bias, state, positions, state_slots, cu_q, out):
+# ----------------------------------------------------------------------------- short convolution
+def short_conv_ref(u, w, bias, state, positions, state_slots, cu_q, out, silu):
     taps, C = w.shape
     for r, a, b in _segments(cu_q, u.shape[0]):
         slot = int(state_slots[r])
@@ -224,30 +304,38 @@ def conv_silu_ref(u, w, bias, state, positions, state_slots, cu_q, out):
             old = old.clone()
             old[: taps - 1 - pos0] = 0
         full = torch.cat([old, u[a:b, :C].float()])
-        y = sum(full[k:k + b - a] * w[k] for k in range(taps)) + bias
-        out[a:b, :C] = F.silu(y).to(out.dtype)
+        y = sum(full[k:k + b - a] * w[k] for k in range(taps))
+        if bias is not None:
+            y = y + bias
+        out[a:b, :C] = (F.silu(y) if silu else y).to(out.dtype)
         if taps > 1:
             state[slot] = full[b - a:].to(state.dtype)
     return out
 
 
-def conv_silu(u, w, bias, state, *, positions, state_slots, q_to_seq=None, cu_q=None):
-    """Causal convolution per channel (``w`` [taps, C], last tap = current token), bias, silu.  u [T, C] (rows of any
-    pitch); ``state`` [slots, taps - 1, C] holds the last inputs of every request and is moved on.  -> [T, pad8(C)]."""
+def short_conv(u, w, bias, state, *, positions, state_slots, q_to_seq=None, cu_q=None, silu=False):
+    """Causal convolution per channel (``w`` [taps, C], last tap = current token), bias (or None), optionally silu.  u [T, C] (rows
+    of any pitch); ``state`` [slots, taps - 1, C] holds the last inputs of every request and is moved on.  -> [T, pad8(C)]."""
     T, (taps, C) = u.shape[0], w.shape
     out = torch.empty(T, pad8(C), dtype=u.dtype, device=u.device)
     if not u.is_cuda:
-        return conv_silu_ref(u, w, bias, state, positions, state_slots, cu_q, out)
+        return short_conv_ref(u, w, bias, state, positions, state_slots, cu_q, out, silu)
     assert u.stride(1) == 1 and state.dtype == u.dtype and w.is_contiguous()
     B = T if cu_q is None else cu_q.shape[0] - 1
-    rc = nat.lib().omni_conv_silu(
+    rc = nat.lib().omni_short_conv(
         nat.ptr(u), nat.c_int(u.stride(0)), nat.c_int(C), nat.c_int(taps), nat.ptr(w), nat.ptr(bias), nat.ptr(state),
         nat.ptr(positions), nat.ptr(q_to_seq), nat.ptr(cu_q), nat.ptr(state_slots), nat.c_int(B), nat.c_int(T), nat.ptr(out),
-        nat.c_int(out.shape[1]), nat.c_int(_f32(u)), nat.stream())
-    nat.check_rc(rc, "omni_conv_silu")
+        nat.c_int(out.shape[1]), nat.c_int(int(silu)), nat.c_int(_f32(u)), nat.stream())
+    nat.check_rc(rc, "omni_short_conv")
     return out
 
 
+def conv_silu(u, w, bias, state, **where):
+    """:func:`short_conv` with a silu on its output, as Mamba-2 has it."""
+    return short_conv(u, w, bias, state, silu=True, **where)
+
+
+# ----------------------------------------------------------------------------- Mamba-2
 def ssm_scan_ref(xbc, dt, A_log, dt_bias, D, state, positions, state_slots, cu_q, H, P, N, G, out):
     inner = H * P
     of = torch.arange(H) // (H // G)

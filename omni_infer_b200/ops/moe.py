@@ -15,13 +15,13 @@ from .gemm import FP8, quant_fp8_block_ref
 
 
 def router_topk_ref(logits, top_k, *, mode="softmax", bias=None, n_group=1, topk_group=1, group_mode="max",
-                    renorm=False, scale=1.0, selector=None, forced_balance=False):
+                    renorm=False, scale=1.0, selector=None, forced_balance=False, logit_bias=None):
     T, E = logits.shape
     if forced_balance:
         ids = (torch.arange(T * top_k, device=logits.device).view(T, top_k)) % E
         w = torch.full((T, top_k), scale / top_k, dtype=torch.float32, device=logits.device)
     else:
-        lf = logits.float()
+        lf = logits.float() if logit_bias is None else logits.float() + logit_bias
         scores = torch.softmax(lf, dim=-1) if mode == "softmax" else torch.sigmoid(lf)
         sel = scores + bias.float() if bias is not None else scores.clone()
         if n_group > 1:
@@ -41,16 +41,17 @@ def router_topk_ref(logits, top_k, *, mode="softmax", bias=None, n_group=1, topk
 
 
 def router_topk(logits, top_k, *, mode="softmax", bias=None, n_group=1, topk_group=1, group_mode="max",
-                renorm=False, scale=1.0, selector=None, counts=None, forced_balance=False, num_valid=None):
+                renorm=False, scale=1.0, selector=None, counts=None, forced_balance=False, num_valid=None, logit_bias=None):
     """logits fp32 [T, E] -> (physical expert ids int32 [T,k], weights fp32 [T,k]).
 
-    ``selector`` int32 [E] maps logical to physical expert ids (OmniPlacement); ``counts`` int64
+    ``bias`` [E] fp32 is added to the scores for the choice only, ``logit_bias`` to the logits.  With ``renorm`` softmax weights
+    are the softmax over the chosen logits.  ``selector`` int32 [E] maps logical to physical expert ids (OmniPlacement); ``counts`` int64
     [n_physical] receives the activation histogram; ``num_valid`` (device int32 scalar) marks rows at or
     beyond it as padding (ids = -1)."""
     if not logits.is_cuda:
         ids, w = router_topk_ref(logits, top_k, mode=mode, bias=bias, n_group=n_group, topk_group=topk_group,
                                  group_mode=group_mode, renorm=renorm, scale=scale, selector=selector,
-                                 forced_balance=forced_balance)
+                                 forced_balance=forced_balance, logit_bias=logit_bias)
         if counts is not None:
             counts += torch.bincount(ids.flatten().long(), minlength=counts.numel()).to(counts.dtype)
         return ids, w
@@ -59,7 +60,7 @@ def router_topk(logits, top_k, *, mode="softmax", bias=None, n_group=1, topk_gro
     ids = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
     rc = nat.lib().omni_router_topk(
-        nat.ptr(logits), nat.ptr(bias), nat.c_int(T), nat.c_int(E), nat.c_int(0 if mode == "softmax" else 1),
+        nat.ptr(logits), nat.ptr(bias), nat.ptr(logit_bias), nat.c_int(T), nat.c_int(E), nat.c_int(0 if mode == "softmax" else 1),
         nat.c_int(n_group), nat.c_int(topk_group), nat.c_int(1 if group_mode == "top2sum" else 0), nat.c_int(top_k),
         nat.c_int(1 if renorm else 0), nat.c_float(scale), nat.ptr(selector), nat.ptr(counts),
         nat.c_int(counts.numel() if counts is not None else 0), nat.c_int(1 if forced_balance else 0), nat.ptr(num_valid),

@@ -83,11 +83,21 @@ class WeightLoader:
         return moe.local_slots_of(expert)
 
     def _store_target(self, name: str, w):
-        """One tensor of a model with ``checkpoint_targets``; columns None: a vector, negative: stored transposed."""
+        """One tensor of a model with ``checkpoint_targets``; columns None: a vector (of one: also a scalar), negative: stored
+        transposed; a pair (store, shape): the layer puts it where it belongs itself."""
         if name not in self.targets:
             raise KeyError(f"checkpoint tensor {name!r} belongs to no parameter of this model")
+        if len(self.targets[name]) == 2:
+            store, want = self.targets[name]
+            if tuple(w.shape) != want:
+                raise ValueError(f"checkpoint tensor {name!r} has shape {tuple(w.shape)}, the configuration asks for {want}")
+            store(w)
+            self.loaded.add(name)
+            return
         p, r0, rows, cols = self.targets[name]
         want = (rows,) if cols is None else ((-cols, rows) if cols < 0 else (rows, cols))
+        if want == (1,) and w.dim() == 0:
+            w = w.view(1)
         if tuple(w.shape) != want:
             raise ValueError(f"checkpoint tensor {name!r} has shape {tuple(w.shape)}, the configuration asks for {want}")
         w = w.t() if cols is not None and cols < 0 else w
