@@ -22,9 +22,36 @@ __device__ __forceinline__ float ex2_fast(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// tanh(z) = 1 - 2 / (1 + e^2z): absolute error of some 1e-7, which the cap multiplies
+__device__ __forceinline__ float rcp_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// tanh(z) = 1 - 2 / (1 + e^2z): absolute error of some 1e-7, which the cap multiplies.  `add` comes on top.
+__device__ __forceinline__ float capped(const ScoreMod& m, float raw, float add) {
+  return fmaf(-2.f * m.cap_log2, rcp_fast(1.f + ex2_fast(raw * m.cap_in)), m.cap_log2 + add);
+}
 __device__ __forceinline__ float cap_score(const ScoreMod& m, float raw) {
-  return m.cap_log2 > 0.f ? m.cap_log2 - __fdividef(2.f * m.cap_log2, 1.f + ex2_fast(raw * m.cap_in)) : raw * m.scale_log2;
+  return m.cap_log2 > 0.f ? capped(m, raw, 0.f) : raw * m.scale_log2;
+}
+
+// two fp32 values in one register pair
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack_f32x2(float a, float b) {
+  f32x2 v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+  return v;
+}
+__device__ __forceinline__ void unpack_f32x2(f32x2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f32x2 fma_f32x2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 v;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(v) : "l"(a), "l"(b), "l"(c));
+  return v;
+}
+__device__ __forceinline__ f32x2 add_f32x2(f32x2 a, f32x2 b) {
+  f32x2 v;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
+  return v;
 }
 
 // First key that a query at `pos` sees through its window (of `window` keys) and in its chunk (of `chunk` positions); 0 = none.

@@ -1,6 +1,6 @@
 // Variable-length causal attention for prefill (tcgen05 + TMEM) and GQA paged decode.
 //
-// omni_fmha_varlen: one CTA per (128-query tile, request, q head).
+// omni_fmha_varlen: one CTA per (q head, request, 128-query tile).
 //   S = Q K^T     A = Q tile (smem, K-major, 64-dim chunks)   B = K tile of 64 keys (smem, K-major)
 //   P = softmax   kept in TMEM as packed bf16                  (thread = query row: no cross-thread reductions)
 //   O += P V      A = P (TMEM)                                 B = V tile (smem, MN-major), 128 output dims
@@ -92,11 +92,12 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
                    const __grid_constant__ CUtensorMap tmap_v, const FmhaParams p) {
   constexpr bool PAGED = MODE == FM_PAGED || MODE == FM_PAGED_MOD;      // keys through the block table
   constexpr bool EXACT = MODE != FM_DENSE;                              // any head sizes, masks, softmax weights as hi + lo
-  const int b = blockIdx.y, h = blockIdx.z;
+  // the last query tiles of the requests see the most keys: they come first, so that the short ones fill the gaps at the end
+  const int b = blockIdx.y, h = blockIdx.x;
   const int q_begin = p.cu_q[b], q_end = p.end_q[b];
   const int k_begin = PAGED ? 0 : p.cu_k[b];
   const int Lq = q_end - q_begin, Lk = PAGED ? p.kv_len[b] : p.end_k[b] - k_begin;
-  const int q0 = blockIdx.x * FM_BQ;
+  const int q0 = (gridDim.z - 1 - blockIdx.z) * FM_BQ;
   if (q0 >= Lq) return;  // uniform for the whole CTA, before any barrier / TMEM use
   const int ctx = Lk - Lq;
   const int hk = h / (p.Hq / p.Hkv);
@@ -249,22 +250,38 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       const int kept = p.keep - kbase;
       float dist_bias = 0.f;                       // of column 0
       if (MODE == FM_PAGED_MOD) dist_bias = slope * (float)(q_pos - kbase);
+      // raw scores (their scale is positive and enters with the subtraction of the maximum), or final ones in log2 units
       float s[FM_BK];
-      float mx = -INFINITY;
-#pragma unroll
-      for (int c0 = 0; c0 < FM_BK; c0 += 32) {
-        uint32_t sv32[32];
-        tmem_ld_x32(lane_addr + L::T_S + (i & 1) * FM_BK + c0, sv32);
+      {
+        uint32_t lo32[32], hi32[32];
+        tmem_ld_x32(lane_addr + L::T_S + (i & 1) * FM_BK, lo32);
+        tmem_ld_x32(lane_addr + L::T_S + (i & 1) * FM_BK + 32, hi32);
         tmem_ld_wait();
 #pragma unroll
-        for (int j = 0; j < 32; ++j) {
-          float v = __uint_as_float(sv32[j]);
-          if (MODE == FM_PAGED_MOD) v = cap_score(p.score, v) - (dist_bias - slope * (float)(c0 + j));
-          else v *= p.scale_log2;
-          s[c0 + j] = (c0 + j < lim && (!EXACT || c0 + j >= low || (PAGED && c0 + j < kept))) ? v : -INFINITY;
-          mx = fmaxf(mx, s[c0 + j]);
+        for (int j = 0; j < 32; ++j) { s[j] = __uint_as_float(lo32[j]); s[32 + j] = __uint_as_float(hi32[j]); }
+      }
+      if (MODE == FM_PAGED_MOD) {
+        if (p.score.cap_log2 > 0.f) {
+#pragma unroll
+          for (int j = 0; j < FM_BK; ++j) s[j] = capped(p.score, s[j], fmaf(slope, (float)j, -dist_bias));
+        } else {
+#pragma unroll
+          for (int j = 0; j < FM_BK; ++j) s[j] = fmaf(s[j], p.scale_log2, fmaf(slope, (float)j, -dist_bias));
         }
       }
+      if (!__all_sync(0xffffffffu, lim >= FM_BK && (!EXACT || low <= 0 || (PAGED && kept >= FM_BK)))) {
+#pragma unroll
+        for (int j = 0; j < FM_BK; ++j)
+          if (!(j < lim && (!EXACT || j >= low || (PAGED && j < kept)))) s[j] = -INFINITY;
+      }
+      float mx4[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+      for (int j = 4; j < FM_BK; j += 4) {
+        mx4[0] = fmaxf(mx4[0], s[j]); mx4[1] = fmaxf(mx4[1], s[j + 1]);
+        mx4[2] = fmaxf(mx4[2], s[j + 2]); mx4[3] = fmaxf(mx4[3], s[j + 3]);
+      }
+      const float unit = MODE == FM_PAGED_MOD ? 1.f : p.scale_log2;
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * unit;
       // A row that has seen no key yet (its window starts in a later tile, or it lies past the end of the request)
       // has nothing accumulated: it takes the maximum over as it is.
       const float m_new = fmaxf(m, mx);
@@ -273,7 +290,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       if (i > 0 && __any_sync(0xffffffffu, grow)) {
         if (!mbar_wait(o_done, (i - 1) & 1, abort_flag, p.status, 18, i)) { ok = false; break; }
         tc_fence_after();
-        const float f = grow ? exp2f(m - m_new) : 1.0f;
+        const float f = grow ? ex2_fast(m - m_new) : 1.0f;
         if (grow) { l *= f; m = m_new; }
 #pragma unroll 1
         for (int c = 0; c < nv * 64; c += 32) {
@@ -287,21 +304,31 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         tmem_st_wait();
       }
       uint32_t pk[32], pl[32];
-      float rs = 0.f;
       const float m_ref = m == -INFINITY ? 0.f : m;
+      const f32x2 unit2 = pack_f32x2(unit, unit), neg_m2 = pack_f32x2(-m_ref, -m_ref), minus2 = pack_f32x2(-1.f, -1.f);
+      f32x2 rs2[2] = {0ull, 0ull};
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
-        const float p0 = exp2f(s[2 * j] - m_ref), p1 = exp2f(s[2 * j + 1] - m_ref);
-        rs += p0 + p1;
+        float p0, p1;
+        unpack_f32x2(fma_f32x2(pack_f32x2(s[2 * j], s[2 * j + 1]), unit2, neg_m2), p0, p1);
+        p0 = ex2_fast(p0);
+        p1 = ex2_fast(p1);
+        const f32x2 pp = pack_f32x2(p0, p1);
+        rs2[j & 1] = add_f32x2(rs2[j & 1], pp);
         __nv_bfloat162 h2 = __floats2bfloat162_rn(p0, p1);
-        pk[j] = *reinterpret_cast<uint32_t*>(&h2);
+        const uint32_t hb = *reinterpret_cast<uint32_t*>(&h2);
+        pk[j] = hb;
         if (EXACT) {      // what the rounding to bf16 left over
-          const float2 hf = __bfloat1622float2(h2);
-          h2 = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
+          unpack_f32x2(fma_f32x2(pack_f32x2(__uint_as_float(hb << 16), __uint_as_float(hb & 0xffff0000u)), minus2, pp), p0, p1);
+          h2 = __floats2bfloat162_rn(p0, p1);
           pl[j] = *reinterpret_cast<uint32_t*>(&h2);
         }
       }
-      l += rs;
+      {
+        float a, b;
+        unpack_f32x2(add_f32x2(rs2[0], rs2[1]), a, b);
+        l += a + b;
+      }
       tmem_st_x32(lane_addr + L::T_P + (i & 1) * L::T_P_STRIDE, pk);
       if (EXACT) tmem_st_x32(lane_addr + L::T_P + FM_BK / 2 + (i & 1) * L::T_P_STRIDE, pl);
       tmem_st_wait();
@@ -392,7 +419,7 @@ extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q
   p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = FM_DV; p.out_ld = Hq * FM_DV;
   p.out_scale = 1.0f;
-  return launch_fmha<FM_DENSE, FM_MAXC, 3>(dim3((max_q + FM_BQ - 1) / FM_BQ, B, Hq), tq, tq, tk, tk2, tv, p, stream);
+  return launch_fmha<FM_DENSE, FM_MAXC, 3>(dim3(Hq, B, (max_q + FM_BQ - 1) / FM_BQ), tq, tq, tk, tk2, tv, p, stream);
 }
 
 // Ragged queries against the paged cache.  q: rows of pitch q_ld holding Hq heads of d_k; k_cache / v_cache
@@ -403,7 +430,7 @@ extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const 
                                float scale, float softcap, const float* slopes, const float* sink, float out_scale, void* out, int out_ld, void* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (d_k < 8 || d_v < 8 || d_k % 8 != 0 || d_v % 8 != 0 || d_k > 64 * FM_MAXC || d_v > FM_DV) return -1;
-  if (Hkv < 1 || Hq % Hkv != 0 || B > 65535 || Hq > 65535 || window < 0 || chunk < 0 || keep < 0) return -2;
+  if (Hkv < 1 || Hq % Hkv != 0 || B > 65535 || max_q > 65535 * FM_BQ || window < 0 || chunk < 0 || keep < 0) return -2;
   if (block_size < FM_BK || block_size % FM_BK != 0 || q_ld % 8 != 0 || out_ld % 8 != 0) return -3;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % 16 != 0) return -4;
   CUtensorMap tq, tk, tv;
@@ -419,7 +446,7 @@ extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const 
   p.dv = d_v; p.out_ld = out_ld; p.kv_len = kv_len; p.block_table = block_table; p.bt_ld = bt_ld;
   p.block_size = block_size; p.window = window; p.chunk = chunk; p.keep = keep; p.sink = sink; p.out_scale = out_scale;
   p.score = make_score_mod(scale, softcap, slopes);
-  const dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, Hq);
+  const dim3 grid(Hq, B, (max_q + FM_BQ - 1) / FM_BQ);
   if (softcap > 0.f || slopes != nullptr) {
     if (p.nk1 <= 2) return launch_fmha<FM_PAGED_MOD, 2, 2>(grid, tq, tq, tk, tk, tv, p, stream);
     return launch_fmha<FM_PAGED_MOD, FM_MAXC, 3>(grid, tq, tq, tk, tk, tv, p, stream);
@@ -438,7 +465,7 @@ extern "C" int omni_fmha_latent(const void* q, long long q_rows, int q_ld, const
   if (B <= 0 || max_q <= 0) return 0;
   const int nk1 = (d1 + 63) / 64, nk2 = (d2 + 63) / 64;
   if (d1 < 8 || d2 < 8 || d_v < 8 || d1 % 8 != 0 || d2 % 8 != 0 || d_v % 8 != 0 || nk1 + nk2 > FM_MAXC || d_v > FM_DV) return -1;
-  if (H < 1 || B > 65535 || H > 65535 || window < 0 || q_rows < 1 || k_rows < 1) return -2;
+  if (H < 1 || B > 65535 || max_q > 65535 * FM_BQ || window < 0 || q_rows < 1 || k_rows < 1) return -2;
   if (q_ld % 8 != 0 || kv_ld % 8 != 0 || k2_ld % 8 != 0 || out_ld % 8 != 0 || q_ld < H * (d1 + d2) || kv_ld < H * (d1 + d_v)) return -3;
   if (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)k2 | (uintptr_t)out) % 16 != 0) return -4;
   CUtensorMap tq, tq2, tk, tk2, tv;
@@ -454,7 +481,7 @@ extern "C" int omni_fmha_latent(const void* q, long long q_rows, int q_ld, const
   p.cu_q = q_start; p.end_q = q_end; p.cu_k = k_start; p.end_k = k_end; p.Hq = H; p.Hkv = H; p.nk1 = nk1; p.nk2 = nk2;
   p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = d_v; p.out_ld = out_ld; p.window = window; p.out_scale = 1.0f; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
-  const dim3 grid((max_q + FM_BQ - 1) / FM_BQ, B, H);
+  const dim3 grid(H, B, (max_q + FM_BQ - 1) / FM_BQ);
   if (nk1 + nk2 <= 2) return launch_fmha<FM_LATENT, 2, 2>(grid, tq, tq2, tk, tk2, tv, p, stream);
   return launch_fmha<FM_LATENT, FM_MAXC, 3>(grid, tq, tq2, tk, tk2, tv, p, stream);
 }
