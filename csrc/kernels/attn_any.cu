@@ -14,7 +14,7 @@
 namespace omni {
 
 constexpr int AA_WARPS = 4;
-constexpr int AA_MAXV = 16;      // value columns per lane: d_v <= 512
+constexpr int AA_MAXV = 64;      // value columns per lane, at most: d_v <= 2048
 
 struct AttnAnyOpts {
   long long k_row, v_row;        // elements from one token's row to the next in the caches
@@ -25,7 +25,8 @@ struct AttnAnyOpts {
   int gate_ld;
 };
 
-template <typename T>
+// MAXV: value columns per lane
+template <typename T, int MAXV>
 __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
     const T* __restrict__ q, int q_ld, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
     const int64_t* __restrict__ positions, const int* __restrict__ q_to_seq, const int64_t* __restrict__ slots,
@@ -48,9 +49,9 @@ __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
   const int lo = first_key(pos, o.window, o.chunk);
   const float slope = o.slopes != nullptr ? o.slopes[h] : 0.f;
   const int* bt = block_table + (size_t)q_to_seq[t] * bt_ld;
-  float m = -INFINITY, l = 0.f, acc[AA_MAXV];
+  float m = -INFINITY, l = 0.f, acc[MAXV];
 #pragma unroll
-  for (int i = 0; i < AA_MAXV; ++i) acc[i] = 0.f;
+  for (int i = 0; i < MAXV; ++i) acc[i] = 0.f;
   const int kept = min(o.keep, lo);                 // keys ahead of the window that stay visible
   for (int k0 = kept > 0 ? 0 : lo; k0 <= pos; k0 = k0 < lo && k0 + 32 >= kept ? lo : k0 + 32) {
     const int key = k0 + lane, end = k0 < lo ? kept : pos + 1;
@@ -74,20 +75,20 @@ __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
     l = l * f + warp_sum32(p);
     m = m_new;
 #pragma unroll
-    for (int i = 0; i < AA_MAXV; ++i) acc[i] *= f;
+    for (int i = 0; i < MAXV; ++i) acc[i] *= f;
     const int n = min(32, end - k0);
     for (int j = 0; j < n; ++j) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const T* vr = v_cache + (size_t)__shfl_sync(0xffffffffu, (unsigned long long)slot, j) * o.v_row + (size_t)hk * dv;
 #pragma unroll
-      for (int i = 0; i < AA_MAXV; ++i)
+      for (int i = 0; i < MAXV; ++i)
         if (i * 32 + lane < dv) acc[i] = fmaf(pj, to_f32(vr[i * 32 + lane]), acc[i]);
     }
   }
   if (sink != nullptr) l += expf(sink[h] - m);      // one more term of the denominator, without a value
   if (o.gate != nullptr) out_scale /= 1.f + expf(-to_f32(((const T*)o.gate)[(size_t)t * o.gate_ld + h]));
 #pragma unroll
-  for (int i = 0; i < AA_MAXV; ++i)
+  for (int i = 0; i < MAXV; ++i)
     if (i * 32 + lane < dv) orow[i * 32 + lane] = from_f32<T>(acc[i] / l * out_scale);
 }
 
@@ -97,7 +98,8 @@ static int launch_attn_any(const void* q, int q_ld, const void* k, const void* v
                            int dk, int dv, int block_size, float scale, const float* sink, float out_scale, void* out,
                            int out_ld, const AttnAnyOpts& o, cudaStream_t st) {
   const long long items = (long long)rows * Hq;
-  attn_any_kernel<T><<<(unsigned)((items + AA_WARPS - 1) / AA_WARPS), AA_WARPS * 32, AA_WARPS * dk * sizeof(float), st>>>(
+  const auto kernel = dv <= 32 * 16 ? attn_any_kernel<T, 16> : attn_any_kernel<T, AA_MAXV>;
+  kernel<<<(unsigned)((items + AA_WARPS - 1) / AA_WARPS), AA_WARPS * 32, AA_WARPS * dk * sizeof(float), st>>>(
       (const T*)q, q_ld, (const T*)k, (const T*)v, positions, q_to_seq, slots, bt, bt_ld, rows, Hq, Hkv, dk, dv, block_size,
       scale, sink, out_scale, (T*)out, out_ld, o);
   return (int)cudaGetLastError();

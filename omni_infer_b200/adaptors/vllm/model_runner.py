@@ -272,8 +272,8 @@ class ModelRunner:
         dt = self.model.model.dtype if hasattr(self.model, "model") else torch.bfloat16
         self.num_blocks = num_blocks
 
-        ipc = (self.kv_connector is not None and getattr(self.kv_connector, "transport", "inproc") != "inproc"
-               and self.device.type == "cuda")
+        ipc_transport = self.kv_connector is not None and getattr(self.kv_connector, "transport", "inproc") != "inproc"
+        ipc = ipc_transport and self.device.type == "cuda"
 
         def zeros(*shape):
             if ipc:     # another process will open this memory through CUDA IPC
@@ -292,7 +292,11 @@ class ModelRunner:
                 num_blocks, bs, self.cfg.max_num_seqs, lambda *shape, dtype: torch.zeros(*shape, dtype=dtype, device=self.device))
             self.drafter_kv = []
             if self.kv_connector is not None:
-                self.kv_connector.register_kv_caches(self.model.paged_caches(self.kv_caches))
+                from ...accelerators.pd.kv_push import flatten_cache
+                pools = self.model.paged_caches(self.kv_caches)
+                if ipc_transport and len({t[0].numel() for t in flatten_cache(pools)}) > 1:
+                    raise ValueError("KV hand-over between processes needs blocks of one size in all layers")
+                self.kv_connector.register_kv_caches(pools)
             return
         self.kv_caches = [one() for _ in range(self.model.num_kv_layers)]
         self.drafter_kv = [[one()] for _ in self.drafters]

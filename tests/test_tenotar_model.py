@@ -338,6 +338,27 @@ def test_caches_by_layer():
     assert m.num_kv_layers == 6 and m.kv_bytes_per_token() == per * 4 and m.state_bytes(4) == 4 * 128 * (2 + 3) * 4
 
 
+def test_hand_over_between_processes_needs_equal_blocks():
+    class Connector:
+        transport, seen = "ipc", None
+
+        def register_kv_caches(self, caches):
+            self.seen = caches
+
+    same, mixed = [cases.latent(mlp=None)] * 2, [cases.latent(mlp=None), cases.window(mlp=None)]
+    for layers, transport, fine in ((same, "ipc", True), (mixed, "ipc", False), (mixed, "inproc", True)):
+        cfg = cases.config(layers)
+        r = build(cfg, cases.weights(cfg), "cpu", "float32", blocks=4, max_model_len=64, max_num_seqs=1).worker.runner
+        r.kv_connector = Connector()
+        r.kv_connector.transport = transport
+        if fine:
+            r.initialize_kv_cache(4)
+            assert len(r.kv_connector.seen) == 2
+        else:
+            with pytest.raises(ValueError, match="one size"):
+                r.initialize_kv_cache(4)
+
+
 def test_what_the_model_does_not_combine_with():
     for kw in (dict(enable_prefix_caching=True), dict(num_speculative_tokens=1), dict(enable_omni_attn=True, omni_attn_config={"sink": 1, "recent": 1})):
         with pytest.raises(ValueError):

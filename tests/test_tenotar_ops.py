@@ -261,7 +261,7 @@ def test_gathered_pages(device, dtype):
 
 
 @pytest.mark.parametrize("device,dtype", RUNS)
-@pytest.mark.parametrize("H,C,R", [(4, 64, 16), (20, 96, 32), (3, 16, 8), (16, 512, 64), (5, 512, 64), (2, 200, 56), (3, 296, 24), (100, 512, 64)])
+@pytest.mark.parametrize("H,C,R", [(4, 64, 16), (20, 96, 32), (3, 16, 8), (16, 512, 64), (5, 512, 64), (2, 200, 56), (3, 296, 24), (100, 512, 64), (2, 600, 8)])
 @pytest.mark.parametrize("window", [0, 1, 37, 64, 65, 200])
 def test_attention_in_latent_space(device, dtype, H, C, R, window):
     """Rows that stand alone, and several rows of a request; values are a part of the keys; a gate per row and head."""
