@@ -127,6 +127,7 @@ class GeGLUMLP(nn.Module):
         self.gate_up_proj = PaddedLinear(hidden, 2 * self.block, dtype=dtype, device=device, bias_column=bias)
         self.down_proj = PaddedLinear(inter, hidden, dtype=dtype, device=device)
         self.out_bias = nn.Parameter(torch.zeros(hidden, dtype=torch.float32, device=device), requires_grad=False) if bias else None
+        self.zero_padding()
 
     @property
     def in_cols(self):
