@@ -122,7 +122,7 @@ class LatentAttention(nn.Module):
     def forward(self, x, md: AttnMetadata, cache, shared=None):
         s, T = self.spec, x.shape[0]
         a = ops.gemm(x, self.in_proj.weight)
-        portions = md.is_prefill and x.is_cuda and latent_prefill_fits(x.dtype, self.d, self.r, self.p)
+        portions = md.is_prefill and x.is_cuda and latent_prefill_fits(x.dtype, self.d, self.r, self.p, s.scale)
         plan = step_plan(md, s.window, x.device) if portions else None
         own_keys = portions and plan.n_long > 0 and plan.gather is None
         cq, rows = latent_prepare(a, s.q_rank, self.kv0, s.kv_rank, s.rot_dim, self.q_norm, self.kv_norm, self.eps, self.cos_sin,

@@ -127,9 +127,9 @@ def latent_attention(q, cache, latent_cols, *, positions, q_to_seq, slots, block
     return out.view(T, H, latent_cols)
 
 
-def latent_prefill_fits(dtype, d1, d2, dv) -> bool:
-    """Do the head sizes fit the tensor-core kernel for portions of prompts?"""
-    return dtype == torch.bfloat16 and (d1 + 63) // 64 + (d2 + 63) // 64 <= 3 and dv <= 128
+def latent_prefill_fits(dtype, d1, d2, dv, scale) -> bool:
+    """Does the tensor-core kernel for portions of prompts take these head sizes and this (positive) scale?"""
+    return scale > 0 and dtype == torch.bfloat16 and (d1 + 63) // 64 + (d2 + 63) // 64 <= 3 and dv <= 128
 
 
 def latent_prefill(q, kv, k2, *, d1, dv, q_start, q_end, k_start, k_end, max_q, scale, window=0, gate=None, out=None):

@@ -242,7 +242,7 @@ def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_ta
     gate_args = (nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0))
     mod = (nat.c_int(window), nat.c_int(chunk), nat.c_int(keep_first), nat.c_float(scale), nat.c_float(softcap), nat.ptr(slopes), nat.ptr(sink))
     tc = not any_shape and not f32 and ld % 8 == 0 and out.data_ptr() % 16 == 0 and dk % 8 == 0 and dv % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
-    if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0 and packed and gate is None:
+    if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0 and packed and gate is None and scale > 0:
         rc = lib.omni_fmha_paged(
             nat.ptr(q), nat.c_int64(T), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache),
             nat.c_int64(k_cache.shape[0] * bs), nat.ptr(cu_q), nat.ptr(seq_lens), nat.ptr(block_table),

@@ -280,7 +280,7 @@ def test_attention_in_latent_space(device, dtype, H, C, R, window):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("H,d1,d2,dv", [(4, 128, 64, 128), (3, 32, 16, 80), (2, 8, 8, 8), (5, 64, 64, 72), (2, 104, 40, 128), (1, 72, 24, 16)])
+@pytest.mark.parametrize("H,d1,d2,dv", [(4, 128, 64, 128), (3, 40, 16, 88), (2, 8, 8, 8), (5, 64, 64, 72), (2, 104, 40, 128), (1, 72, 24, 16)])
 @pytest.mark.parametrize("window", [0, 1, 70, 64, 129])
 def test_attention_over_projected_keys(H, d1, d2, dv, window):
     """Requests anywhere in the rows, some of the step's rows left out, keys of which only the last belong to queries."""
