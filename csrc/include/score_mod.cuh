@@ -4,17 +4,18 @@
 
 namespace omni {
 
-// score = cap tanh(raw scale / cap) - slope distance (each part optional), in units of log 2
+// score = cap tanh(raw scale / cap) - slope distance - r1 ln(1 + r2 distance) (each part optional), in units of log 2
 struct ScoreMod {
   float scale_log2;        // scale * log2(e)
   float cap_in;            // 2 log2(e) scale / cap
   float cap_log2;          // cap * log2(e); 0 = no cap
   const float* slopes;     // [heads] or null
+  const float *r1, *r2;    // [heads] or null
 };
 
-inline ScoreMod make_score_mod(float scale, float cap, const float* slopes) {
+inline ScoreMod make_score_mod(float scale, float cap, const float* slopes, const float* r1 = nullptr, const float* r2 = nullptr) {
   constexpr float kLog2e = 1.4426950408889634f;
-  return {scale * kLog2e, cap > 0.f ? 2.f * kLog2e * scale / cap : 0.f, cap > 0.f ? cap * kLog2e : 0.f, slopes};
+  return {scale * kLog2e, cap > 0.f ? 2.f * kLog2e * scale / cap : 0.f, cap > 0.f ? cap * kLog2e : 0.f, slopes, r1, r2};
 }
 
 __device__ __forceinline__ float ex2_fast(float x) {
@@ -22,6 +23,13 @@ __device__ __forceinline__ float ex2_fast(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float lg2_fast(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// r1 ln(1 + r2 distance) in units of log 2; absolute error of some 1e-7, which r1 multiplies
+__device__ __forceinline__ float log_bias(float r1, float r2, float distance) { return r1 * lg2_fast(fmaf(r2, distance, 1.f)); }
 __device__ __forceinline__ float rcp_fast(float x) {
   float y;
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

@@ -6,7 +6,8 @@
 //   lane = column  P V, value rows read coalesced
 // Scores, softmax and the accumulation over the values are fp32.  `sink` (per head, may be null): exp(sink) stands in the
 // softmax denominator; `out_scale` multiplies the result before it is rounded, and so does sigmoid(gate[row, head]) if there is a
-// gate.  Optionally: the first `keep` keys beside the window, chunks, a soft cap of the scores and a distance bias per head.
+// gate (or of gate[row, head, column]).  Optionally: the first `keep` keys beside the window, chunks, a soft cap of the scores, a linear
+// and a logarithmic distance bias per head.
 // Rows of the caches have a pitch of their own, so that values may be a part of the key rows (latent attention).
 #include "../include/omni_vec.cuh"
 #include "../include/score_mod.cuh"
@@ -21,8 +22,9 @@ struct AttnAnyOpts {
   int window, chunk, keep;
   float softcap;
   const float* slopes;           // [Hq] or null
+  const float *r1, *r2;          // [Hq] or null
   const void* gate;              // [rows, gate_ld] of the activation type, or null
-  int gate_ld;
+  int gate_ld, gate_cols;        // per head: 1, or dv
 };
 
 // MAXV: value columns per lane
@@ -48,6 +50,7 @@ __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
   const int pos = (int)positions[t];
   const int lo = first_key(pos, o.window, o.chunk);
   const float slope = o.slopes != nullptr ? o.slopes[h] : 0.f;
+  const float r1 = o.r1 != nullptr ? o.r1[h] : 0.f, r2 = o.r1 != nullptr ? o.r2[h] : 0.f;
   const int* bt = block_table + (size_t)q_to_seq[t] * bt_ld;
   float m = -INFINITY, l = 0.f, acc[MAXV];
 #pragma unroll
@@ -65,6 +68,7 @@ __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
       s = dot * scale;
       if (o.softcap > 0.f) s = o.softcap * tanhf(s / o.softcap);
       s -= slope * (float)(pos - key);
+      if (o.r1 != nullptr) s -= r1 * log1pf(r2 * (float)(pos - key));
     }
     float mx = s;
 #pragma unroll
@@ -86,10 +90,15 @@ __global__ void __launch_bounds__(AA_WARPS * 32) attn_any_kernel(
     }
   }
   if (sink != nullptr) l += expf(sink[h] - m);      // one more term of the denominator, without a value
-  if (o.gate != nullptr) out_scale /= 1.f + expf(-to_f32(((const T*)o.gate)[(size_t)t * o.gate_ld + h]));
+  const T* gate = o.gate != nullptr ? (const T*)o.gate + (size_t)t * o.gate_ld + h * o.gate_cols : nullptr;
+  if (gate != nullptr && o.gate_cols == 1) out_scale /= 1.f + expf(-to_f32(gate[0]));
 #pragma unroll
   for (int i = 0; i < MAXV; ++i)
-    if (i * 32 + lane < dv) orow[i * 32 + lane] = from_f32<T>(acc[i] / l * out_scale);
+    if (i * 32 + lane < dv) {
+      float v = acc[i] / l * out_scale;
+      if (gate != nullptr && o.gate_cols > 1) v /= 1.f + expf(-to_f32(gate[i * 32 + lane]));
+      orow[i * 32 + lane] = from_f32<T>(v);
+    }
 }
 
 template <typename T>
@@ -112,12 +121,13 @@ using namespace omni;
 extern "C" int omni_attn_any(const void* q, int q_ld, const void* k_cache, const void* v_cache, long long k_row, long long v_row,
                              const int64_t* positions, const int* q_to_seq, const int64_t* slots, const int* block_table, int bt_ld,
                              int rows, int Hq, int Hkv, int dk, int dv, int block_size, int window, int chunk, int keep, float scale,
-                             float softcap, const float* slopes, const float* sink, const void* gate, int gate_ld, float out_scale,
-                             void* out, int out_ld, int f32, cudaStream_t st) {
+                             float softcap, const float* slopes, const float* r1, const float* r2, const float* sink, const void* gate,
+                             int gate_ld, int gate_cols, float out_scale, void* out, int out_ld, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (Hkv < 1 || Hq % Hkv != 0 || dk < 1 || dk > 2048 || dv < 1 || dv > 32 * AA_MAXV || block_size < 1 || window < 0) return -1;
   if (chunk < 0 || keep < 0 || k_row < (long long)Hkv * dk || v_row < (long long)Hkv * dv) return -2;
-  const AttnAnyOpts o = {k_row, v_row, window, chunk, keep, softcap, slopes, gate, gate_ld};
+  if ((r1 == nullptr) != (r2 == nullptr) || (gate != nullptr && ((gate_cols != 1 && gate_cols != dv) || gate_ld < Hq * gate_cols))) return -3;
+  const AttnAnyOpts o = {k_row, v_row, window, chunk, keep, softcap, slopes, r1, r2, gate, gate_ld, gate_cols};
   if (f32)
     return launch_attn_any<float>(q, q_ld, k_cache, v_cache, positions, q_to_seq, slots, block_table, bt_ld, rows, Hq, Hkv, dk,
                                   dv, block_size, scale, sink, out_scale, out, out_ld, o, st);

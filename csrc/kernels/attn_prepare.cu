@@ -1,7 +1,8 @@
 // Between the input projections of an attention layer and the attention itself:
 //   omni_qkv_prepare     optional RMSNorm of every q and k head, rotation of the first dimensions of every head (halves or
-//                        neighbours), values mixed with those of an earlier layer, K/V scatter into the paged cache
-//   omni_latent_prepare  latent attention: RMSNorm of the query latent and of the key/value latent, rotation of the shared key
+//                        neighbours), values mixed with those of an earlier layer or divided by their head's root mean square, K/V
+//                        scatter into the paged cache
+//   omni_latent_prepare  latent attention: RMSNorm of the query latent (if there is one) and of the key/value latent, rotation of the shared key
 //                        part; latent | key part go to the cache and, if asked for, to contiguous rows
 //   omni_rotate_heads    rotation of a part of every head, in place or into another layout
 //   omni_gather_pages    rows of the paged cache to contiguous rows, a range of positions per request
@@ -23,6 +24,7 @@ struct QkvParams {
   const float* mix;            // one value: v <- (1 - mix) v + mix v_first; null: v as it is
   const void* v_first;         // [T, vf_ld]
   int vf_ld;
+  int v_norm;                  // v <- v / rms(v) by head (without mix)
 };
 
 // One CTA per token, one warp per head.  q in place, k and v into the cache.
@@ -99,7 +101,27 @@ __global__ void qkv_prepare_kernel(T* __restrict__ qkv, const QkvParams p, T* __
       store_vec<V>(dst + c, a);
     }
   }
-  if (slot >= 0) {
+  if (slot >= 0 && p.v_norm) {
+    for (int hd = warp; hd < p.Hkv; hd += nwarps) {
+      const T* vr = row + (size_t)(p.Hq + p.Hkv) * D + (size_t)hd * p.DV;
+      T* vd = v_cache + ((size_t)slot * p.Hkv + hd) * p.DV;
+      float ss = 0.f;
+      for (int c = lane * V; c < p.DV; c += 32 * V) {
+        float v[V];
+        load_vec<V>(vr + c, v);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss += v[i] * v[i];
+      }
+      const float r = 1.0f / sqrtf(warp_sum32(ss) / (float)p.DV + p.eps);
+      for (int c = lane * V; c < p.DV; c += 32 * V) {
+        float v[V];
+        load_vec<V>(vr + c, v);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] *= r;
+        store_vec<V>(vd + c, v);
+      }
+    }
+  } else if (slot >= 0) {
     const T* vr = row + (size_t)(p.Hq + p.Hkv) * D;
     const int n = p.Hkv * p.DV;
     T* vd = v_cache + (size_t)slot * n;
@@ -119,7 +141,7 @@ __global__ void qkv_prepare_kernel(T* __restrict__ qkv, const QkvParams p, T* __
 }
 
 struct LatentParams {
-  int a_ld, q_rank, kv0, kv_rank, rot;   // columns of a row: [0, q_rank) query latent, from kv0 on kv_rank latent | rot key part
+  int a_ld, q_rank, kv0, kv_rank, rot;   // columns of a row: [0, q_rank) query latent (0: none), from kv0 on kv_rank latent | rot key part
   const float *qw, *cw;
   float eps;
   const float* cos_sin;
@@ -148,7 +170,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ a, const LatentParam
     for (int i = 0; i < V; ++i) sc += v[i] * v[i];
   }
   const float2 tot = block_sum2(sq, sc);
-  const float rq = 1.0f / sqrtf(tot.x / (float)p.q_rank + p.eps), rc = 1.0f / sqrtf(tot.y / (float)p.kv_rank + p.eps);
+  const float rq = 1.0f / sqrtf(tot.x / (float)max(p.q_rank, 1) + p.eps), rc = 1.0f / sqrtf(tot.y / (float)p.kv_rank + p.eps);
   T* qd = cq + (size_t)t * p.q_cols;
   for (int c = threadIdx.x * V; c < p.q_cols; c += blockDim.x * V) {
     float v[V], g[V];
@@ -243,12 +265,12 @@ static bool aligned16(const void* p) { return (uintptr_t)p % 16 == 0; }
 
 extern "C" int omni_qkv_prepare(void* qkv, int ld, int Hq, int Hkv, int D, int DV, const float* qw, const float* kw, float eps,
                                 const float* cos_sin, int rot, int pairs, const int64_t* positions, const int64_t* slots,
-                                const float* mix, const void* v_first, int vf_ld, void* k_cache, void* v_cache, int T_rows,
+                                const float* mix, const void* v_first, int vf_ld, int v_norm, void* k_cache, void* v_cache, int T_rows,
                                 int f32, cudaStream_t st) {
   if (T_rows <= 0) return 0;
   if (Hq < 1 || Hkv < 1 || D < 1 || DV < 1 || rot < 0 || rot > D || rot % 2 != 0 || (rot > 0 && cos_sin == nullptr)) return -1;
-  if (k_cache == nullptr || v_cache == nullptr || (qw == nullptr) != (kw == nullptr) || (mix != nullptr && v_first == nullptr)) return -2;
-  const QkvParams p = {ld, Hq, Hkv, D, DV, qw, kw, eps, cos_sin, rot, pairs, positions, slots, mix, v_first, vf_ld};
+  if (k_cache == nullptr || v_cache == nullptr || (qw == nullptr) != (kw == nullptr) || (mix != nullptr && (v_first == nullptr || v_norm))) return -2;
+  const QkvParams p = {ld, Hq, Hkv, D, DV, qw, kw, eps, cos_sin, rot, pairs, positions, slots, mix, v_first, vf_ld, v_norm};
   const bool v4 = D % 4 == 0 && DV % 4 == 0 && (rot / 2) % 4 == 0 && ld % 4 == 0 && (mix == nullptr || (vf_ld % 4 == 0 && (uintptr_t)v_first % (f32 ? 16 : 8) == 0)) &&
                   aligned16(qkv);
   if (v4) {
@@ -265,9 +287,10 @@ extern "C" int omni_latent_prepare(const void* a, int a_ld, int q_rank, int kv0,
                                    int q_cols, void* cache, void* rows, int c_cols, int r_cols, int T_rows, int f32,
                                    cudaStream_t st) {
   if (T_rows <= 0) return 0;
-  if (q_rank < 1 || kv_rank < 1 || rot < 2 || rot % 2 != 0 || q_cols < q_rank || c_cols < kv_rank || r_cols < rot || kv0 < q_rank ||
+  if (q_rank < 0 || (q_rank > 0 && (cq == nullptr || qw == nullptr)) || kv_rank < 1 || rot < 2 || rot % 2 != 0 || q_cols < q_rank || c_cols < kv_rank || r_cols < rot || kv0 < q_rank ||
       a_ld < kv0 + kv_rank + rot || cos_sin == nullptr)
     return -1;
+  if (q_rank == 0) q_cols = 0;
   const LatentParams p = {a_ld, q_rank, kv0, kv_rank, rot, qw, cw, eps, cos_sin, positions, slots, q_cols, c_cols, r_cols};
   if (q_rank % 4 == 0 && kv0 % 4 == 0 && kv_rank % 4 == 0 && a_ld % 4 == 0 && q_cols % 4 == 0 && c_cols % 4 == 0 && r_cols % 4 == 0) {
     FOR_TYPE((latent_prepare_kernel<T, 4><<<T_rows, 128, 0, st>>>((const T*)a, p, (T*)cq, (T*)cache, (T*)rows));)

@@ -12,9 +12,9 @@
 // zero-filled), with an optional sliding window - key tiles outside every query's window are never loaded - and with the
 // softmax weights carried as a pair of bf16 values (p = hi + lo, two MMAs), i.e. to 16 bits of mantissa; optionally a sink per
 // head in the softmax denominator and a factor on the result, kept first keys beside the window (their tiles come first), chunks
-// instead of it, and capped or biased scores (an instantiation of its own).
+// instead of it, a gate per output element, and capped or biased scores (an instantiation of its own).
 // omni_fmha_latent: contiguous key rows as in the first form, but with any head sizes, the window, the pair of bf16 weights and a
-// gate per row and head as in the second: latent attention over keys and values that were projected from their latents.
+// gate per row and head, and with the sinks of the second: latent attention over keys and values that were projected from their latents.
 // Causal mask is aligned to the end of the key range (query i of a request with Lq queries and Lk keys sees
 // keys <= Lk - Lq + i), which also covers chunked prefill and prefix-cache hits.
 //
@@ -50,7 +50,9 @@ struct FmhaParams {
   int window;          // a query sees the last `window` keys up to its own; 0 = all
   int chunk, keep;     // see first_key; the first `keep` keys are visible in any case
   ScoreMod score;      // FM_PAGED_MOD
-  const __nv_bfloat16* gate;   // [Tq, gate_ld] or null: the result of head h is multiplied by sigmoid(gate[t, h])
+  // [Tq, gate_ld] or null: the result of head h is multiplied by sigmoid(gate[t, h]) (latent), or of column d of it by
+  // sigmoid(gate[t, h dv + d]) (paged)
+  const __nv_bfloat16* gate;
   int gate_ld;
   const float* sink;   // [Hq] or null: exp(sink) is one more term of the softmax denominator
   float out_scale;     // multiplies the result before it is rounded
@@ -238,6 +240,8 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     const int first = EXACT ? first_key(q_pos, p.window, p.chunk) : 0;
     float slope = 0.f;
     if (MODE == FM_PAGED_MOD && p.score.slopes != nullptr) slope = p.score.slopes[h] * 1.4426950408889634f;
+    float r1 = 0.f, r2 = 0.f;
+    if (MODE == FM_PAGED_MOD && p.score.r1 != nullptr) { r1 = p.score.r1[h]; r2 = p.score.r2[h]; }
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int i = 0; i < n; ++i) {
@@ -267,6 +271,11 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         } else {
 #pragma unroll
           for (int j = 0; j < FM_BK; ++j) s[j] = fmaf(s[j], p.scale_log2, fmaf(slope, (float)j, -dist_bias));
+        }
+        if (p.score.r1 != nullptr) {
+          const float dist = (float)(q_pos - kbase);      // to column 0; keys ahead of the query are masked below
+#pragma unroll
+          for (int j = 0; j < FM_BK; ++j) s[j] -= log_bias(r1, r2, fmaxf(dist - (float)j, 0.f));
         }
       }
       if (!__all_sync(0xffffffffu, lim >= FM_BK && (!EXACT || low <= 0 || (PAGED && kept >= FM_BK)))) {
@@ -341,7 +350,7 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       tc_fence_after();
       const bool row_ok = (q0 + row) < Lq;
       float den = l;
-      if (PAGED && p.sink != nullptr && m != -INFINITY) den += exp2f(p.sink[h] * 1.4426950408889634f - m);
+      if (EXACT && p.sink != nullptr && m != -INFINITY) den += exp2f(p.sink[h] * 1.4426950408889634f - m);
       float inv_l = l > 0.f ? (EXACT ? p.out_scale : 1.0f) / den : 0.f;
       if (MODE == FM_LATENT && p.gate != nullptr && row_ok)
         inv_l /= 1.f + __expf(-__bfloat162float(p.gate[(size_t)(q_begin + q0 + row) * p.gate_ld + h]));
@@ -355,9 +364,22 @@ fmha_varlen_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
             if (EXACT && c + j >= p.dv) break;
+            float g8[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) g8[e] = inv_l;
+            if (PAGED && p.gate != nullptr) {
+              const uint4 gv = *reinterpret_cast<const uint4*>(p.gate + (size_t)(q_begin + q0 + row) * p.gate_ld + h * p.dv + c + j);
+              const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float2 f = __bfloat1622float2(g2[e]);
+                g8[2 * e] = __fdividef(inv_l, 1.f + __expf(-f.x));
+                g8[2 * e + 1] = __fdividef(inv_l, 1.f + __expf(-f.y));
+              }
+            }
             __nv_bfloat16 o8[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) o8[e] = __float2bfloat16(__uint_as_float(ov[j + e]) * inv_l);
+            for (int e = 0; e < 8; ++e) o8[e] = __float2bfloat16(__uint_as_float(ov[j + e]) * g8[e]);
             *reinterpret_cast<uint4*>(orow + c + j) = *reinterpret_cast<uint4*>(o8);
           }
         }
@@ -427,11 +449,13 @@ extern "C" int omni_fmha_varlen(const void* q, long long q_rows, int q_ld, int q
 extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const void* k_cache, const void* v_cache,
                                long long slots, const int* cu_q, const int* kv_len, const int* block_table, int bt_ld, int B,
                                int max_q, int Hq, int Hkv, int d_k, int d_v, int block_size, int window, int chunk, int keep,
-                               float scale, float softcap, const float* slopes, const float* sink, float out_scale, void* out, int out_ld, void* status, cudaStream_t stream) {
+                               float scale, float softcap, const float* slopes, const float* r1, const float* r2, const float* sink,
+                               const void* gate, int gate_ld, float out_scale, void* out, int out_ld, void* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   if (d_k < 8 || d_v < 8 || d_k % 8 != 0 || d_v % 8 != 0 || d_k > 64 * FM_MAXC || d_v > FM_DV) return -1;
   if (Hkv < 1 || Hq % Hkv != 0 || B > 65535 || max_q > 65535 * FM_BQ || window < 0 || chunk < 0 || keep < 0) return -2;
   if (block_size < FM_BK || block_size % FM_BK != 0 || q_ld % 8 != 0 || out_ld % 8 != 0) return -3;
+  if ((r1 == nullptr) != (r2 == nullptr) || (gate != nullptr && (gate_ld % 8 != 0 || (uintptr_t)gate % 16 != 0 || gate_ld < Hq * d_v))) return -5;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % 16 != 0) return -4;
   CUtensorMap tq, tk, tv;
   if (make_tmap_3d(&tq, q, 2, d_k, Hq, (uint64_t)q_rows, (uint64_t)d_k * 2, (uint64_t)q_ld * 2, 64, 1, FM_BQ, true)) return -10;
@@ -445,9 +469,9 @@ extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const 
   p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
   p.dv = d_v; p.out_ld = out_ld; p.kv_len = kv_len; p.block_table = block_table; p.bt_ld = bt_ld;
   p.block_size = block_size; p.window = window; p.chunk = chunk; p.keep = keep; p.sink = sink; p.out_scale = out_scale;
-  p.score = make_score_mod(scale, softcap, slopes);
+  p.score = make_score_mod(scale, softcap, slopes, r1, r2); p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
   const dim3 grid(Hq, B, (max_q + FM_BQ - 1) / FM_BQ);
-  if (softcap > 0.f || slopes != nullptr) {
+  if (softcap > 0.f || slopes != nullptr || r1 != nullptr) {
     if (p.nk1 <= 2) return launch_fmha<FM_PAGED_MOD, 2, 2>(grid, tq, tq, tk, tk, tv, p, stream);
     return launch_fmha<FM_PAGED_MOD, FM_MAXC, 3>(grid, tq, tq, tk, tk, tv, p, stream);
   }
@@ -461,7 +485,7 @@ extern "C" int omni_fmha_paged(const void* q, long long q_rows, int q_ld, const 
 extern "C" int omni_fmha_latent(const void* q, long long q_rows, int q_ld, const void* kv, long long k_rows, int kv_ld,
                                 const void* k2, int k2_ld, const int* q_start, const int* q_end, const int* k_start,
                                 const int* k_end, int B, int max_q, int H, int d1, int d2, int d_v, int window, float scale,
-                                const void* gate, int gate_ld, void* out, int out_ld, void* status, cudaStream_t stream) {
+                                const void* gate, int gate_ld, const float* sink, void* out, int out_ld, void* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return 0;
   const int nk1 = (d1 + 63) / 64, nk2 = (d2 + 63) / 64;
   if (d1 < 8 || d2 < 8 || d_v < 8 || d1 % 8 != 0 || d2 % 8 != 0 || d_v % 8 != 0 || nk1 + nk2 > FM_MAXC || d_v > FM_DV) return -1;
@@ -480,7 +504,7 @@ extern "C" int omni_fmha_latent(const void* q, long long q_rows, int q_ld, const
   memset(&p, 0, sizeof(p));
   p.cu_q = q_start; p.end_q = q_end; p.cu_k = k_start; p.end_k = k_end; p.Hq = H; p.Hkv = H; p.nk1 = nk1; p.nk2 = nk2;
   p.scale_log2 = scale * 1.4426950408889634f; p.causal = 1; p.out = (__nv_bfloat16*)out; p.status = (OmniStatus*)status;
-  p.dv = d_v; p.out_ld = out_ld; p.window = window; p.out_scale = 1.0f; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
+  p.dv = d_v; p.out_ld = out_ld; p.window = window; p.out_scale = 1.0f; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld; p.sink = sink;
   const dim3 grid(H, B, (max_q + FM_BQ - 1) / FM_BQ);
   if (nk1 + nk2 <= 2) return launch_fmha<FM_LATENT, 2, 2>(grid, tq, tq2, tk, tk2, tv, p, stream);
   return launch_fmha<FM_LATENT, FM_MAXC, 3>(grid, tq, tq2, tk, tk2, tv, p, stream);

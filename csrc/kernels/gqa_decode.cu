@@ -24,8 +24,9 @@
 // 8 up to 256; staged rows are DP = 64, 128 or 256 wide and the columns past the real size stay zero), any number of query
 // heads per KV head (16 per CTA), a sliding window (tiles before it are not read), and softmax weights carried as a pair
 // of bf16 values (two MMAs per value tile), i.e. to 16 bits of mantissa.  Beside the window it knows kept first keys and
-// chunks, a soft cap of the scores and a distance bias per head (an instantiation of its own), cache rows of any pitch (latent
-// attention: the values are the first columns of the key rows), rows that share a request (q_to_seq), and a gate per row and head.
+// chunks, a soft cap of the scores, a linear and a logarithmic distance bias per head (an instantiation of its own), cache rows of
+// any pitch (latent attention: the values are the first columns of the key rows), rows that share a request (q_to_seq), and a gate
+// per row and head or per output element.
 //
 // Reference counterpart: the paged decode attention of the GQA backend
 // (omni/models/common/layers/attention/backend/attention.py:507-702).
@@ -59,11 +60,11 @@ struct GqShape {           // used by the general form only
   long long k_row, v_row;  // elements from one token's row to the next in the caches
   const int* q_to_seq;     // [B] block-table row of each q row, or null (identity)
   ScoreMod score;          // GEN 2
-  const __nv_bfloat16* gate;   // [B, gate_ld] or null: the result of head h is multiplied by sigmoid(gate[b, h])
-  int gate_ld;
+  const __nv_bfloat16* gate;   // [B, gate_ld] or null: the result of head h is multiplied by sigmoid(gate[b, h gate_cols (+ d)])
+  int gate_ld, gate_cols;      // per head: 1, or dv
 };
-__device__ __forceinline__ float gq_gate(const __nv_bfloat16* gate, int ld, int b, int h) {
-  return gate == nullptr ? 1.f : 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)b * ld + h])));
+__device__ __forceinline__ float gq_gate(const __nv_bfloat16* gate, int ld, int cols, int b, int h, int d) {
+  return gate == nullptr ? 1.f : 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)b * ld + h * cols + (cols > 1 ? d : 0)])));
 }
 
 __device__ __forceinline__ uint32_t gq_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -161,11 +162,19 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 #pragma unroll
   for (int j = 0; j < JT; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
 
-  float slope[2] = {0.f, 0.f};                                // of the two rows of this lane, in log2 units
+  float slope[2] = {0.f, 0.f}, r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};      // of the two rows of this lane; slopes in log2 units
   if (GEN == 2 && sh.score.slopes != nullptr) {
 #pragma unroll
     for (int r = 0; r < 2; ++r)
       if ((lane >> 2) + 8 * r < G) slope[r] = sh.score.slopes[hk * Gall + g0 + (lane >> 2) + 8 * r] * 1.4426950408889634f;
+  }
+  if (GEN == 2 && sh.score.r1 != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if ((lane >> 2) + 8 * r < G) {
+        r1[r] = sh.score.r1[hk * Gall + g0 + (lane >> 2) + 8 * r];
+        r2[r] = sh.score.r2[hk * Gall + g0 + (lane >> 2) + 8 * r];
+      }
   }
 
   for (int u = u_begin + warp; u < u_end; u += GQ_WARPS) {
@@ -212,7 +221,8 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + j * 8 + (e & 1);
         const bool see = key < L && (!GEN || key >= low || key < sh.keep);
-        const float w = GEN == 2 ? cap_score(sh.score, s[j][e]) - slope[e >> 1] * (float)(L - 1 - key) : s[j][e] * scale_log2;
+        float w = GEN == 2 ? cap_score(sh.score, s[j][e]) - slope[e >> 1] * (float)(L - 1 - key) : s[j][e] * scale_log2;
+        if (GEN == 2 && sh.score.r1 != nullptr) w -= log_bias(r1[e >> 1], r2[e >> 1], (float)max(L - 1 - key, 0));
         const float v = see ? w : -INFINITY;
         s[j][e] = v;
         mt[e >> 1] = fmaxf(mt[e >> 1], v);
@@ -315,7 +325,7 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
     if (splits == 1) {
       float den = ll;
       if (GEN && sh.sink != nullptr && ll > 0.f) den += exp2f(sh.sink[hq] * 1.4426950408889634f - mm);
-      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / den * (GEN ? sh.out_scale * gq_gate(sh.gate, sh.gate_ld, b, hq) : 1.f) : 0.f);
+      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / den * (GEN ? sh.out_scale * gq_gate(sh.gate, sh.gate_ld, sh.gate_cols, b, hq, d) : 1.f) : 0.f);
     } else {
       o_part[(((size_t)b * splits + split) * Hq + hq) * dv + d] = ll > 0.f ? acc / ll : 0.f;
       if (d == 0) lse_part[((size_t)b * splits + split) * Hq + hq] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
@@ -325,7 +335,7 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
 
 __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part, int splits,
                                    int Hq, int dv, int out_ld, const float* __restrict__ sink, float out_scale,
-                                   const __nv_bfloat16* __restrict__ gate, int gate_ld, __nv_bfloat16* out) {
+                                   const __nv_bfloat16* __restrict__ gate, int gate_ld, int gate_cols, __nv_bfloat16* out) {
   const int bh = blockIdx.x;
   const int b = bh / Hq, h = bh - b * Hq;
   const int d = threadIdx.x;
@@ -341,7 +351,7 @@ __global__ void gqa_combine_kernel(const float* __restrict__ o_part, const float
     acc += w * o_part[(((size_t)b * splits + s) * Hq + h) * dv + d];
   }
   if (sink != nullptr && den > 0.f) den += exp2f(sink[h] * 1.4426950408889634f - mx);
-  out[(size_t)b * out_ld + h * dv + d] = __float2bfloat16(den > 0.f ? acc / den * out_scale * gq_gate(gate, gate_ld, b, h) : 0.f);
+  out[(size_t)b * out_ld + h * dv + d] = __float2bfloat16(den > 0.f ? acc / den * out_scale * gq_gate(gate, gate_ld, gate_cols, b, h, d) : 0.f);
 }
 
 }  // namespace omni
@@ -368,7 +378,7 @@ static int launch_gqa(dim3 grid, const void* q, const void* k_cache, const void*
   if (e != cudaSuccess) return (int)e;
   if (splits > 1) {
     gqa_combine_kernel<<<B * Hq, (dv + 31) / 32 * 32, 0, stream>>>(o_part, lse_part, splits, Hq, dv, out_ld, sh.sink,
-                                                                   sh.out_scale, sh.gate, sh.gate_ld, (__nv_bfloat16*)out);
+                                                                   sh.out_scale, sh.gate, sh.gate_ld, sh.gate_cols, (__nv_bfloat16*)out);
     e = cudaGetLastError();
   }
   return (int)e;
@@ -392,16 +402,17 @@ extern "C" int omni_gqa_paged_decode_window(const void* q, int q_ld, const void*
                                             long long v_row, const int* q_to_seq, const int* block_table, int bt_ld,
                                             const int* seq_lens, int B, int Hq, int Hkv, int dk, int dv, int block_size,
                                             int window, int chunk, int keep, float scale, float softcap, const float* slopes,
-                                            const float* sink, const void* gate, int gate_ld, float out_scale, int splits, float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
+                                            const float* r1, const float* r2, const float* sink, const void* gate, int gate_ld, int gate_cols, float out_scale, int splits, float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (Hkv < 1 || Hq % Hkv != 0 || splits < 1 || splits > 65535 || B > 65535 || window < 0) return -1;
   if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;
   if (dk < 8 || dv < 8 || dk % 8 != 0 || dv % 8 != 0 || dk > 256 || dv > 256) return -3;
   if (q_ld % 8 != 0 || ((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16 != 0) return -4;
   if (chunk < 0 || keep < 0 || k_row < (long long)Hkv * dk || v_row < (long long)Hkv * dv || k_row % 8 != 0 || v_row % 8 != 0) return -6;
+  if ((r1 == nullptr) != (r2 == nullptr) || (gate != nullptr && ((gate_cols != 1 && gate_cols != dv) || gate_ld < Hq * gate_cols))) return -7;
   const GqShape sh = {q_ld, out_ld, dk, dv, window, sink, out_scale, chunk, keep, k_row, v_row, q_to_seq,
-                      make_score_mod(scale, softcap, slopes), (const __nv_bfloat16*)gate, gate_ld};
-  const bool mod = softcap > 0.f || slopes != nullptr;
+                      make_score_mod(scale, softcap, slopes, r1, r2), (const __nv_bfloat16*)gate, gate_ld, gate_cols};
+  const bool mod = softcap > 0.f || slopes != nullptr || r1 != nullptr;
   const dim3 grid(Hkv * ((Hq / Hkv + 15) / 16), splits, B);
   const int d = dk > dv ? dk : dv;
 #define GQA_CASE(DP)                                                                                                     \

@@ -1,8 +1,10 @@
-// Mixers whose state is a matrix per head, between their projections: the matrix memory of xLSTM (mLSTM) and WKV.
+// Mixers whose state is a matrix per head, between their projections: the matrix memory of xLSTM (mLSTM), WKV and gated linear
+// attention (GLA).
 //
 //   mLSTM   S <- keep S + add k v^T,  n <- keep n + add k,  o = S^T q / (max(|n . q|, exp(-m)) + 1e-6)
 //           with m the running maximum of the log gates, keep = exp(f + m' - m), add = exp(i - m)
 //   WKV     o = (S + diag(u) k v^T)^T r,  S <- diag(w) S + k v^T,  w = exp(-exp(z + w0)) per head and key channel
+//   GLA     S <- diag(a) S + k v^T,  o = S^T q,  a = sigmoid(z + w0)^(1 / tau) per head and key channel
 //
 // State slots (fp32): S [slots, H, P or P + 1, N] with N the key size and P the value size; the last row of the mLSTM's is n,
 // which is what a value of one would accumulate.  m [slots, H].  A request whose first token of the call is at position 0
@@ -13,7 +15,7 @@
 //   omni_state_rows    token by token, the state in registers: a warp owns a few rows of P, N lies across its lanes.  One token
 //                      per request (decode) makes it a stream over the state; fp32 runs and short portions take it too
 //   omni_head_norm     o of every head divided by its root mean square, times a weight, a gate and a constant
-// The chunked forms for portions of prompts: ssd_sm100.cu (mLSTM), wkv_chunk.cu (WKV).
+// The chunked forms for portions of prompts: ssd_sm100.cu (mLSTM), wkv_chunk.cu (WKV, GLA).
 #include "../include/omni_vec.cuh"
 
 namespace omni {
@@ -133,12 +135,13 @@ __global__ void __launch_bounds__(GT_THREADS) mlstm_gates_kernel(const MlstmGate
 struct StateParams {
   const void *a, *b, *v;     // query, key [T, ld] with head h at column h N, value with head h at column h P
   int a_ld, b_ld, v_ld;
-  float a_scale;             // mLSTM: multiplies the query
+  float a_scale;             // mLSTM, GLA: multiplies the query
   const float2* ka;          // mLSTM [T, H]
   float* den;                // mLSTM [T, H]: n . q
-  const float* z;            // WKV [T, z_ld]
+  const float* z;            // WKV, GLA [T, z_ld]
   int z_ld;
-  const float *w0, *u;       // WKV [H N]
+  const float *w0, *u;       // WKV, GLA (w0 alone) [H N]
+  float inv_tau;             // GLA
   float* state;
   const int* cu_q;           // [B + 1], null = one row per request
   const int64_t* positions;
@@ -150,12 +153,15 @@ struct StateParams {
   int vec;                   // rows allow NV-wide loads
 };
 
+enum { ST_MLSTM = 0, ST_WKV = 1, ST_GLA = 2 };
+
 // NV values of N per lane (VECN: neighbours, otherwise 32 apart), R rows of the state per warp.
-template <typename T, bool WKV, int NV, int R, bool VECN>
+template <typename T, int KIND, int NV, int R, bool VECN>
 __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
+  constexpr bool MLSTM = KIND == ST_MLSTM;         // the others have a decay per channel
   const int h = blockIdx.x, r = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int p0 = (blockIdx.y * 4 + warp) * R, PR = WKV ? p.P : p.P + 1;
+  const int p0 = (blockIdx.y * 4 + warp) * R, PR = MLSTM ? p.P + 1 : p.P;
   if (p0 >= PR) return;
   const int row0 = p.cu_q ? p.cu_q[r] : r, row1 = p.cu_q ? p.cu_q[r + 1] : r + 1;
   if (row1 <= row0 || (p.max_rows > 0 && row1 - row0 > p.max_rows)) return;
@@ -165,7 +171,7 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
     for (int t = row0; t < row1; ++t)
       for (int i = lane; i < R; i += 32) {
         if (p0 + i < p.P) y[(size_t)t * p.y_ld + h * p.P + p0 + i] = from_f32<T>(0.f);
-        if (!WKV && p0 + i == p.P) p.den[(size_t)t * p.H + h] = 0.f;
+        if (MLSTM && p0 + i == p.P) p.den[(size_t)t * p.H + h] = 0.f;
       }
     return;
   }
@@ -191,23 +197,23 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
       for (int j = 0; j < NV; ++j) S[i][j] = (!fresh && p0 + i < PR && n_of(j) < p.N) ? st[(size_t)i * p.N + n_of(j)] : 0.f;
     }
   }
-  float w0[WKV ? NV : 1], u[WKV ? NV : 1];
-  if constexpr (WKV) {
+  float w0[MLSTM ? 1 : NV], u[KIND == ST_WKV ? NV : 1];
+  if constexpr (!MLSTM) {
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
       const bool in = n_of(j) < p.N;
       w0[j] = in ? p.w0[h * p.N + n_of(j)] : 0.f;
-      u[j] = in ? p.u[h * p.N + n_of(j)] : 0.f;
+      if constexpr (KIND == ST_WKV) u[j] = in ? p.u[h * p.N + n_of(j)] : 0.f;
     }
   }
   struct Tok {
-    float a[NV], b[NV], z[WKV ? NV : 1], x;
+    float a[NV], b[NV], z[MLSTM ? 1 : NV], x;
     float2 ka;
   };
   auto fetch = [&](int t, Tok& k) {
     const T* ar = (const T*)p.a + (size_t)t * p.a_ld + h * p.N;
     const T* br = (const T*)p.b + (size_t)t * p.b_ld + h * p.N;
-    const float* zr = WKV ? p.z + (size_t)t * p.z_ld + h * p.N : nullptr;
+    const float* zr = MLSTM ? nullptr : p.z + (size_t)t * p.z_ld + h * p.N;
     bool done = false;
     if constexpr (VECN && NV <= 4) {
       if (p.vec) {
@@ -215,12 +221,12 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
           k.a[j] = k.b[j] = 0.f;
-          if constexpr (WKV) k.z[j] = 0.f;
+          if constexpr (!MLSTM) k.z[j] = 0.f;
         }
         if (lane * NV < p.N) {
           load_vec<NV>(ar + lane * NV, k.a);
           load_vec<NV>(br + lane * NV, k.b);
-          if constexpr (WKV) load_vec<NV>(zr + lane * NV, k.z);
+          if constexpr (!MLSTM) load_vec<NV>(zr + lane * NV, k.z);
         }
       }
     }
@@ -230,12 +236,12 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
         const bool in = n_of(j) < p.N;
         k.a[j] = in ? to_f32(ar[n_of(j)]) : 0.f;
         k.b[j] = in ? to_f32(br[n_of(j)]) : 0.f;
-        if constexpr (WKV) k.z[j] = in ? zr[n_of(j)] : 0.f;
+        if constexpr (!MLSTM) k.z[j] = in ? zr[n_of(j)] : 0.f;
       }
     }
     const int pr = p0 + lane;                      // lane i holds the value of row i
     k.x = (lane < R && pr < p.P) ? to_f32(((const T*)p.v)[(size_t)t * p.v_ld + h * p.P + pr]) : 0.f;
-    if constexpr (!WKV) {
+    if constexpr (MLSTM) {
       if (lane < R && pr == p.P) k.x = 1.f;
       k.ka = p.ka[(size_t)t * p.H + h];
     }
@@ -245,7 +251,25 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
   for (int t = row0; t < row1; ++t) {
     if (t + 1 < row1) fetch(t + 1, nxt);
     float v[R];
-    if constexpr (WKV) {
+    if constexpr (KIND == ST_GLA) {
+      float dec[NV];
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        dec[j] = expf(log_sigmoid(cur.z[j] + w0[j]) * p.inv_tau);
+        cur.a[j] *= p.a_scale;
+      }
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const float x = __shfl_sync(0xffffffffu, cur.x, i);
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          S[i][j] = fmaf(dec[j], S[i][j], x * cur.b[j]);
+          s = fmaf(S[i][j], cur.a[j], s);
+        }
+        v[i] = s;
+      }
+    } else if constexpr (KIND == ST_WKV) {
       float dec[NV], uk = 0.f;
 #pragma unroll
       for (int j = 0; j < NV; ++j) {
@@ -296,7 +320,7 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
     const int i = lane / (32 / R);
     if (lane % (32 / R) == 0) {
       if (p0 + i < p.P) y[(size_t)t * p.y_ld + h * p.P + p0 + i] = from_f32<T>(s);
-      if (!WKV && p0 + i == p.P) p.den[(size_t)t * p.H + h] = s;
+      if (MLSTM && p0 + i == p.P) p.den[(size_t)t * p.H + h] = s;
     }
     cur = nxt;
   }
@@ -321,16 +345,16 @@ __global__ void __launch_bounds__(128) state_rows_kernel(const StateParams p) {
   }
 }
 
-template <typename T, bool WKV>
+template <typename T, int KIND>
 static int launch_state_rows(StateParams p, int B, cudaStream_t stream) {
-  const int PR = WKV ? p.P : p.P + 1;
+  const int PR = KIND == ST_MLSTM ? p.P + 1 : p.P;
 #define ST_CASE(NV, R, VECN)                                                                                              \
   {                                                                                                                       \
     const uintptr_t al = NV * sizeof(T) - 1;                                                                              \
     p.vec = VECN && p.N % NV == 0 && ((p.a_ld | p.b_ld) % NV) == 0 && (((uintptr_t)p.a | (uintptr_t)p.b) & al) == 0 &&     \
-            (!WKV || (p.z_ld % NV == 0 && ((uintptr_t)p.z & (NV * 4 - 1)) == 0));                                          \
+            (KIND == ST_MLSTM || (p.z_ld % NV == 0 && ((uintptr_t)p.z & (NV * 4 - 1)) == 0));                                          \
     const dim3 grid(p.H, (PR + 4 * R - 1) / (4 * R), B);                                                                  \
-    state_rows_kernel<T, WKV, NV, R, VECN><<<grid, 128, 0, stream>>>(p);                                                  \
+    state_rows_kernel<T, KIND, NV, R, VECN><<<grid, 128, 0, stream>>>(p);                                                  \
     return (int)cudaGetLastError();                                                                                       \
   }
   if (p.N <= 32) ST_CASE(1, 8, true)
@@ -418,17 +442,18 @@ extern "C" int omni_mlstm_gates(const float* z, int z_ld, int f_col, const void*
   return (int)cudaGetLastError();
 }
 
-// kind 0: mLSTM (ka, den), 1: WKV (z, w0, u).
+// kind 0: mLSTM (ka, den), 1: WKV (z, w0, u), 2: GLA (z, w0, inv_tau).
 extern "C" int omni_state_rows(int kind, const void* a, int a_ld, float a_scale, const void* b, int b_ld, const void* v, int v_ld,
-                               const void* ka, float* den, const float* z, int z_ld, const void* w0, const void* u, void* state,
-                               const int* cu_q, const int64_t* positions, const int* state_slots, int B, void* y, int y_ld, int H,
-                               int P, int N, int f32, int max_rows, cudaStream_t st) {
+                               const void* ka, float* den, const float* z, int z_ld, const void* w0, const void* u, float inv_tau,
+                               void* state, const int* cu_q, const int64_t* positions, const int* state_slots, int B, void* y, int y_ld,
+                               int H, int P, int N, int f32, int max_rows, cudaStream_t st) {
   if (B <= 0) return 0;
-  if (H < 1 || P < 1 || N < 1 || B > 65535 || P > 65535 * 8) return -1;
+  if (H < 1 || P < 1 || N < 1 || B > 65535 || P > 65535 * 8 || kind < 0 || kind > 2) return -1;
   StateParams p = {a, b, v, a_ld, b_ld, v_ld, a_scale, (const float2*)ka, den, z, z_ld, (const float*)w0, (const float*)u,
-                   (float*)state, cu_q, positions, state_slots, y, y_ld, H, P, N, max_rows, 0};
-  if (kind == 0) return f32 ? launch_state_rows<float, false>(p, B, st) : launch_state_rows<bf16, false>(p, B, st);
-  return f32 ? launch_state_rows<float, true>(p, B, st) : launch_state_rows<bf16, true>(p, B, st);
+                   inv_tau, (float*)state, cu_q, positions, state_slots, y, y_ld, H, P, N, max_rows, 0};
+  if (kind == ST_MLSTM) return f32 ? launch_state_rows<float, ST_MLSTM>(p, B, st) : launch_state_rows<bf16, ST_MLSTM>(p, B, st);
+  if (kind == ST_WKV) return f32 ? launch_state_rows<float, ST_WKV>(p, B, st) : launch_state_rows<bf16, ST_WKV>(p, B, st);
+  return f32 ? launch_state_rows<float, ST_GLA>(p, B, st) : launch_state_rows<bf16, ST_GLA>(p, B, st);
 }
 
 // y, gate, out: head h at column h P of rows of their pitches.  den / m [T, H] null: y is what is normed.  act 0 sigmoid, 1 silu.

@@ -26,7 +26,8 @@
 //
 // The exact form (omni_mla_decode_window: latent attention layers of layer-list models) adds a sliding window - tiles ahead of it
 // are not read -, carries the softmax weights as a pair of bf16 values (p = hi + lo, two MMAs per value tile), i.e. to 16 bits of
-// mantissa, and multiplies the result of every head by a sigmoid gate.
+// mantissa, multiplies the result of every head by a sigmoid gate, and knows a sink per head (one more term of the softmax
+// denominator).
 //
 // Stands where the reference calls npu_fused_infer_attention_score on the absorbed path
 // (omni/models/common/layers/attention/deepseek_mla.py:533-560, 625-650).
@@ -53,6 +54,7 @@ struct MlaDecodeParams {
   int window;            // exact form: a row sees its last `window` tokens; 0 = all
   const __nv_bfloat16* gate;   // exact form: [Bq, gate_ld] logits or null
   int gate_ld;
+  const float* sink;     // exact form: [H] or null
   OmniStatus* status;
 };
 
@@ -516,7 +518,9 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       }
       if (ok) {
         tc_fence_after();
-        float inv_l = 1.0f / (sm_sum[row] + sm_sum[128 + row]);
+        float den = sm_sum[row] + sm_sum[128 + row];
+        if (EXACT && p.sink != nullptr && p.num_splits == 1 && row < p.H) den += exp2f(p.sink[row] * 1.4426950408889634f - m);
+        float inv_l = 1.0f / den;
         if (EXACT && p.num_splits == 1 && row < p.H) inv_l *= mla_gate(p.gate, p.gate_ld, bq, row);
         const float l_tot = sm_sum[row] + sm_sum[128 + row];
         const bool row_ok = row < p.H;
@@ -604,7 +608,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
 // out[bq, h, :] = sum_s w_s * o_part[bq, s, h, :],  w_s = 2^(lse_s - max) / sum
 __global__ void mla_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part,
                                    int splits, int H, const __nv_bfloat16* __restrict__ gate, int gate_ld,
-                                   __nv_bfloat16* out) {
+                                   const float* __restrict__ sink, __nv_bfloat16* out) {
   const int bh = blockIdx.x;  // bq * H + h
   const int bq = bh / H, h = bh - bq * H;
   float mx = -INFINITY;
@@ -614,6 +618,7 @@ __global__ void mla_combine_kernel(const float* __restrict__ o_part, const float
     const float v = lse_part[((size_t)bq * splits + s) * H + h];
     den += (v == -INFINITY) ? 0.f : exp2f(v - mx);
   }
+  if (sink != nullptr && den > 0.f) den += exp2f(sink[h] * 1.4426950408889634f - mx);
   const float inv = den > 0.f ? mla_gate(gate, gate_ld, bq, h) / den : 0.f;
   for (int c = threadIdx.x * 4; c < 512; c += blockDim.x * 4) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -646,8 +651,8 @@ extern "C" int omni_mla_debug_read(int* out32) {
 template <bool EXACT>
 static int mla_decode_launch(const void* q, const void* cache, int cache_ld, long long num_slots,
                              const int* block_table, int bt_ld, const int* seq_lens, const int* q_to_seq, int Bq,
-                             int H, int block_size, float scale, int window, const void* gate, int gate_ld, int num_splits,
-                             void* out, float* o_part, float* lse_part, void* status, cudaStream_t stream) {
+                             int H, int block_size, float scale, int window, const void* gate, int gate_ld, const float* sink,
+                             int num_splits, void* out, float* o_part, float* lse_part, void* status, cudaStream_t stream) {
   if (Bq <= 0) return 0;
   if (H < 1 || H > 128) return -1;
   if (block_size != 32 && block_size % 64 != 0) return -2;
@@ -661,7 +666,7 @@ static int mla_decode_launch(const void* q, const void* cache, int cache_ld, lon
   p.q = (const __nv_bfloat16*)q; p.H = H; p.block_size = block_size; p.block_table = block_table; p.bt_ld = bt_ld; p.seq_lens = seq_lens;
   p.q_to_seq = q_to_seq; p.scale_log2 = scale * 1.4426950408889634f; p.num_splits = num_splits;
   p.out = (__nv_bfloat16*)out; p.o_part = o_part; p.lse_part = lse_part; p.status = (OmniStatus*)status;
-  p.window = window; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
+  p.window = window; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld; p.sink = sink;
   static bool configured[64] = {false};
   if (int e = ensure_dyn_smem((const void*)mla_decode_kernel<EXACT>, MLA_SMEM, configured)) return e;
   dim3 grid(2, num_splits, Bq);
@@ -669,7 +674,7 @@ static int mla_decode_launch(const void* q, const void* cache, int cache_ld, lon
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   if (num_splits > 1) {
-    mla_combine_kernel<<<Bq * H, 128, 0, stream>>>(o_part, lse_part, num_splits, H, p.gate, gate_ld, (__nv_bfloat16*)out);
+    mla_combine_kernel<<<Bq * H, 128, 0, stream>>>(o_part, lse_part, num_splits, H, p.gate, gate_ld, sink, (__nv_bfloat16*)out);
     e = cudaGetLastError();
   }
   return (int)e;
@@ -681,18 +686,18 @@ extern "C" int omni_mla_decode(const void* q, const void* cache, int cache_ld, l
                                int H, int block_size, float scale, int num_splits, void* out, float* o_part,
                                float* lse_part, void* status, cudaStream_t stream) {
   return mla_decode_launch<false>(q, cache, cache_ld, num_slots, block_table, bt_ld, seq_lens, q_to_seq, Bq, H, block_size, scale,
-                                  0, nullptr, 0, num_splits, out, o_part, lse_part, status, stream);
+                                  0, nullptr, 0, nullptr, num_splits, out, o_part, lse_part, status, stream);
 }
 
 // The exact form.
 extern "C" int omni_mla_decode_window(const void* q, const void* cache, int cache_ld, long long num_slots,
                                       const int* block_table, int bt_ld, const int* seq_lens, const int* q_to_seq, int Bq,
                                       int H, int block_size, float scale, int window, const void* gate, int gate_ld,
-                                      int num_splits, void* out, float* o_part, float* lse_part, void* status,
+                                      const float* sink, int num_splits, void* out, float* o_part, float* lse_part, void* status,
                                       cudaStream_t stream) {
   if (window < 0 || (gate != nullptr && gate_ld < H)) return -5;
   return mla_decode_launch<true>(q, cache, cache_ld, num_slots, block_table, bt_ld, seq_lens, q_to_seq, Bq, H, block_size, scale,
-                                 window, gate, gate_ld, num_splits, out, o_part, lse_part, status, stream);
+                                 window, gate, gate_ld, sink, num_splits, out, o_part, lse_part, status, stream);
 }
 
 // -------------------------------------------------------------------------------------------------------

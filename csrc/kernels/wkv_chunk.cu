@@ -1,16 +1,22 @@
-// WKV over portions of prompts: o_t = (S + diag(u) k_t v_t^T)^T r_t, S <- diag(w_t) S + k_t v_t^T with a decay per head and key
-// channel, w = exp(-exp(z + w0)).  bf16 activations, head sizes up to 128 that are multiples of 8.  (matrix_state.cu holds the
-// token-by-token form.)
+// Recurrences with a decay per head and key channel over portions of prompts, bf16 activations (matrix_state.cu holds the
+// token-by-token forms):
+//   WKV  o_t = (S + diag(u) k_t v_t^T)^T r_t, S <- diag(w_t) S + k_t v_t^T with w = exp(-exp(z + w0)); head sizes up to 128 that are
+//        multiples of 8
+//   GLA  S <- diag(w_t) S + k_t v_t^T, o_t = S^T r_t with w = sigmoid(z + w0)^(1 / tau); key sizes up to 256 and value sizes that are
+//        multiples of 8
 //
 // Chunks of 16 tokens.  With c_t the running sum of log2 w inside the chunk (c_-1 = 0),
 //   O = (r 2^(c_t-1)) S + A v,   A_ij = sum over channels r_i k_j 2^(c_i-1 - c_j) for j < i, r_i u k_i on the diagonal
 //   S <- 2^(c_15) S + (k 2^(c_15 - c_t))^T v
+// for WKV; in GLA a token's own decay and pair come ahead of its output: c_t and c_i stand where c_t-1 and c_i-1 do, and r_i k_i is
+// on the diagonal.
 // A decay per channel leaves no common factor to take out of a block of scores, and k 2^(-c_j) alone may overflow: every
 // exponent that is taken here is a difference whose sign makes it at most zero.  A is made of 4 x 4 tiles: below the diagonal
 // tiles both sides refer to the tile's first row (8 exponentials for 16 products), on it every pair has its own.
 //
-// One CTA walks the chunks of one (request, head); two kinds of warps, stages of shared memory between them:
-//   prep   (two or three groups of 4 warps that take turns) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
+// One CTA walks the chunks of one (request, head) and up to 128 of its value columns; two kinds of warps, stages of shared memory
+// between them:
+//   prep   (one to three groups of 4 warps that take turns) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
 //          the tiles of A with lanes over channels
 //   state  (one warp per 16 value columns) S^T in fp32 accumulators; O^T = S^T R^T + V^T A^T and S^T += V^T K on mma.sync, S^T being
 //          its own A operand.  A chunk of 16 tokens is too short for tcgen05: the chain from S to S would go through tensor memory
@@ -28,14 +34,15 @@ struct WkvParams {
   int r_ld, k_ld, v_ld;
   const float* z;                      // [T, z_ld]
   int z_ld;
-  const float *w0, *u;                 // [H D]
-  float* state;                        // [slots, H, D (value), D (key)]
+  const float *w0, *u;                 // [H D]; u: WKV
+  float r_scale, inv_tau;              // GLA: multiplies r; 1 / tau
+  float* state;                        // [slots, H, P (value), D (key)]
   const int* cu_q;
   const int64_t* positions;
   const int* state_slots;
   __nv_bfloat16* y;
   int y_ld;
-  int H, D, min_rows;
+  int H, D, P, min_rows;
   OmniStatus* status;
 };
 
@@ -43,13 +50,14 @@ constexpr int WK_L = 16;                           // tokens per chunk
 constexpr int WK_PREP = 4;                         // warps of a prep group
 constexpr int WK_TP = 20;                          // floats per channel of the arrays [channel][token]
 constexpr int WK_APITCH = 48;                      // bytes per row of A
-template <int DP>
+template <int DP, int VP>                            // key channels, value columns of a CTA
 struct WkLayout {
-  static constexpr int GROUPS = DP > 64 ? 2 : 3;   // prep groups, as many as fit
+  static constexpr int GROUPS = DP > 128 ? 1 : (DP > 64 || VP > 64 ? 2 : 3);   // prep groups, as many as fit
   static constexpr int STAGES = 2 * GROUPS;
   static constexpr int PITCH = DP * 2 + 16;        // bytes per token row; ldmatrix rows fall into different banks
   static constexpr int TILE = WK_L * PITCH;
-  static constexpr int A_OFF = 5 * TILE;           // after R hi, R lo, K hi, K lo, V
+  static constexpr int VPITCH = VP * 2 + 16;
+  static constexpr int A_OFF = 4 * TILE + WK_L * VPITCH;      // after R hi, R lo, K hi, K lo, V
   static constexpr int DS_OFF = A_OFF + 2 * WK_L * WK_APITCH;
   static constexpr int STAGE = DS_OFF + DP * 4;
   static constexpr int T_OFF = STAGES * STAGE;  // per group r, k, c: [DP][WK_TP] floats each
@@ -57,7 +65,7 @@ struct WkLayout {
   static constexpr int U_OFF = T_OFF + GROUPS * 3 * T_ARR;
   static constexpr int BAR_OFF = U_OFF + DP * 4;
   static constexpr int SMEM = BAR_OFF + 128;
-  static constexpr int STATE_WARPS = DP / 16;
+  static constexpr int STATE_WARPS = VP / 16;
   static constexpr int THREADS = 32 * (GROUPS * WK_PREP + STATE_WARPS);
 };
 
@@ -110,10 +118,17 @@ __device__ __forceinline__ void wk_group_sum(float (&v)[16], int lane) {
   }
 }
 
-template <int DP>
-__global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const WkvParams p) {
-  using L = WkLayout<DP>;
-  const int h = blockIdx.x, q = blockIdx.y;
+// log2 of the decay, from z + w0
+template <bool GLA>
+__device__ __forceinline__ float wk_log2_decay(float z, float inv_tau) {
+  if (GLA) return 1.4426950408889634f * (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau;
+  return -1.4426950408889634f * expf(z);
+}
+
+template <int DP, int VP, bool GLA>
+__global__ void __launch_bounds__(WkLayout<DP, VP>::THREADS) wkv_chunk_kernel(const WkvParams p) {
+  using L = WkLayout<DP, VP>;
+  const int h = blockIdx.x, q = blockIdx.y, v_col0 = blockIdx.z * VP, P = p.P;
   const int row0 = p.cu_q[q], n_rows = p.cu_q[q + 1] - row0, slot = p.state_slots[q];
   if (n_rows <= 0 || n_rows < p.min_rows || slot < 0) return;
   const int n = (n_rows + WK_L - 1) / WK_L, D = p.D;
@@ -131,7 +146,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
   // what is never written later: A above the diagonal, channels past the head size
   for (int i = threadIdx.x; i < L::BAR_OFF / 4; i += L::THREADS) reinterpret_cast<uint32_t*>(wk_smem)[i] = 0u;
   __syncthreads();
-  for (int c = threadIdx.x; c < D; c += L::THREADS) reinterpret_cast<float*>(wk_smem + L::U_OFF)[c] = p.u[h * D + c];
+  for (int c = threadIdx.x; c < D; c += L::THREADS) reinterpret_cast<float*>(wk_smem + L::U_OFF)[c] = GLA ? 1.f : p.u[h * D + c];
   __syncthreads();
 
   if (warp < L::GROUPS * WK_PREP) {
@@ -161,7 +176,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           const bool ok = e < left;
           rn[a][e] = ok ? *rp : zero;
           kn[a][e] = ok ? *kp : zero;
-          zn[a][e] = ok ? *zp : -INFINITY;               // no decay
+          zn[a][e] = ok ? *zp : (GLA ? INFINITY : -INFINITY);      // no decay
           rp += p.r_ld; kp += p.k_ld; zp += p.z_ld;
         }
       }
@@ -172,21 +187,22 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
       uint8_t* st = wk_smem + s * L::STAGE;
       float* rT = reinterpret_cast<float*>(wk_smem + L::T_OFF + grp * 3 * L::T_ARR);
       float* kT = rT + DP * WK_TP;
-      float* cT = kT + DP * WK_TP;                       // cT[channel][t] = c_t-1, t = 0 .. 16
+      float* cT = kT + DP * WK_TP;                       // cT[channel][t] = c_t-1, t = 0 .. 16; GLA: c_t
       float w2[PASS][8];
 #pragma unroll
       for (int a = 0; a < PASS; ++a)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) w2[a][e] = fmaxf(-1.4426950408889634f * expf(zn[a][e] + w0[a]), -256.f);   // log2 w; 2^-256 is 0
+        for (int e = 0; e < 8; ++e) w2[a][e] = fmaxf(wk_log2_decay<GLA>(zn[a][e] + w0[a], p.inv_tau), -256.f);   // 2^-256 is 0
       if (!mbar_wait(&empty[s], ph ^ 1, abort_flag, p.status, 71, ch)) break;
       // ---- v rows
-      for (int i = tid; i < WK_L * (D / 8); i += 32 * WK_PREP) {
-        const int t = i / (D / 8), c8 = i % (D / 8);
+      const int v8 = min(VP, P - v_col0) / 8;
+      for (int i = tid; i < WK_L * v8; i += 32 * WK_PREP) {
+        const int t = i / v8, c8 = i % v8;
         const bool ok = ch * WK_L + t < n_rows;
-        const __nv_bfloat16* src = p.v + (size_t)(row0 + (ok ? ch * WK_L + t : 0)) * p.v_ld + h * D + c8 * 8;
+        const __nv_bfloat16* src = p.v + (size_t)(row0 + (ok ? ch * WK_L + t : 0)) * p.v_ld + h * P + v_col0 + c8 * 8;
         const int bytes = ok ? 16 : 0;                   // the rest is zero-filled
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;"
-                     ::"r"(smem_u32(st + 4 * L::TILE + t * L::PITCH + c8 * 16)), "l"(src), "r"(bytes) : "memory");
+                     ::"r"(smem_u32(st + 4 * L::TILE + t * L::VPITCH + c8 * 16)), "l"(src), "r"(bytes) : "memory");
       }
       // ---- elementwise; the arrays are free once the whole group has handed over its chunk before
       if (ch >= L::GROUPS && !mbar_wait(&full[(ch - L::GROUPS) % L::STAGES], ((ch - L::GROUPS) / L::STAGES) & 1, abort_flag, p.status, 74, ch)) break;
@@ -203,9 +219,9 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           uint8_t* o = st + half * 8 * L::PITCH + c * 2;
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
-            rf[e] = __bfloat162float(rn[a][e]);
+            rf[e] = __bfloat162float(rn[a][e]) * (GLA ? p.r_scale : 1.f);
             kf[e] = __bfloat162float(kn[a][e]);
-            pv[e] = base + (e ? cum[e - 1] : 0.f);
+            pv[e] = GLA ? base + cum[e] : base + (e ? cum[e - 1] : 0.f);
             const float R = rf[e] * wk_ex2(pv[e]), K = kf[e] * wk_ex2(fminf(tot - (base + cum[e]), 0.f));
             const __nv_bfloat16 rh = __float2bfloat16(R), kh = __float2bfloat16(K);
             *reinterpret_cast<__nv_bfloat16*>(o + e * L::PITCH) = rh;
@@ -221,7 +237,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           *reinterpret_cast<float4*>(cT + at) = make_float4(pv[0], pv[1], pv[2], pv[3]);
           *reinterpret_cast<float4*>(cT + at + 4) = make_float4(pv[4], pv[5], pv[6], pv[7]);
           if (half) {
-            cT[c * WK_TP + 16] = base + cum[7];
+            if (!GLA) cT[c * WK_TP + 16] = base + cum[7];
             reinterpret_cast<float*>(st + L::DS_OFF)[c] = wk_ex2(tot);
           }
         }
@@ -253,8 +269,10 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           for (int i = 0; i < 4; ++i) {
             acc[i * 4 + i] = fmaf(rv[i] * uc, kv[i], acc[i * 4 + i]);
 #pragma unroll
-            for (int j = 0; j < i; ++j)                  // c_i-1 - c_j
-              acc[i * 4 + j] = fmaf(rv[i] * kv[j], j + 1 == i ? 1.f : wk_ex2(fminf(cv[i] - cv[j + 1], 0.f)), acc[i * 4 + j]);
+            for (int j = 0; j < i; ++j) {                // c_i-1 - c_j; GLA: c_i - c_j
+              if (GLA) acc[i * 4 + j] = fmaf(rv[i] * kv[j], wk_ex2(fminf(cv[i] - cv[j], 0.f)), acc[i * 4 + j]);
+              else acc[i * 4 + j] = fmaf(rv[i] * kv[j], j + 1 == i ? 1.f : wk_ex2(fminf(cv[i] - cv[j + 1], 0.f)), acc[i * 4 + j]);
+            }
           }
         }
         wk_group_sum<8>(acc, lane);
@@ -271,10 +289,11 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
           const int c = cc + (lane & 15);
           const float4 r4 = *reinterpret_cast<const float4*>(rT + c * WK_TP + I * 4), k4 = *reinterpret_cast<const float4*>(kT + c * WK_TP + J * 4);
           const float4 pi = *reinterpret_cast<const float4*>(cT + c * WK_TP + I * 4), pj = *reinterpret_cast<const float4*>(cT + c * WK_TP + J * 4);
-          const float ref = pi.x, pj4 = cT[c * WK_TP + J * 4 + 4];
+          const float ref = pi.x, pj4 = GLA ? 0.f : cT[c * WK_TP + J * 4 + 4];
+          const float cj[4] = {GLA ? pj.x : pj.y, GLA ? pj.y : pj.z, GLA ? pj.z : pj.w, GLA ? pj.w : pj4};      // c of the tile's keys
           const float rv[4] = {r4.x, r4.y * wk_ex2(fminf(pi.y - ref, 0.f)), r4.z * wk_ex2(fminf(pi.z - ref, 0.f)), r4.w * wk_ex2(fminf(pi.w - ref, 0.f))};
-          const float kv[4] = {k4.x * wk_ex2(fminf(ref - pj.y, 0.f)), k4.y * wk_ex2(fminf(ref - pj.z, 0.f)), k4.z * wk_ex2(fminf(ref - pj.w, 0.f)),
-                               k4.w * wk_ex2(fminf(ref - pj4, 0.f))};
+          const float kv[4] = {k4.x * wk_ex2(fminf(ref - cj[0], 0.f)), k4.y * wk_ex2(fminf(ref - cj[1], 0.f)),
+                               k4.z * wk_ex2(fminf(ref - cj[2], 0.f)), k4.w * wk_ex2(fminf(ref - cj[3], 0.f))};
 #pragma unroll
           for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -290,9 +309,9 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
     }
   } else {
     // ------------------------------------------------------------------ state
-    const int p0 = (warp - L::GROUPS * WK_PREP) * 16, g = lane >> 2, t2 = (lane & 3) * 2;
+    const int vc0 = (warp - L::GROUPS * WK_PREP) * 16, p0 = v_col0 + vc0, g = lane >> 2, t2 = (lane & 3) * 2;
     float S[DP / 8][4];                                  // rows p0 + g (+ 8) of S^T, channels nt * 8 + t2 (+ 1)
-    float* gs = p.state + ((size_t)slot * p.H + h) * D * D;
+    float* gs = p.state + ((size_t)slot * p.H + h) * P * D;
     const bool fresh = p.positions[row0] == 0;
 #pragma unroll
     for (int nt = 0; nt < DP / 8; ++nt)
@@ -300,7 +319,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
       for (int e = 0; e < 4; e += 2) {
         const int pr = p0 + g + e * 4, c = nt * 8 + t2;
         float2 v = make_float2(0.f, 0.f);
-        if (!fresh && pr < D && c < D) v = *reinterpret_cast<const float2*>(gs + (size_t)pr * D + c);
+        if (!fresh && pr < P && c < D) v = *reinterpret_cast<const float2*>(gs + (size_t)pr * D + c);
         S[nt][e] = v.x;
         S[nt][e + 1] = v.y;
       }
@@ -337,7 +356,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
       }
       // ---- + V^T A^T
       uint32_t va[4];
-      wk_ldsm4t(st + 4 * L::TILE + lrow * L::PITCH + p0 * 2 + lcol, va);      // (tokens, values) 00 01 10 11 transposed: a0 a1 a2 a3
+      wk_ldsm4t(st + 4 * L::TILE + lrow * L::VPITCH + vc0 * 2 + lcol, va);      // (tokens, values) 00 01 10 11 transposed: a0 a1 a2 a3
       {
         uint32_t bh[4], bl[4];
         const uint32_t at = st + L::A_OFF + lrow * WK_APITCH + lcol;
@@ -375,7 +394,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int t = ch * WK_L + i * 8 + t2 + (e & 1), pr = p0 + g + (e >> 1) * 8;
-          if (t < n_rows && pr < D) p.y[(size_t)(row0 + t) * p.y_ld + h * D + pr] = __float2bfloat16(o[i][e] + (o2[i][e] + o3[i][e]));
+          if (t < n_rows && pr < P) p.y[(size_t)(row0 + t) * p.y_ld + h * P + pr] = __float2bfloat16(o[i][e] + (o2[i][e] + o3[i][e]));
         }
     }
     if (ok) {
@@ -384,7 +403,7 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
 #pragma unroll
         for (int e = 0; e < 4; e += 2) {
           const int pr = p0 + g + e * 4, c = nt * 8 + t2;
-          if (pr < D && c < D) *reinterpret_cast<float2*>(gs + (size_t)pr * D + c) = make_float2(S[nt][e], S[nt][e + 1]);
+          if (pr < P && c < D) *reinterpret_cast<float2*>(gs + (size_t)pr * D + c) = make_float2(S[nt][e], S[nt][e + 1]);
         }
     }
   }
@@ -393,12 +412,12 @@ __global__ void __launch_bounds__(WkLayout<DP>::THREADS) wkv_chunk_kernel(const 
   if (threadIdx.x == 0 && *abort_flag) report_abort(abort_flag, p.status);
 }
 
-template <int DP>
+template <int DP, int VP, bool GLA>
 static int launch_wkv(const WkvParams& p, int B, cudaStream_t stream) {
-  using L = WkLayout<DP>;
+  using L = WkLayout<DP, VP>;
   static bool configured[64] = {false};
-  if (int e = ensure_dyn_smem((const void*)wkv_chunk_kernel<DP>, L::SMEM, configured)) return e;
-  wkv_chunk_kernel<DP><<<dim3(p.H, B), L::THREADS, L::SMEM, stream>>>(p);
+  if (int e = ensure_dyn_smem((const void*)wkv_chunk_kernel<DP, VP, GLA>, L::SMEM, configured)) return e;
+  wkv_chunk_kernel<DP, VP, GLA><<<dim3(p.H, B, (p.P + VP - 1) / VP), L::THREADS, L::SMEM, stream>>>(p);
   return (int)cudaGetLastError();
 }
 
@@ -415,9 +434,31 @@ extern "C" int omni_wkv_chunks(const void* r, int r_ld, const void* k, int k_ld,
   if (H < 1 || B > 65535 || min_rows < 1 || D < 8 || D % 8 != 0 || D > 128) return -1;
   if (v_ld % 8 != 0 || (uintptr_t)v % 16 != 0 || (uintptr_t)state % 16 != 0) return -2;
   WkvParams p = {(const __nv_bfloat16*)r, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, r_ld, k_ld, v_ld, z, z_ld, (const float*)w0,
-                 (const float*)u, (float*)state, cu_q, positions, state_slots, (__nv_bfloat16*)y, y_ld, H, D, min_rows,
+                 (const float*)u, 1.f, 0.f, (float*)state, cu_q, positions, state_slots, (__nv_bfloat16*)y, y_ld, H, D, D, min_rows,
                  (OmniStatus*)status};
-  if (D <= 32) return launch_wkv<32>(p, B, stream);
-  if (D <= 64) return launch_wkv<64>(p, B, stream);
-  return launch_wkv<128>(p, B, stream);
+  if (D <= 32) return launch_wkv<32, 32, false>(p, B, stream);
+  if (D <= 64) return launch_wkv<64, 64, false>(p, B, stream);
+  return launch_wkv<128, 128, false>(p, B, stream);
+}
+
+// q, k with head h at column h N, v and y at column h P, z and bias [H N], state [slots, H, P, N].
+extern "C" int omni_gla_chunks(const void* q, int q_ld, const void* k, int k_ld, const void* v, int v_ld, const float* z, int z_ld,
+                               const float* bias, float q_scale, float inv_tau, void* state, const int* cu_q, const int64_t* positions,
+                               const int* state_slots, int B, int max_q, void* y, int y_ld, int H, int P, int N, int min_rows,
+                               void* status, cudaStream_t stream) {
+  if (B <= 0 || max_q < min_rows) return 0;
+  if (H < 1 || B > 65535 || min_rows < 1 || N < 8 || N % 8 != 0 || N > 256 || P < 8 || P % 8 != 0 || P > 65535 || !(inv_tau > 0.f)) return -1;
+  if (v_ld % 8 != 0 || (uintptr_t)v % 16 != 0 || (uintptr_t)state % 16 != 0) return -2;
+  WkvParams p = {(const __nv_bfloat16*)q, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, q_ld, k_ld, v_ld, z, z_ld, bias, nullptr,
+                 q_scale, inv_tau, (float*)state, cu_q, positions, state_slots, (__nv_bfloat16*)y, y_ld, H, N, P, min_rows,
+                 (OmniStatus*)status};
+#define GLA_CASE(DP)                                                \
+  if (N <= DP) {                                                    \
+    if (P <= 32) return launch_wkv<DP, 32, true>(p, B, stream);     \
+    if (P <= 64) return launch_wkv<DP, 64, true>(p, B, stream);     \
+    return launch_wkv<DP, 128, true>(p, B, stream);                 \
+  }
+  GLA_CASE(32) GLA_CASE(64) GLA_CASE(128) GLA_CASE(256)
+#undef GLA_CASE
+  return -3;
 }

@@ -60,6 +60,8 @@ ARCH_KERNELS = {
                 "post_norm_ops", "sampler_misc", "ssd_sm100", "stream_ops", "wkv_chunk"),
     "Tenotar": ("attn_any", "attn_prepare", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "mla_decode", "moe_route",
                 "norm_rope", "post_norm_ops", "sampler_misc", "short_conv"),
+    "Zusotar": ("attn_any", "attn_prepare", "depth_average", "fmha_sm100", "gemm_sm100", "gemm_tokmajor_sm100", "gqa_decode", "matrix_state",
+                "mla_decode", "moe_route", "norm_rope", "post_norm_ops", "sampler_misc", "wkv_chunk"),
 }
 
 

@@ -8,7 +8,7 @@ import logging
 import os
 import time
 from concurrent.futures import ThreadPoolExecutor
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Optional
 
 import torch
@@ -67,6 +67,9 @@ class EngineCore:
                  kv_connector_pair=None):
         self.cfg = cfg
         self.model_cfg = model_cfg or get_config(cfg.model, **cfg.model_overrides)
+        if 0 < self.model_cfg.learned_positions < cfg.max_model_len:
+            logger.info("the context is bounded by the model's %d learned positions", self.model_cfg.learned_positions)
+            cfg = self.cfg = replace(cfg, max_model_len=self.model_cfg.learned_positions)
         if cfg.shared_expert_ranks:
             self.model_cfg.shared_expert_ranks = int(cfg.shared_expert_ranks)
         rc = RunnerConfig(block_size=cfg.block_size, num_kv_blocks=cfg.num_kv_blocks,

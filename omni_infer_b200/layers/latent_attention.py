@@ -1,10 +1,14 @@
-"""Latent attention of the layer-list models: queries through a latent of their own, keys and values projected from one cached
-latent per token, a rotated key part that all heads share, a sliding window, and a sigmoid gate per head.
+"""Latent attention of the layer-list models: queries through a latent of their own or straight from the input, keys and values
+projected from one cached latent per token, a rotated key part that all heads share, a sliding window or none, and optionally a
+sigmoid gate per head and a sink per head in the softmax.
 
 Single tokens (and fp32 runs, and head sizes that the kernel for portions does not take) attend in latent space: the key
 projection is absorbed into the query and the value projection follows.  Portions of prompts project the latents of the keys
 they can see - those of the step itself, or gathered from the pages.  Blocks of the weights are padded to multiples of 8 with
-zeros, so all sizes can be TMA operands."""
+zeros, so all sizes can be TMA operands.
+
+The kernels rotate dimension i together with i + rot_dim / 2.  Where neighbours turn together, the rows of the weights that make the
+rotated parts are stored even ones first: queries and keys change alike, so their products stay."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -80,14 +84,16 @@ class LatentAttention(nn.Module):
         self.spec, self.hidden, self.eps, self.cos_sin = spec, hidden, eps, cos_sin
         s = spec
         self.d, self.r, self.p, self.c = pad8(s.dim), s.rot_cols, pad8(s.vdim), s.latent_cols
-        # rows of the input projection: query latent | key/value latent, key part | gates, each block from a multiple of 8 on
-        self.kv0 = pad8(s.q_rank)
+        # rows of the input projection: query latent, or per head unrotated | rotated query | key/value latent, key part | gates,
+        # each block from a multiple of 8 on
+        self.kv0 = pad8(s.q_rank) if s.q_rank else s.heads * (self.d + self.r)
         self.g0 = self.kv0 + pad8(s.kv_rank + s.rot_dim)
         self.in_proj = PaddedLinear(hidden, self.g0 + (s.heads if s.gate else 0), dtype=dtype, device=device)
         par = lambda *n: nn.Parameter(torch.zeros(*n, dtype=dtype, device=device), requires_grad=False)       # noqa: E731
         one = lambda n: nn.Parameter(torch.ones(n, dtype=torch.float32, device=device), requires_grad=False)  # noqa: E731
-        self.q_norm, self.kv_norm = one(s.q_rank), one(s.kv_rank)
-        self.w_uq = par(s.heads * (self.d + self.r), pad8(s.q_rank))            # per head unrotated | rotated
+        self.q_norm, self.kv_norm = one(s.q_rank) if s.q_rank else None, one(s.kv_rank)
+        self.w_uq = par(s.heads * (self.d + self.r), pad8(s.q_rank)) if s.q_rank else None            # per head unrotated | rotated
+        self.sink = nn.Parameter(torch.zeros(s.heads, dtype=torch.float32, device=device), requires_grad=False) if s.sink else None
         self.w_kv = par(s.heads * (self.d + self.p), self.c)                    # per head key | value
         self.o_proj = par(pad8(hidden), s.heads * self.p)
         self.w_uk = self.w_uv = None                                            # [H, c, d], [H, p, c] for the absorbed form
@@ -97,20 +103,22 @@ class LatentAttention(nn.Module):
         return self.in_proj.in_features
 
     def _blocks(self):
-        """Views by head of the padded weights."""
+        """Views by head of the padded weights: queries, keys and values, output."""
         s = self.spec
-        return (self.w_uq.data.view(s.heads, self.d + self.r, -1), self.w_kv.data.view(s.heads, self.d + self.p, -1),
+        q = self.w_uq.data if self.w_uq is not None else self.in_proj.weight.data[:self.kv0]
+        return (q.view(s.heads, self.d + self.r, -1), self.w_kv.data.view(s.heads, self.d + self.p, -1),
                 self.o_proj.data.view(-1, s.heads, self.p))
 
     def zero_padding(self):
         s = self.spec
         uq, kv, o = self._blocks()
         a = self.in_proj.weight.data
-        a[s.q_rank:self.kv0] = 0
+        if s.q_rank:
+            a[s.q_rank:self.kv0] = 0
+            uq[..., s.q_rank:] = 0
         a[self.kv0 + s.kv_rank + s.rot_dim:self.g0] = 0
         uq[:, s.dim:self.d] = 0
         uq[:, self.d + s.rot_dim:] = 0
-        uq[..., s.q_rank:] = 0
         kv[:, s.dim:self.d] = 0
         kv[:, self.d + s.vdim:] = 0
         kv[..., s.kv_rank:] = 0
@@ -127,7 +135,7 @@ class LatentAttention(nn.Module):
         own_keys = portions and plan.n_long > 0 and plan.gather is None
         cq, rows = latent_prepare(a, s.q_rank, self.kv0, s.kv_rank, s.rot_dim, self.q_norm, self.kv_norm, self.eps, self.cos_sin,
                                   md.positions, md.slot_mapping, cache, self.c, pad8(s.q_rank), want_rows=own_keys)
-        q = ops.gemm(cq, self.w_uq).view(T, s.heads, self.d + self.r)
+        q = (ops.gemm(cq, self.w_uq) if s.q_rank else a[:, :self.kv0]).unflatten(1, (s.heads, self.d + self.r))
         gate = a[:, self.g0:self.g0 + s.heads] if s.gate else None
         if not portions:
             lens = md.q_seq_lens if not md.is_prefill else self._visible(md)
@@ -146,7 +154,7 @@ class LatentAttention(nn.Module):
                 rows = gather_pages(cache, md.block_table, req, pos0, plan.k_start, plan.k_end, total, longest)
             kv = ops.gemm(rows[:, :self.c], self.w_kv)
             o = latent_prefill(q, kv, rows[:, self.c:], d1=self.d, dv=self.p, q_start=plan.q_start, q_end=plan.q_end, k_start=plan.k_start,
-                               k_end=plan.k_end, max_q=plan.max_q, scale=s.scale, window=s.window, gate=gate)
+                               k_end=plan.k_end, max_q=plan.max_q, scale=s.scale, window=s.window, gate=gate, sink=self.sink)
             if part is not None:
                 o[plan.rows] = part
         return ops.gemm(o, self.o_proj)
@@ -164,18 +172,27 @@ class LatentAttention(nn.Module):
         ops.bmm_heads(q[..., :self.d], self.w_uk, out=qa)
         rotate_heads(q[..., self.d:], s.rot_dim, self.cos_sin, positions, qa[..., self.c:])
         lat = latent_attention(qa, cache, self.c, positions=positions, q_to_seq=q_to_seq, slots=slots, block_table=md.block_table,
-                               seq_lens=lens, scale=s.scale, window=s.window, gate=gate, max_seq_len=md.max_seq_len or md.max_k)
+                               seq_lens=lens, scale=s.scale, window=s.window, gate=gate, sink=self.sink,
+                               max_seq_len=md.max_seq_len or md.max_k)
         return ops.bmm_heads(lat, self.w_uv).reshape(T, s.heads * self.p)
 
     def checkpoint_targets(self):
         """{checkpoint suffix: (parameter, first row, rows, columns)}, columns None: a vector; or (store, shape)."""
         s, h, a = self.spec, self.hidden, self.in_proj.weight
         uq, kv, o = self._blocks()
+        q_in = s.q_rank or h
+        order = torch.arange(s.rot_dim)
+        if s.rot_pairs:
+            order = torch.cat([order[0::2], order[1::2]])
 
         def store_uq(w):
-            w = w.view(s.heads, s.dim + s.rot_dim, s.q_rank)
-            uq[:, :s.dim, :s.q_rank] = w[:, :s.dim]
-            uq[:, self.d:self.d + s.rot_dim, :s.q_rank] = w[:, s.dim:]
+            w = w.view(s.heads, s.dim + s.rot_dim, q_in)
+            uq[:, :s.dim, :q_in] = w[:, :s.dim]
+            uq[:, self.d:self.d + s.rot_dim, :q_in] = w[:, s.dim:][:, order]
+
+        def store_dkv(w):
+            a.data[self.kv0:self.kv0 + s.kv_rank, :h] = w[:s.kv_rank]
+            a.data[self.kv0 + s.kv_rank:self.kv0 + s.kv_rank + s.rot_dim, :h] = w[s.kv_rank:][order]
 
         def store_kv(row, n):
             def store(w):
@@ -185,10 +202,14 @@ class LatentAttention(nn.Module):
         def store_o(w):
             o[:h, :, :s.vdim] = w.view(h, s.heads, s.vdim)
 
-        t = {"dq": (a, 0, s.q_rank, h), "dkv": (a, self.kv0, s.kv_rank + s.rot_dim, h), "dq.norm": (self.q_norm, 0, s.q_rank, None),
-             "dkv.norm": (self.kv_norm, 0, s.kv_rank, None), "uq": (store_uq, (s.heads * (s.dim + s.rot_dim), s.q_rank)),
+        t = {"dkv": (store_dkv, (s.kv_rank + s.rot_dim, h)), "dkv.norm": (self.kv_norm, 0, s.kv_rank, None),
+             "uq" if s.q_rank else "q": (store_uq, (s.heads * (s.dim + s.rot_dim), q_in)),
              "uk": (store_kv(0, s.dim), (s.heads * s.dim, s.kv_rank)), "uv": (store_kv(self.d, s.vdim), (s.heads * s.vdim, s.kv_rank)),
              "o": (store_o, (h, s.heads * s.vdim))}
+        if s.q_rank:
+            t.update({"dq": (a, 0, s.q_rank, h), "dq.norm": (self.q_norm, 0, s.q_rank, None)})
         if s.gate:
             t["g"] = (a, self.g0, s.heads, h)
+        if s.sink:
+            t["sink"] = (self.sink, 0, s.heads, None)
         return t

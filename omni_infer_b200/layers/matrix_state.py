@@ -1,4 +1,5 @@
-"""Mixers with a matrix per head as their state: WKV time mixing, and attention beside the matrix memory of xLSTM.
+"""Mixers with a matrix per head as their state: WKV time mixing, gated linear attention, and attention beside the matrix memory
+of xLSTM.
 A request's state lives in its state slot, the attention's keys and values in its pages."""
 from __future__ import annotations
 
@@ -6,9 +7,9 @@ import torch
 from torch import nn
 
 from .. import ops
-from ..models.config import MLSTMSpec, ParallelSpec, WkvSpec
+from ..models.config import GLASpec, MLSTMSpec, ParallelSpec, WkvSpec
 from ..ops.layer_list import pad8
-from ..ops.matrix_state import CHUNK_MIN_ROWS, head_norm, mlstm_chunked, mlstm_gates, mlstm_scan, wkv_scan
+from ..ops.matrix_state import CHUNK_MIN_ROWS, gla_scan, head_norm, mlstm_chunked, mlstm_gates, mlstm_scan, wkv_scan
 from ..ops.streams import tanh_split, token_shift
 from .common import AttnMetadata, PaddedLinear
 from .windowed_attention import WindowedAttention
@@ -178,4 +179,69 @@ class WkvMixer(nn.Module):
         t.update({"w1": (self.w1, 0, s.rank, h), "w2": (self.w2, 0, n, s.rank), "w0": (self.w0, 0, n, None),
                   "u": (self.u.data.view(s.heads, s.dim), 0, s.heads, s.dim), "norm": (self.norm_weight, 0, n, None),
                   "o": (self.o_proj.weight, 0, h, n)})
+        return t
+
+
+class GlaMixer(nn.Module):
+    """Gated linear attention.  One input projection with rows q | k | v | output gate | first half of the decay's projection, each
+    block from a multiple of 8 on; the second half's values stay fp32."""
+    out_bias = None
+    ones = False
+
+    def __init__(self, spec: GLASpec, hidden: int, eps: float, *, dtype, device=None):
+        super().__init__()
+        self.spec, self.hidden, self.eps = spec, hidden, eps
+        s = spec
+        if s.rank < 1:
+            raise ValueError("the rank of the decay's projection is not known: it is the number of rows of mix.a1")
+        self.nk, self.nv, self.half = s.heads * s.dim, s.heads * s.vdim, pad8(s.rank)
+        self.k0 = pad8(self.nk)
+        self.v0 = 2 * self.k0
+        self.g0 = self.v0 + pad8(self.nv)
+        self.a0 = self.g0 + pad8(self.nv)
+        self.in_proj = PaddedLinear(hidden, self.a0 + self.half, dtype=dtype, device=device)
+        self.a2 = nn.Parameter(torch.zeros(self.k0, self.half, dtype=dtype, device=device), requires_grad=False)
+        self.o_proj = PaddedLinear(self.nv, hidden, dtype=dtype, device=device)
+        self.decay_bias = _f32(self.nk, device=device, value=2.0)
+        self.norm_weight = nn.Parameter(torch.ones(self.nv, dtype=torch.float32, device=device), requires_grad=False)      # of every head
+
+    @property
+    def in_cols(self):
+        return self.in_proj.in_features
+
+    def _parts(self):
+        return (("q", 0, self.nk), ("k", self.k0, self.nk), ("v", self.v0, self.nv), ("g", self.g0, self.nv), ("a1", self.a0, self.spec.rank))
+
+    def zero_padding(self):
+        w = self.in_proj.weight.data
+        for _, a, n in self._parts():
+            w[a + n:a + pad8(n)] = 0
+        self.a2.data[self.nk:] = 0
+        self.a2.data[:, self.spec.rank:] = 0
+
+    def state_shapes(self, slots: int, dtype):
+        s = self.spec
+        return (((slots, s.heads, s.vdim, s.dim), torch.float32),)
+
+    def forward(self, x, md: AttnMetadata, state, shared=None):
+        s, nk = self.spec, self.nk
+        u = ops.gemm(x, self.in_proj.weight)
+        z = ops.gemm(u[:, self.a0:], self.a2, out_dtype=torch.float32)
+        y = gla_scan(u[:, :nk], u[:, self.k0:self.k0 + nk], u[:, self.v0:self.v0 + self.nv], z, self.decay_bias, 1.0 / s.tau, state[0],
+                     H=s.heads, P=s.vdim, N=s.dim, **_ragged(md), **_rows_of(md))
+        K = self.o_proj.in_features
+        out = (torch.empty if K == self.nv else torch.zeros)(x.shape[0], K, dtype=x.dtype, device=x.device)
+        head_norm(y, u[:, self.g0:self.a0], self.norm_weight, out, H=s.heads, P=s.vdim, eps=self.eps, act="silu")
+        return ops.gemm(out, self.o_proj.weight)
+
+    def checkpoint_targets(self):
+        """{checkpoint suffix: (parameter or a view of one, first row, rows, columns)}; columns None: a vector; or (store, shape)."""
+        s, h, w = self.spec, self.hidden, self.in_proj.weight
+
+        def store_norm(v):
+            self.norm_weight.data.view(s.heads, s.vdim).copy_(v.float())
+
+        t = {name: (w, a, n, h) for name, a, n in self._parts()}
+        t.update({"a2": (self.a2, 0, self.nk, s.rank), "a2.b": (self.decay_bias, 0, self.nk, None), "norm": (store_norm, (s.vdim,)),
+                  "o": (self.o_proj.weight, 0, h, self.nv)})
         return t

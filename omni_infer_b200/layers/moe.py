@@ -251,8 +251,9 @@ class MoELayer(nn.Module):
 class ExpertMixture(nn.Module):
     """Mixture of gated experts of a layer-list model, with a shared expert.  Either softmax scores over the experts and the
     identity experts (whose output is the input), the choice by score + correction, weights = scores * scale without
-    renormalising; or the choice by logit + bias and the softmax over the chosen.  Every rank holds all experts.  The parts are
-    returned unsummed; the residual kernel adds them up."""
+    renormalising; or the choice by logit + bias and the softmax over the chosen; or sigmoid scores that choose and weight, the
+    choice limited to the best groups of experts.  Every rank holds all experts.  The parts are returned unsummed; the residual
+    kernel adds them up."""
     out_bias = None
     ones = False
 
@@ -263,9 +264,11 @@ class ExpertMixture(nn.Module):
         self.block = pad8(s.ff)
         zeros = lambda *n, dt=dtype: nn.Parameter(torch.zeros(*n, dtype=dt, device=device), requires_grad=False)  # noqa: E731
         self.router = zeros(s.experts + s.identity, W)
-        self.correction = zeros(s.experts + s.identity, dt=torch.float32)      # of the scores, or the bias of the logits
-        self.correction.init_value = 0.0
-        self.chosen = s.weighting == "chosen"
+        self.chosen, self.sigmoid = s.weighting == "chosen", s.weighting == "sigmoid"
+        self.correction = None
+        if not self.sigmoid:
+            self.correction = zeros(s.experts + s.identity, dt=torch.float32)      # of the scores, or the bias of the logits
+            self.correction.init_value = 0.0
         self.w13, self.w2 = zeros(s.experts, 2 * self.block, W), zeros(s.experts, W, self.block)
         self.shared = None
         if s.shared_ff and s.act == "clamped_glu":
@@ -295,8 +298,11 @@ class ExpertMixture(nn.Module):
             else:
                 shared = self.shared(x)
         logits = ops.gemm(x, self.router, out_dtype=torch.float32)
-        how = dict(logit_bias=self.correction, renorm=True) if self.chosen else dict(bias=self.correction)
-        ids, w = ops.router_topk(logits, s.top, mode="softmax", scale=s.scale, num_valid=num_valid, **how)
+        if self.sigmoid:
+            how = dict(mode="sigmoid", n_group=s.groups, topk_group=s.keep_groups, group_mode="top2sum")
+        else:
+            how = dict(mode="softmax", **(dict(logit_bias=self.correction, renorm=True) if self.chosen else dict(bias=self.correction)))
+        ids, w = ops.router_topk(logits, s.top, scale=s.scale, num_valid=num_valid, **how)
         perm = ops.moe_permute(x, ids, w, 0, s.experts)
         kw = dict(seg_start=perm.seg_start, seg_len=perm.seg_len, t_hint=max(16, (T * s.top + s.experts - 1) // s.experts))
         act = ops.gemm(perm.x, self.w13, epi=s.act, glu_limit=s.limit, **kw)
@@ -309,7 +315,9 @@ class ExpertMixture(nn.Module):
         """{checkpoint suffix: (parameter or a view of one, first row, rows, columns)}; columns None: a vector."""
         s, H, b = self.spec, self.hidden, self.block
         n = s.experts + s.identity
-        t = {"router": (self.router, 0, n, H), "router.b" if self.chosen else "correction": (self.correction, 0, n, None)}
+        t = {"router": (self.router, 0, n, H)}
+        if self.correction is not None:
+            t["router.b" if self.chosen else "correction"] = (self.correction, 0, n, None)
         for e in range(s.experts):
             t[f"e{e}.gate"], t[f"e{e}.up"] = (self.w13.data[e], 0, s.ff, H), (self.w13.data[e], b, s.ff, H)
             t[f"e{e}.down"] = (self.w2.data[e], 0, H, s.ff)

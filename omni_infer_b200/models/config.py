@@ -12,6 +12,8 @@ from typing import Any, Optional
 
 # architectures of layer-list models with one residual and norms ahead of the sublayers
 NORM_FIRST = ("Tenotar",)
+# and those with norms on both sides of them
+NORM_BOTH = ("Zusotar",)
 
 
 @dataclass
@@ -39,6 +41,9 @@ class AttentionSpec:
     bias: bool = False                       # of the four projections
     conv: int = 0                            # taps of a short convolution of q, k and v; 0 = none
     v_mix: bool = False                      # values are mixed with those of the first layer that has this set
+    v_norm: bool = False                     # every value head is divided by its root mean square
+    log_bias: bool = False                   # learned r1 ln(1 + r2 distance) per head is taken off the scores
+    out_gate: bool = False                   # a sigmoid gate per element on the output, projected from the layer's input
 
     @property
     def owns_kv(self) -> bool:
@@ -54,18 +59,20 @@ class AttentionSpec:
 
 @dataclass
 class LatentSpec:
-    """Softmax attention through a query and a key/value latent of one layer of a layer-list model.  The cache holds the normed
-    latent and one rotated key part that all heads share."""
+    """Softmax attention through a key/value latent, and a query latent or none, of one layer of a layer-list model.  The cache
+    holds the normed latent and one rotated key part that all heads share."""
     heads: int
     dim: int                                 # unrotated query / key size per head
     rot_dim: int                             # rotated query / key size per head
     vdim: int
-    q_rank: int
+    q_rank: int                              # 0 = queries are projected from the layer's input
     kv_rank: int
     scale: float
     window: int = 0                          # a query sees itself and the window - 1 tokens before it; 0 = all
     rot_base: float = 10000.0
     gate: bool = True                        # a sigmoid gate per head on the output
+    sink: bool = False                       # a learned term per head in the softmax denominator
+    rot_pairs: bool = False                  # neighbouring dimensions are rotated together (else i with i + rot_dim / 2)
 
     kv_from = None
     owns_kv = True
@@ -135,6 +142,16 @@ class WkvSpec:
 
 
 @dataclass
+class GLASpec:
+    """Gated linear attention of one layer of a layer-list model."""
+    heads: int
+    dim: int                                 # query / key size per head
+    vdim: int                                # value size per head
+    tau: float                               # the decay is sigmoid(z)^(1 / tau)
+    rank: int = 0                            # of the decay's projection; 0 = as the checkpoint has it
+
+
+@dataclass
 class ParallelSpec:
     """Attention and a matrix memory side by side on the same input."""
     left: AttentionSpec
@@ -155,8 +172,11 @@ class ExpertsSpec:
     shared_ff: int = 0                       # expert that runs for every token, 0 = none
     shared_limit: float = 0.0
     act: str = "clamped_glu"                 # or "swiglu"
-    # "scores": softmax over all outputs, chosen by score + correction; "chosen": by logit + bias, softmax over the chosen ones
+    # "scores": softmax over all outputs, chosen by score + correction; "chosen": by logit + bias, softmax over the chosen ones;
+    # "sigmoid": sigmoid scores, chosen by them
     weighting: str = "scores"
+    groups: int = 1                          # equal groups of neighbours, scored by the sum of their two best experts ...
+    keep_groups: int = 1                     # ... of which the choice is made from this many
 
 
 @dataclass
@@ -172,6 +192,7 @@ class LayerSpec:
     latent: Optional[LatentSpec] = None
     act: str = "geglu"                       # of the dense feed-forward: or "swiglu"
     ff_bias: bool = False                    # of its three projections
+    gla: Optional[GLASpec] = None
 
     @property
     def paged(self):
@@ -182,7 +203,7 @@ class LayerSpec:
 
     @property
     def recurrent(self) -> bool:
-        return (self.mamba2 is not None or self.parallel is not None or self.wkv is not None
+        return (self.mamba2 is not None or self.parallel is not None or self.wkv is not None or self.gla is not None
                 or (self.attention is not None and self.attention.conv > 0))
 
     @staticmethod
@@ -225,12 +246,40 @@ class LayerSpec:
         return s
 
     @classmethod
-    def from_dict(cls, i: int, d: dict, norm_first: bool = False) -> "LayerSpec":
-        """Entry ``i`` of the ``layers`` list of a config.json.  The type may carry a running number (several mixers of
-        one kind with sizes of their own)."""
+    def _norm_both_entry(cls, i: int, d: dict) -> "LayerSpec":
+        """Entry ``i`` of a design with norms on both sides of the sublayers: latent attention with a sink and queries of their
+        own projection; windowed attention with normed values, a logarithmic distance bias and an output gate; gated linear
+        attention.  The type may carry a running number."""
         kind, m = re.sub(r"_\d+$", "", d["type"]), d["mixer"]
-        s = cls._norm_first_entry(i, d) if norm_first else cls(weights_of=d.get("weights_of"))
-        if norm_first:
+        rot, mask, s = m.get("rot") or {}, m.get("mask") or {}, cls(act="swiglu")
+        if kind == "latent_attention":
+            s.latent = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], q_rank=0, kv_rank=m["kv_rank"],
+                                  scale=float(m["scale"]), rot_base=float(rot.get("base", 10000.0)), gate=False, sink=True, rot_pairs=True)
+            if s.latent.rot_dim % 2 or rot.get("dims", s.latent.rot_dim) != s.latent.rot_dim:
+                raise ValueError(f"layer {i}: the rotated part must be even and rotated as a whole")
+        elif kind == "attention":
+            s.attention = AttentionSpec(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]),
+                                        window=int(mask.get("size") or 0), qk_norm=False, v_norm=True, log_bias=True, out_gate=True)
+        elif kind == "gla":
+            s.gla = GLASpec(heads=m["heads"], dim=m["dim"], vdim=m["vdim"], tau=float(m["tau"]))
+            if not s.gla.tau > 0:
+                raise ValueError(f"layer {i}: tau must be positive")
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {d['type']!r}")
+        return s
+
+    @classmethod
+    def from_dict(cls, i: int, d: dict, norms: str = "") -> "LayerSpec":
+        """Entry ``i`` of the ``layers`` list of a config.json.  The type may carry a running number (several mixers of
+        one kind with sizes of their own).  ``norms``: "first" and "both" for the designs of ``NORM_FIRST`` and ``NORM_BOTH``."""
+        kind, m = re.sub(r"_\d+$", "", d["type"]), d["mixer"]
+        if norms == "first":
+            s = cls._norm_first_entry(i, d)
+        elif norms == "both":
+            s = cls._norm_both_entry(i, d)
+        else:
+            s = cls(weights_of=d.get("weights_of"))
+        if norms:
             pass
         elif kind == "attention":
             rot = m.get("rot") or {}
@@ -265,9 +314,16 @@ class LayerSpec:
                 if not mlp.get("router") or not mlp.get("expert"):
                     raise ValueError(f"layer {i}: a feed-forward of kind 'moe' needs a router and an expert")
                 r, e, sh = mlp["router"], mlp["expert"], mlp.get("shared") or {}
-                if norm_first:
+                if norms == "first":
                     s.experts = ExpertsSpec(experts=r["experts"], top=r["top"], ff=e["ff"], shared_ff=int(sh.get("ff", 0)),
                                             act="swiglu", weighting="chosen")
+                elif norms == "both":
+                    g = r.get("groups") or {}
+                    s.experts = ExpertsSpec(experts=r["experts"], top=r["top"], ff=e["ff"], shared_ff=int(sh.get("ff", 0)), act="swiglu",
+                                            weighting="sigmoid", groups=int(g.get("count", 1)), keep_groups=int(g.get("keep", 1)))
+                    n, k = s.experts.groups, s.experts.keep_groups
+                    if not 0 < k <= n <= 32 or s.experts.experts % n or s.experts.top > s.experts.experts // n * k:
+                        raise ValueError(f"layer {i}: {s.experts.top} of {s.experts.experts} experts from {k} of {n} groups")
                 else:
                     s.experts = ExpertsSpec(experts=r["experts"], top=r["top"], ff=e["ff"], limit=float(e["limit"]),
                                             identity=int(r.get("identity") or 0), scale=float(r.get("scale", 1.0)),
@@ -291,6 +347,15 @@ class ModelConfig:
     # layer-list models: one residual with RMS norms ahead of the sublayers
     norm_first: bool = False
     logit_scale: float = 1.0
+    # ... on both sides of them, with what a sublayer adds times residual_mult
+    norm_both: bool = False
+    residual_mult: float = 1.0
+    # what checkpoints leave out of the weights of those norms (1: they are stored around zero)
+    norm_offset: float = 0.0
+    # after every layer the residual is a learned sum of the embedding output and all layers' results so far
+    depth_average: bool = False
+    # rows of the table of learned positions, which bounds the context; 0 = none
+    learned_positions: int = 0
     # tensor-parallel attention: heads sharded over attn_tp_size ranks, hidden states sharded by token rows between
     # layers (set by the model runner; 1 = every rank runs whole attention layers on its own requests)
     attn_tp_size: int = 1
@@ -432,8 +497,8 @@ class ModelConfig:
     @classmethod
     def from_layer_list(cls, arch: str, d: dict[str, Any]) -> "ModelConfig":
         """config.json whose ``layers`` list describes every layer (mixer and feed-forward sizes of its own)."""
-        norm_first = arch in NORM_FIRST
-        layers = [LayerSpec.from_dict(i, e, norm_first) for i, e in enumerate(d["layers"])]
+        norm_first, norm_both = arch in NORM_FIRST, arch in NORM_BOTH
+        layers = [LayerSpec.from_dict(i, e, "first" if norm_first else ("both" if norm_both else "")) for i, e in enumerate(d["layers"])]
         for i, s in enumerate(layers):
             a = s.attention
             if a is None or a.owns_kv:
@@ -448,7 +513,7 @@ class ModelConfig:
             mixed = {s.attention.kv_heads * s.attention.vdim for s in layers if s.attention is not None and s.attention.v_mix}
             if len(mixed) > 1:
                 raise ValueError("layers that mix their values must have equally many of them")
-        elif any((s.parallel or s.wkv or s.experts) is not None if not streams else (s.attention or s.mamba2) is not None or s.ff for s in layers):
+        elif not norm_both and any((s.parallel or s.wkv or s.experts) is not None if not streams else (s.attention or s.mamba2) is not None or s.ff for s in layers):
             raise ValueError("attention, mamba2 and dense layers run on one residual with norms on the outputs, parallel, wkv and "
                              "mixture-of-experts layers on residual streams with norms ahead")
         for i, s in enumerate(layers):
@@ -465,9 +530,11 @@ class ModelConfig:
                 layers[i].weights_of = next(j for j, o in enumerate(layers) if o is s)
         return cls(architecture=arch, layers=layers, vocab_size=d["vocab"], hidden_size=d["width"],
                    num_hidden_layers=len(layers), rms_norm_eps=float(d["norm"]["eps"]), use_mla=False,
-                   tie_word_embeddings=not norm_first, n_routed_experts=0, name=arch, streams=streams,
+                   tie_word_embeddings=not (norm_first or norm_both), n_routed_experts=0, name=arch, streams=streams,
                    embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)), norm_first=norm_first,
-                   logit_scale=float(d.get("logit_scale", 1.0)))
+                   logit_scale=float(d.get("logit_scale", 1.0)), norm_both=norm_both, residual_mult=float(d.get("residual_mult", 1.0)),
+                   norm_offset=1.0 if norm_both else 0.0, depth_average=norm_both,
+                   learned_positions=int(d["max_positions"]) if norm_both else 0)
 
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
@@ -479,16 +546,18 @@ class ModelConfig:
 
     def unresolved_sizes(self) -> bool:
         """Are there sizes that only the checkpoint's tensors tell?"""
-        return any(s.wkv is not None and s.wkv.rank == 0 for s in self.layers or ())
+        return any(r is not None and r.rank == 0 for s in self.layers or () for r in (s.wkv, s.gla))
 
     def resolve_sizes(self, shapes: dict) -> None:
         """``shapes``: checkpoint tensor name -> shape."""
         for i, s in enumerate(self.layers or ()):
-            if s.wkv is not None and s.wkv.rank == 0:
-                name = f"l{i if s.weights_of is None else s.weights_of}.mix.w1"
+            for r, tensor in ((s.wkv, "w1"), (s.gla, "a1")):
+                if r is None or r.rank != 0:
+                    continue
+                name = f"l{i if s.weights_of is None else s.weights_of}.mix.{tensor}"
                 if name not in shapes:
                     raise KeyError(f"checkpoint lacks {name}")
-                s.wkv.rank = int(shapes[name][0])
+                r.rank = int(shapes[name][0])
 
 
 # ------------------------------------------------------------------------------------------------
@@ -673,6 +742,44 @@ def tiny_tenotar(**kw) -> ModelConfig:
                    chunk=48, conv=3, ff=96, experts=6, top=2, expert_ff=24, shared_ff=40, **kw)
 
 
+def zusotar(width=2048, layers=12, vocab=32768, heads=16, kv_heads=4, dim=128, kv_rank=512, rot_dim=64, window=1024, g_heads=16, g_dim=64,
+            g_vdim=128, g_rank=16, ff=5632, experts=32, groups=4, keep=2, top=4, expert_ff=768, shared_ff=1536, positions=16384,
+            **kw) -> ModelConfig:
+    """Layer-list model with norms on both sides of its sublayers: latent attention, gated linear attention and windowed attention
+    in turn, the first layer with a dense feed-forward and the others with a mixture of experts."""
+    specs = []
+    for i in range(layers):
+        if i % 3 == 0:
+            s = LayerSpec(latent=LatentSpec(heads, dim, rot_dim, dim, 0, kv_rank, (dim + rot_dim) ** -0.5, rot_base=5e5, gate=False, sink=True,
+                                            rot_pairs=True))
+        elif i % 3 == 1:
+            s = LayerSpec(gla=GLASpec(g_heads, g_dim, g_vdim, 16.0, g_rank))
+        else:
+            s = LayerSpec(AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window, qk_norm=False, v_norm=True, log_bias=True,
+                                        out_gate=True))
+        s.act = "swiglu"
+        if i == 0:
+            s.ff = ff
+        else:
+            s.experts = ExpertsSpec(experts, top, expert_ff, shared_ff=shared_ff, act="swiglu", weighting="sigmoid", groups=groups,
+                                    keep_groups=keep)
+        specs.append(s)
+    c = ModelConfig(architecture="Zusotar", name="zusotar", layers=specs, vocab_size=vocab, hidden_size=width,
+                    num_hidden_layers=layers, use_mla=False, tie_word_embeddings=False, rms_norm_eps=1e-5, norm_both=True,
+                    residual_mult=0.4, norm_offset=1.0, depth_average=True, learned_positions=positions)
+    for k, v in kw.items():
+        setattr(c, k, v)
+    return c
+
+
+def tiny_zusotar(**kw) -> ModelConfig:
+    """CPU-sized layer-list model with norms on both sides of its sublayers."""
+    kw.setdefault("dtype", "float32")
+    kw.setdefault("name", "tiny-zusotar")
+    return zusotar(width=64, layers=6, vocab=512, heads=4, kv_heads=2, dim=16, kv_rank=40, rot_dim=8, window=40, g_heads=2, g_dim=16,
+                   g_vdim=24, g_rank=8, ff=96, experts=8, groups=4, keep=2, top=2, expert_ff=24, shared_ff=40, positions=512, **kw)
+
+
 def tiny_forovik(**kw) -> ModelConfig:
     """CPU-sized layer-list model."""
     kw.setdefault("dtype", "float32")
@@ -686,6 +793,8 @@ PRESETS = {
     "tiny-forovik": tiny_forovik,
     "tenotar": tenotar,
     "tiny-tenotar": tiny_tenotar,
+    "zusotar": zusotar,
+    "tiny-zusotar": tiny_zusotar,
     "fimudra": fimudra,
     "tiny-fimudra": tiny_fimudra,
     "tiny-deepseek-v3": tiny_deepseek_v3,

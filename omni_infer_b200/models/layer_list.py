@@ -1,5 +1,5 @@
 """Models described layer by layer: ``ModelConfig.layers`` lists a mixer and an optional feed-forward per layer, each with sizes
-of its own.  Three ways to connect them:
+of its own.  Four ways to connect them:
 
 One residual, norms on the outputs (``cfg.streams == 0``; windowed attention, Mamba-2, gated dense feed-forward): sublayers read
 the residual stream itself, ``x <- x + norm1(mixer(x))``, ``x <- x + norm2(ff(x))``.  Every addition, its norm and the activation
@@ -14,6 +14,11 @@ One residual, norms ahead (``cfg.norm_first``; latent, windowed and chunked atte
 experts): ``x <- x + mixer(norm1(x))``, ``x <- x + ff(norm2(x))``.  Addition, output bias and the norm for the next sublayer are
 one kernel.  The head is a matrix of its own; its factor enters with the last norm.
 
+One residual, norms on both sides (``cfg.norm_both``; latent attention, windowed attention, gated linear attention, dense
+feed-forwards and mixtures of experts): ``x <- x + m norm1b(mixer(norm1(x)))``, ``x <- x + m norm2b(ff(norm2(x)))``, learned positions
+added to the embeddings, and after every layer a learned average of the embedding output and all layers' results so far.  Norm
+behind, addition, average and the norm for the next sublayer are one kernel.
+
 The residual is fp32 in all of them, and the embedding table is also the LM head in the first two.
 
 A layer's entry in ``kv_caches`` is what its mixer reads: the (k, v) page pools of an attention layer - the same tensors for a
@@ -27,10 +32,11 @@ from .. import ops
 from ..layers.common import GeGLUMLP, PaddedLinear, PostNorm, _dtype
 from ..layers.latent_attention import LatentAttention
 from ..layers.mamba2 import Mamba2Mixer
-from ..layers.matrix_state import ParallelMixer, WkvMixer
+from ..layers.matrix_state import GlaMixer, ParallelMixer, WkvMixer
 from ..layers.moe import ExpertMixture
 from ..layers.vocab_parallel import lm_logits
 from ..layers.windowed_attention import WindowedAttention
+from ..ops.depth import both_norms_step, embed_positions
 from ..ops.layer_list import add_norm, embed_norm, embed_residual, pad8, rmsnorm_residual
 from ..ops.streams import embed_streams, stream_step
 from .config import ModelConfig
@@ -46,6 +52,8 @@ def _mixer(s, width, eps, **kw):
         return ParallelMixer(s.parallel, width, eps, cos_sin=cos_sin, **kw)
     if s.wkv is not None:
         return WkvMixer(s.wkv, width, eps, **kw)
+    if s.gla is not None:
+        return GlaMixer(s.gla, width, eps, **kw)
     return Mamba2Mixer(s.mamba2, width, eps, **kw)
 
 
@@ -136,6 +144,38 @@ class NormFirstLayer(nn.Module):
         return out
 
 
+class NormBothLayer(NormFirstLayer):
+    """One residual, norms on both sides, an average over depth behind.  The model runs the sublayers; this holds their weights,
+    those of the norms complete (``norm_offset`` added)."""
+
+    def __init__(self, cfg: ModelConfig, i: int, *, dtype, device=None, cos_sin=None):
+        super().__init__(cfg, i, dtype=dtype, device=device, cos_sin=cos_sin)
+        self.offset = cfg.norm_offset
+        norm = lambda: nn.Parameter(torch.ones(cfg.hidden_size, dtype=torch.float32, device=device), requires_grad=False)      # noqa: E731
+        self.norm1b, self.norm2b = norm(), norm() if self.mlp is not None else None
+        self.dwa = None
+        if cfg.depth_average:
+            self.dwa = nn.Parameter(torch.zeros(i + 2, dtype=torch.float32, device=device), requires_grad=False)
+            self.dwa.data[-1] = 1.0
+            self.dwa.init_value = self.dwa.data.clone()
+
+    def checkpoint_targets(self):
+        out = super().checkpoint_targets()
+        for name in ("norm1", "norm1b", "norm2", "norm2b"):
+            if getattr(self, name) is not None:
+                out[name] = _offset_target(getattr(self, name), self.offset)
+        if self.dwa is not None:
+            out["dwa"] = (self.dwa, 0, self.dwa.shape[0], None)
+        return out
+
+
+def _offset_target(p, offset: float):
+    """Checkpoint target of a norm weight that is stored without its offset."""
+    def store(w):
+        p.data.copy_(w.float() + offset)
+    return store, tuple(p.shape)
+
+
 class LayerListModel(nn.Module):
     def __init__(self, cfg: ModelConfig, *, device=None):
         super().__init__()
@@ -154,7 +194,12 @@ class LayerListModel(nn.Module):
 
         self.embed_tokens = nn.Embedding(cfg.vocab_size, pad8(cfg.hidden_size), dtype=self.dtype, device=device)
         self.embed_tokens.weight.requires_grad_(False)
-        kind = StreamLayer if cfg.streams else (NormFirstLayer if cfg.norm_first else LayerListLayer)
+        self.pos_embedding = None
+        if cfg.learned_positions:
+            self.pos_embedding = nn.Parameter(torch.zeros(cfg.learned_positions, pad8(cfg.hidden_size), dtype=self.dtype, device=device),
+                                              requires_grad=False)
+        kind = (StreamLayer if cfg.streams else NormFirstLayer if cfg.norm_first else NormBothLayer if cfg.norm_both
+                else LayerListLayer)
         built: list = []
         for i, s in enumerate(cfg.layers):      # a layer with another's weights is that layer's module
             built.append(None if s.weights_of is not None else
@@ -170,6 +215,8 @@ class LayerListModel(nn.Module):
             return self._forward_streams(input_ids, md, kv_caches)
         if self.cfg.norm_first:
             return self._forward_norm_first(input_ids, md, kv_caches)
+        if self.cfg.norm_both:
+            return self._forward_norm_both(input_ids, md, kv_caches)
         x, xa = embed_residual(input_ids, self.embed_tokens.weight)
         for layer, cache in zip(self.layers, kv_caches):
             xa = layer(x, xa, md, cache)
@@ -191,7 +238,6 @@ class LayerListModel(nn.Module):
             h = stream_step(x, run(h), link.mix, link.out, inw, norm, eps, self.dtype, last=last)
         return h
 
-
     def _forward_norm_first(self, input_ids, md, kv_caches):
         eps, width, shared, subs = self.cfg.rms_norm_eps, pad8(self.cfg.hidden_size), {}, []
         for layer, cache in zip(self.layers, kv_caches):
@@ -208,6 +254,29 @@ class LayerListModel(nn.Module):
                 h = add_norm(x, run(h), norm, eps, self.dtype, ld=nxt.in_cols, ones=nxt.ones, bias=sub.out_bias)
             else:
                 h = add_norm(x, run(h), self.norm, eps, self.dtype, ld=width, bias=sub.out_bias, scale=self.cfg.logit_scale)
+        return h
+
+    def _forward_norm_both(self, input_ids, md, kv_caches):
+        cfg, eps, m, width, n = self.cfg, self.cfg.rms_norm_eps, self.cfg.residual_mult, pad8(self.cfg.hidden_size), len(self.layers)
+        T, dev = input_ids.shape[0], self.embed_tokens.weight.device
+        # the embedding output and what every layer but the last one gave; the residual itself is overwritten
+        results = torch.empty(n if cfg.depth_average else 1, T, width, dtype=torch.float32, device=dev)
+        src, x = results[0], torch.empty(T, width, dtype=torch.float32, device=dev)
+        first = self.layers[0]
+        h = embed_positions(input_ids, self.embed_tokens.weight, md.positions, self.pos_embedding, src, first.norm1, eps,
+                            ld=first.mixer.in_cols)
+        for i, (layer, cache) in enumerate(zip(self.layers, kv_caches)):
+            nxt = self.layers[i + 1] if i + 1 < n else None
+            behind = dict(w=self.norm, ld=width) if nxt is None else dict(w=nxt.norm1, ld=nxt.mixer.in_cols)
+            if layer.dwa is not None:
+                behind.update(results=results, average=layer.dwa)
+            y, norm = layer.mixer(h, md, cache), layer.norm1b
+            if layer.mlp is not None:
+                h = both_norms_step(src, x, y, norm, m, layer.norm2, eps, self.dtype, ld=layer.mlp.in_cols)
+                y = layer.mlp(h, md.num_valid) if isinstance(layer.mlp, ExpertMixture) else layer.mlp(h)
+                src, norm = x, layer.norm2b
+            h = both_norms_step(src, x, y, norm, m, behind.pop("w"), eps, self.dtype, **behind)
+            src = x
         return h
 
 
@@ -273,6 +342,8 @@ class LayerListForCausalLM(nn.Module):
     def process_weights_after_loading(self):
         """Padding rows and columns hold zeros whatever the loader or the random initialisation put there."""
         self.model.embed_tokens.weight.data[:, self.cfg.hidden_size:] = 0
+        if self.model.pos_embedding is not None:
+            self.model.pos_embedding.data[:, self.cfg.hidden_size:] = 0
         if self.lm_head is not None:
             self.lm_head.data[:, self.cfg.hidden_size:] = 0
         mods = [m for m in self.modules() if hasattr(m, "zero_padding")]
@@ -287,6 +358,10 @@ class LayerListForCausalLM(nn.Module):
         """{checkpoint tensor: (parameter, first row, rows, columns)} for the weight loader."""
         H = self.cfg.hidden_size
         out = {"embed": (self.model.embed_tokens.weight, 0, self.cfg.vocab_size, H), "final.norm": (self.model.norm, 0, H, None)}
+        if self.cfg.norm_both:
+            out["final.norm"] = _offset_target(self.model.norm, self.cfg.norm_offset)
+        if self.model.pos_embedding is not None:
+            out["pos"] = (self.model.pos_embedding, 0, self.cfg.learned_positions, H)
         if self.lm_head is not None:
             out["head"] = (self.lm_head, 0, self.cfg.vocab_size, H)
         for i, layer in enumerate(self.model.layers):

@@ -30,6 +30,7 @@ def _lazy():
         "Forovik": LayerListForCausalLM,
         "Fimudra": LayerListForCausalLM,
         "Tenotar": LayerListForCausalLM,
+        "Zusotar": LayerListForCausalLM,
     }
     if any(os.environ.get(k) == "1" for k in ("RANDOM_MODE", "CAPTURE_MODE", "REPLAY_MODE")):
         from .mock import mock_model_class_factory

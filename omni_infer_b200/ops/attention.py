@@ -42,10 +42,11 @@ def _mla_scratch(dev, n_o, n_l):
 
 
 def mla_decode(q, cache, block_table, seq_lens, scale, q_to_seq=None, num_splits=0, max_seq_len=None, kv_lora=512, exact=False,
-               window=0, gate=None):
+               window=0, gate=None, sink=None):
     """Absorbed MLA decode attention.  ``seq_lens[b]`` is the number of cache tokens q row b attends to
     (MTP rows of one request get consecutive lengths); ``q_to_seq`` maps q rows to block-table rows.  ``exact`` (GPU only): softmax
-    weights to 16 bits of mantissa, optionally a sliding ``window`` and a factor sigmoid(``gate`` [Bq, H]) on the heads."""
+    weights to 16 bits of mantissa, optionally a sliding ``window``, a factor sigmoid(``gate`` [Bq, H]) on the heads and one more term
+    exp(``sink`` [H]) in their softmax denominators."""
     if not q.is_cuda:
         assert not exact
         return mla_decode_ref(q, cache, block_table, seq_lens, scale, q_to_seq, kv_lora)
@@ -65,8 +66,8 @@ def mla_decode(q, cache, block_table, seq_lens, scale, q_to_seq=None, num_splits
     o_part = lse = None
     if num_splits > 1:
         o_part, lse = _mla_scratch(q.device, Bq * num_splits * H * 512, Bq * num_splits * H)
-    assert exact or (window == 0 and gate is None)
-    extra = (nat.c_int(window), nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0)) if exact else ()
+    assert exact or (window == 0 and gate is None and sink is None)
+    extra = (nat.c_int(window), nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0), nat.ptr(sink)) if exact else ()
     rc = (nat.lib().omni_mla_decode_window if exact else nat.lib().omni_mla_decode)(
         nat.ptr(q), nat.ptr(cache2), nat.c_int(cache2.stride(0)), nat.ctypes.c_longlong(cache2.shape[0]),
         nat.ptr(block_table), nat.c_int(block_table.stride(0)), nat.ptr(seq_lens), nat.ptr(q_to_seq), nat.c_int(Bq),

@@ -21,11 +21,13 @@ def _rotate_pairs_ref(x, cos_sin, positions, rot):
     return torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., rot:]], -1)
 
 
-def qkv_prepare(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, pairs, positions, slots, k_cache, v_cache, mix=None, v_first=None):
+def qkv_prepare(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, pairs, positions, slots, k_cache, v_cache, mix=None, v_first=None,
+                v_norm=False):
     """``qkv`` rows are q heads | k heads | v heads.  RMSNorm of every q and k head with one weight for all (``q_w=None``: none),
     rotation of the first ``rot`` dimensions of every head (``pairs``: neighbours, else halves); q in place, k and v into the caches
     [blocks, block, hkv, d] at ``slots`` (-1: not stored).  ``mix`` (one value) with ``v_first`` [T, hkv dv]: (1 - mix) v + mix v_first
-    is stored."""
+    is stored; ``v_norm``: every v head divided by its root mean square (not both)."""
+    assert not (v_norm and mix is not None)
     T, nq, nk, nv = qkv.shape[0], hq * dk, hkv * dk, hkv * dv
     if not qkv.is_cuda:
         turn = _rotate_pairs_ref if pairs else _rotate_half_ref
@@ -36,6 +38,8 @@ def qkv_prepare(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, pairs, positi
         v = qkv[:, nq + nk:nq + nk + nv].float()
         if mix is not None:
             v = (1 - mix) * v + mix * v_first.float()
+        if v_norm:
+            v = rms_ref(v.view(T, hkv, dv), 1.0, eps)
         ok = slots >= 0
         k_cache.view(-1, hkv, dk)[slots[ok]] = k[ok].to(k_cache.dtype)
         v_cache.view(-1, hkv, dv)[slots[ok]] = v.view(T, hkv, dv)[ok].to(v_cache.dtype)
@@ -44,19 +48,21 @@ def qkv_prepare(qkv, hq, hkv, dk, dv, q_w, k_w, eps, cos_sin, rot, pairs, positi
     rc = nat.lib().omni_qkv_prepare(
         nat.ptr(qkv), nat.c_int(qkv.stride(0)), nat.c_int(hq), nat.c_int(hkv), nat.c_int(dk), nat.c_int(dv), nat.ptr(q_w), nat.ptr(k_w),
         nat.c_float(eps), nat.ptr(cos_sin), nat.c_int(rot), nat.c_int(int(pairs)), nat.ptr(positions), nat.ptr(slots), nat.ptr(mix),
-        nat.ptr(v_first if mix is not None else None), nat.c_int(v_first.stride(0) if mix is not None else 0), nat.ptr(k_cache),
-        nat.ptr(v_cache), nat.c_int(T), nat.c_int(_f32(qkv)), nat.stream())
+        nat.ptr(v_first if mix is not None else None), nat.c_int(v_first.stride(0) if mix is not None else 0), nat.c_int(int(v_norm)),
+        nat.ptr(k_cache), nat.ptr(v_cache), nat.c_int(T), nat.c_int(_f32(qkv)), nat.stream())
     nat.check_rc(rc, "omni_qkv_prepare")
 
 
 def latent_prepare(a, q_rank, kv0, kv_rank, rot, q_w, kv_w, eps, cos_sin, positions, slots, cache, latent_cols, q_cols, want_rows=False):
-    """``a`` rows: q_rank columns of the query latent, and from column ``kv0`` on kv_rank of the key/value latent | rot of the shared
-    key part.  Both latents are normed, the key part rotated; latent | key part (``latent_cols`` and the rest of the cache's
-    columns, zeros past the real sizes) are cached at ``slots``.  -> (query latent [T, q_cols], the cached rows or None)."""
+    """``a`` rows: q_rank columns of the query latent (0: there is none), and from column ``kv0`` on kv_rank of the key/value latent | rot
+    of the shared key part.  The latents are normed, the key part rotated; latent | key part (``latent_cols`` and the rest of the cache's
+    columns, zeros past the real sizes) are cached at ``slots``.  -> (query latent [T, q_cols] or None, the cached rows or None)."""
     T, D = a.shape[0], cache.shape[-1]
     if not a.is_cuda:
-        cq = torch.zeros(T, q_cols, dtype=a.dtype)
-        cq[:, :q_rank] = rms_ref(a[:, :q_rank].float(), q_w, eps).to(a.dtype)
+        cq = None
+        if q_rank:
+            cq = torch.zeros(T, q_cols, dtype=a.dtype)
+            cq[:, :q_rank] = rms_ref(a[:, :q_rank].float(), q_w, eps).to(a.dtype)
         rows = torch.zeros(T, D, dtype=a.dtype)
         rows[:, :kv_rank] = rms_ref(a[:, kv0:kv0 + kv_rank].float(), kv_w, eps).to(a.dtype)
         kr = _rotate_half_ref(a[:, None, kv0 + kv_rank:kv0 + kv_rank + rot].float(), cos_sin, positions, rot)
@@ -65,7 +71,7 @@ def latent_prepare(a, q_rank, kv0, kv_rank, rot, q_w, kv_w, eps, cos_sin, positi
         cache.view(-1, D)[slots[ok]] = rows[ok]
         return cq, rows if want_rows else None
     assert a.stride(1) == 1 and cache.is_contiguous() and cache.dtype == a.dtype
-    cq = torch.empty(T, q_cols, dtype=a.dtype, device=a.device)
+    cq = torch.empty(T, q_cols, dtype=a.dtype, device=a.device) if q_rank else None
     rows = torch.empty(T, D, dtype=a.dtype, device=a.device) if want_rows else None
     rc = nat.lib().omni_latent_prepare(
         nat.ptr(a), nat.c_int(a.stride(0)), nat.c_int(q_rank), nat.c_int(kv0), nat.c_int(kv_rank), nat.c_int(rot), nat.ptr(q_w),
@@ -112,18 +118,19 @@ def gather_pages(cache, block_table, requests, pos0, first, end, total, longest)
     return out
 
 
-def latent_attention(q, cache, latent_cols, *, positions, q_to_seq, slots, block_table, seq_lens, scale, window=0, gate=None, max_seq_len=0):
+def latent_attention(q, cache, latent_cols, *, positions, q_to_seq, slots, block_table, seq_lens, scale, window=0, gate=None, max_seq_len=0,
+                     sink=None):
     """Attention in latent space: q [T, H, D] (latent part | rotated part) against the cached rows [blocks, block, D] that the rows'
     requests (``q_to_seq``) hold, row t seeing the last ``window`` of its first ``seq_lens[t]``; values are the first ``latent_cols``
-    of the rows.  ``gate`` [T, H]: as in :func:`paged_attention`.  -> [T, H, latent_cols]."""
+    of the rows.  ``gate`` [T, H], ``sink`` [H]: as in :func:`paged_attention`.  -> [T, H, latent_cols]."""
     T, H, D = q.shape
     if q.is_cuda and q.dtype == torch.bfloat16 and (D, latent_cols) == (576, 512) and H <= 128 and (cache.shape[1] == 32 or cache.shape[1] % 64 == 0):
         from .attention import mla_decode
         return mla_decode(q, cache, block_table, seq_lens, scale, q_to_seq=q_to_seq, max_seq_len=max_seq_len, exact=True, window=window,
-                          gate=gate)
+                          gate=gate, sink=sink)
     kv = cache.unsqueeze(2)
     out = paged_attention(q, kv, kv[..., :latent_cols], positions=positions, q_to_seq=q_to_seq, slots=slots, block_table=block_table,
-                          seq_lens=seq_lens, scale=scale, window=window, gate=gate, max_seq_len=max_seq_len, rows_share=True)
+                          seq_lens=seq_lens, scale=scale, window=window, gate=gate, max_seq_len=max_seq_len, rows_share=True, sink=sink)
     return out.view(T, H, latent_cols)
 
 
@@ -132,7 +139,7 @@ def latent_prefill_fits(dtype, d1, d2, dv, scale) -> bool:
     return scale > 0 and dtype == torch.bfloat16 and (d1 + 63) // 64 + (d2 + 63) // 64 <= 3 and dv <= 128
 
 
-def latent_prefill(q, kv, k2, *, d1, dv, q_start, q_end, k_start, k_end, max_q, scale, window=0, gate=None, out=None):
+def latent_prefill(q, kv, k2, *, d1, dv, q_start, q_end, k_start, k_end, max_q, scale, window=0, gate=None, sink=None, out=None):
     """Attention over projected keys: q [T, H, d1 + d2], ``kv`` [K, H (d1 + dv)] = per head keys | values, ``k2`` [K, d2] key columns
     of all heads.  Request b has query rows q_start[b]:q_end[b] and key rows k_start[b]:k_end[b], whose last ones are its queries'.
     Writes those rows of ``out`` [T, H dv]."""
@@ -145,7 +152,7 @@ def latent_prefill(q, kv, k2, *, d1, dv, q_start, q_end, k_start, k_end, max_q, 
         nat.ptr(q), nat.c_int64(T), nat.c_int(q.stride(0)), nat.ptr(kv), nat.c_int64(kv.shape[0]), nat.c_int(kv.stride(0)), nat.ptr(k2),
         nat.c_int(k2.stride(0)), nat.ptr(q_start), nat.ptr(q_end), nat.ptr(k_start), nat.ptr(k_end), nat.c_int(q_start.shape[0]),
         nat.c_int(max_q), nat.c_int(H), nat.c_int(d1), nat.c_int(d2), nat.c_int(dv), nat.c_int(window), nat.c_float(scale),
-        nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0), nat.ptr(out), nat.c_int(out.stride(0)),
+        nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0), nat.ptr(sink), nat.ptr(out), nat.c_int(out.stride(0)),
         nat.ptr(nat.status_buffer(q.device)), nat.stream())
     nat.check_rc(rc, "omni_fmha_latent")
     return out

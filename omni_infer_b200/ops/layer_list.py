@@ -175,7 +175,7 @@ def first_visible(pos: int, window: int, chunk: int) -> int:
 
 
 def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out, keep_first=0,
-                        chunk=0, softcap=0.0, slopes=None, gate=None):
+                        chunk=0, softcap=0.0, slopes=None, gate=None, log_bias=None):
     hq, dk = q.shape[1], q.shape[2]
     bs, hkv, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     kf, vf = k_cache.flatten(0, 1), v_cache.flatten(0, 1)
@@ -195,11 +195,13 @@ def paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_t
             s = softcap * torch.tanh(s / softcap)
         if slopes is not None:
             s = s - slopes[:, None] * (p - pos)
+        if log_bias is not None:
+            s = s - log_bias[0][:, None] * torch.log1p(log_bias[1][:, None] * (p - pos))
         if sink is not None:
             s = torch.cat([s, sink[:, None]], 1)
         o = torch.einsum("hl,lhd->hd", torch.softmax(s, -1)[:, :len(pos)], v) * out_scale
         if gate is not None:
-            o = o * torch.sigmoid(gate[t].float())[:, None]
+            o = o * torch.sigmoid(gate[t].float()).view(hq, -1)
         out[t, :hq * dv] = o.reshape(-1).to(out.dtype)
     return out
 
@@ -213,12 +215,12 @@ def _splits(ctas: int, keys: int) -> int:
 
 def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_table, seq_lens, scale, window=0, cu_q=None,
                     max_q=1, max_seq_len=0, sink=None, out_scale=1.0, out=None, any_shape=False, keep_first=0, chunk=0, softcap=0.0,
-                    slopes=None, gate=None, rows_share=False):
+                    slopes=None, gate=None, rows_share=False, log_bias=None):
     """q [T, hq, dk] (rows of any pitch) against the cached keys of the rows' requests, each row seeing the ``window``
     positions up to its own (0: all of them), only those of its own ``chunk`` of positions (0: no chunks), and the ``keep_first``
-    first ones in any case.  A score is ``softcap tanh(q k scale / softcap) - slopes[head] distance`` (each part optional).  ``sink``
-    [hq] fp32: exp(sink) is one more term of the head's softmax denominator; ``out_scale`` multiplies the result, and so does the
-    sigmoid of ``gate`` [T, hq].  Returns [T, pad8(hq * dv)], or writes the first columns of ``out``.  The value cache may be a
+    first ones in any case.  A score is ``softcap tanh(q k scale / softcap) - slopes[head] distance``, less ``r1[head]
+    ln(1 + r2[head] distance)`` with ``log_bias`` = (r1, r2) (each part optional).  ``sink`` [hq] fp32: exp(sink) is one more term of
+    the head's softmax denominator; ``out_scale`` multiplies the result, and so does the sigmoid of ``gate``, [T, hq] or [T, hq * dv].  Returns [T, pad8(hq * dv)], or writes the first columns of ``out``.  The value cache may be a
     column slice of the key cache (one key/value head).
 
     bf16 portions of prompts run on tcgen05 (``omni_fmha_paged``), bf16 single tokens on the split-KV decode kernel; fp32
@@ -232,22 +234,26 @@ def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_ta
     ld = out.stride(0)
     if not q.is_cuda:
         return paged_attention_ref(q, k_cache, v_cache, positions, q_to_seq, slots, block_table, scale, window, sink, out_scale, out,
-                                   keep_first, chunk, softcap, slopes, gate)
+                                   keep_first, chunk, softcap, slopes, gate, log_bias)
     assert q.stride(2) == 1 and q.stride(1) == dk and k_cache.dtype == q.dtype and block_table.stride(1) == 1
     k_row, v_row = k_cache.stride(1), v_cache.stride(1)
-    assert k_cache.stride(0) == bs * k_row and v_cache.stride(0) == bs * v_row and (gate is None or gate.stride(1) == 1)
+    assert k_cache.stride(0) == bs * k_row and v_cache.stride(0) == bs * v_row
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape[1] in (hq, hq * dv))
+    r1, r2 = log_bias if log_bias is not None else (None, None)
     packed = k_row == hkv * dk and v_row == hkv * dv
     f32 = _f32(q)
     lib = nat.lib()
-    gate_args = (nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0))
-    mod = (nat.c_int(window), nat.c_int(chunk), nat.c_int(keep_first), nat.c_float(scale), nat.c_float(softcap), nat.ptr(slopes), nat.ptr(sink))
+    gate_args = (nat.ptr(gate), nat.c_int(gate.stride(0) if gate is not None else 0), nat.c_int(gate.shape[1] // hq if gate is not None else 1))
+    mod = (nat.c_int(window), nat.c_int(chunk), nat.c_int(keep_first), nat.c_float(scale), nat.c_float(softcap), nat.ptr(slopes), nat.ptr(r1),
+           nat.ptr(r2), nat.ptr(sink))
     tc = not any_shape and not f32 and ld % 8 == 0 and out.data_ptr() % 16 == 0 and dk % 8 == 0 and dv % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
-    if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0 and packed and gate is None and scale > 0:
+    vec_gate = gate is None or (gate.shape[1] == hq * dv and gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)
+    if tc and cu_q is not None and dk <= 192 and dv <= 128 and bs % 64 == 0 and packed and vec_gate and scale > 0:
         rc = lib.omni_fmha_paged(
             nat.ptr(q), nat.c_int64(T), nat.c_int(q.stride(0)), nat.ptr(k_cache), nat.ptr(v_cache),
             nat.c_int64(k_cache.shape[0] * bs), nat.ptr(cu_q), nat.ptr(seq_lens), nat.ptr(block_table),
             nat.c_int(block_table.stride(0)), nat.c_int(cu_q.shape[0] - 1), nat.c_int(max_q), nat.c_int(hq), nat.c_int(hkv),
-            nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), *mod, nat.c_float(out_scale), nat.ptr(out), nat.c_int(ld),
+            nat.c_int(dk), nat.c_int(dv), nat.c_int(bs), *mod, *gate_args[:2], nat.c_float(out_scale), nat.ptr(out), nat.c_int(ld),
             nat.ptr(nat.status_buffer(q.device)), nat.stream())
         nat.check_rc(rc, "omni_fmha_paged")
         return out

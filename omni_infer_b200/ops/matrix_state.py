@@ -1,7 +1,8 @@
-"""Mixers whose state is a matrix per head, between their projections: the matrix memory of xLSTM (mLSTM) and WKV.
+"""Mixers whose state is a matrix per head, between their projections: the matrix memory of xLSTM (mLSTM), WKV and gated linear
+attention (GLA).
 
 CUDA tensors run ``csrc/kernels/matrix_state.cu`` (gates, token by token, norm), ``ssd_sm100.cu`` (mLSTM portions of prompts on
-tcgen05) and ``wkv_chunk.cu`` (WKV portions); CPU tensors the fp32 references here.  Ragged batches as in :mod:`.layer_list`.
+tcgen05) and ``wkv_chunk.cu`` (WKV and GLA portions); CPU tensors the fp32 references here.  Ragged batches as in :mod:`.layer_list`.
 
 State: [slots, H, P, N] fp32 (N key size, P value size; the mLSTM's has one more row, its normaliser) and for the mLSTM
 m [slots, H], the running maximum of its log gates.  A request that starts at position 0 starts from zeros."""
@@ -71,12 +72,12 @@ def _tma(*ts) -> bool:
     return all(t.stride(1) == 1 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in ts)
 
 
-def _rows(kind, a, a_scale, b, v, gates, z, w0, u, state, out, H, P, N, positions, state_slots, cu_q, max_rows):
+def _rows(kind, a, a_scale, b, v, gates, z, w0, u, state, out, H, P, N, positions, state_slots, cu_q, max_rows, inv_tau=0.0):
     B = a.shape[0] if cu_q is None else cu_q.shape[0] - 1
     rc = nat.lib().omni_state_rows(
         nat.c_int(kind), nat.ptr(a), nat.c_int(a.stride(0)), nat.c_float(a_scale), nat.ptr(b), nat.c_int(b.stride(0)), nat.ptr(v),
         nat.c_int(v.stride(0)), nat.ptr(gates.keep_add if gates else None), nat.ptr(gates.den if gates else None), nat.ptr(z),
-        nat.c_int(z.stride(0) if z is not None else 0), nat.ptr(w0), nat.ptr(u), nat.ptr(state), nat.ptr(cu_q), nat.ptr(positions),
+        nat.c_int(z.stride(0) if z is not None else 0), nat.ptr(w0), nat.ptr(u), nat.c_float(inv_tau), nat.ptr(state), nat.ptr(cu_q), nat.ptr(positions),
         nat.ptr(state_slots), nat.c_int(B), nat.ptr(out), nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N),
         nat.c_int(_f32(a)), nat.c_int(max_rows), nat.stream())
     nat.check_rc(rc, "omni_state_rows")
@@ -148,6 +149,46 @@ def wkv_scan(r, k, v, z, w0, u, state, *, H, N, positions, state_slots, cu_q=Non
             return out
         max_rows = CHUNK_MIN_ROWS - 1
     _rows(1, r, 1.0, k, v, None, z, w0, u, state, out, H, N, N, positions, state_slots, cu_q, max_rows)
+    return out
+
+
+def gla_chunked(dtype, N: int, P: int) -> bool:
+    """Do portions of prompts run in chunks at these sizes?"""
+    return dtype == torch.bfloat16 and N % 8 == 0 and N <= 256 and P % 8 == 0
+
+
+def gla_scan(q, k, v, z, bias, inv_tau, state, *, H, P, N, positions, state_slots, cu_q=None, min_q=1, max_q=0, by_rows=False):
+    """S <- diag(a) S + k v^T, o = S^T q N^-1/2 with a = sigmoid(z + bias)^inv_tau per head and key channel; q, k [T, H N],
+    v [T, H P], z fp32 [T, >= H N] (rows of any pitch) -> o [T, H P]."""
+    T, scale = q.shape[0], N ** -0.5
+    out = torch.empty(T, H * P, dtype=q.dtype, device=q.device)
+    if not q.is_cuda:
+        a = torch.exp(F.logsigmoid(z[:, :H * N].float() + bias) * inv_tau).view(T, H, 1, N)
+        for r, first, end in _segments(cu_q, T):
+            slot = int(state_slots[r])
+            if slot < 0:
+                out[first:end] = 0
+                continue
+            S = state[slot].clone() if int(positions[first]) > 0 else torch.zeros_like(state[slot])      # [H, P, N]
+            for t in range(first, end):
+                S = a[t] * S + v[t].float().view(H, P, 1) * k[t].float().view(H, 1, N)
+                out[t] = torch.einsum("hpn,hn->hp", S, q[t].float().view(H, N) * scale).reshape(-1).to(out.dtype)
+            state[slot] = S
+        return out
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and state.dtype == torch.float32
+    max_rows = 0
+    if cu_q is not None and not by_rows and gla_chunked(q.dtype, N, P) and _tma(v):
+        rc = nat.lib().omni_gla_chunks(
+            nat.ptr(q), nat.c_int(q.stride(0)), nat.ptr(k), nat.c_int(k.stride(0)), nat.ptr(v), nat.c_int(v.stride(0)), nat.ptr(z),
+            nat.c_int(z.stride(0)), nat.ptr(bias), nat.c_float(scale), nat.c_float(inv_tau), nat.ptr(state), nat.ptr(cu_q),
+            nat.ptr(positions), nat.ptr(state_slots), nat.c_int(cu_q.shape[0] - 1), nat.c_int(max_q or T), nat.ptr(out),
+            nat.c_int(out.stride(0)), nat.c_int(H), nat.c_int(P), nat.c_int(N), nat.c_int(CHUNK_MIN_ROWS),
+            nat.ptr(nat.status_buffer(q.device)), nat.stream())
+        nat.check_rc(rc, "omni_gla_chunks")
+        if min_q >= CHUNK_MIN_ROWS:
+            return out
+        max_rows = CHUNK_MIN_ROWS - 1
+    _rows(2, q, scale, k, v, None, z, bias, None, state, out, H, P, N, positions, state_slots, cu_q, max_rows, inv_tau)
     return out
 
 
