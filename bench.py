@@ -46,10 +46,11 @@ def parse():
                          "(input + output / 2), 0 = time right after the prefill")
     ap.add_argument("--layer-list", default=None, 
                     choices=["kernels", "model", "all", "fimudra-kernels", "fimudra-model", "fimudra", "tenotar-kernels", "tenotar-model",
-                             "tenotar"],
+                             "tenotar", "zusotar-kernels", "zusotar-model", "zusotar"],
                     help="instead of the headline: layer-list models (windowed attention + Mamba-2; fimudra: attention beside a "
-                         "matrix memory, WKV, expert mixtures; tenotar: latent, windowed and chunked attention, expert mixtures) "
-                         "beside the closest models at equal sizes, per kernel and whole, one JSON line each")
+                         "matrix memory, WKV, expert mixtures; tenotar: latent, windowed and chunked attention, expert mixtures; "
+                         "zusotar: latent, windowed and gated linear attention, averages over depth) beside the closest models at equal sizes, "
+                         "per kernel and whole, one JSON line each")
     ap.add_argument("--no-breakdown", action="store_true", help="skip the untimed per-module timing step")
     ap.add_argument("--no-nccl-arm", action="store_true", help="skip the untimed NCCL all-to-all comparison steps (N > 1)")
     return ap.parse_args()
@@ -212,6 +213,8 @@ def main():
             from benchmarks.fimudra_bench import main as layer_list_main
         elif args.layer_list.startswith("tenotar"):
             from benchmarks.tenotar_bench import main as layer_list_main
+        elif args.layer_list.startswith("zusotar"):
+            from benchmarks.zusotar_bench import main as layer_list_main
         else:
             from benchmarks.layer_list_bench import main as layer_list_main
         return layer_list_main(args.layer_list)

@@ -183,69 +183,81 @@ def kernels(out) -> None:
             torch.cuda.empty_cache()
 
 
-def models(out, steps=20, warmup=5) -> None:
+def mla_like(c, **kw):
+    """The MLA expert model (DeepSeek-V3 architecture) at the sizes ``c``."""
+    from omni_infer_b200.models.config import ModelConfig
+    return ModelConfig(architecture="DeepseekV3ForCausalLM", name="mla-moe", num_key_value_heads=c["heads"], q_lora_rank=c.get("q_rank", 0),
+                       kv_lora_rank=c["kv_rank"], qk_nope_head_dim=c["dim"], qk_rope_head_dim=c["rot_dim"], v_head_dim=c["dim"],
+                       n_shared_experts=c["shared_ff"] // c["expert_ff"], first_k_dense_replace=1, **_common(c), **kw)
+
+
+def qwen_like(c):
+    """The GQA expert model (Qwen3-MoE architecture) at the sizes ``c``."""
+    from omni_infer_b200.models.config import ModelConfig
+    return ModelConfig(architecture="Qwen3MoeForCausalLM", name="qwen3-moe", num_key_value_heads=c["kv_heads"], head_dim=c["dim"],
+                       use_mla=False, n_shared_experts=0, first_k_dense_replace=0, qk_norm=True, rope_theta=1e6, **_common(c))
+
+
+def _common(c):
+    return dict(vocab_size=c["vocab"], hidden_size=c["width"], num_hidden_layers=c["layers"], num_attention_heads=c["heads"],
+                intermediate_size=c["ff"], moe_intermediate_size=c["expert_ff"], n_routed_experts=c["experts"],
+                num_experts_per_tok=c["top"], scoring_func="softmax", topk_method="greedy", norm_topk_prob=True,
+                max_position_embeddings=9216)
+
+
+def models(out) -> None:
+    from omni_infer_b200.models.config import tenotar
+    for size, c in SIZES.items():
+        for name, mc in (("tenotar", tenotar(**c)), ("mla-moe", mla_like(c)), ("qwen3-moe", qwen_like(c))):
+            throughput(out, size, c, name, mc)
+
+
+def throughput(out, size, c, name, mc, steps=20, warmup=5) -> None:
+    """Prefill and decode of a whole model through the engine."""
     import torch
 
     from omni_infer_b200.engine.engine_core import EngineConfig, EngineCore
     from omni_infer_b200.engine.request import SamplingParams
-    from omni_infer_b200.models.config import ModelConfig, tenotar
     from omni_infer_b200.ops import _native as nat
 
-    def common(c):
-        return dict(vocab_size=c["vocab"], hidden_size=c["width"], num_hidden_layers=c["layers"], num_attention_heads=c["heads"],
-                    intermediate_size=c["ff"], moe_intermediate_size=c["expert_ff"], n_routed_experts=c["experts"],
-                    num_experts_per_tok=c["top"], scoring_func="softmax", topk_method="greedy", norm_topk_prob=True,
-                    max_position_embeddings=9216)
-
-    def mla(c):
-        return ModelConfig(architecture="DeepseekV3ForCausalLM", name="mla-moe", num_key_value_heads=c["heads"], q_lora_rank=c["q_rank"],
-                           kv_lora_rank=c["kv_rank"], qk_nope_head_dim=c["dim"], qk_rope_head_dim=c["rot_dim"], v_head_dim=c["dim"],
-                           n_shared_experts=c["shared_ff"] // c["expert_ff"], first_k_dense_replace=1, **common(c))
-
-    def qwen(c):
-        return ModelConfig(architecture="Qwen3MoeForCausalLM", name="qwen3-moe", num_key_value_heads=c["kv_heads"], head_dim=c["dim"],
-                           use_mla=False, n_shared_experts=0, first_k_dense_replace=0, qk_norm=True, rope_theta=1e6, **common(c))
-
-    for size, c in SIZES.items():
-        for name, mc in (("tenotar", tenotar(**c)), ("mla-moe", mla(c)), ("qwen3-moe", qwen(c))):
-            for B, L in ((64, 1024), (256, 1024)):
-                per = L + steps + warmup + 16
-                eng = EngineCore(EngineConfig(model=name, block_size=128, num_kv_blocks=B * ((per + 127) // 128 + 1) + 1, max_num_seqs=B,
-                                              max_num_batched_tokens=8192, max_model_len=per + 128, decode_gear_list=[B]), model_cfg=mc)
-                g = torch.Generator().manual_seed(1)
-                prompts = torch.randint(0, c["vocab"], (B, L), generator=g)
-                sp = SamplingParams(max_tokens=10 ** 6, ignore_eos=True)
-                for p in prompts:
-                    eng.add_request(p.tolist(), sp)
-                ts = []
-                while eng.scheduler.num_waiting:
-                    n0 = eng.scheduler.stats["scheduled_prefill_tokens"]
-                    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                    torch.cuda.synchronize()
-                    a.record()
-                    eng.step()
-                    b.record()
-                    torch.cuda.synchronize()
-                    ts.append((eng.scheduler.stats["scheduled_prefill_tokens"] - n0, a.elapsed_time(b)))
-                ts = ts[2:] if len(ts) > 4 else ts[1:]
-                n_tok, ms = sum(t[0] for t in ts), sum(t[1] for t in ts)
-                for _ in range(warmup):
-                    eng.step()
-                torch.cuda.synchronize()
-                a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                a.record()
-                for _ in range(steps):
-                    eng.step()
-                b.record()
-                torch.cuda.synchronize()
-                nat.check_status()
-                dec = a.elapsed_time(b) / steps
-                nparam = sum(p.numel() for p in eng.worker.runner.model.parameters())
-                out({"size": size, "model": name, "layers": c["layers"], "params_M": round(nparam / 1e6), "batch": B, "prompt": L,
-                     "prefill_tok_s": round(n_tok / ms * 1e3), "decode_ms_per_step": round(dec, 3), "decode_tok_s": round(B / dec * 1e3),
-                     "cuda_graph": eng.worker.runner.graphs is not None})
-                del eng
-                torch.cuda.empty_cache()
+    for B, L in ((64, 1024), (256, 1024)):
+        per = L + steps + warmup + 16
+        eng = EngineCore(EngineConfig(model=name, block_size=128, num_kv_blocks=B * ((per + 127) // 128 + 1) + 1, max_num_seqs=B,
+                                      max_num_batched_tokens=8192, max_model_len=per + 128, decode_gear_list=[B]), model_cfg=mc)
+        g = torch.Generator().manual_seed(1)
+        prompts = torch.randint(0, c["vocab"], (B, L), generator=g)
+        sp = SamplingParams(max_tokens=10 ** 6, ignore_eos=True)
+        for p in prompts:
+            eng.add_request(p.tolist(), sp)
+        ts = []
+        while eng.scheduler.num_waiting:
+            n0 = eng.scheduler.stats["scheduled_prefill_tokens"]
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            a.record()
+            eng.step()
+            b.record()
+            torch.cuda.synchronize()
+            ts.append((eng.scheduler.stats["scheduled_prefill_tokens"] - n0, a.elapsed_time(b)))
+        ts = ts[2:] if len(ts) > 4 else ts[1:]
+        n_tok, ms = sum(t[0] for t in ts), sum(t[1] for t in ts)
+        for _ in range(warmup):
+            eng.step()
+        torch.cuda.synchronize()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        for _ in range(steps):
+            eng.step()
+        b.record()
+        torch.cuda.synchronize()
+        nat.check_status()
+        dec = a.elapsed_time(b) / steps
+        nparam = sum(p.numel() for p in eng.worker.runner.model.parameters())
+        out({"size": size, "model": name, "layers": c["layers"], "params_M": round(nparam / 1e6), "batch": B, "prompt": L,
+             "prefill_tok_s": round(n_tok / ms * 1e3), "decode_ms_per_step": round(dec, 3), "decode_tok_s": round(B / dec * 1e3),
+             "cuda_graph": eng.worker.runner.graphs is not None})
+        del eng
+        torch.cuda.empty_cache()
 
 
 def main(which: str) -> int:

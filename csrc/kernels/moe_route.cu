@@ -103,7 +103,7 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const RouterParams p) 
         const float v = sel[lane * gs + j];
         if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
       }
-      gscore = p.group_mode == 1 ? b1 + b2 : b1;
+      gscore = p.group_mode == 1 && gs > 1 ? b1 + b2 : b1;
     }
     unsigned keep = 0;
     for (int r = 0; r < p.topk_group; ++r) {

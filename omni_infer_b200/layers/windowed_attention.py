@@ -42,6 +42,8 @@ class WindowedAttention(nn.Module):
         self.ones, self.out_bias = s.bias, f32(hidden) if s.bias else None       # the output's bias is added with the residual
         self.conv_weight = f32(s.conv, self.proj_rows) if s.conv else None       # taps first: channels are contiguous
         self.r1, self.r2 = (f32(s.heads), f32(s.heads)) if s.log_bias else (None, None)
+        if s.log_bias:
+            self.r1.init_value, self.r2.init_value = 0.5, 0.1
         self.vmix = f32(1) if s.v_mix else None
         if s.v_mix:
             self.vmix.init_value = 0.5

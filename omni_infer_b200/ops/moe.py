@@ -26,7 +26,7 @@ def router_topk_ref(logits, top_k, *, mode="softmax", bias=None, n_group=1, topk
         sel = scores + bias.float() if bias is not None else scores.clone()
         if n_group > 1:
             g = sel.view(T, n_group, E // n_group)
-            gs = g.topk(2, dim=-1).values.sum(-1) if group_mode == "top2sum" else g.max(-1).values
+            gs = g.topk(min(2, g.shape[-1]), dim=-1).values.sum(-1) if group_mode == "top2sum" else g.max(-1).values
             keep = torch.zeros_like(gs, dtype=torch.bool)
             keep.scatter_(1, gs.topk(topk_group, dim=-1).indices, True)
             sel = sel.masked_fill(~keep.unsqueeze(-1).expand(T, n_group, E // n_group).reshape(T, E), float("-inf"))

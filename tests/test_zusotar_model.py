@@ -1,0 +1,404 @@
+"""The Zusotar design through the engine - weight loading, pages and state slots, ragged and decode steps, scheduler, sampling,
+trace replay - against the plain whole-sequence implementation."""
+import copy
+import functools
+import io
+import json
+
+import pytest
+import torch
+
+import zusotar_cases as cases
+import zusotar_oracle as oracle
+from layer_list_cases import row_errors, tokens, write_model
+from omni_infer_b200.engine.engine_core import LLM, EngineConfig, EngineCore
+from omni_infer_b200.engine.request import SamplingParams
+from omni_infer_b200.engine.trace_replay import TraceReplay
+from omni_infer_b200.models.config import ModelConfig, get_config
+from test_layer_list_model import RUNS, portions, run
+from zusotar_cases import CONFIGS, expected
+
+# Most rows / all rows / the typical row.  In 16 bits a close choice of experts may fall the other way, which moves that row and a
+# little those that attend to it: all rows are held to rounding where every expert is chosen.
+TOL = {"float32": (1e-5, 3e-5, 5e-6), "bfloat16": (0.08, 0.12, 0.03)}
+CLOSE_CHOICE = (0.12, None, 0.045)
+EXACT_CHOICE = ("odd", "wide", "deep")
+
+
+@pytest.fixture(autouse=True)
+def _one_thread():
+    n = torch.get_num_threads()
+    torch.set_num_threads(1)
+    yield
+    torch.set_num_threads(n)
+
+
+def build(cfg, w, device, dtype, blocks=24, block_size=64, **kw):
+    mc = ModelConfig.from_hf_dict(cfg)
+    mc.dtype = dtype
+    kw.setdefault("max_num_seqs", 4)
+    kw.setdefault("max_model_len", 512)
+    return EngineCore(EngineConfig(model="x", device=device, block_size=block_size, num_kv_blocks=blocks, **kw), model_cfg=mc,
+                      weights=list(w.items()))
+
+
+def engine(name, device, dtype, seed=0, **kw):
+    return build(CONFIGS[name], cases.weights(CONFIGS[name], seed), device, dtype, **kw)
+
+
+def check(got, want, dtype, exact_choice=True):
+    e = row_errors(got, want)
+    most, every, typical = TOL[dtype] if exact_choice or dtype == "float32" else CLOSE_CHOICE
+    assert float(e.median()) < typical and float(e.quantile(0.7)) < most, (float(e.max()), float(e.median()))
+    if exact_choice or dtype == "float32":
+        assert float(e.max()) < every, (float(e.max()), int(e.argmax()))
+
+
+# ----------------------------------------------------------------------------- the same logits however they are computed
+@pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("name", CONFIGS)
+def test_cuts_of_one_sequence(name, device, dtype):
+    """Whole prompt; one token at a time from the start; a prompt and long decoding; portions down to two tokens."""
+    n = 150
+    toks = tokens(n, CONFIGS[name]["vocab"], 1)
+    eng = engine(name, device, dtype)
+    for sizes in ([n], [1], [100] + [1] * 50, [2, 3], [65, 1, 64, 2], [63, 17], [29, 8, 9, 1]):
+        got = run(eng, {"a": toks}, [[("a", m)] for m in portions(n, sizes)])["a"]
+        check(got, expected(name, 0, toks), dtype, name in EXACT_CHOICE)
+    assert eng.kv.num_free_blocks == 23 and len(eng.kv.free_state_slots) == 4
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("name", CONFIGS)
+def test_batches_of_unequal_requests(name, device, dtype):
+    """Portions beside single tokens, requests that pause and come back, pages and slots used again; each as if it were alone."""
+    V = CONFIGS[name]["vocab"]
+    seqs = {"a": tokens(140, V, 1), "b": tokens(33, V, 2), "c": tokens(1, V, 3), "d": tokens(90, V, 4), "e": tokens(67, V, 5)}
+    plan = [[("a", 64), ("b", 1), ("c", 1), ("d", 30)], [("b", 1), ("a", 2)], [("d", 2), ("b", 17)], [("a", 1), ("b", 1), ("d", 1), ("e", 1)],
+            [("e", 3), ("b", 13), ("a", 40)], [("e", 40), ("d", 1), ("a", 3)], [("a", 1), ("d", 1), ("e", 1)], [("a", 29), ("d", 55), ("e", 1)],
+            [("e", 21), ("c", 1)], [("b", 33), ("c", 1)]]
+    eng = engine(name, device, dtype, blocks=10)
+    got = run(eng, seqs, plan)
+    for i, t in seqs.items():
+        for k in range(0, len(got[i]), len(t)):
+            if len(t) > 1 or dtype == "float32":
+                check(got[i][k:k + len(t)], expected(name, 0, t), dtype, name in EXACT_CHOICE)
+    assert eng.kv.num_free_blocks == 9
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+def test_other_page_sizes(device, dtype):
+    """Long sequences cut at and around page and window edges; pages of 16 and of 128 tokens."""
+    toks = tokens(330, CONFIGS["wide"]["vocab"], 7)
+    for bs, sizes in ((16, [330]), (64, [128, 1, 127, 74]), (128, [129, 1, 1, 126, 73]), (64, [255, 2, 73])):
+        eng = engine("wide", device, dtype, block_size=bs, blocks=24 if bs > 16 else 40)
+        got = run(eng, {"a": toks}, [[("a", m)] for m in portions(330, sizes)])["a"]
+        check(got, expected("wide", 0, toks), dtype)
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("kind", ["latent", "window", "gla"])
+def test_stacks_of_one_kind(device, dtype, kind):
+    """The pool sized by the engine; without pages or without state slots; the last layer without a feed-forward."""
+    make = {"latent": cases.latent, "window": cases.window, "gla": cases.gla}[kind]
+    cfg = cases.config([make(mlp=cases.all_of()), make(mlp=cases.dense()), make(mlp=None)])
+    w = cases.weights(cfg, 8)
+    mc = ModelConfig.from_hf_dict(cfg)
+    mc.dtype = dtype
+    eng = EngineCore(EngineConfig(model="x", device=device, block_size=64, max_num_seqs=2, max_model_len=256), model_cfg=mc, weights=list(w.items()))
+    assert mc.has_recurrent_state == (kind == "gla")
+    toks = tokens(90, 97, 3)
+    got = run(eng, {"a": toks}, [[("a", m)] for m in (40, 2, 1, 1, 46)])["a"]
+    check(got, oracle.forward(cfg, w, toks), dtype)
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+def test_one_layer_alone(device, dtype):
+    """There is no earlier layer to average with but the embedding output."""
+    cfg = cases.config([cases.window(mlp=None)])
+    w, toks = cases.weights(cfg, 2), tokens(50, 97, 1)
+    got = run(build(cfg, w, device, dtype), {"a": toks}, [[("a", m)] for m in (30, 1, 19)])["a"]
+    check(got, oracle.forward(cfg, w, toks), dtype)
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+def test_residual_after_every_layer(device, dtype):
+    name = "plain" if dtype == "float32" else "wide"
+    cfg = CONFIGS[name]
+    eng, seen, toks = engine(name, device, dtype), [], tokens(23, cfg["vocab"], 2)
+    from omni_infer_b200.models import layer_list as mod
+    step = mod.both_norms_step
+
+    def spy(x_in, x_out, *a, **k):
+        h = step(x_in, x_out, *a, **k)
+        if k.get("average") is not None:
+            seen.append(x_out[:, :cfg["width"]].double().cpu())
+        return h
+
+    mod.both_norms_step = spy
+    try:
+        run(eng, {"a": toks}, [[("a", len(toks))]])
+    finally:
+        mod.both_norms_step = step
+    _, want = oracle.forward(cfg, cases.weights(cfg), toks, True)
+    assert len(seen) == len(want)
+    for got, w in zip(seen, want):
+        err = (got - w).pow(2).mean().sqrt() / w.pow(2).mean().sqrt()
+        assert float(err) < (5e-6 if dtype == "float32" else 0.02)
+
+
+# ----------------------------------------------------------------------------- far tokens, edges, first tokens
+def sharp(kind, **kw):
+    """A one-layer model whose queries look for token 9 alone: where it lies shows in the logits."""
+    make = {"latent": cases.latent, "window": cases.window, "gla": cases.gla}[kind]
+    cfg = cases.config([make(mlp=None, **kw)], width=32, vocab=16, mult=1.0)
+    w = cases.weights(cfg, 3)
+    w["embed"][:, 0], w["embed"][:, 5] = 2.0, 0.0
+    w["pos"].mul_(0.02)
+    w["pos"][:, 0] = w["pos"][:, 5] = 0.0
+    w["embed"][9, 5] = 4.0
+    w["l0.norm1"].zero_()
+    w["l0.norm1"][5] = 1.0
+    p, m = "l0.mix.", cfg["layers"][0]["mixer"]
+    if kind == "latent":
+        w[p + "q"].zero_()
+        w[p + "q"].view(m["heads"], m["dim"] + m["rot_dim"], 32)[:, 0, 0] = 1.2
+        w[p + "dkv"].mul_(0.3)
+        w[p + "dkv"][0] = 0.0
+        w[p + "dkv"][0, 5] = 2.0
+        w[p + "dkv.norm"].fill_(1.0)
+        w[p + "uk"].mul_(0.1)
+        w[p + "uk"].view(m["heads"], m["dim"], -1)[:, 0, 0] = 5.0
+        w[p + "sink"].fill_(3.0)
+    elif kind == "window":
+        w[p + "q"].zero_()
+        w[p + "k"].mul_(0.05)
+        w[p + "q"].view(-1, m["dim"], 32)[:, m["dim"] - 1, 0] = 3.0
+        w[p + "k"].view(-1, m["dim"], 32)[:, m["dim"] - 1, 5] = 3.0
+    else:       # one slow channel that only token 9 writes
+        n = m["dim"]
+        for c in "qk":
+            w[p + c].view(-1, n, 32)[:, 0] = 0.0
+        w[p + "q"].view(-1, n, 32)[:, 0, 0] = 3.0
+        w[p + "k"].view(-1, n, 32)[:, 0, 5] = 3.0
+        w[p + "a2"].view(-1, n, w[p + "a2"].shape[1])[:, 0] = 0.0
+        w[p + "a2.b"].view(-1, n)[:, 0] = 7.0
+    return cfg, w
+
+
+FAR = [("latent", dict(), [(0, True), (63, True), (64, True), (200, True)]), ("latent", dict(heads=2, kv_rank=300, rot=16), [(0, True), (127, True)]),
+       ("window", dict(size=70), [(227, True), (226, False), (0, False)]), ("window", dict(size=64), [(233, True), (232, False)]),
+       ("window", dict(size=128), [(169, True), (168, False)]), ("gla", dict(tau=16.0), [(0, True), (150, True)]), ("gla", dict(dim=7, tau=16.0), [(3, True)])]
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("decode", [False, True], ids=["prompt", "decoded"])
+@pytest.mark.parametrize("case", range(len(FAR)))
+def test_a_rare_token_far_back_and_at_the_edges(device, dtype, decode, case):
+    """The first token, page edges, just inside the window: it decides the last row; just outside it changes nothing."""
+    kind, kw, places = FAR[case]
+    cfg, w = sharp(kind, **kw)
+    eng = build(cfg, w, device, dtype, blocks=8, max_num_seqs=2)
+    n = 297
+    base = [t % 8 for t in tokens(n, 16, 4)]
+    plain = oracle.forward(cfg, w, base)[-1:]
+    for at, seen in places:
+        toks = list(base)
+        toks[at] = 9
+        got = run(eng, {"a": toks}, [[("a", n - 2)], [("a", 1)], [("a", 1)]] if decode else [[("a", 100)], [("a", n - 100)]])["a"]
+        want = oracle.forward(cfg, w, toks)
+        assert float(row_errors(got, want).max()) < (2e-5 if dtype == "float32" else 0.08)
+        moved = float(row_errors(plain, want[-1:])[0])
+        assert moved > 0.25 if seen else moved < 0.02, ("the case does not show the token", moved)
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+def test_sinks_positions_and_averages_show(device, dtype):
+    """Each of them changed in the weights changes the logits as in the plain implementation."""
+    name = "deep"
+    cfg, toks = CONFIGS[name], tokens(60, CONFIGS[name]["vocab"], 5)
+    base = expected(name, 0, toks)
+    for key, change in (("l0.mix.sink", lambda v: v + 4), ("pos", lambda v: -v), ("l1.dwa", lambda v: v.flip(0)), ("l2.norm1b", lambda v: v + 1)):
+        w = cases.weights(cfg)
+        w[key] = change(w[key])
+        want = oracle.forward(cfg, w, toks)
+        assert float(row_errors(base, want).median()) > 0.15, key
+        check(run(build(cfg, w, device, dtype), {"a": toks}, [[("a", 40)], [("a", 1)], [("a", 19)]])["a"], want, dtype)
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+def test_a_fresh_request_starts_from_an_empty_state(device, dtype):
+    cfg = cases.config([cases.gla(tau=16.0, mlp=None)], width=32, vocab=16)
+    w = cases.weights(cfg, 5)
+    eng = build(cfg, w, device, dtype, blocks=4, max_num_seqs=1)
+    a, b = tokens(20, 16, 1), tokens(7, 16, 2)
+    for toks, sizes in ((a, [20]), (b, [1]), (a, [2, 1]), (b, [3, 1, 3])):
+        got = run(eng, {"a": toks}, [[("a", m)] for m in portions(len(toks), sizes)])["a"]
+        assert float(row_errors(got, oracle.forward(cfg, w, toks)).max()) < (2e-5 if dtype == "float32" else 0.08)
+
+
+# ----------------------------------------------------------------------------- generation
+@functools.lru_cache(maxsize=None)
+def safe_greedy(name, prompt, n, margin):
+    """Greedy continuation of the oracle, cut where the two best logits come closer than ``margin``."""
+    toks, w = list(prompt), cases.weights(CONFIGS[name], 0)
+    for _ in range(n):
+        last = oracle.forward(CONFIGS[name], w, toks)[-1]
+        top = last.topk(2).values
+        if float(top[0] - top[1]) < margin * float(last.std()):
+            break
+        toks.append(int(last.argmax()))
+    return toks[len(prompt):]
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("mode", ["plain", "chunked", "mixed", "preempted", "multi-step"])
+def test_greedy_generation(device, dtype, mode):
+    name = "plain" if dtype == "float32" else "wide"
+    kw = {"plain": {}, "chunked": dict(enable_chunked_prefill=True, max_num_batched_tokens=24),
+          "mixed": dict(enable_chunked_prefill=True, mixed_batches=True, max_num_batched_tokens=24),
+          "preempted": dict(block_size=16, blocks=9, enable_chunked_prefill=True, mixed_batches=True, max_num_batched_tokens=40),
+          "multi-step": dict(num_step=3)}[mode]
+    eng = engine(name, device, dtype, **kw)
+    V = CONFIGS[name]["vocab"]
+    prompts = [tokens(n, V, seed) for n, seed in ((1, 68), (30, 76), (47, 66), (5, 51), (19, 60))]      # several tokens are clear
+    ids = [eng.add_request(p, SamplingParams(max_tokens=12, ignore_eos=True)) for p in prompts]
+    outs = eng.run_until_done(2000)
+    compared = 0
+    for i, p in zip(ids, prompts):
+        want = safe_greedy(name, tuple(p), 12, 0.002 if dtype == "float32" else 0.15)
+        assert len(outs[i]) == 12 and outs[i][: len(want)] == want
+        compared += len(want)
+    assert compared > 30
+    assert len(eng.kv.free_state_slots) == 4
+    if mode == "preempted":
+        assert eng.scheduler.stats["preemptions"] > 0
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+@pytest.mark.parametrize("num_step", [1, 3])
+def test_learned_positions_bound_the_context(device, dtype, num_step):
+    cfg = cases.config([cases.gla(mlp=None), cases.latent(mlp=None)], width=32, vocab=16, positions=50)
+    eng = build(cfg, cases.weights(cfg, 1), device, dtype, blocks=8, max_model_len=300, num_step=num_step)
+    assert eng.cfg.max_model_len == 50
+    i = eng.add_request([1] * 45, SamplingParams(max_tokens=100, ignore_eos=True))
+    assert len(eng.run_until_done(200)[i]) == 5
+    with pytest.raises(RuntimeError, match="outgrows"):
+        TraceReplay(eng).step([{"id": "s", "tokens": [1] * 51, "want": []}])
+
+
+def test_sampling_and_llm_front_end():
+    llm = LLM("tiny-zusotar", model_config=get_config("tiny-zusotar"), device="cpu", num_kv_blocks=16, block_size=16, max_model_len=128, max_num_seqs=2)
+    outs = llm.generate([[1, 2, 3], [4] * 30], SamplingParams(max_tokens=6, temperature=0.8, top_k=20, ignore_eos=True, repetition_penalty=1.1))
+    assert [len(o) for o in outs] == [6, 6] and all(0 <= t < 512 for o in outs for t in o)
+
+
+# ----------------------------------------------------------------------------- configuration, loading, caches, replay
+def test_configuration_reader():
+    d = CONFIGS["plain"]
+    c = ModelConfig.from_hf_dict(d)
+    assert c.architecture == "Zusotar" and c.norm_both and not c.norm_first and not c.streams and not c.tie_word_embeddings
+    assert (c.residual_mult, c.norm_offset, c.depth_average, c.learned_positions, c.rms_norm_eps) == (0.6, 1.0, True, 512, 1e-5)
+    s = c.layers[0].latent
+    assert (s.heads, s.dim, s.rot_dim, s.vdim, s.q_rank, s.kv_rank, s.window, s.rot_base) == (3, 16, 8, 24, 0, 32, 0, 300.0)
+    assert s.sink and s.rot_pairs and not s.gate
+    assert c.layers[0].ff == 40 and not c.layers[0].ff_bias and c.layers[0].act == "swiglu" and c.layers[0].experts is None
+    g = c.layers[1].gla
+    assert (g.heads, g.dim, g.vdim, g.tau, g.rank) == (3, 16, 24, 5.0, 0)
+    a = c.layers[2].attention
+    assert (a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.rot_dims, a.chunk, a.softcap) == (4, 2, 24, 16, 20, 0, 0, 0.0)
+    assert a.v_norm and a.log_bias and a.out_gate and not (a.qk_norm or a.sink or a.bias or a.v_mix or a.distance_bias)
+    assert c.layers[3].latent.dim == 24 and c.layers[4].attention.window == 9       # types with running numbers
+    e = c.layers[1].experts
+    assert (e.experts, e.top, e.ff, e.shared_ff, e.act, e.weighting, e.groups, e.keep_groups, e.scale) == (6, 2, 24, 40, "swiglu", "sigmoid", 3, 2, 1.0)
+    assert c.has_recurrent_state and c.unresolved_sizes()
+    c.resolve_sizes({k: tuple(v.shape) for k, v in cases.weights(d).items()})
+    assert [s.gla.rank for s in c.layers if s.gla is not None] == [12, 8] and not c.unresolved_sizes()
+    odd = ModelConfig.from_hf_dict(CONFIGS["odd"])
+    assert odd.layers[0].experts.groups == 1 and odd.layers[0].experts.shared_ff == 0 and odd.layers[1].experts is None and not odd.layers[1].ff
+
+    def bad(match, change):
+        d = copy.deepcopy(CONFIGS["plain"])
+        change(d)
+        with pytest.raises(ValueError, match=match):
+            ModelConfig.from_hf_dict(d)
+
+    bad("unknown mixer", lambda d: d["layers"][1].update(type="mamba2"))
+    bad("rotated", lambda d: d["layers"][0]["mixer"]["rot"].update(dims=4))
+    bad("heads must divide", lambda d: d["layers"][2]["mixer"].update(kv_heads=3))
+    bad("tau", lambda d: d["layers"][1]["mixer"].update(tau=0.0))
+    bad("groups", lambda d: d["layers"][2]["mlp"]["router"].update(top=5))
+    bad("groups", lambda d: d["layers"][2]["mlp"]["router"].update(groups={"count": 4, "keep": 2}))
+    bad("experts", lambda d: d["layers"][2]["mlp"]["router"].update(top=0))
+
+
+def test_loader_wants_every_tensor_and_no_other():
+    cfg = CONFIGS["odd"]
+    w = cases.weights(cfg)
+    small = dict(device="cpu", dtype="float32", blocks=4, max_model_len=64, max_num_seqs=1)
+    model = build(cfg, w, **small).worker.runner.model
+    targets = model.checkpoint_targets()
+    assert set(targets) == set(w)
+    for k, t in targets.items():
+        if len(t) == 4:
+            p, r0, rows, cols = t
+            assert torch.equal((p.data[r0:r0 + rows] if cols is None else p.data[r0:r0 + rows, :cols]).float(), w[k].float())
+    assert torch.equal(model.model.norm, 1 + w["final.norm"].float()) and torch.equal(model.model.layers[0].norm2b, 1 + w["l0.norm2b"].float())
+    for missing in ("l2.mix.uk", "pos", "l1.dwa", "l0.norm1b", "l0.mix.a1"):
+        with pytest.raises(KeyError, match="lacks"):
+            build(cfg, {k: v for k, v in w.items() if k != missing}, **small)
+    with pytest.raises(KeyError, match="no parameter"):
+        build(cfg, dict(w, **{"l1.norm2": w["l0.norm1"]}), **small)
+    for key in ("l2.mix.q", "pos", "l0.mix.norm", "l2.norm2", "l3.mix.r1"):
+        with pytest.raises(ValueError, match="shape"):
+            build(cfg, dict(w, **{key: w[key][:-1].contiguous()}), **small)
+
+
+def test_caches_by_layer():
+    eng = engine("plain", "cpu", "float32")
+    c = eng.worker.runner.kv_caches
+    assert c[0].shape == (24, 64, 40) and c[3].shape == (24, 64, 56)
+    assert [tuple(t.shape) for t in c[1]] == [(4, 3, 24, 16)] and [tuple(t.shape) for t in c[5]] == [(4, 2, 16, 24)] and c[1][0].dtype == torch.float32
+    (k, v) = c[2]
+    assert k.shape == (24, 64, 2, 24) and v.shape == (24, 64, 2, 16)
+    m = eng.worker.runner.model
+    assert m.num_kv_layers == 4 and m.kv_bytes_per_token() == (40 + 56 + 2 * (24 + 16) + 2 * (16 + 16)) * 4
+    assert m.state_bytes(4) == 4 * (3 * 24 * 16 + 2 * 16 * 24) * 4
+
+
+def test_what_the_model_does_not_combine_with():
+    for kw in (dict(enable_prefix_caching=True), dict(num_speculative_tokens=1), dict(enable_omni_attn=True, omni_attn_config={"sink": 1, "recent": 1})):
+        with pytest.raises(ValueError):
+            engine("plain", "cpu", "float32", **kw)
+
+
+@pytest.mark.parametrize("device,dtype", RUNS)
+def test_trace_runner_on_a_model_folder(device, dtype, tmp_path):
+    from omni_infer_b200.cli.trace_run import build_engine, replay
+    name = "wide"
+    cfg = CONFIGS[name]
+    write_model(tmp_path, {k: v for k, v in cfg.items() if k != "_ranks"}, cases.weights(cfg))
+    seqs = {"p": tokens(70, cfg["vocab"], 1), "q": tokens(20, cfg["vocab"], 2)}
+    steps = [{"step": 0, "entries": [{"id": "p", "tokens": seqs["p"][:50], "want": [49, 0]}, {"id": "q", "tokens": seqs["q"][:1], "want": []}],
+              "end": []},
+             {"step": 1, "entries": [{"id": "p", "tokens": seqs["p"][50:51], "want": [0]}, {"id": "q", "tokens": seqs["q"][1:2], "want": [0]}]},
+             {"step": 2, "entries": [{"id": "q", "tokens": seqs["q"][2:], "want": []}], "end": ["q"]},
+             {"step": 3, "entries": [{"id": "p", "tokens": seqs["p"][51:], "want": [18]}], "end": ["p"]}]
+    eng = build_engine(str(tmp_path), dtype, 192, device=device)
+    done = []
+    replay(eng, io.StringIO("\n".join(json.dumps(s) for s in steps)), str(tmp_path), done.append)
+    assert done == [0, 1, 2, 3] and not (tmp_path / "2.f32").exists()
+
+    def rows(k):
+        return torch.frombuffer(bytearray((tmp_path / f"{k}.f32").read_bytes()), dtype=torch.float32).view(-1, cfg["vocab"])
+
+    p, q = expected(name, 0, seqs["p"]), expected(name, 0, seqs["q"])
+    for got, want in ((rows(0), p[[49, 0]]), (rows(1), torch.stack([p[50], q[1]])), (rows(3), p[[69]])):
+        assert float(row_errors(got, want).max()) < TOL[dtype][1]
+
+
+def test_kernel_build_takes_the_architecture_sources_only():
+    from omni_infer_b200 import build as b
+    _, every = b._kernel_inputs()
+    _, some = b._kernel_inputs(b.ARCH_KERNELS["Zusotar"])
+    assert {s.stem for s in some} == set(b.ARCH_KERNELS["Zusotar"]) < {s.stem for s in every}
