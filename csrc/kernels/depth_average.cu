@@ -102,7 +102,7 @@ struct StepParams {
   int H, ld, h_ld;
 };
 
-template <typename T, int V, int KEEP>
+template <typename T, int V, int KEEP, bool AVG>
 __global__ void both_norms_step_kernel(const StepParams p, int T_rows) {
   const int t = blockIdx.x;
   __shared__ int rows[32];
@@ -117,7 +117,7 @@ __global__ void both_norms_step_kernel(const StepParams p, int T_rows) {
     else load_vec<V>((const T*)p.y + (size_t)t * p.y_ld + c, y);
   };
   // what does not wait for the norm: x, or (with an average) x apart from the part of the earlier results
-  float yk[KEEP][V], xk[KEEP][V], past[KEEP][V], ss = 0.f;
+  float yk[KEEP][V], xk[KEEP][V], past[AVG ? KEEP : 1][V], ss = 0.f;
   auto earlier = [&](int c, float (&a)[V]) {
 #pragma unroll
     for (int i = 0; i < V; ++i) a[i] = 0.f;
@@ -135,7 +135,7 @@ __global__ void both_norms_step_kernel(const StepParams p, int T_rows) {
     if (c < p.H) {
       sublayer(c, yk[k]);
       load_vec<V>(p.x_in + row + c, xk[k]);
-      if (p.results != nullptr) earlier(c, past[k]);
+      if constexpr (AVG) earlier(c, past[k]);
 #pragma unroll
       for (int i = 0; i < V; ++i) ss += yk[k][i] * yk[k][i];
     }
@@ -147,14 +147,14 @@ __global__ void both_norms_step_kernel(const StepParams p, int T_rows) {
     for (int i = 0; i < V; ++i) ss += y[i] * y[i];
   }
   const float r = p.mult / sqrtf(block_sum2(ss, 0.f).x / (float)p.H + p.eps);
-  const float last = p.results != nullptr ? p.average[p.n] : 1.f;
+  const float last = AVG ? p.average[p.n] : 1.f;
   ss = 0.f;
   auto update = [&](int c, float (&y)[V], float (&x)[V], float (&a)[V]) {      // leaves the new residual in x
     float g[V];
     load_vec<V>(p.w_out + c, g);
 #pragma unroll
     for (int i = 0; i < V; ++i) x[i] = fmaf(y[i] * r, g[i], x[i]);
-    if (p.results != nullptr) {
+    if constexpr (AVG) {
       if (p.store) store_vec<V>(p.results + p.n * layer + row + c, x);
 #pragma unroll
       for (int i = 0; i < V; ++i) x[i] = fmaf(last, x[i], a[i]);
@@ -166,13 +166,13 @@ __global__ void both_norms_step_kernel(const StepParams p, int T_rows) {
 #pragma unroll
   for (int k = 0; k < KEEP; ++k) {
     const int c = threadIdx.x * V + k * step;
-    if (c < p.H) update(c, yk[k], xk[k], past[k]);
+    if (c < p.H) update(c, yk[k], xk[k], past[AVG ? k : 0]);
   }
   for (int c = threadIdx.x * V + KEEP * step; c < p.H; c += step) {
     float y[V], x[V], a[V];
     sublayer(c, y);
     load_vec<V>(p.x_in + row + c, x);
-    if (p.results != nullptr) earlier(c, a);
+    if constexpr (AVG) earlier(c, a);
     update(c, y, x, a);
   }
   const float rn = 1.0f / sqrtf(block_sum2(ss, 0.f).x / (float)p.H + p.eps);
@@ -199,7 +199,7 @@ __global__ void both_norms_step_kernel(const StepParams p, int T_rows) {
 
 static inline int da_threads(int n, int v) {
   const int th = ((n + v - 1) / v + 31) / 32 * 32;
-  return th > 512 ? 512 : (th < 32 ? 32 : th);
+  return th > 256 ? 256 : (th < 32 ? 32 : th);
 }
 
 }  // namespace omni
@@ -215,8 +215,8 @@ extern "C" int omni_embed_positions(const int64_t* ids, const void* table, int r
   if (T_rows <= 0) return 0;
   if (H < 1 || ld < H || h_ld < H || table_ld < H || (pos_table != nullptr && (pos_ld < H || positions == nullptr))) return -1;
   const EmbedParams p = {ids, table, rows, table_ld, positions, pos_table, pos_rows, pos_ld, (float*)x, H, ld, w, eps, h, h_ld};
-  if (H % 4 == 0 && ld % 4 == 0 && h_ld % 4 == 0 && table_ld % 4 == 0 && (pos_table == nullptr || pos_ld % 4 == 0)) {
-    FOR_TYPE((embed_positions_kernel<T, 4, 2><<<T_rows, da_threads(H, 4), 0, st>>>(p));)
+  if (H % 8 == 0 && ld % 8 == 0 && h_ld % 8 == 0 && table_ld % 8 == 0 && (pos_table == nullptr || pos_ld % 8 == 0)) {
+    FOR_TYPE((embed_positions_kernel<T, 8, 2><<<T_rows, da_threads(H, 8), 0, st>>>(p));)
   } else {
     FOR_TYPE((embed_positions_kernel<T, 1, 2><<<T_rows, da_threads(H, 1), 0, st>>>(p));)
   }
@@ -233,11 +233,14 @@ extern "C" int omni_both_norms_step(const void* x_in, void* x_out, int T_rows, i
   if (results != nullptr && (average == nullptr || n < 1)) return -3;
   const StepParams p = {(const float*)x_in, (float*)x_out, y, y_ld, row_of, top_k, shared, w_out, mult, (float*)results, average, n, store,
                         w, eps, h, H, ld, h_ld};
-  if (H % 4 == 0 && ld % 4 == 0 && h_ld % 4 == 0 && y_ld % 4 == 0) {
-    FOR_TYPE((both_norms_step_kernel<T, 4, 2><<<T_rows, da_threads(H, 4), 0, st>>>(p, T_rows));)
-  } else {
-    FOR_TYPE((both_norms_step_kernel<T, 1, 2><<<T_rows, da_threads(H, 1), 0, st>>>(p, T_rows));)
-  }
+#define STEP(V, KEEP)                                                                                                            \
+  if (results != nullptr) { FOR_TYPE((both_norms_step_kernel<T, V, KEEP, true><<<T_rows, da_threads(H, V), 0, st>>>(p, T_rows));) } \
+  else { FOR_TYPE((both_norms_step_kernel<T, V, KEEP, false><<<T_rows, da_threads(H, V), 0, st>>>(p, T_rows));) }
+  const bool v8 = H % 8 == 0 && ld % 8 == 0 && h_ld % 8 == 0 && y_ld % 8 == 0;
+  if (v8 && H <= 2048) { STEP(8, 1) }
+  else if (v8) { STEP(8, 2) }
+  else { STEP(1, 2) }
+#undef STEP
   return (int)cudaGetLastError();
 }
 #undef FOR_TYPE

@@ -14,7 +14,7 @@
 // exponent that is taken here is a difference whose sign makes it at most zero.  A is made of 4 x 4 tiles: below the diagonal
 // tiles both sides refer to the tile's first row (8 exponentials for 16 products), on it every pair has its own.
 //
-// One CTA walks the chunks of one (request, head) and up to 128 of its value columns; two kinds of warps, stages of shared memory
+// One CTA walks the chunks of one (request, head) and 32, 64 or 128 of its value columns; two kinds of warps, stages of shared memory
 // between them:
 //   prep   (one to three groups of 4 warps that take turns) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
 //          the tiles of A with lanes over channels
@@ -52,7 +52,7 @@ constexpr int WK_TP = 20;                          // floats per channel of the 
 constexpr int WK_APITCH = 48;                      // bytes per row of A
 template <int DP, int VP>                            // key channels, value columns of a CTA
 struct WkLayout {
-  static constexpr int GROUPS = DP > 128 ? 1 : (DP > 64 || VP > 64 ? 2 : 3);   // prep groups, as many as fit
+  static constexpr int GROUPS = DP > 128 ? 1 : (DP > 64 && VP != 64 ? 2 : 3);   // prep groups, as many as fit
   static constexpr int STAGES = 2 * GROUPS;
   static constexpr int PITCH = DP * 2 + 16;        // bytes per token row; ldmatrix rows fall into different banks
   static constexpr int TILE = WK_L * PITCH;
@@ -64,7 +64,8 @@ struct WkLayout {
   static constexpr int T_ARR = DP * WK_TP * 4;
   static constexpr int U_OFF = T_OFF + GROUPS * 3 * T_ARR;
   static constexpr int BAR_OFF = U_OFF + DP * 4;
-  static constexpr int SMEM = BAR_OFF + 128;
+  static constexpr int SMEM = BAR_OFF + ((2 * STAGES + GROUPS) * 8 + 4 + 15) / 16 * 16;      // barriers, abort flag
+  static_assert(SMEM <= 232448, "exceeds the 227 KB shared-memory limit of one CTA");
   static constexpr int STATE_WARPS = VP / 16;
   static constexpr int THREADS = 32 * (GROUPS * WK_PREP + STATE_WARPS);
 };
@@ -121,7 +122,12 @@ __device__ __forceinline__ void wk_group_sum(float (&v)[16], int lane) {
 // log2 of the decay, from z + w0
 template <bool GLA>
 __device__ __forceinline__ float wk_log2_decay(float z, float inv_tau) {
-  if (GLA) return 1.4426950408889634f * (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau;
+  if (GLA) {      // log2 of the sigmoid; its absolute error of some 1e-7 is what a whole sequence multiplies at most
+    const float z2 = z * 1.4426950408889634f;
+    float l;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(l) : "f"(1.f + wk_ex2(-fabsf(z2))));
+    return (fminf(z2, 0.f) - l) * inv_tau;
+  }
   return -1.4426950408889634f * expf(z);
 }
 
@@ -452,11 +458,13 @@ extern "C" int omni_gla_chunks(const void* q, int q_ld, const void* k, int k_ld,
   WkvParams p = {(const __nv_bfloat16*)q, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, q_ld, k_ld, v_ld, z, z_ld, bias, nullptr,
                  q_scale, inv_tau, (float*)state, cu_q, positions, state_slots, (__nv_bfloat16*)y, y_ld, H, N, P, min_rows,
                  (OmniStatus*)status};
-#define GLA_CASE(DP)                                                \
-  if (N <= DP) {                                                    \
-    if (P <= 32) return launch_wkv<DP, 32, true>(p, B, stream);     \
-    if (P <= 64) return launch_wkv<DP, 64, true>(p, B, stream);     \
-    return launch_wkv<DP, 128, true>(p, B, stream);                 \
+  // every CTA prepares its chunks anew: 64 columns each only where that leaves no SM with two CTAs
+  const bool narrow = (long long)H * B * ((P + 63) / 64) <= 148;
+#define GLA_CASE(DP)                                                       \
+  if (N <= DP) {                                                           \
+    if (P <= 32) return launch_wkv<DP, 32, true>(p, B, stream);            \
+    if (P <= 64 || narrow) return launch_wkv<DP, 64, true>(p, B, stream);  \
+    return launch_wkv<DP, 128, true>(p, B, stream);                        \
   }
   GLA_CASE(32) GLA_CASE(64) GLA_CASE(128) GLA_CASE(256)
 #undef GLA_CASE

@@ -19,10 +19,11 @@ from test_layer_list_model import RUNS, portions, run
 from zusotar_cases import CONFIGS, expected
 
 # Most rows / all rows / the typical row.  In 16 bits a close choice of experts may fall the other way, which moves that row and a
-# little those that attend to it: all rows are held to rounding where every expert is chosen.
+# little those that attend to it: all rows are held to rounding where every expert is chosen and heads are wide enough for their
+# norms not to blow rounding up.
 TOL = {"float32": (1e-5, 3e-5, 5e-6), "bfloat16": (0.08, 0.12, 0.03)}
-CLOSE_CHOICE = (0.12, None, 0.045)
-EXACT_CHOICE = ("odd", "wide", "deep")
+LOOSE = (0.12, None, 0.045)
+EXACT = ("wide", "deep")
 
 
 @pytest.fixture(autouse=True)
@@ -46,11 +47,11 @@ def engine(name, device, dtype, seed=0, **kw):
     return build(CONFIGS[name], cases.weights(CONFIGS[name], seed), device, dtype, **kw)
 
 
-def check(got, want, dtype, exact_choice=True):
+def check(got, want, dtype, exact=True):
     e = row_errors(got, want)
-    most, every, typical = TOL[dtype] if exact_choice or dtype == "float32" else CLOSE_CHOICE
+    most, every, typical = TOL[dtype] if exact or dtype == "float32" else LOOSE
     assert float(e.median()) < typical and float(e.quantile(0.7)) < most, (float(e.max()), float(e.median()))
-    if exact_choice or dtype == "float32":
+    if exact or dtype == "float32":
         assert float(e.max()) < every, (float(e.max()), int(e.argmax()))
 
 
@@ -64,7 +65,7 @@ def test_cuts_of_one_sequence(name, device, dtype):
     eng = engine(name, device, dtype)
     for sizes in ([n], [1], [100] + [1] * 50, [2, 3], [65, 1, 64, 2], [63, 17], [29, 8, 9, 1]):
         got = run(eng, {"a": toks}, [[("a", m)] for m in portions(n, sizes)])["a"]
-        check(got, expected(name, 0, toks), dtype, name in EXACT_CHOICE)
+        check(got, expected(name, 0, toks), dtype, name in EXACT)
     assert eng.kv.num_free_blocks == 23 and len(eng.kv.free_state_slots) == 4
 
 
@@ -82,7 +83,7 @@ def test_batches_of_unequal_requests(name, device, dtype):
     for i, t in seqs.items():
         for k in range(0, len(got[i]), len(t)):
             if len(t) > 1 or dtype == "float32":
-                check(got[i][k:k + len(t)], expected(name, 0, t), dtype, name in EXACT_CHOICE)
+                check(got[i][k:k + len(t)], expected(name, 0, t), dtype, name in EXACT)
     assert eng.kv.num_free_blocks == 9
 
 
