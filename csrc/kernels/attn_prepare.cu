@@ -150,29 +150,32 @@ struct LatentParams {
   int c_cols, r_cols;                    // latent and key part in a cache row
 };
 
-template <typename T, int V>
+// A CTA per token, or (ONE_WARP) a warp per token.
+template <typename T, int V, bool ONE_WARP>
 __global__ void latent_prepare_kernel(const T* __restrict__ a, const LatentParams p, T* __restrict__ cq, T* __restrict__ cache,
-                                      T* __restrict__ rows) {
-  const int t = blockIdx.x;
+                                      T* __restrict__ rows, int T_rows) {
+  const int t = ONE_WARP ? blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.x;
+  if (ONE_WARP && t >= T_rows) return;
+  const int tid = ONE_WARP ? threadIdx.x & 31 : threadIdx.x, nt = ONE_WARP ? 32 : blockDim.x;
   const T* ar = a + (size_t)t * p.a_ld;
   const T* cr = ar + p.kv0;
   float sq = 0.f, sc = 0.f;
-  for (int c = threadIdx.x * V; c < p.q_rank; c += blockDim.x * V) {
+  for (int c = tid * V; c < p.q_rank; c += nt * V) {
     float v[V];
     load_vec<V>(ar + c, v);
 #pragma unroll
     for (int i = 0; i < V; ++i) sq += v[i] * v[i];
   }
-  for (int c = threadIdx.x * V; c < p.kv_rank; c += blockDim.x * V) {
+  for (int c = tid * V; c < p.kv_rank; c += nt * V) {
     float v[V];
     load_vec<V>(cr + c, v);
 #pragma unroll
     for (int i = 0; i < V; ++i) sc += v[i] * v[i];
   }
-  const float2 tot = block_sum2(sq, sc);
+  const float2 tot = ONE_WARP ? make_float2(warp_sum32(sq), warp_sum32(sc)) : block_sum2(sq, sc);
   const float rq = 1.0f / sqrtf(tot.x / (float)max(p.q_rank, 1) + p.eps), rc = 1.0f / sqrtf(tot.y / (float)p.kv_rank + p.eps);
   T* qd = cq + (size_t)t * p.q_cols;
-  for (int c = threadIdx.x * V; c < p.q_cols; c += blockDim.x * V) {
+  for (int c = tid * V; c < p.q_cols; c += nt * V) {
     float v[V], g[V];
 #pragma unroll
     for (int i = 0; i < V; ++i) v[i] = 0.f;
@@ -188,7 +191,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ a, const LatentParam
   const int D = p.c_cols + p.r_cols;
   T* d0 = slot >= 0 ? cache + (size_t)slot * D : nullptr;
   T* d1 = rows != nullptr ? rows + (size_t)t * D : nullptr;
-  for (int c = threadIdx.x * V; c < p.c_cols; c += blockDim.x * V) {
+  for (int c = tid * V; c < p.c_cols; c += nt * V) {
     float v[V], g[V];
 #pragma unroll
     for (int i = 0; i < V; ++i) v[i] = 0.f;
@@ -203,7 +206,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ a, const LatentParam
   }
   const int half = p.rot >> 1;
   const float* cs = p.cos_sin + (size_t)p.positions[t] * p.rot;
-  for (int c = threadIdx.x; c < p.r_cols; c += blockDim.x) {
+  for (int c = tid; c < p.r_cols; c += nt) {
     float v = 0.f;
     if (c < p.rot) {
       const int i = c < half ? c : c - half;
@@ -292,11 +295,14 @@ extern "C" int omni_latent_prepare(const void* a, int a_ld, int q_rank, int kv0,
     return -1;
   if (q_rank == 0) q_cols = 0;
   const LatentParams p = {a_ld, q_rank, kv0, kv_rank, rot, qw, cw, eps, cos_sin, positions, slots, q_cols, c_cols, r_cols};
-  if (q_rank % 4 == 0 && kv0 % 4 == 0 && kv_rank % 4 == 0 && a_ld % 4 == 0 && q_cols % 4 == 0 && c_cols % 4 == 0 && r_cols % 4 == 0) {
-    FOR_TYPE((latent_prepare_kernel<T, 4><<<T_rows, 128, 0, st>>>((const T*)a, p, (T*)cq, (T*)cache, (T*)rows));)
-  } else {
-    FOR_TYPE((latent_prepare_kernel<T, 1><<<T_rows, 128, 0, st>>>((const T*)a, p, (T*)cq, (T*)cache, (T*)rows));)
-  }
+#define LATENT(V)                                                                                                                     \
+  if (q_rank == 0) { FOR_TYPE((latent_prepare_kernel<T, V, true><<<(T_rows + 3) / 4, 128, 0, st>>>((const T*)a, p, (T*)cq, (T*)cache, (T*)rows, T_rows));) } \
+  else { FOR_TYPE((latent_prepare_kernel<T, V, false><<<T_rows, 128, 0, st>>>((const T*)a, p, (T*)cq, (T*)cache, (T*)rows, T_rows));) }
+  const int sizes = q_rank | kv0 | kv_rank | a_ld | q_cols | c_cols | r_cols;
+  if (q_rank == 0 && sizes % 8 == 0) { LATENT(8) }
+  else if (sizes % 4 == 0) { LATENT(4) }
+  else { LATENT(1) }
+#undef LATENT
   return (int)cudaGetLastError();
 }
 
