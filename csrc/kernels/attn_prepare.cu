@@ -2,8 +2,8 @@
 //   omni_qkv_prepare     optional RMSNorm of every q and k head, rotation of the first dimensions of every head (halves or
 //                        neighbours), values mixed with those of an earlier layer or divided by their head's root mean square, K/V
 //                        scatter into the paged cache
-//   omni_latent_prepare  latent attention: RMSNorm of the query latent (if there is one) and of the key/value latent, rotation of the shared key
-//                        part; latent | key part go to the cache and, if asked for, to contiguous rows
+//   omni_latent_prepare  latent attention: RMSNorm of the query latent (if there is one) and of the key/value latent, rotation of
+//                        the shared key part; latent | key part go to the cache and, if asked for, to contiguous rows
 //   omni_rotate_heads    rotation of a part of every head, in place or into another layout
 //   omni_gather_pages    rows of the paged cache to contiguous rows, a range of positions per request
 // Activations are bf16 or fp32 (`f32`), norm weights and angles fp32; every value between two roundings is fp32.  cos_sin
@@ -290,7 +290,8 @@ extern "C" int omni_latent_prepare(const void* a, int a_ld, int q_rank, int kv0,
                                    int q_cols, void* cache, void* rows, int c_cols, int r_cols, int T_rows, int f32,
                                    cudaStream_t st) {
   if (T_rows <= 0) return 0;
-  if (q_rank < 0 || (q_rank > 0 && (cq == nullptr || qw == nullptr)) || kv_rank < 1 || rot < 2 || rot % 2 != 0 || q_cols < q_rank || c_cols < kv_rank || r_cols < rot || kv0 < q_rank ||
+  if (q_rank < 0 || (q_rank > 0 && (cq == nullptr || qw == nullptr))) return -2;
+  if (kv_rank < 1 || rot < 2 || rot % 2 != 0 || q_cols < q_rank || c_cols < kv_rank || r_cols < rot || kv0 < q_rank ||
       a_ld < kv0 + kv_rank + rot || cos_sin == nullptr)
     return -1;
   if (q_rank == 0) q_cols = 0;

@@ -325,7 +325,8 @@ gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __re
     if (splits == 1) {
       float den = ll;
       if (GEN && sh.sink != nullptr && ll > 0.f) den += exp2f(sh.sink[hq] * 1.4426950408889634f - mm);
-      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / den * (GEN ? sh.out_scale * gq_gate(sh.gate, sh.gate_ld, sh.gate_cols, b, hq, d) : 1.f) : 0.f);
+      const float f = GEN ? sh.out_scale * gq_gate(sh.gate, sh.gate_ld, sh.gate_cols, b, hq, d) : 1.f;
+      out[(size_t)b * out_ld + hq * dv + d] = __float2bfloat16(ll > 0.f ? acc / den * f : 0.f);
     } else {
       o_part[(((size_t)b * splits + split) * Hq + hq) * dv + d] = ll > 0.f ? acc / ll : 0.f;
       if (d == 0) lse_part[((size_t)b * splits + split) * Hq + hq] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
@@ -402,7 +403,8 @@ extern "C" int omni_gqa_paged_decode_window(const void* q, int q_ld, const void*
                                             long long v_row, const int* q_to_seq, const int* block_table, int bt_ld,
                                             const int* seq_lens, int B, int Hq, int Hkv, int dk, int dv, int block_size,
                                             int window, int chunk, int keep, float scale, float softcap, const float* slopes,
-                                            const float* r1, const float* r2, const float* sink, const void* gate, int gate_ld, int gate_cols, float out_scale, int splits, float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
+                                            const float* r1, const float* r2, const float* sink, const void* gate, int gate_ld,
+                                            int gate_cols, float out_scale, int splits, float* o_part, float* lse_part, void* out, int out_ld, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (Hkv < 1 || Hq % Hkv != 0 || splits < 1 || splits > 65535 || B > 65535 || window < 0) return -1;
   if (splits > 1 && (o_part == nullptr || lse_part == nullptr)) return -2;

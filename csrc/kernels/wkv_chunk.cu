@@ -16,8 +16,8 @@
 //
 // One CTA walks the chunks of one (request, head) and 32, 64 or 128 of its value columns; two kinds of warps, stages of shared memory
 // between them:
-//   prep   (one to three groups of 4 warps that take turns) elementwise part with a thread per channel and 8 tokens, the next chunk's inputs already in registers, then
-//          the tiles of A with lanes over channels
+//   prep   (one to three groups of 4 warps that take turns) elementwise part with a thread per channel and 8 tokens, the next
+//          chunk's inputs already in registers, then the tiles of A with lanes over channels
 //   state  (one warp per 16 value columns) S^T in fp32 accumulators; O^T = S^T R^T + V^T A^T and S^T += V^T K on mma.sync, S^T being
 //          its own A operand.  A chunk of 16 tokens is too short for tcgen05: the chain from S to S would go through tensor memory
 //          and two commits per chunk, where it is a handful of dependent MMAs here.

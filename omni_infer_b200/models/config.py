@@ -513,7 +513,8 @@ class ModelConfig:
             mixed = {s.attention.kv_heads * s.attention.vdim for s in layers if s.attention is not None and s.attention.v_mix}
             if len(mixed) > 1:
                 raise ValueError("layers that mix their values must have equally many of them")
-        elif not norm_both and any((s.parallel or s.wkv or s.experts) is not None if not streams else (s.attention or s.mamba2) is not None or s.ff for s in layers):
+        elif not norm_both and any((s.parallel or s.wkv or s.experts) is not None if not streams
+                                   else (s.attention or s.mamba2) is not None or s.ff for s in layers):
             raise ValueError("attention, mamba2 and dense layers run on one residual with norms on the outputs, parallel, wkv and "
                              "mixture-of-experts layers on residual streams with norms ahead")
         for i, s in enumerate(layers):

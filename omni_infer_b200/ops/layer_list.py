@@ -220,7 +220,8 @@ def paged_attention(q, k_cache, v_cache, *, positions, q_to_seq, slots, block_ta
     positions up to its own (0: all of them), only those of its own ``chunk`` of positions (0: no chunks), and the ``keep_first``
     first ones in any case.  A score is ``softcap tanh(q k scale / softcap) - slopes[head] distance``, less ``r1[head]
     ln(1 + r2[head] distance)`` with ``log_bias`` = (r1, r2) (each part optional).  ``sink`` [hq] fp32: exp(sink) is one more term of
-    the head's softmax denominator; ``out_scale`` multiplies the result, and so does the sigmoid of ``gate``, [T, hq] or [T, hq * dv].  Returns [T, pad8(hq * dv)], or writes the first columns of ``out``.  The value cache may be a
+    the head's softmax denominator; ``out_scale`` multiplies the result, and so does the sigmoid of ``gate``, [T, hq]
+    or [T, hq * dv].  Returns [T, pad8(hq * dv)], or writes the first columns of ``out``.  The value cache may be a
     column slice of the key cache (one key/value head).
 
     bf16 portions of prompts run on tcgen05 (``omni_fmha_paged``), bf16 single tokens on the split-KV decode kernel; fp32
